@@ -171,10 +171,8 @@ struct Engine {
   bool stack_capturing = false;  // a decode pass is being captured: nothing in it may wait for the device
   struct StackSpanH { int tok0, len, pos0, slot; bool products; };
   std::vector<StackSpanH> stack_spans_h;  // spans of the pass being built; products: its latent attention runs as matrix products
-  int stack_lat_split = 1, stack_lat_keys = 0;  // slicing of the history in latent attention for the pass being built
   int stack_abq = 0;          // tokens per query block of paged attention (0: the model has none); smallest over its layers
   int stack_kb = 0;           // its query blocks in the pass being built
-  int stack_att_split = 1, stack_att_keys = 0;  // its slicing of the history (layers without a chunked mask)
   std::vector<std::pair<int, int>> stack_att_plan;  // per layer: (slices, keys per slice) of paged attention in the pass being built;
                                                     // a chunked mask bounds the history a block walks, so its layers slice on their own
   std::map<std::vector<uint64_t>, uint64_t> stack_graph_ids;  // (pass shape, slicing of every layer) -> key into `graphs`

@@ -54,7 +54,7 @@ template <int BN, bool kDual>
 __global__ void __launch_bounds__(kGemmThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
                     float *__restrict__ out_partial, uint16_t *__restrict__ out_act, int T, int N, int K,
-                    int w_row0, int up_row_off, int kb_per_split, int tile_rows, int n_stages, int early_tma, int act_kind) {
+                    int w_row0, int up_row_off, int kb_per_split, int tile_rows, int n_stages, int early_tma, int act_kind, int ld_act) {
   using Cfg = GemmCfg<BN, kDual>;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t smem_base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -173,7 +173,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
               // act_kind 0: silu(gate) * up; 1: gelu_tanh(gate) * up
               const float av = act_kind == 1 ? 0.5f * gv * (1.f + tanhf(0.7978845608028654f * (gv + 0.044715f * gv * gv * gv)))
                                              : gv / (1.0f + expf(-gv));
-              out_act[(size_t)t * N + n] = float_to_bf16_bits(av * uv);
+              out_act[(size_t)t * ld_act + n] = float_to_bf16_bits(av * uv);
             }
           }
         }
@@ -253,7 +253,7 @@ int gemm_pick_split_k(int T, int N, int K) {
 
 template <int BN, bool kDual>
 static cudaError_t gemm_launch(const TmaMap &w_map, const TmaMap &x_map, float *out, uint16_t *act, int T, int N,
-                               int K, int w_row0, int up_off, int split_k, int tile_rows, cudaStream_t st, int act_kind = 0) {
+                               int K, int w_row0, int up_off, int split_k, int tile_rows, cudaStream_t st, int act_kind = 0, int ld_act = 0) {
   using Cfg = GemmCfg<BN, kDual>;
   auto kern = gemm_tcgen05_kernel<BN, kDual>;
   static DeviceOnce once;
@@ -283,7 +283,7 @@ static cudaError_t gemm_launch(const TmaMap &w_map, const TmaMap &x_map, float *
   static int early = -1;
   if (early < 0) { const char *e = getenv("DIS_GEMM_EARLY_TMA"); early = (e && atoi(e) == 0) ? 0 : 1; }
   return launch_k(kern, grid, dim3(kGemmThreads), (size_t)smem, st, *reinterpret_cast<const CUtensorMap *>(&w_map),
-                  *reinterpret_cast<const CUtensorMap *>(&x_map), out, act, T, N, K, w_row0, up_off, per, tile_rows, stages, early, act_kind);
+                  *reinterpret_cast<const CUtensorMap *>(&x_map), out, act, T, N, K, w_row0, up_off, per, tile_rows, stages, early, act_kind, ld_act > 0 ? ld_act : N);
 }
 
 cudaError_t launch_gemm_partial(const TmaMap &w_map, const TmaMap &x_map, float *out, int T, int N, int K,
@@ -307,13 +307,13 @@ int gemm_pick_tile_rows(int N) {
 }
 
 cudaError_t launch_gemm_glu(const TmaMap &w_map, const TmaMap &x_map, uint16_t *act, int T, int I, int K,
-                            int w_row0, int tile_rows, int act_kind, cudaStream_t st) {
+                            int w_row0, int tile_rows, int act_kind, cudaStream_t st, int ld_act) {
   if (T <= 0) return cudaSuccess;
   switch (gemm_token_tile(T)) {
-    case 32: return gemm_launch<32, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind);
-    case 64: return gemm_launch<64, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind);
-    case 128: return gemm_launch<128, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind);
-    default: return gemm_launch<256, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind);
+    case 32: return gemm_launch<32, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind, ld_act);
+    case 64: return gemm_launch<64, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind, ld_act);
+    case 128: return gemm_launch<128, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind, ld_act);
+    default: return gemm_launch<256, true>(w_map, x_map, nullptr, act, T, I, K, w_row0, I, 1, tile_rows, st, act_kind, ld_act);
   }
 }
 cudaError_t launch_gemm_silu(const TmaMap &w_map, const TmaMap &x_map, uint16_t *act, int T, int I, int K,

@@ -524,18 +524,19 @@ cudaError_t launch_stack_final_ln(const float *x, const int *row_map, const floa
   return cudaGetLastError();
 }
 
-// Pre-norm boundary over residual streams, one block per token.  xs [T][S][W].  y = bias + the n_part slices of the product before.
+// Pre-norm boundary over residual streams, one block per token.  xs [T][S][W].  y = mult * (bias + the n_part slices of the
+// product before).
 // prev (or null) = the coefficients of the sublayer that made y, laid out in[S] | out[S] | mix[S][S] (mix indexed [from][to]):
 // every stream becomes x_t <- sum_s mix[s][t] x_s + out[t] y, all from the old streams; prev == null: the one stream gets x += y.
 // Then, with pre_w: u = sum_s next[s] x_s (next = the coming sublayer's coefficients, their first S numbers; null: u = x_0), and
 // h = u / sqrt(mean(u^2) + eps) * pre_w goes to hc in the compute type.  Everything is fp32.
 constexpr int kHcMaxStreams = 8;
-// SS: the number of streams when the compiler may know it (2, 4), else 0 and S counts at run time up to kHcMaxStreams.
+// SS: the number of streams when the compiler may know it (1, 2, 4), else 0 and S counts at run time up to kHcMaxStreams.
 // VEC: W is a multiple of 4 and every pointer 16-byte aligned, so a thread moves four neighbouring columns per access.
 template <bool F32, int SS, bool VEC>
 __global__ void __launch_bounds__(256) stack_boundary_hc_kernel(float *xs, int S_rt, const float *__restrict__ y, int n_part, long long stride,
                                                                 const float *__restrict__ bias, const float *prev, const float *next,
-                                                                const float *__restrict__ pre_w, void *hc, int W, float eps) {
+                                                                const float *__restrict__ pre_w, void *hc, int W, float eps, float mult) {
   extern __shared__ __align__(16) float row[];  // [W]: u
   __shared__ float sh[32];
   __shared__ float cf[2 * kHcMaxStreams + kHcMaxStreams * kHcMaxStreams];  // out[S] | mix[S][S] of prev, then in[S] of next
@@ -586,6 +587,8 @@ __global__ void __launch_bounds__(256) stack_boundary_hc_kernel(float *xs, int S
         for (int e = 0; e < V; e++) v[e] += p[e];
       }
 #pragma unroll
+      for (int e = 0; e < V; e++) v[e] *= mult;
+#pragma unroll
       for (int to = 0; to < SM; to++) {
         if (to < S) {
           float nv[V];
@@ -635,22 +638,22 @@ __global__ void __launch_bounds__(256) stack_boundary_hc_kernel(float *xs, int S
 }
 template <bool F32, int SS, bool VEC>
 static cudaError_t boundary_hc_go(float *xs, int streams, const float *y, int n_part, long long stride, const float *bias, const float *prev,
-                                  const float *next, const float *pre_w, void *hc, int T, int W, float eps, cudaStream_t st) {
+                                  const float *next, const float *pre_w, void *hc, int T, int W, float eps, float mult, cudaStream_t st) {
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_boundary_hc_kernel<F32, SS, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); }));
-  stack_boundary_hc_kernel<F32, SS, VEC><<<T, 256, (size_t)W * 4, st>>>(xs, streams, y, n_part, stride, bias, prev, next, pre_w, hc, W, eps);
+  stack_boundary_hc_kernel<F32, SS, VEC><<<T, 256, (size_t)W * 4, st>>>(xs, streams, y, n_part, stride, bias, prev, next, pre_w, hc, W, eps, mult);
   return cudaGetLastError();
 }
 cudaError_t launch_stack_boundary_hc(float *xs, int streams, const float *y, int n_part, long long stride, const float *bias,
                                      const float *prev, const float *next, const float *pre_w, void *hc, bool f32, int T, int W, float eps,
-                                     cudaStream_t st) {
+                                     float mult, cudaStream_t st) {
   if (streams < 1 || streams > kHcMaxStreams || (size_t)W * 4 > 160 * 1024) return cudaErrorInvalidValue;
   if (T <= 0) return cudaSuccess;
   if (n_part < 1) n_part = 1;
   auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const bool vec = W % 4 == 0 && stride % 4 == 0 && al(xs) && al(y) && al(bias) && al(pre_w) && al(hc);
-#define DIS_HC(F, SSV, VV) return boundary_hc_go<F, SSV, VV>(xs, streams, y, n_part, stride, bias, prev, next, pre_w, hc, T, W, eps, st)
-#define DIS_HC_S(F, VV) do { if (streams == 2) DIS_HC(F, 2, VV); if (streams == 4) DIS_HC(F, 4, VV); DIS_HC(F, 0, VV); } while (0)
+#define DIS_HC(F, SSV, VV) return boundary_hc_go<F, SSV, VV>(xs, streams, y, n_part, stride, bias, prev, next, pre_w, hc, T, W, eps, mult, st)
+#define DIS_HC_S(F, VV) do { if (streams == 1) DIS_HC(F, 1, VV); if (streams == 2) DIS_HC(F, 2, VV); if (streams == 4) DIS_HC(F, 4, VV); DIS_HC(F, 0, VV); } while (0)
   if (f32) { if (vec) DIS_HC_S(true, true); else DIS_HC_S(true, false); }
   else { if (vec) DIS_HC_S(false, true); else DIS_HC_S(false, false); }
 #undef DIS_HC_S
@@ -815,14 +818,14 @@ __device__ __forceinline__ float glu_unit(float g, float u, float limit) {
   return g * sigmoid_precise(1.702f * g) * (u + 1.f);
 }
 // VEC: ff is a multiple of 4 and every base pointer 16-byte aligned: a thread takes four neighbouring columns (16-byte loads of
-// gate and up, one 8- or 16-byte store).  An ungated activation (DIS_ACT_RELU2) reads rows of ff columns, not 2 ff.
+// gate and up, one 8- or 16-byte store).  An ungated activation (DIS_ACT_RELU2) reads ff columns of a row, not 2 ff.
 template <bool F32, int ACT, bool VEC>
 __global__ void stack_glu_kernel(const float *__restrict__ gu, int n_part, long long stride, const float *__restrict__ bias,
-                                 void *__restrict__ act, const int *rows_ptr, int M, int ff, float limit) {
+                                 void *__restrict__ act, const int *rows_ptr, int M, int ff, float limit, long long ld_gu, long long ld_act) {
   const int rows = rows_ptr ? min(M, rows_ptr[0]) : M;
   for (int r = blockIdx.x; r < rows; r += gridDim.x) {
     constexpr bool GATED = ACT != DIS_ACT_RELU2;
-    const float *gr = gu + (long long)r * (GATED ? 2 : 1) * ff;
+    const float *gr = gu + (long long)r * ld_gu;
     if (VEC) {
       for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4; c < ff; c += gridDim.y * blockDim.x * 4) {
         const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -838,32 +841,34 @@ __global__ void stack_glu_kernel(const float *__restrict__ gu, int n_part, long 
         }
         const float v0 = glu_unit<ACT>(g.x, u.x, limit), v1 = glu_unit<ACT>(g.y, u.y, limit), v2 = glu_unit<ACT>(g.z, u.z, limit),
                     v3 = glu_unit<ACT>(g.w, u.w, limit);
-        if (F32) *reinterpret_cast<float4 *>(reinterpret_cast<float *>(act) + (long long)r * ff + c) = make_float4(v0, v1, v2, v3);
+        if (F32) *reinterpret_cast<float4 *>(reinterpret_cast<float *>(act) + (long long)r * ld_act + c) = make_float4(v0, v1, v2, v3);
         else {
           uint2 o;
           o.x = (uint32_t)float_to_bf16_bits(v0) | ((uint32_t)float_to_bf16_bits(v1) << 16);
           o.y = (uint32_t)float_to_bf16_bits(v2) | ((uint32_t)float_to_bf16_bits(v3) << 16);
-          *reinterpret_cast<uint2 *>(reinterpret_cast<uint16_t *>(act) + (long long)r * ff + c) = o;
+          *reinterpret_cast<uint2 *>(reinterpret_cast<uint16_t *>(act) + (long long)r * ld_act + c) = o;
         }
       }
     } else {
       for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ff; c += gridDim.y * blockDim.x) {
         float g = gr[c] + (bias ? bias[c] : 0.f), u = GATED ? gr[ff + c] + (bias ? bias[ff + c] : 0.f) : 0.f;
         for (int k = 1; k < n_part; k++) { g += gr[(long long)k * stride + c]; if (GATED) u += gr[(long long)k * stride + ff + c]; }
-        st_el<F32>(act, (long long)r * ff + c, glu_unit<ACT>(g, u, limit));
+        st_el<F32>(act, (long long)r * ld_act + c, glu_unit<ACT>(g, u, limit));
       }
     }
   }
 }
 cudaError_t launch_stack_glu(const float *gu, int n_part, long long stride, const float *bias, void *act, bool f32, const int *rows_ptr,
-                             int M, int ff, float limit, int kind, cudaStream_t st) {
+                             int M, int ff, float limit, int kind, cudaStream_t st, long long ld_gu, long long ld_act) {
   if (M <= 0) return cudaSuccess;
-  const bool vec = ff % 4 == 0 && stride % 4 == 0 && reinterpret_cast<uintptr_t>(gu) % 16 == 0 && reinterpret_cast<uintptr_t>(act) % 16 == 0 &&
+  if (ld_gu <= 0) ld_gu = (long long)(kind == DIS_ACT_RELU2 ? 1 : 2) * ff;
+  if (ld_act <= 0) ld_act = ff;
+  const bool vec = ff % 4 == 0 && stride % 4 == 0 && ld_gu % 4 == 0 && ld_act % 4 == 0 && reinterpret_cast<uintptr_t>(gu) % 16 == 0 && reinterpret_cast<uintptr_t>(act) % 16 == 0 &&
                    reinterpret_cast<uintptr_t>(bias) % 16 == 0;
   const int per = vec ? 4 : 1;
   // few rows: the columns are spread over grid.y as well
   const dim3 grid(std::min(M, 148 * 16), M >= 512 ? 1 : std::min((ff + 256 * per - 1) / (256 * per), 16));
-#define DIS_GLU(F, A, V) stack_glu_kernel<F, A, V><<<grid, 256, 0, st>>>(gu, n_part, stride, bias, act, rows_ptr, M, ff, limit)
+#define DIS_GLU(F, A, V) stack_glu_kernel<F, A, V><<<grid, 256, 0, st>>>(gu, n_part, stride, bias, act, rows_ptr, M, ff, limit, ld_gu, ld_act)
 #define DIS_GLU_ACT(A)                     \
   do {                                     \
     if (f32 && vec) DIS_GLU(true, A, true); \

@@ -14,15 +14,16 @@ namespace dis {
 // the keys).  `bias` (or null): one entry per column of the projection, added here when the product left it out.
 // kpool == null: the layer reads another layer's cache; only the queries are prepared.
 // n_part > 1: the projection comes as split-K slices (slice stride `stride`); the block first sums its token's row of n_cols
-// columns (and the bias) into shared memory and works from there.  gate_out (or null): receives columns gate_off .. + H of the
-// row (the logits of the output gates, which the attention kernel reads from memory).
+// columns (and the bias) into shared memory and works from there.  gate_out (or null): receives columns gate_off .. of the row, H or
+// (DIS_ATTN_GATE_FULL) H*dv of them (the logits of the output gates, which the attention kernel reads from memory).
+// mix: DIS_ATTN_V_MIX -- the first such layer of a pass leaves its values in mix.save, the later ones blend theirs with them.
 template <bool F32>
 __global__ void __launch_bounds__(128) stack_attn_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
                                                               int gate_off, float *gate_out, long long ld_gate, int q_off, int k_off, int v_off,
                                                               const float *bias, const float *qn, const float *kn, const double *freq,
                                                               const double *vfreq, StackAttn c, StackSpans sp, float *qf, void *kpool,
                                                               void *vpool, float *vrot, const int *page_table, int max_pages,
-                                                              int page_size) {
+                                                              int page_size, StackVMix mix) {
   extern __shared__ __align__(16) float tab[];  // cos [half], sin [half], value cos [dv/2], value sin [dv/2], per-head factors [H + G], summed row
   const int srow_off = (c.rot_dims + c.dv + c.H + c.G + 3) & ~3;  // the summed row starts on a 16-byte boundary
   __shared__ float sh[32];
@@ -51,23 +52,16 @@ __global__ void __launch_bounds__(128) stack_attn_prep_kernel(const float *proj,
     __syncthreads();
   }
   if (gate_out)
-    for (int i = threadIdx.x; i < c.H; i += blockDim.x) gate_out[(long long)t * ld_gate + i] = row[gate_off + i];
+    for (int i = threadIdx.x, n = (c.flags & DIS_ATTN_GATE_FULL) ? c.H * c.dv : c.H; i < n; i += blockDim.x) gate_out[(long long)t * ld_gate + i] = row[gate_off + i];
   const int pos = sp.pos[t], slot = sp.slot[t];
   const int half = c.rot_dims >> 1, vhalf = c.dv >> 1;
   const bool rot_v = (c.flags & DIS_ATTN_ROT_V) != 0, own = kpool != nullptr;
   float *cs = tab, *sn = tab + half, *vcs = sn + half, *vsn = vcs + vhalf, *hr = vsn + vhalf;
-  // the angle pos * f is formed and brought into [-pi, pi] in double (position 100000 is then as exact as position 5); sine and
-  // cosine of the reduced angle are float
-  auto angle = [](int p, double f, float *sn_out, float *cs_out) {
-    const double a = (double)p * f;
-    const double r = a - 6.283185307179586476925 * rint(a * 0.15915494309189533577);
-    sincosf((float)r, sn_out, cs_out);
-  };
-  for (int i = threadIdx.x; i < half; i += blockDim.x) angle(pos, freq[i], &sn[i], &cs[i]);
+  for (int i = threadIdx.x; i < half; i += blockDim.x) angle_sincos(pos, freq[i], &sn[i], &cs[i]);
   if (rot_v)
     for (int i = threadIdx.x; i < vhalf; i += blockDim.x) {
       float s_, c_;
-      angle(pos, vfreq[i], &s_, &c_);
+      angle_sincos(pos, vfreq[i], &s_, &c_);
       vcs[i] = c_; vsn[i] = s_;
       vrot[(long long)t * c.dv + i] = c_;
       vrot[(long long)t * c.dv + vhalf + i] = s_;
@@ -124,6 +118,8 @@ __global__ void __launch_bounds__(128) stack_attn_prep_kernel(const float *proj,
       auto vv = [&](int j) { return row[v_off + j] + (vb ? vb[j] : 0.f); };
       v = e < vhalf ? vv(i) * vcs[e] - vv(i + vhalf) * vsn[e] : vv(i) * vcs[e - vhalf] + vv(i - vhalf) * vsn[e - vhalf];
     }
+    if (mix.save) mix.save[(long long)t * nv + i] = v;
+    if (mix.first) { const float lam = mix.lam[0]; v = (1.f - lam) * v + lam * mix.first[(long long)t * nv + i]; }
     st_el<F32>(vpool, prow * nv + i, v);
   }
 }
@@ -131,7 +127,7 @@ cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, 
                                    long long ld_gate, int q_off, int k_off, int v_off, const float *bias, const float *qn,
                                    const float *kn, const double *freq, const double *vfreq, const StackAttn &c, const StackSpans &sp,
                                    float *qf, void *kpool, void *vpool, float *vrot, bool f32, const int *page_table, int max_pages,
-                                   int page_size, cudaStream_t st) {
+                                   int page_size, const StackVMix &mix, cudaStream_t st) {
   if (sp.T <= 0) return cudaSuccess;
   if (n_part < 1) n_part = 1;
   const size_t sh = (size_t)(((c.rot_dims + c.dv + c.H + c.G + 3) & ~3) + (n_part > 1 ? n_cols : 0)) * sizeof(float);
@@ -141,8 +137,8 @@ cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, 
     cudaError_t e = cudaFuncSetAttribute(stack_attn_prep_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_attn_prep_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   }));
-  if (f32) stack_attn_prep_kernel<true><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size);
-  else stack_attn_prep_kernel<false><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size);
+  if (f32) stack_attn_prep_kernel<true><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
+  else stack_attn_prep_kernel<false><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
   return cudaGetLastError();
 }
 
@@ -152,6 +148,15 @@ cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, 
 // coordinates.  SIG: weight = sigmoid(score * temp[h] + pb[h]), plain sums.  Otherwise an online softmax (running maximum and
 // denominator per pair).  Epilogue (whole history in one CTA) or merge kernel (slices): normalise, rotate the output back by
 // the query's position when values were rotated, scale, and store into the mixer's output row.
+// A block walks the keys any of its tokens may see: the kept first positions below its window, then everything from the window's
+// start k_lo on.  Both runs are numbered through: index v < n_keep is position v, index v >= n_keep is position v + shift, so tiles
+// and slices are cut over one gapless range [0, total) and no tile is spent on a short run of kept keys.
+struct AttnWalk {
+  int n_keep, shift;
+  __device__ __forceinline__ AttnWalk(const StackAttn &c, int k_lo) : n_keep(min(c.keep, k_lo)), shift(k_lo - n_keep) {}
+  __device__ __forceinline__ int key(int v) const { return v < n_keep ? v : v + shift; }
+  __device__ __forceinline__ int total(int last_pos) const { return last_pos + 1 - shift; }
+};
 constexpr int kAtTile = 32, kAtWarps = 8, kAtMaxSplit = 64;
 bool stack_attn_mma_ok(const StackAttn &c, bool f32);
 int stack_attn_mma_block_tokens(const StackAttn &c);
@@ -164,6 +169,7 @@ struct AttnOut {
   const float *vrot;  // [T][dv]: cos | sin of the query position's value angles, or null
   const float *gate;  // [T][ldg]: logit of head h's output gate at column h, or null
   long long ldg;
+  const float *gate_full;  // [T][ldg]: logit of the gate of head h's coordinate j at column h * dv + j, or null
 };
 // factor on head h's output at token tok: the mixer's weight times the head's sigmoid gate
 __device__ __forceinline__ float attn_out_factor(const AttnOut &o, int tok, int h) {
@@ -178,6 +184,7 @@ __device__ __forceinline__ void attn_store(const AttnOut &o, const float *a, flo
     const float *cs = o.vrot + (long long)tok * dv, *sn = cs + hf;
     v = j < hf ? (a[j] * cs[j] + a[j + hf] * sn[j]) * inv : (a[j] * cs[j - hf] - a[j - hf] * sn[j - hf]) * inv;
   }
+  if (o.gate_full) v *= sigmoid_precise(o.gate_full[(long long)tok * o.ldg + (long long)h * dv + j]);
   st_el<F32>(o.out, (long long)tok * o.ld + o.off + (long long)h * dv + j, v * attn_out_factor(o, tok, h));
 }
 
@@ -221,20 +228,22 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) { mx[i] = with_sink ? sink[g * R + i % R] : -INFINITY; dn[i] = with_sink ? 1.f : 0.f; }
   const int *pt = page_table + (long long)slot * max_pages;
   const int k_lo = stack_attn_row_lo(c, sp.pos[tok0]);
-  const int k_begin = part ? k_lo + (int)blockIdx.z * keys_per_split : k_lo;
-  const int k_end = part ? min(last_pos + 1, k_begin + keys_per_split) : last_pos + 1;
+  const AttnWalk wk(c, k_lo);
+  const int k_begin = part ? (int)blockIdx.z * keys_per_split : 0;  // indices of the walk
+  const int k_end = part ? min(wk.total(last_pos), k_begin + keys_per_split) : wk.total(last_pos);
   const long long krow = (long long)c.G * d, vrow = (long long)c.G * dv;
+  const bool dist = !SIG && (c.flags & DIS_ATTN_DISTANCE);
   const float inv_cap = c.softcap > 0.f ? 1.f / c.softcap : 0.f;
   for (int k0 = k_begin; k0 < k_end; k0 += kAtTile) {
     const int nk = min(kAtTile, k_end - k0);
     __syncthreads();
     for (int i = threadIdx.x; i < nk * d; i += blockDim.x) {
-      const int kk = i / d, cc = i - kk * d, kp = k0 + kk;
+      const int kk = i / d, cc = i - kk * d, kp = wk.key(k0 + kk);
       const long long prow = (long long)pt[kp / page_size] * page_size + kp % page_size;
       kt[(size_t)kk * DP + cc] = ld_el<F32>(kpool, prow * krow + (long long)g * d + cc);
     }
     for (int i = threadIdx.x; i < nk * dv; i += blockDim.x) {
-      const int kk = i / dv, cc = i - kk * dv, kp = k0 + kk;
+      const int kk = i / dv, cc = i - kk * dv, kp = wk.key(k0 + kk);
       const long long prow = (long long)pt[kp / page_size] * page_size + kp % page_size;
       vt[(size_t)kk * VP + cc] = ld_el<F32>(vpool, prow * vrow + (long long)g * dv + cc);
     }
@@ -244,7 +253,8 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
       const int qlo = stack_attn_row_lo(c, qpos);
       const float *q = qs + (size_t)p * d;
       float sc = -INFINITY;
-      if (l < nk && k0 + l <= qpos && k0 + l >= qlo) {
+      const int kp = wk.key(k0 + l);
+      if (l < nk && kp <= qpos && (kp >= qlo || kp < c.keep)) {
         const float *kr = kt + (size_t)l * DP;
         float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;  // four chains, added at the end: the sum's order is fixed by d alone
         int i = 0;
@@ -255,6 +265,7 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
         for (; i < d; i++) s0 = fmaf(q[i], kr[i], s0);
         sc = ((s0 + s1) + (s2 + s3)) * c.scale;
         if (c.softcap > 0.f) sc = c.softcap * tanhf(sc * inv_cap);
+        if (dist) sc -= stack_attn_slope(h, c.H) * (float)(qpos - kp);
       }
       float pr, corr = 1.f, psum = 0.f, m_new = 0.f;
       if (SIG) {
@@ -375,17 +386,21 @@ __device__ __forceinline__ float ex2_(float x) {  // 2^x, flushing results below
 // skip the checks.
 // cap2 > 0 (softmax only): the scaled score s passes cap tanh(s / cap) first; scale2 is then the plain scale over the cap, and
 // tanh x = 1 - 2 / (1 + e^(2x)) is formed with one ex2 and one reciprocal (absolute error of the order of 1e-7, times the cap).
-template <bool SIG, bool MASKED>
+// k0: index of the tile's first key in the walk `wk`; keep: positions below it are always visible.  DIST: the score is lowered by
+// slope2[e] per position of distance (slope in units of log 2).
+template <bool SIG, bool MASKED, bool DIST>
 __device__ __forceinline__ void attn_tile_weights(float (&sacc)[kMmKeys / 8][4], float (&mnew)[2], int k0, int qd, const int (&r_pos)[2],
-                                                  const int (&r_lo)[2], int k_end, const float (&tmp_h)[2], const float (&pb_h)[2],
-                                                  float scale2, float cap2) {
+                                                  const int (&r_lo)[2], int k_end, const AttnWalk &wk, int keep, const float (&tmp_h)[2],
+                                                  const float (&pb_h)[2], const float (&slope2)[2], float scale2, float cap2) {
 #pragma unroll
   for (int j = 0; j < kMmKeys / 8; j++)
 #pragma unroll
     for (int q4 = 0; q4 < 4; q4++) {
       const int e = q4 >> 1;
       bool vis = true;
-      if (MASKED) { const int kp = k0 + j * 8 + qd * 2 + (q4 & 1); vis = kp <= r_pos[e] && kp < k_end && kp >= r_lo[e]; }
+      const int v = k0 + j * 8 + qd * 2 + (q4 & 1);
+      int kp = v + wk.shift;  // (a tile that needs no mask holds no kept keys from below the window)
+      if (MASKED) { kp = wk.key(v); vis = kp <= r_pos[e] && v < k_end && (kp >= r_lo[e] || kp < keep); }
       float sv = sacc[j][q4];
       if (SIG) {
         float rc;
@@ -398,6 +413,7 @@ __device__ __forceinline__ void attn_tile_weights(float (&sacc)[kMmKeys / 8][4],
           asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(rc) : "f"(1.f + ex2_(sv * (2.f * kLog2e))));
           sv = cap2 * fmaf(-2.f, rc, 1.f);
         }
+        if (DIST) sv = fmaf(-slope2[e], (float)(r_pos[e] - kp), sv);
         sv = vis ? sv : -INFINITY;
         mnew[e] = fmaxf(mnew[e], sv);
       }
@@ -410,7 +426,7 @@ bool stack_attn_mma_ok(const StackAttn &c, bool f32) {
 }
 int stack_attn_mma_block_tokens(const StackAttn &c) { return std::max(1, kMmRows / (c.H / c.G)); }
 
-template <int DMAX, bool SIG>
+template <int DMAX, bool SIG, bool DIST>
 __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const float *__restrict__ qf, const uint16_t *__restrict__ kpool,
                                                                        const uint16_t *__restrict__ vpool, const float *temp,
                                                                        const float *pb, const float *sink, StackAttn c, StackSpans sp, const int *qb_tok0,
@@ -430,8 +446,9 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
   const int *pt = page_table + (long long)slot * max_pages;
   // chunked or windowed mask: the first token's bound is where the block's history starts (later rows may start later still)
   const int k_lo = stack_attn_row_lo(c, pos_first);
-  const int k_begin = part ? k_lo + (int)blockIdx.z * keys_per_split : k_lo;
-  const int k_end = part ? min(last_pos + 1, k_begin + keys_per_split) : last_pos + 1;
+  const AttnWalk wk(c, k_lo);
+  const int k_begin = part ? (int)blockIdx.z * keys_per_split : 0;  // indices of the walk
+  const int k_end = part ? min(wk.total(last_pos), k_begin + keys_per_split) : wk.total(last_pos);
   const int nk16 = (d + 15) >> 4, nv8 = dv >> 3, dc = d >> 3, vc = dv >> 3;  // k-steps of Q K^T, n-tiles of P V, 16-byte chunks per row
   // columns d .. 16 nk16 of the K stages are read by the last k-step: zero them once (cp.async never touches them)
   if (d & 15)
@@ -479,6 +496,11 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
 #pragma unroll
     for (int e = 0; e < 2; e++) { tmp_h[e] = temp[r_head[e]] * c.scale * kLog2e; pb_h[e] = pb[r_head[e]] * kLog2e; }
   }
+  float slope2[2] = {0.f, 0.f};
+  if (DIST) {
+#pragma unroll
+    for (int e = 0; e < 2; e++) slope2[e] = stack_attn_slope(r_head[e], c.H) * kLog2e;
+  }
   // with a soft cap the scores are first brought to units of the cap (scale / cap), and the capped score to units of log 2
   const float cap2 = !SIG && c.softcap > 0.f ? c.softcap * kLog2e : 0.f;
   const float scale2 = cap2 > 0.f ? c.scale / c.softcap : c.scale * kLog2e;
@@ -493,11 +515,11 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
   const int ld_row = threadIdx.x >> 1, ld_part = threadIdx.x & 1;
   const int pshift = 31 - __clz(page_size);  // page_size is a power of two
   // the page of this thread's row is read one tile ahead of the copy that needs it
-  auto page_of = [&](int k0) { const int kp = k0 + ld_row; return kp < k_end ? pt[kp >> pshift] : 0; };
+  auto page_of = [&](int k0) { const int v = k0 + ld_row; return v < k_end ? pt[wk.key(v) >> pshift] : 0; };
   int page_next = page_of(k_begin);
   auto load_tile = [&](int k0, int stage) {
-    const int kp = k0 + ld_row;
-    const bool ok = kp < k_end;
+    const int kp = wk.key(k0 + ld_row);
+    const bool ok = k0 + ld_row < k_end;
     const long long prow = ok ? (long long)page_next * page_size + (kp & (page_size - 1)) : 0;
     page_next = page_of(k0 + kMmKeys);
     const uint16_t *ksrc = kpool + prow * krow + (long long)kvh * d, *vsrc = vpool + prow * vrow + (long long)kvh * dv;
@@ -519,7 +541,8 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    if (warp_live && k0 <= warp_last_pos && k0 + kMmKeys > warp_lo) {
+    const int key_a = wk.key(k0), key_z = wk.key(k0 + kMmKeys - 1);  // positions of the tile's first and last key
+    if (warp_live && key_a <= warp_last_pos && (key_z >= warp_lo || key_a < c.keep)) {
       // S = Q K^T: k-steps outside, key tiles inside, so that consecutive products go to different accumulators; one ldmatrix
       // brings the fragments of two key tiles (lane l: matrix l / 8 = (tile, column half), row l % 8)
       const uint32_t kt = ks_base + (uint32_t)(stage * kMmKeys * PITCH * 2);
@@ -540,10 +563,10 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
       }
       // ---- weights, fp32.  Scores are carried in units of log 2 (the factor 1 / ln 2 is folded into the scale), so every
       // exponential is one ex2.  Only a tile that reaches past a row's position or the slice's end needs the mask.
-      const bool masked = k0 + kMmKeys - 1 > warp_first_pos || k0 + kMmKeys > k_end || k0 < warp_lo_max;
+      const bool masked = key_z > warp_first_pos || k0 + kMmKeys > k_end || key_a < warp_lo_max;
       float mnew[2] = {mrow[0], mrow[1]};
-      if (masked) attn_tile_weights<SIG, true>(sacc, mnew, k0, qd, r_pos, r_lo, k_end, tmp_h, pb_h, scale2, cap2);
-      else attn_tile_weights<SIG, false>(sacc, mnew, k0, qd, r_pos, r_lo, k_end, tmp_h, pb_h, scale2, cap2);
+      if (masked) attn_tile_weights<SIG, true, DIST>(sacc, mnew, k0, qd, r_pos, r_lo, k_end, wk, c.keep, tmp_h, pb_h, slope2, scale2, cap2);
+      else attn_tile_weights<SIG, false, DIST>(sacc, mnew, k0, qd, r_pos, r_lo, k_end, wk, c.keep, tmp_h, pb_h, slope2, scale2, cap2);
       if (!SIG) {
         float corr[2];
 #pragma unroll
@@ -618,8 +641,13 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
       const float *cs = o.vrot + (long long)tok * dv, *sn = cs + hf;
       const float u = ot[rr * (dv + 1) + m], w = ot[rr * (dv + 1) + m + hf], inv = ot[rr * (dv + 1) + dv];
       uint16_t *orow = reinterpret_cast<uint16_t *>(o.out) + (long long)tok * o.ld + o.off + (long long)head * dv;
-      orow[m] = float_to_bf16_bits((u * cs[m] + w * sn[m]) * inv);
-      orow[m + hf] = float_to_bf16_bits((w * cs[m] - u * sn[m]) * inv);
+      float a0 = (u * cs[m] + w * sn[m]) * inv, a1 = (w * cs[m] - u * sn[m]) * inv;
+      if (o.gate_full) {
+        const float *gr = o.gate_full + (long long)tok * o.ldg + (long long)head * dv;
+        a0 *= sigmoid_precise(gr[m]); a1 *= sigmoid_precise(gr[m + hf]);
+      }
+      orow[m] = float_to_bf16_bits(a0);
+      orow[m + hf] = float_to_bf16_bits(a1);
     }
     return;
   }
@@ -636,9 +664,14 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
     }
     const float inv = attn_out_factor(o, r_tok[e], r_head[e]) * (SIG ? 1.f : 1.f / lrow[e]);
     uint16_t *orow = reinterpret_cast<uint16_t *>(o.out) + (long long)r_tok[e] * o.ld + o.off + (long long)r_head[e] * dv;
+    const float *gr = o.gate_full ? o.gate_full + (long long)r_tok[e] * o.ldg + (long long)r_head[e] * dv + qd * 2 : nullptr;
 #pragma unroll
     for (int j = 0; j < DMAX / 8; j++)
-      if (j < nv8) *reinterpret_cast<uint32_t *>(orow + j * 8 + qd * 2) = pack_bf16(oacc[j][e * 2] * inv, oacc[j][e * 2 + 1] * inv);
+      if (j < nv8) {
+        float a0 = oacc[j][e * 2] * inv, a1 = oacc[j][e * 2 + 1] * inv;
+        if (gr) { a0 *= sigmoid_precise(gr[j * 8]); a1 *= sigmoid_precise(gr[j * 8 + 1]); }
+        *reinterpret_cast<uint32_t *>(orow + j * 8 + qd * 2) = pack_bf16(a0, a1);
+      }
   }
 }
 
@@ -649,6 +682,7 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
                               int keys_per_split, float *part, cudaStream_t st) {
   if (n_qb <= 0) return cudaSuccess;
   if (!(c.flags & (DIS_ATTN_SINK | DIS_ATTN_SINK_UNIT))) sink = nullptr;  // the unit sink is a vector of zero logits
+  const float *gate_full = (c.flags & DIS_ATTN_GATE_FULL) ? gate : nullptr;
   if (!(c.flags & DIS_ATTN_GATE)) gate = nullptr;
   if (n_split <= 1 || !part) { n_split = 1; part = nullptr; }
   if (n_split > kAtMaxSplit) return cudaErrorInvalidValue;
@@ -662,7 +696,7 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
     if (e == cudaSuccess) e = cudaFuncSetAttribute(stack_attn_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_attn_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
   }));
-  const AttnOut o{out, ld_out, out_off, out_scale, (c.flags & DIS_ATTN_ROT_V) ? vrot : nullptr, gate, ld_gate};
+  const AttnOut o{out, ld_out, out_off, out_scale, (c.flags & DIS_ATTN_ROT_V) ? vrot : nullptr, gate, ld_gate, gate_full};
   const dim3 grid(n_qb, c.G, n_split);
   static int use_mma = -1;
   if (use_mma < 0) { const char *e = getenv("DIS_STACK_ATTN_MMA"); use_mma = (e && atoi(e) == 0) ? 0 : 1; }
@@ -670,20 +704,28 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
   if (use_mma && stack_attn_mma_ok(c, f32) && bq <= stack_attn_mma_block_tokens(c) && ld_out % 2 == 0 && out_off % 2 == 0) {
     static DeviceOnce once_mma;
     DIS_CUDA_TRY(once_mma.run([&] {
-      cudaError_t e = cudaFuncSetAttribute(stack_attn_mma_kernel<64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-      if (e == cudaSuccess) e = cudaFuncSetAttribute(stack_attn_mma_kernel<64, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-      if (e == cudaSuccess) e = cudaFuncSetAttribute(stack_attn_mma_kernel<128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-      return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_attn_mma_kernel<128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+      cudaError_t e = cudaSuccess;
+      auto allow = [&](auto kern) { if (e == cudaSuccess) e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); };
+      allow(stack_attn_mma_kernel<64, true, false>);
+      allow(stack_attn_mma_kernel<64, false, false>);
+      allow(stack_attn_mma_kernel<64, false, true>);
+      allow(stack_attn_mma_kernel<128, true, false>);
+      allow(stack_attn_mma_kernel<128, false, false>);
+      allow(stack_attn_mma_kernel<128, false, true>);
+      return e;
     }));
     const bool small = c.d <= 64 && c.dv <= 64;
     const size_t shm = (size_t)4 * kMmKeys * ((small ? 64 : 128) + 8) * sizeof(uint16_t);
     const uint16_t *kp = reinterpret_cast<const uint16_t *>(kpool), *vp = reinterpret_cast<const uint16_t *>(vpool);
-#define DIS_ATTN_MMA(D, S) \
-  stack_attn_mma_kernel<D, S><<<grid, kMmWarps * 32, shm, st>>>(qf, kp, vp, temp, pb, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, o, keys_per_split, part)
-    if (small && sig) DIS_ATTN_MMA(64, true);
-    else if (small) DIS_ATTN_MMA(64, false);
-    else if (sig) DIS_ATTN_MMA(128, true);
-    else DIS_ATTN_MMA(128, false);
+    const bool dist = (c.flags & DIS_ATTN_DISTANCE) != 0;
+#define DIS_ATTN_MMA(D, S, B) \
+  stack_attn_mma_kernel<D, S, B><<<grid, kMmWarps * 32, shm, st>>>(qf, kp, vp, temp, pb, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, o, keys_per_split, part)
+    if (small && sig) DIS_ATTN_MMA(64, true, false);
+    else if (small && dist) DIS_ATTN_MMA(64, false, true);
+    else if (small) DIS_ATTN_MMA(64, false, false);
+    else if (sig) DIS_ATTN_MMA(128, true, false);
+    else if (dist) DIS_ATTN_MMA(128, false, true);
+    else DIS_ATTN_MMA(128, false, false);
 #undef DIS_ATTN_MMA
     if (part) {
       const size_t msh = (size_t)(c.dv + n_split) * sizeof(float);

@@ -12,13 +12,13 @@ __device__ __forceinline__ float silu_(float v) { return v / (1.f + expf(-v)); }
 // One CTA per (span, head).  S [d][dv] lives in shared memory for the whole span; per token: S = a S + k v^T, o = S^T q.
 // Warp w owns rows i = w, w + nw, ...; lanes own columns.  The partial o of every warp goes through shared memory and is added
 // in warp order, so the sum's order is fixed.  A span that starts at position 0 starts from S = 0 (the slot is not read).
-// GATE false: one decay per head, q, k, v through SiLU.  GATE true: the decay is a vector per token (dec [T][H*d], one factor per
-// row of S), q is multiplied by qscale, no activation.
+// GATE 0: one decay per head, q, k, v through SiLU.  GATE 1: the decay is a vector per token (dec [T][H*d], one factor per
+// row of S), q is multiplied by qscale, no activation.  GATE 3: one decay per head, no activation.
 // first column of head 0's q, k, v in a row of proj.  hpg > 1: q and k are shared by groups of hpg consecutive heads (head h reads
 // block h / hpg).  dec_head (gated form): the decay is one factor per token and head, dec [T][H], not one per key channel.
 // vscale (or null): [T][H], a factor per token and head on the values as they are staged.
 struct LightCols { int q, k, v; int hpg = 1; int dec_head = 0; const float *vscale = nullptr; };
-template <bool GATE>
+template <int GATE>
 __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj, long long ld, LightCols col, const float *decay,
                                                               const float *dec, float qscale, float *state, StackSpans sp, float *o, int H,
                                                               int d, int dv) {
@@ -33,7 +33,8 @@ __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj,
   float *part = vs + dv;          // [nw][dv]
   float *as = part + (size_t)nw * dv;  // [d] (GATE)
   float *st = state + ((long long)slot * H + h) * d * dv;
-  const float a = GATE ? 1.f : decay[h];
+  constexpr bool DEC = GATE == 1;
+  const float a = DEC ? 1.f : decay[h];
   for (int i = threadIdx.x; i < d * dv; i += blockDim.x) S[i] = pos0 > 0 ? st[i] : 0.f;
   for (int t = 0; t < len; t++) {
     const float *row = proj + (long long)(tok0 + t) * ld;
@@ -42,7 +43,7 @@ __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj,
       const float qv = row[col.q + (long long)(h / col.hpg) * d + i], kv = row[col.k + (long long)(h / col.hpg) * d + i];
       qs[i] = GATE ? qv * qscale : silu_(qv);
       ks[i] = GATE ? kv : silu_(kv);
-      if (GATE) as[i] = col.dec_head ? dec[(long long)(tok0 + t) * H + h] : dec[(long long)(tok0 + t) * H * d + (long long)h * d + i];
+      if (DEC) as[i] = col.dec_head ? dec[(long long)(tok0 + t) * H + h] : dec[(long long)(tok0 + t) * H * d + (long long)h * d + i];
     }
     for (int j = threadIdx.x; j < dv; j += blockDim.x) {
       const float vv = row[col.v + (long long)h * dv + j];
@@ -53,7 +54,7 @@ __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj,
       const float vj = vs[j];
       float acc = 0.f;
       for (int i = w; i < d; i += nw) {
-        const float sv = fmaf(GATE ? as[i] : a, S[(size_t)i * dv + j], ks[i] * vj);
+        const float sv = fmaf(DEC ? as[i] : a, S[(size_t)i * dv + j], ks[i] * vj);
         S[(size_t)i * dv + j] = sv;
         acc = fmaf(sv, qs[i], acc);
       }
@@ -85,6 +86,7 @@ __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj,
 // GATE 2 (state-space mixer): one decay per token and head, dec [T][H], and a factor per token and head on the values,
 // col.vscale [T][H]; both are staged as one number per token (the first two entries of the token's decay row), so the inner loop
 // reads them once instead of a vector per group of rows.
+// GATE 3 (retention): one decay per head as in GATE 0, but q, k and v enter as they are.
 // Rows and columns beyond d and dv: shared memory starts as zeros and nobody writes those entries, so their k, q and decays are
 // zero and their part of S stays zero; the inner loop needs no bounds checks.
 constexpr int kLightTok = 8, kLightSeg = 64;
@@ -95,6 +97,7 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
                                                                      int dv, float *seg, float *seg_a, int max_seg) {
   extern __shared__ __align__(16) float shm[];
   constexpr int DP = RI * 8, DVP = RJ * 32;
+  constexpr bool DEC = GATE == 1 || GATE == 2;  // decays come per token
   // heads vary fastest over the grid: the CTAs that run at the same time then read whole rows of the projections rather than
   // one head's columns at a stride of a row, which would keep most memory channels idle
   const int h = blockIdx.x % H, sc = blockIdx.x / H;
@@ -108,7 +111,7 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
     first = tok0 + c * kLightSeg;
     n = min(kLightSeg, len - c * kLightSeg);
     sg = seg + ((size_t)(tok0 / kLightSeg + s + c) * H + h) * d * dv;
-    if (GATE) sga = seg_a + ((size_t)(tok0 / kLightSeg + s + c) * H + h) * d;
+    if (DEC) sga = seg_a + ((size_t)(tok0 / kLightSeg + s + c) * H + h) * d;
   }
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, i0 = w * RI;
   float *qs = shm;                             // [tok][DP]
@@ -116,9 +119,9 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
   float *vs = ks + kLightTok * DP;             // [tok][DVP]
   float *part = vs + kLightTok * DVP;          // [tok][8][DVP]
   float *as = part + kLightTok * 8 * DVP;      // [tok][DP] (GATE)
-  for (int i = threadIdx.x; i < kLightTok * ((GATE ? 3 : 2) * DP + 9 * DVP); i += blockDim.x) shm[i] = 0.f;  // (the loop's first barrier follows)
+  for (int i = threadIdx.x; i < kLightTok * ((DEC ? 3 : 2) * DP + 9 * DVP); i += blockDim.x) shm[i] = 0.f;  // (the loop's first barrier follows)
   float *st = state + ((long long)slot * H + h) * d * dv;
-  const float a = GATE ? 1.f : decay[h];
+  const float a = DEC ? 1.f : decay[h];
   float S[RI][RJ];
   float A[GATE == 1 ? RI : 1];  // MODE 1: running product of the decays of this thread's rows (GATE 2: of the head)
 #pragma unroll
@@ -154,7 +157,7 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
       src[u] = (c == 2 * d + dv ? dec : col.vscale) + h;
       sstride[u] = H;
       sdst[u] = as + (c - 2 * d - dv);
-    } else if (c < per) {  // one decay per key channel, or the head's one decay copied to every channel
+    } else if (DEC && c < per) {  // one decay per key channel, or the head's one decay copied to every channel
       src[u] = col.dec_head ? dec + h : dec + (long long)h * d + (c - 2 * d - dv);
       sstride[u] = col.dec_head ? (long long)H : (long long)H * d;
       sdst[u] = as + (c - 2 * d - dv);
@@ -232,7 +235,7 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
       const int i = i0 + ii, j = l + jj * 32;
       if (i < d && j < dv) dst[(size_t)i * dv + j] = S[ii][jj];
     }
-  if (GATE && MODE == 1 && l == 0) {
+  if (DEC && MODE == 1 && l == 0) {
 #pragma unroll
     for (int ii = 0; ii < RI; ii++)
       if (i0 + ii < d) sga[i0 + ii] = A[GATE == 1 ? ii : 0];
@@ -318,20 +321,21 @@ template <int RI, int RJ, int GATE>
 static cudaError_t lightning_reg(const float *proj, long long ld, LightCols col, const float *decay, const float *dec, float qscale,
                                  float *state, const StackSpans &sp, float *o, int H, int d, int dv, float *seg, float *seg_a,
                                  int max_len, cudaStream_t st) {
-  const size_t sh = (size_t)kLightTok * ((GATE ? 3 : 2) * RI * 8 + RJ * 32 + 8 * RJ * 32) * sizeof(float);
+  constexpr bool DEC = GATE == 1 || GATE == 2;
+  const size_t sh = (size_t)kLightTok * ((DEC ? 3 : 2) * RI * 8 + RJ * 32 + 8 * RJ * 32) * sizeof(float);
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] {
     cudaError_t e = cudaFuncSetAttribute(stack_lightning_reg_kernel<RI, RJ, 0, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(stack_lightning_reg_kernel<RI, RJ, 1, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_lightning_reg_kernel<RI, RJ, 2, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
   }));
-  if (!seg || (GATE && !seg_a) || max_len <= kLightSeg) {
+  if (!seg || (DEC && !seg_a) || max_len <= kLightSeg) {
     stack_lightning_reg_kernel<RI, RJ, 0, GATE><<<sp.n_spans * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, nullptr, nullptr, 1);
     return cudaGetLastError();
   }
   const int max_seg = (max_len + kLightSeg - 1) / kLightSeg;
   stack_lightning_reg_kernel<RI, RJ, 1, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg);
-  stack_lightning_carry_kernel<<<sp.n_spans * H * ((d * dv + 255) / 256), 256, 0, st>>>(decay, GATE ? seg_a : nullptr, state, sp, seg, H, d, dv);
+  stack_lightning_carry_kernel<<<sp.n_spans * H * ((d * dv + 255) / 256), 256, 0, st>>>(decay, DEC ? seg_a : nullptr, state, sp, seg, H, d, dv);
   stack_lightning_reg_kernel<RI, RJ, 2, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg);
   return cudaGetLastError();
 }
@@ -340,13 +344,106 @@ cudaError_t launch_stack_lightning(const float *proj, long long ld, const float 
                                    float *o, int H, int d, int dv, float *seg, int max_len, cudaStream_t st) {
   const int threads = 256;
   const LightCols col{0, H * d, 2 * H * d};
-  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, false>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
-  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, false>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, 0>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, 0>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
   const size_t sh = ((size_t)d * dv + 2 * d + dv + (size_t)(threads / 32) * dv) * sizeof(float);
   if (sh > 220 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
-  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
-  stack_lightning_kernel<false><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv);
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
+  stack_lightning_kernel<0><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv);
+  return cudaGetLastError();
+}
+
+// ------------------------------------------------------------------------------------------------ retention
+// In front of the recurrence, one block per token: q and k [H][d] of the token's row are rotated over the first rot_dims
+// coordinates of every head (pairs i, i + rot_dims/2, angle pos * freq[i]), k is multiplied by kscale.  The row comes as n_part
+// slices of n_cols columns (n_part 1: it may be dst itself); every column lands in dst.  Cosine and sine are formed once per token.
+__global__ void __launch_bounds__(256) stack_retention_prep_kernel(const float *src, long long ld_src, int n_part, long long stride,
+                                                                   int n_cols, float *dst, long long ld_dst, int q_off, int k_off, int H,
+                                                                   int d, const double *__restrict__ freq, int rot_dims, float kscale,
+                                                                   const int *__restrict__ pos) {
+  extern __shared__ __align__(16) float rsh[];  // cos [half], sin [half], then (n_part > 1) the summed row
+  const int t = blockIdx.x, half = rot_dims >> 1;
+  float *cs = rsh, *sn = rsh + half;
+  const float *row = src + (long long)t * ld_src;
+  float *out = dst + (long long)t * ld_dst;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) angle_sincos(pos[t], freq[i], &sn[i], &cs[i]);
+  if (n_part > 1) {
+    float *srow = rsh + ((rot_dims + 3) & ~3);
+    const bool v4 = ((n_cols | (int)(ld_src & 3) | (int)(stride & 3)) & 3) == 0;
+    if (v4) {
+      for (int i = threadIdx.x * 4; i < n_cols; i += blockDim.x * 4) {
+        float4 v = *reinterpret_cast<const float4 *>(row + i);
+#pragma unroll 4
+        for (int k = 1; k < n_part; k++) {
+          const float4 p = *reinterpret_cast<const float4 *>(row + (long long)k * stride + i);
+          v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+        }
+        *reinterpret_cast<float4 *>(srow + i) = v;
+      }
+    } else
+      for (int i = threadIdx.x; i < n_cols; i += blockDim.x) {
+        float v = row[i];
+        for (int k = 1; k < n_part; k++) v += row[(long long)k * stride + i];
+        srow[i] = v;
+      }
+    row = srow;
+  }
+  __syncthreads();
+  const int n = H * d;
+  auto rotate = [&](int off, float scale) {  // a thread owns a pair (or an unrotated coordinate), so working in place is safe
+    const int per = half + (d - rot_dims);  // work items of a head
+    for (int e = threadIdx.x; e < H * per; e += blockDim.x) {
+      const int h = e / per, i = e - h * per, base = off + h * d;
+      if (i < half) {
+        const float u = row[base + i], v = row[base + i + half];
+        out[base + i] = (u * cs[i] - v * sn[i]) * scale;
+        out[base + i + half] = (v * cs[i] + u * sn[i]) * scale;
+      } else out[base + i + half] = row[base + i + half] * scale;
+    }
+  };
+  rotate(q_off, 1.f);
+  rotate(k_off, kscale);
+  if (row != out)
+    for (int i = threadIdx.x; i < n_cols; i += blockDim.x)
+      if (!((i >= q_off && i < q_off + n) || (i >= k_off && i < k_off + n))) out[i] = row[i];
+}
+cudaError_t launch_stack_retention_prep(const float *src, long long ld_src, int n_part, long long stride, int n_cols, float *dst,
+                                        long long ld_dst, int q_off, int k_off, int H, int d, const double *freq, int rot_dims, float kscale,
+                                        const StackSpans &sp, cudaStream_t st) {
+  if (sp.T <= 0) return cudaSuccess;
+  const size_t sh = (size_t)(((rot_dims + 3) & ~3) + (n_part > 1 ? n_cols : 0)) * sizeof(float);
+  if (sh > 200 * 1024) return cudaErrorInvalidValue;
+  static DeviceOnce once;
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_retention_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); }));
+  stack_retention_prep_kernel<<<sp.T, 256, sh, st>>>(src, ld_src, n_part, stride, n_cols, dst, ld_dst, q_off, k_off, H, d, freq, rot_dims, kscale, sp.pos);
+  return cudaGetLastError();
+}
+
+// The value columns of a head are independent of each other, so a head whose values are wider than the register kernel takes
+// runs as `blocks` heads of dv / blocks columns that share q, k and the decay; the state is laid out that way as well.
+int stack_retention_blocks(int d, int dv) {
+  if (d > 128) return 1;  // shared-memory form
+  int nb = (dv + 127) / 128;
+  while (dv % nb) nb++;
+  return nb;
+}
+cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *decay, float *state,
+                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, cudaStream_t st) {
+  const int nb = stack_retention_blocks(d, dv);
+  LightCols col{q_off, k_off, v_off};
+  col.hpg = nb;
+  H *= nb; dv /= nb;
+  if (d <= 32 && dv <= 64) return lightning_reg<4, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  if (d <= 128 && dv <= 64) return lightning_reg<16, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  const int threads = 256;
+  const size_t sh = ((size_t)d * dv + 2 * d + dv + (size_t)(threads / 32) * dv) * sizeof(float);
+  if (sh > 220 * 1024) return cudaErrorInvalidValue;
+  static DeviceOnce once;
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
+  stack_lightning_kernel<3><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv);
   return cudaGetLastError();
 }
 
@@ -402,17 +499,17 @@ cudaError_t launch_stack_gla(const float *proj, long long ld, int q_off, int k_o
   const LightCols col{q_off, k_off, v_off};
   const float qscale = 1.f / sqrtf((float)d);
   // rows of S per warp (RI) and columns per lane (RJ) chosen so that all eight warps own rows: d <= 8 RI, dv <= 32 RJ
-  if (d <= 32 && dv <= 64) return lightning_reg<4, 2, true>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
-  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, true>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
-  if (d <= 64 && dv <= 128) return lightning_reg<8, 4, true>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
-  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, true>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
+  if (d <= 32 && dv <= 64) return lightning_reg<4, 2, 1>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
+  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, 1>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
+  if (d <= 64 && dv <= 128) return lightning_reg<8, 4, 1>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
+  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, 1>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_len, st);
   // larger heads: the state of one head in shared memory, one CTA per (span, head)
   const int threads = 256;
   const size_t sh = ((size_t)d * dv + 3 * d + dv + (size_t)(threads / 32) * dv) * sizeof(float);
   if (sh > 220 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
-  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
-  stack_lightning_kernel<true><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv);
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
+  stack_lightning_kernel<1><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, nullptr, dec, qscale, state, sp, o, H, d, dv);
   return cudaGetLastError();
 }
 
@@ -436,8 +533,8 @@ cudaError_t launch_stack_ssd(const float *buf, long long ld_b, int c_off, int b_
   const size_t sh = ((size_t)d * dv + 3 * d + dv + (size_t)(threads / 32) * dv) * sizeof(float);
   if (sh > 220 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
-  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
-  stack_lightning_kernel<true><<<dim3(sp.n_spans, H), threads, sh, st>>>(buf, ld_b, col, nullptr, dec, 1.f, state, sp, o, H, d, dv);
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
+  stack_lightning_kernel<1><<<dim3(sp.n_spans, H), threads, sh, st>>>(buf, ld_b, col, nullptr, dec, 1.f, state, sp, o, H, d, dv);
   return cudaGetLastError();
 }
 
@@ -695,7 +792,7 @@ cudaError_t launch_stack_ssm_out(const float *o, const float *buf, long long ld_
 }
 
 // out[t][off + h*dv + j] = scale * o[t][h][j] / rms(o[t][h]) * w[j] * silu(gate[t][h*dv + j]): the norm runs over one head's dv
-// outputs, its gain vector is shared by the heads.  One warp per (token, head).
+// outputs, its gain vector (null: ones) is shared by the heads.  One warp per (token, head).
 template <bool F32>
 __global__ void __launch_bounds__(256) stack_headnorm_silu_kernel(const float *o, const float *w, const float *gate, long long ldg, void *out,
                                                                   long long ldo, int off, float scale, int rows, int H, int dv, float eps) {
@@ -709,7 +806,7 @@ __global__ void __launch_bounds__(256) stack_headnorm_silu_kernel(const float *o
   const float k = rsqrtf(s / (float)dv + eps) * scale;
   for (int j = l; j < dv; j += 32) {
     const float g = gate[(long long)t * ldg + (long long)h * dv + j];
-    st_el<F32>(out, (long long)t * ldo + off + (long long)h * dv + j, r[j] * k * w[j] * silu_(g));
+    st_el<F32>(out, (long long)t * ldo + off + (long long)h * dv + j, r[j] * k * (w ? w[j] : 1.f) * silu_(g));
   }
 }
 cudaError_t launch_stack_headnorm_silu(const float *o, const float *w, const float *gate, long long ldg, void *out, long long ldo,
@@ -744,21 +841,22 @@ cudaError_t launch_stack_norm_gate(const float *o, const float *w, const float *
 // heads > 0: o is laid out head by head, [heads][T][n / heads] (the per-head tensor-core products write it so)
 template <bool F32>
 __global__ void stack_gate_kernel(const float *__restrict__ o, const float *__restrict__ gate, long long ldg, void *__restrict__ out, int T,
-                                  int n, int heads) {
+                                  int n, int heads, long long ldo) {
   const int hw = heads > 0 ? n / heads : n;
   for (int t = blockIdx.x; t < T; t += gridDim.x) {
     for (int c = threadIdx.x; c < n; c += blockDim.x) {
       const float v = heads > 0 ? o[((long long)(c / hw) * T + t) * hw + c % hw] : o[(long long)t * n + c];
-      st_el<F32>(out, (long long)t * n + c, v * sigmoid_precise(gate[t * ldg + c]));
+      st_el<F32>(out, t * ldo + c, gate ? v * sigmoid_precise(gate[t * ldg + c]) : v);
     }
   }
 }
 cudaError_t launch_stack_gate(const float *o, const float *gate, long long ldg, void *out, bool f32, int T, int n, int heads,
-                              cudaStream_t st) {
+                              cudaStream_t st, long long ldo) {
   if (T <= 0) return cudaSuccess;
+  if (ldo <= 0) ldo = n;
   const int grid = std::min(T, 148 * 16);
-  if (f32) stack_gate_kernel<true><<<grid, 256, 0, st>>>(o, gate, ldg, out, T, n, heads);
-  else stack_gate_kernel<false><<<grid, 256, 0, st>>>(o, gate, ldg, out, T, n, heads);
+  if (f32) stack_gate_kernel<true><<<grid, 256, 0, st>>>(o, gate, ldg, out, T, n, heads, ldo);
+  else stack_gate_kernel<false><<<grid, 256, 0, st>>>(o, gate, ldg, out, T, n, heads, ldo);
   return cudaGetLastError();
 }
 
@@ -895,30 +993,70 @@ cudaError_t launch_stack_mingru(const float *proj, long long ld, const float *bi
 }
 
 // ------------------------------------------------------------------------------------------------ latent attention
-// Rotation of coordinates (i, i + rot_dims/2), i < rot_dims/2, by the angle pos * base^(-2i/rot_dims); the rest passes.  The angle
-// is formed in double so that position 5000 is as exact as position 5.
-__device__ __forceinline__ float rotated(const float *v, int i, int rot_dims, int pos, float base) {
-  const int half = rot_dims >> 1;
-  if (i >= rot_dims) return v[i];
-  const int p = i < half ? i : i - half;
-  const double f = exp2(-2.0 * (double)p / (double)rot_dims * log2((double)base));
-  double sn, cs;
-  sincos((double)pos * f, &sn, &cs);
-  return i < half ? (float)((double)v[i] * cs - (double)v[i + half] * sn) : (float)((double)v[i] * cs + (double)v[i - half] * sn);
+// Preparation, one block per token.  Rotation over the first rot_dims coordinates of the rotated parts: coordinate i turns with
+// i + rot_dims/2, or (rot_pairs) 2i with 2i + 1, by the angle pos * freq[i] formed in double; the rest passes.  Cosine and sine are
+// formed once per token and shared by the heads and the key.
+__device__ __forceinline__ float latent_rotated(const float *v, int i, const StackLatent &c, const float *cs, const float *sn) {
+  if (i >= c.rot_dims) return v[i];
+  if (c.rot_pairs) {
+    const int p = i >> 1;
+    return (i & 1) ? v[i] * cs[p] + v[i - 1] * sn[p] : v[i] * cs[p] - v[i + 1] * sn[p];
+  }
+  const int half = c.rot_dims >> 1;
+  return i < half ? v[i] * cs[i] - v[i + half] * sn[i] : v[i] * cs[i - half] + v[i - half] * sn[i - half];
 }
-
+// Columns of the row: queries (rotated parts go to qf) at q_off when qf is given; latent and rotated key part at dkv_off when pool is
+// given; the query latent at dq_off when cq is given (RMS-normed with the gain dq_norm into cq [T][q_rank], compute type).  The row may
+// come as n_part slices of n_cols columns; columns keep_off .. keep_off + keep_n of their sum then go to keep [T][ld_keep] as well.
 template <bool F32>
-__global__ void __launch_bounds__(128) stack_latent_prep_kernel(const float *proj, long long ld, int q_off, int dkv_off,
-                                                                const float *dkv_norm, StackLatent c, StackSpans sp, float *qf,
-                                                                void *pool, const int *page_table, int max_pages, int page_size) {
+__global__ void __launch_bounds__(256) stack_latent_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
+                                                                int q_off, int dkv_off, const float *dkv_norm, int dq_off,
+                                                                const float *dq_norm, void *cq, float *keep, long long ld_keep,
+                                                                int keep_off, int keep_n, const double *__restrict__ freq,
+                                                                StackLatent c, StackSpans sp, float *qf, void *pool,
+                                                                const int *page_table, int max_pages, int page_size) {
+  extern __shared__ __align__(16) float lsh[];  // cos [half], sin [half], then (n_part > 1) the summed row
   __shared__ float sh[32];
   const int t = blockIdx.x;
   const float *row = proj + (long long)t * ld;
-  const int pos = sp.pos[t];
+  const int pos = sp.pos[t], half = c.rot_dims >> 1;
   const int D = c.r + c.dr;
-  for (int i = threadIdx.x; i < c.H * c.dr; i += blockDim.x) {
-    const int h = i / c.dr, k = i % c.dr;
-    qf[((long long)t * c.H + h) * D + c.r + k] = rotated(row + q_off + (long long)h * (c.d + c.dr) + c.d, k, c.rot_dims, pos, c.rot_base);
+  float *cs = lsh, *sn = lsh + half;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) angle_sincos(pos, freq[i], &sn[i], &cs[i]);
+  if (n_part > 1) {
+    float *srow = lsh + ((c.rot_dims + 3) & ~3);
+    if (((n_cols | (int)(ld & 3) | (int)(stride & 3)) & 3) == 0) {
+      for (int i = threadIdx.x * 4; i < n_cols; i += blockDim.x * 4) {
+        float4 v = *reinterpret_cast<const float4 *>(row + i);
+#pragma unroll 4
+        for (int k = 1; k < n_part; k++) {
+          const float4 p = *reinterpret_cast<const float4 *>(row + (long long)k * stride + i);
+          v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+        }
+        *reinterpret_cast<float4 *>(srow + i) = v;
+      }
+    } else
+      for (int i = threadIdx.x; i < n_cols; i += blockDim.x) {
+        float v = row[i];
+        for (int k = 1; k < n_part; k++) v += row[(long long)k * stride + i];
+        srow[i] = v;
+      }
+    row = srow;
+  }
+  __syncthreads();
+  if (keep)
+    for (int i = threadIdx.x; i < keep_n; i += blockDim.x) keep[(long long)t * ld_keep + i] = row[keep_off + i];
+  if (qf)
+    for (int i = threadIdx.x; i < c.H * c.dr; i += blockDim.x) {
+      const int h = i / c.dr, k = i % c.dr;
+      qf[((long long)t * c.H + h) * D + c.r + k] = latent_rotated(row + q_off + (long long)h * (c.d + c.dr) + c.d, k, c, cs, sn);
+    }
+  if (cq) {
+    const float *dq = row + dq_off;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < c.q_rank; i += blockDim.x) s += dq[i] * dq[i];
+    const float k = rsqrtf(block_sum(s, sh) / (float)c.q_rank + c.eps);
+    for (int i = threadIdx.x; i < c.q_rank; i += blockDim.x) st_el<F32>(cq, (long long)t * c.q_rank + i, dq[i] * k * dq_norm[i]);
   }
   if (!pool) return;
   const int slot = sp.slot[t];
@@ -929,13 +1067,25 @@ __global__ void __launch_bounds__(128) stack_latent_prep_kernel(const float *pro
   s = block_sum(s, sh);
   const float k = rsqrtf(s / (float)c.r + c.eps);
   for (int i = threadIdx.x; i < c.r; i += blockDim.x) st_el<F32>(pool, prow * D + i, dk[i] * k * dkv_norm[i]);
-  for (int i = threadIdx.x; i < c.dr; i += blockDim.x) st_el<F32>(pool, prow * D + c.r + i, rotated(dk + c.r, i, c.rot_dims, pos, c.rot_base));
+  for (int i = threadIdx.x; i < c.dr; i += blockDim.x) st_el<F32>(pool, prow * D + c.r + i, latent_rotated(dk + c.r, i, c, cs, sn));
 }
-cudaError_t launch_stack_latent_prep(const float *proj, long long ld, int q_off, int dkv_off, const float *dkv_norm,
-                                     const StackLatent &c, const StackSpans &sp, float *qf, void *pool, bool f32,
-                                     const int *page_table, int max_pages, int page_size, cudaStream_t st) {
-  if (f32) stack_latent_prep_kernel<true><<<sp.T, 128, 0, st>>>(proj, ld, q_off, dkv_off, dkv_norm, c, sp, qf, pool, page_table, max_pages, page_size);
-  else stack_latent_prep_kernel<false><<<sp.T, 128, 0, st>>>(proj, ld, q_off, dkv_off, dkv_norm, c, sp, qf, pool, page_table, max_pages, page_size);
+cudaError_t launch_stack_latent_prep(const StackLatentPrep &a, const StackLatent &c, const StackSpans &sp, bool f32, const int *page_table,
+                                     int max_pages, int page_size, cudaStream_t st) {
+  if (sp.T <= 0) return cudaSuccess;
+  const int n_part = std::max(1, a.n_part);
+  const size_t sh = (size_t)(((c.rot_dims + 3) & ~3) + (n_part > 1 ? a.n_cols : 0)) * sizeof(float);
+  if (sh > 200 * 1024) return cudaErrorInvalidValue;
+  static DeviceOnce once;
+  DIS_CUDA_TRY(once.run([&] {
+    cudaError_t e = cudaFuncSetAttribute(stack_latent_prep_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_latent_prep_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+  }));
+#define DIS_LAT_PREP(F)                                                                                                                      \
+  stack_latent_prep_kernel<F><<<sp.T, 256, sh, st>>>(a.proj, a.ld, n_part, a.stride, a.n_cols, a.q_off, a.dkv_off, a.dkv_norm, a.dq_off, a.dq_norm, \
+                                                     a.cq, a.keep, a.ld_keep, a.keep_off, a.keep_n, a.freq, c, sp, a.qf, a.pool, page_table, max_pages, page_size)
+  if (f32) DIS_LAT_PREP(true);
+  else DIS_LAT_PREP(false);
+#undef DIS_LAT_PREP
   return cudaGetLastError();
 }
 
@@ -976,9 +1126,12 @@ __global__ void __launch_bounds__(kLatWarps * 32) stack_latent_attn_kernel(const
   for (int i = threadIdx.x; i < pairs * r; i += blockDim.x) acc[i] = 0.f;
   // the whole history in one CTA: the running maximum starts at the head's sink and the denominator at exp(sink - max) = 1;
   // one slice of the history (blockIdx.y, keys_per_split keys): both start empty and the sink joins when the slices are merged
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) { mx[i] = part ? -INFINITY : sink[i % c.H]; dn[i] = part ? 0.f : 1.f; }
+  // (no sink: both start empty)
+  const bool with_sink = !part && sink;
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) { mx[i] = with_sink ? sink[i % c.H] : -INFINITY; dn[i] = with_sink ? 1.f : 0.f; }
   const int *pt = page_table + (long long)slot * max_pages;
-  const int k_begin = part ? (int)blockIdx.y * keys_per_split : 0;
+  const int k_lo = stack_latent_row_lo(c, sp.pos[tok0]);  // a windowed block's history starts at its first token's bound
+  const int k_begin = part ? k_lo + (int)blockIdx.y * keys_per_split : k_lo;
   const int k_end = part ? min(last_pos + 1, k_begin + keys_per_split) : last_pos + 1;
   for (int k0 = k_begin; k0 < k_end; k0 += kLatTile) {
     const int nk = min(kLatTile, k_end - k0);
@@ -1009,7 +1162,7 @@ __global__ void __launch_bounds__(kLatWarps * 32) stack_latent_attn_kernel(const
       const int qpos = sp.pos[tok0 + p / c.H];
       const float *q = qs + (size_t)p * D;
       float sc = -INFINITY;
-      if (l < nk && k0 + l <= qpos) {
+      if (l < nk && k0 + l <= qpos && k0 + l >= stack_latent_row_lo(c, qpos)) {
         const float *kr = tile + (size_t)l * DP;
         float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;  // four chains, added at the end: the sum's order is fixed by D alone
         int i = 0;
@@ -1055,8 +1208,8 @@ __global__ void __launch_bounds__(kLatWarps * 32) stack_latent_attn_kernel(const
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) { rec[(long long)i * (r + 2) + r] = mx[i]; rec[(long long)i * (r + 2) + r + 1] = dn[i]; }
 }
 
-// ---- the same attention on mma.sync (bf16 compute type, kv_rank a multiple of 8, kv_rank + rot_dim a multiple of 16, at most 16
-// (token, head) pairs per query block): the pairs are the 16 rows of m16n8k16 products.  A CTA stages 64 latents of its slice
+// ---- the same attention on mma.sync (bf16 compute type, kv_rank a multiple of 8, kv_rank + rot_dim a multiple of 16; query blocks
+// of at most 16 (token, head) pairs, or of one token whose heads are taken 16 at a time): the pairs are the 16 rows of m16n8k16 products.  A CTA stages 64 latents of its slice
 // as bf16, warp w scores keys 8w .. 8w+7 against all pairs (K = kv_rank + rot_dim), the scores go through shared memory for the
 // online softmax (fp32, two rows per warp, starting at the sink as above), and each warp then adds P C into the output
 // coordinates it owns (n-tiles w, w + 8, ...), which stay in registers over the whole slice.
@@ -1066,12 +1219,12 @@ __device__ __forceinline__ void mma_bf16_m16n8k16(float (&c)[4], uint32_t a0, ui
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 constexpr int kMmaKeys = 64, kMmaRows = 16, kMmaPS = 72;
-bool stack_latent_mma_ok(const StackLatent &c, bool f32) {
-  return !f32 && c.r % 8 == 0 && (c.r + c.dr) % 16 == 0 && c.r <= kLatMaxR && c.H <= kMmaRows;
-}
 static size_t latent_mma_smem(const StackLatent &c) {
   const size_t DS = (size_t)c.r + c.dr + 8;
   return (kMmaRows + kMmaKeys) * DS * 2 + (size_t)kMmaRows * kMmaKeys * 4 + (size_t)kMmaRows * kMmaPS * 2 + 4 * kMmaRows * 4;
+}
+bool stack_latent_mma_ok(const StackLatent &c, bool f32) {
+  return !f32 && c.r % 8 == 0 && (c.r + c.dr) % 16 == 0 && c.r <= kLatMaxR && latent_mma_smem(c) <= 220 * 1024;
 }
 template <int NTW>
 __global__ void __launch_bounds__(256) stack_latent_attn_mma_kernel(const float *qf, const uint16_t *pool, const float *sink, StackLatent c,
@@ -1088,15 +1241,18 @@ __global__ void __launch_bounds__(256) stack_latent_attn_mma_kernel(const float 
   float *dn = mx + kMmaRows, *cr = dn + kMmaRows;                      // [16] each
   int *qp = reinterpret_cast<int *>(cr + kMmaRows);                    // [16] position of the row's query, -1 for a padding row
   __shared__ long long prow_s[kMmaKeys];
+  __shared__ int qlo[kMmaRows];  // first key the row's query sees
   const int tok0 = qb_tok0[blockIdx.x], nq = qb_len[blockIdx.x];
-  const int pairs = nq * c.H;
+  // at most 16 heads: every head of the block's tokens; more: blocks of one token, blockIdx.z takes 16 of its heads
+  const int h0 = (int)blockIdx.z * kMmaRows, Hb = c.H <= kMmaRows ? c.H : min(kMmaRows, c.H - h0);
+  const int pairs = nq * Hb;
   if (pairs > kMmaRows) return;  // the host cuts query blocks to fit
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, g = l >> 2, tig = l & 3;
   const int slot = sp.slot[tok0];
   const int last_pos = sp.pos[tok0 + nq - 1];
   {  // queries: four floats per load, four loads in flight per thread before the first is converted and stored
     const int n4 = kMmaRows * D / 4;
-    const float4 *src = reinterpret_cast<const float4 *>(qf + (long long)tok0 * c.H * D);
+    const float4 *src = reinterpret_cast<const float4 *>(qf + ((long long)tok0 * c.H + h0) * D);
     for (int i0 = threadIdx.x; i0 < n4; i0 += 4 * blockDim.x) {
       float4 v[4];
 #pragma unroll
@@ -1116,15 +1272,18 @@ __global__ void __launch_bounds__(256) stack_latent_attn_mma_kernel(const float 
   }
   if (threadIdx.x < kMmaRows) {
     const int row = threadIdx.x;
-    mx[row] = part ? -INFINITY : (row < pairs ? sink[row % c.H] : 0.f);
-    dn[row] = part ? 0.f : 1.f;
-    qp[row] = row < pairs ? sp.pos[tok0 + row / c.H] : -1;
+    const bool with_sink = !part && sink;
+    mx[row] = with_sink ? (row < pairs ? sink[h0 + row % Hb] : 0.f) : -INFINITY;
+    dn[row] = with_sink ? 1.f : 0.f;
+    qp[row] = row < pairs ? sp.pos[tok0 + row / Hb] : -1;
+    qlo[row] = row < pairs ? stack_latent_row_lo(c, qp[row]) : 0;
   }
   float acc[NTW][4];
 #pragma unroll
   for (int nt = 0; nt < NTW; nt++) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
   const int *pt = page_table + (long long)slot * max_pages;
-  const int k_begin = part ? (int)blockIdx.y * keys_per_split : 0;
+  const int k_lo = stack_latent_row_lo(c, sp.pos[tok0]);
+  const int k_begin = part ? k_lo + (int)blockIdx.y * keys_per_split : k_lo;
   const int k_end = part ? min(last_pos + 1, k_begin + keys_per_split) : last_pos + 1;
   const int vpr = D >> 3;
   for (int k0 = k_begin; k0 < k_end; k0 += kMmaKeys) {
@@ -1170,7 +1329,7 @@ __global__ void __launch_bounds__(256) stack_latent_attn_mma_kernel(const float 
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const int row = g + (e >> 1) * 8, col = w * 8 + 2 * tig + (e & 1);
-        const bool seen = col < nk && k0 + col <= qp[row];
+        const bool seen = col < nk && k0 + col <= qp[row] && k0 + col >= qlo[row];
         S[row * kMmaKeys + col] = seen ? sa[e] * c.scale : -INFINITY;
       }
     }
@@ -1221,12 +1380,12 @@ __global__ void __launch_bounds__(256) stack_latent_attn_mma_kernel(const float 
     for (int e = 0; e < 4; e++) {
       const int row = g + (e >> 1) * 8, col = n0 + 2 * tig + (e & 1);
       if (row >= pairs) continue;
-      if (!part) ol[((long long)tok0 * c.H + row) * r + col] = acc[nt][e] / dn[row];
-      else part[((long long)blockIdx.y * sp.T * c.H + (long long)tok0 * c.H + row) * (r + 2) + col] = acc[nt][e];
+      if (!part) ol[((long long)tok0 * c.H + h0 + row) * r + col] = acc[nt][e] / dn[row];
+      else part[((long long)blockIdx.y * sp.T * c.H + (long long)tok0 * c.H + h0 + row) * (r + 2) + col] = acc[nt][e];
     }
   }
   if (part && threadIdx.x < pairs) {
-    float *rec = part + ((long long)blockIdx.y * sp.T * c.H + (long long)tok0 * c.H + threadIdx.x) * (r + 2);
+    float *rec = part + ((long long)blockIdx.y * sp.T * c.H + (long long)tok0 * c.H + h0 + threadIdx.x) * (r + 2);
     rec[r] = mx[threadIdx.x]; rec[r + 1] = dn[threadIdx.x];
   }
 }
@@ -1236,7 +1395,7 @@ __global__ void stack_latent_merge_kernel(const float *part, const float *sink, 
   __shared__ float ws[kLatMaxSplit];  // per slice e^(m_s - M), 0 for an empty slice
   __shared__ float inv_den;
   const int p = blockIdx.x;
-  const float sk = sink[p % H];
+  const float sk = sink ? sink[p % H] : -INFINITY;
   float M = sk;
   for (int s = 0; s < n_split; s++) M = fmaxf(M, part[((long long)s * pairs_total + p) * (r + 2) + r]);
   for (int s = threadIdx.x; s < n_split; s += blockDim.x) {
@@ -1245,7 +1404,7 @@ __global__ void stack_latent_merge_kernel(const float *part, const float *sink, 
   }
   __syncthreads();
   if (threadIdx.x == 0) {
-    float den = expf(sk - M);
+    float den = sink ? expf(sk - M) : 0.f;
     for (int s = 0; s < n_split; s++) den += part[((long long)s * pairs_total + p) * (r + 2) + r + 1] * ws[s];
     inv_den = 1.f / den;
   }
@@ -1261,9 +1420,9 @@ __global__ void stack_latent_merge_kernel(const float *part, const float *sink, 
 // are copied out of their pages into one contiguous matrix and its transpose, scores = Q C^T and outputs = P C run on the
 // tensor-core product, and the kernel between them turns a block of score rows into softmax weights (fp32, causal, sink).
 __global__ void stack_latent_gather_kernel(const uint16_t *pool, const int *pt, int page_size, int D, int r, int ctx, int ctx8,
-                                           uint16_t *cg, uint16_t *cgt) {
-  const int kp = blockIdx.x;
-  const long long prow = kp < ctx ? (long long)pt[kp / page_size] * page_size + kp % page_size : 0;
+                                           uint16_t *cg, uint16_t *cgt, int first) {
+  const int kp = blockIdx.x, key = first + kp;  // row kp holds the latent of position first + kp
+  const long long prow = kp < ctx ? (long long)pt[key / page_size] * page_size + key % page_size : 0;
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     const uint16_t v = kp < ctx ? pool[prow * D + c] : (uint16_t)0;
     cg[(long long)kp * D + c] = v;
@@ -1271,38 +1430,40 @@ __global__ void stack_latent_gather_kernel(const uint16_t *pool, const int *pt, 
   }
 }
 cudaError_t launch_stack_latent_gather(const void *pool, const int *pt_row, int page_size, int D, int r, int ctx, int ctx8,
-                                       uint16_t *cg, uint16_t *cgt, cudaStream_t st) {
-  stack_latent_gather_kernel<<<ctx8, 128, 0, st>>>(reinterpret_cast<const uint16_t *>(pool), pt_row, page_size, D, r, ctx, ctx8, cg, cgt);
+                                       uint16_t *cg, uint16_t *cgt, int first, cudaStream_t st) {
+  stack_latent_gather_kernel<<<ctx8, 128, 0, st>>>(reinterpret_cast<const uint16_t *>(pool), pt_row, page_size, D, r, ctx, ctx8, cg, cgt, first);
   return cudaGetLastError();
 }
 
-// Row (t, h) of S [rows][ld] holds the raw scores of the query at position pos_first + t against keys 0 .. ld-1.
+// Row (t, h) of S [rows][ld] holds the raw scores of the query at position pos_first + t against keys 0 .. ld-1 (positions count
+// from the first gathered key; window > 0: only the last `window` keys up to the query's own are seen).
 __global__ void __launch_bounds__(256) stack_latent_softmax_kernel(const float *S, int ld, const float *sink, int H, int pos_first,
-                                                                   float scale, uint16_t *P) {
+                                                                   float scale, uint16_t *P, int window) {
   __shared__ float sh[32];
   const long long row = blockIdx.x;
   const int h = (int)(row % H), qpos = pos_first + (int)(row / H);
   const float *s = S + row * ld;
   const int nk = min(ld, qpos + 1);
-  const float sk = sink[h];
+  const int lo = window > 0 ? max(0, qpos - window + 1) : 0;
+  const float sk = sink ? sink[h] : -INFINITY;
   float m = sk;
-  for (int k = threadIdx.x; k < nk; k += blockDim.x) m = fmaxf(m, s[k] * scale);
+  for (int k = lo + threadIdx.x; k < nk; k += blockDim.x) m = fmaxf(m, s[k] * scale);
   m = warp_max(m);
   __syncthreads();
   if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = m;
   __syncthreads();
   for (int i = 0; i < (int)(blockDim.x >> 5); i++) m = fmaxf(m, sh[i]);
   float sum = 0.f;
-  for (int k = threadIdx.x; k < nk; k += blockDim.x) sum += expf(s[k] * scale - m);
-  sum = block_sum(sum, sh) + expf(sk - m);
+  for (int k = lo + threadIdx.x; k < nk; k += blockDim.x) sum += expf(s[k] * scale - m);
+  sum = block_sum(sum, sh) + (sink ? expf(sk - m) : 0.f);
   const float inv = 1.f / sum;
   uint16_t *p = P + row * ld;
-  for (int k = threadIdx.x; k < ld; k += blockDim.x) p[k] = k < nk ? float_to_bf16_bits(expf(s[k] * scale - m) * inv) : (uint16_t)0;
+  for (int k = threadIdx.x; k < ld; k += blockDim.x) p[k] = k < nk && k >= lo ? float_to_bf16_bits(expf(s[k] * scale - m) * inv) : (uint16_t)0;
 }
 cudaError_t launch_stack_latent_softmax(const float *S, int rows, int ld, const float *sink, int H, int pos_first, float scale,
-                                        uint16_t *P, cudaStream_t st) {
+                                        uint16_t *P, int window, cudaStream_t st) {
   if (rows <= 0) return cudaSuccess;
-  stack_latent_softmax_kernel<<<rows, 256, 0, st>>>(S, ld, sink, H, pos_first, scale, P);
+  stack_latent_softmax_kernel<<<rows, 256, 0, st>>>(S, ld, sink, H, pos_first, scale, P, window);
   return cudaGetLastError();
 }
 
@@ -1324,7 +1485,7 @@ cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32
       return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_latent_attn_mma_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
     }));
     if (shm > 220 * 1024) return cudaErrorInvalidValue;
-    const dim3 grid(n_qb, n_split);
+    const dim3 grid(n_qb, n_split, (c.H + kMmaRows - 1) / kMmaRows);
     const uint16_t *pl = reinterpret_cast<const uint16_t *>(pool);
     if (c.r <= 512) stack_latent_attn_mma_kernel<8><<<grid, 256, shm, st>>>(qf, pl, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);
     else stack_latent_attn_mma_kernel<16><<<grid, 256, shm, st>>>(qf, pl, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);

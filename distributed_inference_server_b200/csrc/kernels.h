@@ -121,12 +121,12 @@ cudaError_t launch_gemm_persist_relu2(const TmaMap &w_map128, const TmaMap &x_ma
 cudaError_t launch_gemm_persist_silu(const TmaMap &w_map64, const TmaMap &x_map256, uint16_t *act, int T, int I, int K,
                                      int w_row0, cudaStream_t st);
 cudaError_t launch_gemm_persist_glu(const TmaMap &w_map64, const TmaMap &x_map256, uint16_t *act, int T, int I, int K,
-                                    int w_row0, int act_kind, cudaStream_t st);
+                                    int w_row0, int act_kind, cudaStream_t st, int ld_act = 0);  // ld_act: row stride of act (0: I)
 cudaError_t launch_gemm_silu(const TmaMap &w_map, const TmaMap &x_map, uint16_t *act, int T, int I, int K,
                              int w_row0, int tile_rows, cudaStream_t st);
 // the same with the gate's activation chosen: act_kind 0 = silu, 1 = gelu_tanh
 cudaError_t launch_gemm_glu(const TmaMap &w_map, const TmaMap &x_map, uint16_t *act, int T, int I, int K, int w_row0,
-                            int tile_rows, int act_kind, cudaStream_t st);
+                            int tile_rows, int act_kind, cudaStream_t st, int ld_act = 0);
 int gemm_pick_split_k(int T, int N, int K);
 
 }  // namespace dis

@@ -28,6 +28,14 @@ namespace dis {
     if (_e != cudaSuccess) return _e; \
   } while (0)
 
+static StackLatent stack_latent_shape(const dis_layer_config &lc, float eps) {
+  StackLatent c{lc.heads, lc.dim, lc.rot_dim, lc.vdim, lc.kv_rank, lc.rot_dims, lc.scale, eps};
+  c.window = lc.mask_window;
+  c.rot_pairs = (lc.latent_flags & DIS_LATENT_ROT_PAIRS) ? 1 : 0;
+  c.q_rank = lc.q_rank;
+  return c;
+}
+
 static size_t align_up16(size_t v) { return (v + 15) / 16 * 16; }
 
 void Engine::free_stack() {
@@ -103,6 +111,10 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   StackModel &M = *stack;
   M.c = *sc;
   M.f32 = sc->compute_dtype == DIS_F32;
+  const bool gain_from_one = sc->norm_kind == DIS_NORM_RMS_ONE;  // stored norm vectors get 1 added as they are loaded; the kernels see plain gains
+  if (gain_from_one) M.c.norm_kind = DIS_NORM_RMS;
+  if (M.c.residual_mult == 0.f) M.c.residual_mult = 1.f;
+  const bool par_frame = (sc->frame_flags & DIS_FRAME_PARALLEL) != 0;
   M.max_rows = std::max(sc->max_logit_rows > 0 ? sc->max_logit_rows : max_batch, max_batch);
   M.layers.resize((size_t)sc->n_layers);
   const int W = sc->width, taps = sc->canon_taps;
@@ -135,10 +147,13 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
           return fail(DIS_ERR_INVALID_ARGUMENT, at + "kv_from must name a latent layer with a cache of its own and the same kv_rank and rot_dim");
       }
       L.q_off = 0;
-      L.dkv_off = lc.heads * (lc.dim + lc.rot_dim);
+      L.dkv_off = lc.q_rank > 0 ? lc.q_rank : lc.heads * (lc.dim + lc.rot_dim);  // rows: queries (or their latent) | latent, rotated key part | gate
       L.g_off = L.dkv_off + (lc.kv_from < 0 ? lc.kv_rank + lc.rot_dim : 0);
-      L.n_in = L.g_off + lc.heads * lc.vdim;
-      StackLatent sl{lc.heads, lc.dim, lc.rot_dim, lc.vdim, lc.kv_rank, lc.rot_dims, lc.rot_base, lc.scale, sc->norm_eps};
+      L.n_in = L.g_off + ((lc.latent_flags & DIS_LATENT_NO_GATE) ? 0 : lc.heads * lc.vdim);
+      L.n_act = lc.heads * lc.vdim;
+      if (lc.mask_window < 0 || lc.mask_chunk != 0 || lc.mask_keep != 0 || lc.q_rank < 0)
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "latent attention: mask_window and q_rank must not be negative; it has no chunked mask and no kept positions");
+      const StackLatent sl = stack_latent_shape(lc, sc->norm_eps);
       if (((size_t)32 * (lc.kv_rank + lc.rot_dim + 9) + (size_t)lc.heads * (2 * lc.kv_rank + lc.rot_dim + 2)) * 4 > 200 * 1024)
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "heads * kv_rank does not fit shared memory");
       stack_bq = std::min(stack_bq, stack_latent_block_tokens(sl));
@@ -159,6 +174,15 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       if ((fl & DIS_ATTN_QK_NORM) && (fl & DIS_ATTN_QK_NORM_HEAD)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "query/key norm: whole projection or per head, not both");
       if ((fl & DIS_ATTN_BIAS) && (fl & DIS_ATTN_BIAS_QKV)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "biases: q, k, o or q, k, v, not both");
       if (lc.mask_chunk < 0 || lc.mask_window < 0) return fail(DIS_ERR_INVALID_ARGUMENT, at + "mask_chunk and mask_window must not be negative");
+      if (lc.mask_keep < 0) return fail(DIS_ERR_INVALID_ARGUMENT, at + "mask_keep must not be negative");
+      if ((fl & DIS_ATTN_GATE) && (fl & DIS_ATTN_GATE_FULL)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "output gate: one per head or one per coordinate, not both");
+      if ((fl & DIS_ATTN_DISTANCE) && (fl & DIS_ATTN_SIGMOID)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "the distance term belongs to softmax weights");
+      if (fl & DIS_ATTN_V_MIX) {
+        if ((fl & (DIS_ATTN_V_IS_K | DIS_ATTN_ROT_V)) || lc.kv_from >= 0) return fail(DIS_ERR_INVALID_ARGUMENT, at + "value mixing needs value projections of the layer's own, unrotated");
+        const int n = lc.kv_heads * lc.vdim;
+        if (M.vmix_cols && M.vmix_cols != n) return fail(DIS_ERR_INVALID_ARGUMENT, at + "layers that mix values must agree in kv_heads * vdim");
+        M.vmix_cols = n;
+      }
       if (!(lc.score_softcap >= 0.f)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "score_softcap must not be negative");
       if ((fl & DIS_ATTN_SIGMOID) && (lc.score_softcap > 0.f || (fl & DIS_ATTN_SINK_UNIT))) return fail(DIS_ERR_INVALID_ARGUMENT, at + "a score soft cap and a sink belong to softmax weights");
       if ((fl & DIS_ATTN_SINK) && (fl & DIS_ATTN_SINK_UNIT)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "sink: a learned logit per head or the unit term, not both");
@@ -171,7 +195,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
           return fail(DIS_ERR_INVALID_ARGUMENT, at + "kv_from must name an attention layer with a cache of its own and the same kv_heads, dim, vdim and rotation");
       }
       const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
-      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, sc->norm_eps, lc.mask_chunk, lc.mask_window, lc.score_softcap};
+      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, sc->norm_eps, lc.mask_chunk, lc.mask_window, lc.score_softcap, lc.mask_keep};
       const int bq = stack_attn_block_tokens(sa, sc->compute_dtype == DIS_F32);
       if (((size_t)32 * (d + dv + 10) + (size_t)(H / G) * (d + dv + 2)) * 4 > 200 * 1024) return fail(DIS_ERR_INVALID_ARGUMENT, at + "dim + vdim does not fit shared memory");
       stack_abq = stack_abq ? std::min(stack_abq, bq) : bq;
@@ -183,6 +207,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       L.n_in = lc.kv_from >= 0 ? H * d : L.v_off + ((lc.attn_flags & DIS_ATTN_V_IS_K) ? 0 : G * dv);
       if (lc.kv_from >= 0) L.k_off = L.v_off = 0;
       if (fl & DIS_ATTN_GATE) { L.g_off = L.n_in; L.n_in += H; }
+      if (fl & DIS_ATTN_GATE_FULL) { L.g_off = L.n_in; L.n_in += H * dv; }
       L.n_act = H * dv;
       if (lc.mixer == DIS_MIX_PARALLEL) {
         const int Hr = lc.gla_heads, dr = lc.gla_dim, dvr = lc.gla_vdim;
@@ -207,6 +232,17 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       L.conv_ch = H * P + 2 * G * N;
       L.x_off = H * P; L.dt_off = L.x_off + L.conv_ch;
       L.n_in = L.dt_off + H;
+    } else if (lc.mixer == DIS_MIX_RETENTION) {
+      if (lc.heads <= 0 || lc.dim <= 0 || lc.vdim <= 0 || !lc.decay || lc.rot_dims < 0 || lc.rot_dims > lc.dim || (lc.rot_dims & 1))
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "retention needs heads, dim, vdim, decay and an even rot_dims <= dim");
+      L.decay.assign(lc.decay, lc.decay + lc.heads);
+      L.c.decay = nullptr;
+      const int H = lc.heads, nb = stack_retention_blocks(lc.dim, lc.vdim), dvb = lc.vdim / nb;
+      if ((lc.dim > 128 || dvb > 128) && ((size_t)lc.dim * dvb + 2 * lc.dim + 9 * dvb) * 4 > 220 * 1024) return fail(DIS_ERR_INVALID_ARGUMENT, at + "dim * vdim does not fit shared memory");
+      // rows of the input projection: q | k | v | g
+      L.k_off = H * lc.dim; L.v_off = 2 * H * lc.dim; L.g_off = L.v_off + H * lc.vdim;
+      L.n_in = L.g_off + H * lc.vdim;
+      L.n_act = H * lc.vdim;
     } else return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown mixer");
     if (lc.mlp_act != DIS_ACT_CLAMPED && lc.mlp_act != DIS_ACT_GELU_TANH && lc.mlp_act != DIS_ACT_SILU && lc.mlp_act != DIS_ACT_RELU2) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown feed-forward activation");
     L.gu_rows = lc.mlp_act == DIS_ACT_RELU2 ? 1 : 2;
@@ -222,14 +258,26 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       }
       if (lc.shared_ff < 0) return fail(DIS_ERR_INVALID_ARGUMENT, at + "shared_ff");
     } else if (lc.mlp != DIS_MLP_NONE) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown feed-forward kind");
+    if (par_frame) {  // the feed-forward's rows follow the mixer's in both projections
+      if (lc.mixer != DIS_MIX_ATTENTION && lc.mixer != DIS_MIX_PARALLEL && lc.mixer != DIS_MIX_LATENT && lc.mixer != DIS_MIX_RETENTION)
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "the parallel frame takes the mixers attention, parallel, latent and retention");
+      if (lc.mlp == DIS_MLP_MOE || (lc.mlp == DIS_MLP_DENSE && lc.mlp_act == DIS_ACT_CLAMPED))
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "the parallel frame takes dense feed-forwards without biases");
+      L.par_ff = lc.mlp == DIS_MLP_DENSE ? lc.ff : 0;
+    }
+    L.n_rows = L.n_in + L.gu_rows * L.par_ff;
+    L.ld_act = L.n_act + L.par_ff;
   }
-  if (sc->norm_kind != DIS_NORM_RMS_SCALAR && sc->norm_kind != DIS_NORM_LAYER && sc->norm_kind != DIS_NORM_RMS) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: norm_kind");
+  if (sc->norm_kind != DIS_NORM_RMS_SCALAR && sc->norm_kind != DIS_NORM_LAYER && sc->norm_kind != DIS_NORM_RMS && !gain_from_one) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: norm_kind");
   if (sc->logit_softcap < 0.f) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: logit_softcap must not be negative");
   const bool pre_frame = (sc->frame_flags & DIS_FRAME_PRE_NORM) != 0;
-  if (pre_frame && (sc->norm_kind != DIS_NORM_RMS || sc->canon_taps != 0))
+  if (pre_frame && (M.c.norm_kind != DIS_NORM_RMS || sc->canon_taps != 0))
     return fail(DIS_ERR_INVALID_ARGUMENT, "stack: the pre-norm frame is built for RMS norms with gain vectors and no input convolution");
   if (sc->streams < 0 || sc->streams > 8 || (sc->streams > 0 && !pre_frame))
     return fail(DIS_ERR_INVALID_ARGUMENT, "stack: residual streams (at most 8) need the pre-norm frame");
+  if (!pre_frame && (M.c.residual_mult != 1.f || par_frame || gain_from_one))
+    return fail(DIS_ERR_INVALID_ARGUMENT, "stack: residual_mult, the parallel frame and gains stored around zero need the pre-norm frame");
+  if (par_frame && sc->streams > 0) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: the parallel frame has one residual");
   const bool loop_proj = sc->loop_times > 0 && !(sc->frame_flags & DIS_FRAME_LOOP_PLAIN);
   const int n_streams = std::max(1, sc->streams);
   if (sc->loop_times < 0 || (sc->loop_times > 0 && !(0 <= sc->loop_start && sc->loop_start < sc->loop_stop && sc->loop_stop <= sc->n_layers)))
@@ -293,11 +341,12 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     name("head", &M.head, 0, {sc->vocab, W}, -1);
   }
   ENG_CUDA(alloc(reinterpret_cast<void **>(&M.final_g), 4));
-  const bool ln = sc->norm_kind == DIS_NORM_LAYER || sc->norm_kind == DIS_NORM_RMS;  // norms with vectors
+  const bool ln = M.c.norm_kind == DIS_NORM_LAYER || M.c.norm_kind == DIS_NORM_RMS;  // norms with vectors
+  const int gain_tr = gain_from_one ? 3 : 0;
   const bool ln_bias = sc->norm_kind == DIS_NORM_LAYER;
   if (ln) {
     ENG_CUDA(tensor(M.final_w, (size_t)W, true));
-    name("final.norm", &M.final_w, 0, {W}, -1);
+    name("final.norm", &M.final_w, 0, {W}, -1, gain_tr);
     if (ln_bias) {
       ENG_CUDA(tensor(M.final_b, (size_t)W, true));
       name("final.norm.b", &M.final_b, 0, {W}, -1);
@@ -311,7 +360,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   static StackTensor dummy;  // scalars are written through their own small tensors below
   (void)dummy;
-  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0;
+  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0;
   int max_top = 0, max_e = 0;
   bool any_shared = false;
   size_t max_sff = 0;
@@ -331,8 +380,9 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       for (int k = 0; k < 4; k++) {
         if (k >= 2 && lc.mlp == DIS_MLP_NONE) continue;
         if (pre_frame && (k & 1)) continue;  // no norms behind the sublayers
+        if (par_frame && k >= 2) continue;   // one norm for both
         ENG_CUDA(tensor(L.ln_w[k], (size_t)W, true));
-        name(pre + gn[k], &L.ln_w[k], 0, {W}, i);
+        name(pre + gn[k], &L.ln_w[k], 0, {W}, i, gain_tr);
         if (!ln_bias) continue;
         ENG_CUDA(tensor(L.ln_b[k], (size_t)W, true));
         name(pre + gn[k] + ".b", &L.ln_b[k], 0, {W}, i);
@@ -346,8 +396,22 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       name(hp + "out", &L.hc[q], (size_t)S, {S}, i);
       name(hp + "mix", &L.hc[q], (size_t)2 * S, {S, S}, i);
     }
-    ENG_CUDA(tensor(L.w_in, (size_t)L.n_in * W, M.f32));
-    max_proj = std::max(max_proj, (size_t)L.n_in);
+    ENG_CUDA(tensor(L.w_in, (size_t)L.n_rows * W, M.f32));
+    max_proj = std::max(max_proj, (size_t)L.n_rows);
+    auto freq_table = [&](std::vector<double> f) -> cudaError_t {  // rotary frequencies of the layer, on the device
+      f.push_back(0.0);
+      const cudaError_t e = alloc(reinterpret_cast<void **>(&L.freq), f.size() * 8);
+      return e != cudaSuccess ? e : cudaMemcpy(L.freq, f.data(), f.size() * 8, cudaMemcpyHostToDevice);
+    };
+    auto plain_freq = [&]() {  // base^(-2i/n), formed in double
+      std::vector<double> f((size_t)lc.rot_dims / 2);
+      for (int k = 0; k < lc.rot_dims / 2; k++) f[(size_t)k] = std::pow((double)lc.rot_base, -2.0 * k / (double)lc.rot_dims);
+      return f;
+    };
+    auto out_block = [&](const std::string &nm, size_t off, int cols) {  // a block of columns of the output projection
+      name(nm, &L.w_o, off, {W, cols}, i, 2);
+      stack_names[nm].ld = L.ld_act;
+    };
     if (lc.mixer == DIS_MIX_LIGHTNING) {
       const int H = lc.heads, d = lc.dim, dv = lc.vdim;
       name(pre + "mix.q", &L.w_in, 0, {H * d, W}, i);
@@ -370,20 +434,22 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       if (own) name(a + "k", &L.w_in, (size_t)L.k_off * W, {G * d, W}, i);
       if (own && !(lc.attn_flags & DIS_ATTN_V_IS_K)) name(a + "v", &L.w_in, (size_t)L.v_off * W, {G * dv, W}, i);
       if (lc.attn_flags & DIS_ATTN_GATE) name(a + "g", &L.w_in, (size_t)L.g_off * W, {H, W}, i);
-      ENG_CUDA(tensor(L.w_o, (size_t)W * L.n_act, M.f32));
-      {
-        name(a + "o", &L.w_o, 0, {W, H * dv}, i, 2);
-        stack_names[a + "o"].ld = L.n_act;
+      if (lc.attn_flags & DIS_ATTN_GATE_FULL) name(a + "g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
+      if (lc.attn_flags & DIS_ATTN_V_MIX) {
+        ENG_CUDA(tensor(L.vmix, 1, true));
+        name(a + "vmix", &L.vmix, 0, {}, i);
       }
+      ENG_CUDA(tensor(L.w_o, (size_t)W * L.ld_act, M.f32));
+      out_block(a + "o", 0, H * dv);
       if (lc.attn_flags & DIS_ATTN_BIAS) {
-        ENG_CUDA(tensor(L.b_in, (size_t)L.n_in, true));
+        ENG_CUDA(tensor(L.b_in, (size_t)L.n_rows, true));
         name(a + "q.b", &L.b_in, 0, {H * d}, i);
         name(a + "k.b", &L.b_in, (size_t)L.k_off, {G * d}, i);
         ENG_CUDA(tensor(L.b_o, (size_t)W, true));
         name(a + "o.b", &L.b_o, 0, {W}, i);
       }
       if (lc.attn_flags & DIS_ATTN_BIAS_QKV) {
-        ENG_CUDA(tensor(L.b_in, (size_t)L.n_in, true));
+        ENG_CUDA(tensor(L.b_in, (size_t)L.n_rows, true));
         name(a + "q.b", &L.b_in, 0, {H * d}, i);
         if (own) {
           name(a + "k.b", &L.b_in, (size_t)L.k_off, {G * d}, i);
@@ -426,8 +492,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
           f[(size_t)k] = v;
         }
         for (int k = 0; k < dv / 2; k++) fv[(size_t)k] = std::pow((double)lc.rot_base, -2.0 * k / (double)dv);
-        ENG_CUDA(alloc(reinterpret_cast<void **>(&L.freq), f.size() * 8));
-        ENG_CUDA(cudaMemcpy(L.freq, f.data(), f.size() * 8, cudaMemcpyHostToDevice));
+        ENG_CUDA(freq_table(f));
         if (lc.attn_flags & DIS_ATTN_ROT_V) {
           ENG_CUDA(alloc(reinterpret_cast<void **>(&L.vfreq), fv.size() * 8));
           ENG_CUDA(cudaMemcpy(L.vfreq, fv.data(), fv.size() * 8, cudaMemcpyHostToDevice));
@@ -443,8 +508,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         name(r + "v", &L.w_in, (size_t)L.gv_off * W, {Hr * dvr, W}, i);
         name(r + "g", &L.w_in, (size_t)L.gg_off * W, {Hr * dvr, W}, i);
         name(r + "a1", &L.w_in, (size_t)L.ga_off * W, {rk, W}, i);
-        name(r + "o", &L.w_o, (size_t)H * dv, {W, Hr * dvr}, i, 2);
-        stack_names[r + "o"].ld = L.n_act;
+        out_block(r + "o", (size_t)H * dv, Hr * dvr);
         ENG_CUDA(tensor(L.a2, (size_t)Hr * dr * rk, M.f32));
         name(r + "a2", &L.a2, 0, {Hr * dr, rk}, i);
         ENG_CUDA(tensor(L.a2_b, (size_t)Hr * dr, true));
@@ -454,7 +518,6 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         max_mix = std::max(max_mix, (size_t)Hr * dvr);
         max_dec = std::max(max_dec, (size_t)Hr * dr);
       }
-      max_act = std::max(max_act, (size_t)L.n_act);
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, C = L.conv_ch, inner = H * P;
       name(pre + "mix.in", &L.w_in, 0, {L.n_in, W}, i);
@@ -474,6 +537,20 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       max_act = std::max(max_act, (size_t)inner);
       max_ssm = std::max(max_ssm, (size_t)C);
       max_dec = std::max(max_dec, (size_t)2 * H);  // decays, then step sizes
+    } else if (lc.mixer == DIS_MIX_RETENTION) {
+      const int H = lc.heads, d = lc.dim, dv = lc.vdim, nb = stack_retention_blocks(d, dv);
+      name(pre + "mix.q", &L.w_in, 0, {H * d, W}, i);
+      name(pre + "mix.k", &L.w_in, (size_t)L.k_off * W, {H * d, W}, i);
+      name(pre + "mix.v", &L.w_in, (size_t)L.v_off * W, {H * dv, W}, i);
+      name(pre + "mix.g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
+      ENG_CUDA(tensor(L.w_o, (size_t)W * L.ld_act, M.f32));
+      out_block(pre + "mix.o", 0, H * dv);
+      std::vector<float> dec;
+      for (float a : L.decay) dec.insert(dec.end(), (size_t)nb, a);  // one entry per block of value columns
+      ENG_CUDA(tensor(L.decay_d, dec.size(), true));
+      ENG_CUDA(cudaMemcpy(L.decay_d.ptr, dec.data(), dec.size() * 4, cudaMemcpyHostToDevice));
+      ENG_CUDA(freq_table(plain_freq()));
+      max_mix = std::max(max_mix, (size_t)H * dv);
     } else if (lc.mixer == DIS_MIX_MINGRU) {
       const int n = lc.width;
       name(pre + "mix.z", &L.w_in, 0, {n, W}, i);
@@ -487,28 +564,46 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       max_act = std::max(max_act, (size_t)n);
     } else {
       const int H = lc.heads, d = lc.dim, dr = lc.rot_dim, dv = lc.vdim, r = lc.kv_rank;
-      name(pre + "mix.q", &L.w_in, 0, {H * (d + dr), W}, i);
+      if (lc.q_rank > 0) {
+        name(pre + "mix.dq", &L.w_in, 0, {lc.q_rank, W}, i);
+        ENG_CUDA(tensor(L.q_norm, (size_t)lc.q_rank, true));
+        name(pre + "mix.dq.norm", &L.q_norm, 0, {lc.q_rank}, i);
+        ENG_CUDA(tensor(L.w_uq, (size_t)H * (d + dr) * lc.q_rank, M.f32));
+        name(pre + "mix.uq", &L.w_uq, 0, {H * (d + dr), lc.q_rank}, i);
+        max_cq = std::max(max_cq, (size_t)lc.q_rank);
+        max_ql = std::max(max_ql, (size_t)H * (d + dr));
+      } else name(pre + "mix.q", &L.w_in, 0, {H * (d + dr), W}, i);
+      ENG_CUDA(freq_table(plain_freq()));
       if (lc.kv_from < 0) {
         name(pre + "mix.dkv", &L.w_in, (size_t)L.dkv_off * W, {r + dr, W}, i);
         ENG_CUDA(tensor(L.norm_w, (size_t)r, true));
         name(pre + "mix.dkv.norm", &L.norm_w, 0, {r}, i);
       }
-      name(pre + "mix.g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
+      if (!(lc.latent_flags & DIS_LATENT_NO_GATE)) name(pre + "mix.g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
       ENG_CUDA(tensor(L.ukT, (size_t)H * r * d, M.f32));
       name(pre + "mix.uk", &L.ukT, 0, {H * d, r}, i, /*transpose each head's [d][r] block*/ 1);
       ENG_CUDA(tensor(L.uv, (size_t)H * dv * r, M.f32));
       name(pre + "mix.uv", &L.uv, 0, {H * dv, r}, i);
-      ENG_CUDA(tensor(L.sink, (size_t)H, true));
-      name(pre + "mix.sink", &L.sink, 0, {H}, i);
-      ENG_CUDA(tensor(L.w_o, (size_t)W * H * dv, M.f32));
-      name(pre + "mix.o", &L.w_o, 0, {W, H * dv}, i);
+      if (!(lc.latent_flags & DIS_LATENT_NO_SINK)) {
+        ENG_CUDA(tensor(L.sink, (size_t)H, true));
+        name(pre + "mix.sink", &L.sink, 0, {H}, i);
+      }
+      ENG_CUDA(tensor(L.w_o, (size_t)W * L.ld_act, M.f32));
+      out_block(pre + "mix.o", 0, H * dv);
       max_mix = std::max(max_mix, (size_t)H * std::max(r, dv));
-      max_act = std::max(max_act, (size_t)H * dv);
       max_qf = std::max(max_qf, (size_t)H * (r + dr));
       stack_lat_rec = std::max(stack_lat_rec, (size_t)H * (r + 2));
       stack_lat_heads = std::max(stack_lat_heads, H);
     }
-    if (lc.mlp == DIS_MLP_DENSE) {
+    max_act = std::max(max_act, (size_t)L.ld_act);
+    if (L.par_ff > 0) {  // gate | up: the rows of the input projection behind the mixer's; down: columns of the output projection
+      const size_t at = (size_t)L.n_in * W;
+      L.w_gu.f32 = M.f32; L.w_gu.n = (size_t)L.gu_rows * lc.ff * W;
+      L.w_gu.ptr = reinterpret_cast<char *>(L.w_in.ptr) + at * esz;
+      if (L.gu_rows == 2) name(pre + "mlp.gate", &L.w_in, at, {lc.ff, W}, i);
+      name(pre + "mlp.up", &L.w_in, at + (size_t)(L.gu_rows - 1) * lc.ff * W, {lc.ff, W}, i);
+      out_block(pre + "mlp.down", (size_t)L.n_act, lc.ff);
+    } else if (lc.mlp == DIS_MLP_DENSE) {
       const int ff = lc.ff, gr = L.gu_rows;
       ENG_CUDA(tensor(L.w_gu, (size_t)gr * ff * W, M.f32));
       ENG_CUDA(tensor(L.w_down, (size_t)W * ff, M.f32));
@@ -599,7 +694,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       ENG_CUDA(alloc(reinterpret_cast<void **>(&R.cstate1), slots * (taps - 1) * W * 4));
       if (lc.mlp != DIS_MLP_NONE) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.cstate2), slots * (taps - 1) * W * 4));
     }
-    if (lc.mixer == DIS_MIX_LIGHTNING) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.heads * lc.dim * lc.vdim * 4));
+    if (lc.mixer == DIS_MIX_LIGHTNING || lc.mixer == DIS_MIX_RETENTION) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.heads * lc.dim * lc.vdim * 4));
     else if (lc.mixer == DIS_MIX_MINGRU) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.width * 4));
     else if (lc.mixer == DIS_MIX_PARALLEL) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.gla_heads * lc.gla_dim * lc.gla_vdim * 4));
     else if (lc.mixer == DIS_MIX_SSM) {
@@ -633,6 +728,11 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     ENG_CUDA(alloc(&M.xcat, cap * 2 * W * esz));
   }
   if (max_dec) ENG_CUDA(alloc(reinterpret_cast<void **>(&M.dec), cap * max_dec * 4));
+  if (max_cq) {
+    ENG_CUDA(alloc(&M.cq, cap * max_cq * esz));
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.ql), cap * max_ql * 4));
+  }
+  if (M.vmix_cols) ENG_CUDA(alloc(reinterpret_cast<void **>(&M.vfirst), cap * M.vmix_cols * 4));
   if (max_vrot) ENG_CUDA(alloc(reinterpret_cast<void **>(&M.vrot), cap * max_vrot * 4));
   if (stack_att_rec) {
     M.attn_part_elems = (size_t)2048 * stack_att_rec;  // (tokens x slices) of one pass
@@ -664,6 +764,8 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     for (auto &L : M.layers) {
       if (L.c.mixer == DIS_MIX_LIGHTNING && L.c.dim <= 128 && L.c.vdim <= 128)
         seg = std::max(seg, stack_lightning_seg_floats(cap_tokens, max_batch, L.c.heads, L.c.dim, L.c.vdim));
+      if (L.c.mixer == DIS_MIX_RETENTION && L.c.dim <= 128)
+        seg = std::max(seg, stack_lightning_seg_floats(cap_tokens, max_batch, L.c.heads, L.c.dim, L.c.vdim));
       if (L.c.mixer == DIS_MIX_PARALLEL) {
         seg = std::max(seg, stack_lightning_seg_floats(cap_tokens, max_batch, L.c.gla_heads, L.c.gla_dim, L.c.gla_vdim));
         seg_a = std::max(seg_a, stack_lightning_seg_decay_floats(cap_tokens, max_batch, L.c.gla_heads, L.c.gla_dim));
@@ -684,7 +786,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   if (const char *g = getenv("DIS_STACK_TC")) stack_tc = atoi(g) != 0;
   if (const char *g = getenv("DIS_STACK_PERSIST")) stack_persist = atoi(g) != 0;
   if (!M.f32 && stack_tc) {
-    M.scratch_elems = 2 * cap * std::max(max_proj, (size_t)W);
+    M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), (size_t)W);
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.scratch), M.scratch_elems * 4));
   }
   ENG_CUDA(alloc(reinterpret_cast<void **>(&M.logits), (size_t)M.max_rows * sc->vocab * 4));
@@ -788,6 +890,7 @@ int Engine::load_named(const char *nm, const void *host, int dtype, const int64_
   std::vector<float> f(n);
   if (dtype == DIS_F32) memcpy(f.data(), host, n * 4);
   else for (size_t i = 0; i < n; i++) f[i] = bf16_bits_to_float(reinterpret_cast<const uint16_t *>(host)[i]);
+  if (t.transform == 3) for (float &v : f) v += 1.f;  // a gain stored as its distance from one
   if (t.transform == 1) {  // [H*d][r] -> per head [r][d]
     const dis_layer_config &lc = stack->layers[(size_t)t.layer].c;
     const size_t H = (size_t)lc.heads, d = (size_t)lc.dim, r = (size_t)lc.kv_rank;
@@ -951,13 +1054,15 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
   }
   ENG_CUDA(cudaMemcpyAsync(mt.dev, mt.host, mt.bytes, cudaMemcpyHostToDevice, stream));
   // latent attention: with few query blocks the history is cut into slices so that about two CTAs per SM run
-  stack_lat_split = 1; stack_lat_keys = 0;
-  if (QB > 0 && QB < kNumSMs && stack_max_ctx >= 256 && stack_lat_rec) {
-    int sp = std::min(std::min((2 * kNumSMs + QB - 1) / QB, stack_max_ctx / (stack_lat_mma ? 64 : 32)), 64);  // a slice holds at least one tile of keys
-    const int keys = ((stack_max_ctx + sp - 1) / sp + 31) / 32 * 32;
-    sp = (stack_max_ctx + keys - 1) / keys;
-    if (sp > 1 && (size_t)sp * T * stack_lat_rec <= M.lat_part_elems) { stack_lat_split = sp; stack_lat_keys = keys; }
-  }
+  // (a windowed layer walks at most its window plus the block's own tokens)
+  auto lat_slices = [&](int ctx) -> std::pair<int, int> {
+    if (!(QB > 0 && QB < kNumSMs && ctx >= 256 && stack_lat_rec)) return {1, 0};
+    int sp = std::min(std::min((2 * kNumSMs + QB - 1) / QB, ctx / (stack_lat_mma ? 64 : 32)), 64);  // a slice holds at least one tile of keys
+    const int keys = ((ctx + sp - 1) / sp + 31) / 32 * 32;
+    sp = (ctx + keys - 1) / keys;
+    if (sp > 1 && (size_t)sp * T * stack_lat_rec <= M.lat_part_elems) return {sp, keys};
+    return {1, 0};
+  };
   // paged attention likewise: one CTA per (query block, key/value head, slice).  A layer with a chunked mask walks at most
   // its chunk (plus the block's own tokens) whatever the history's length, so it slices by that bound.
   stack_kb = KB;
@@ -972,14 +1077,18 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
   };
   {
     const std::pair<int, int> whole = att_slices(stack_max_ctx);
-    stack_att_split = whole.first; stack_att_keys = whole.second;
     stack_att_plan.assign(M.layers.size(), whole);
     for (size_t li = 0; li < M.layers.size(); li++) {
       const dis_layer_config &lc = M.layers[li].c;
+      if (lc.mixer == DIS_MIX_LATENT) {
+        stack_att_plan[li] = lat_slices(lc.mask_window > 0 ? (int)std::min<long long>(stack_max_ctx, (long long)lc.mask_window + stack_bq) : stack_max_ctx);
+        continue;
+      }
       if (!(lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL)) continue;
       long long bound = stack_max_ctx;  // keys a query block can reach at most
       if (lc.mask_chunk > 0) bound = std::min(bound, (long long)lc.mask_chunk + stack_abq);
       if (lc.mask_window > 0) bound = std::min(bound, (long long)lc.mask_window + stack_abq);
+      if (bound < stack_max_ctx) bound = std::min(bound + lc.mask_keep, (long long)stack_max_ctx);
       if (bound < stack_max_ctx) stack_att_plan[li] = att_slices((int)bound);
     }
   }
@@ -990,7 +1099,7 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
     ENG_CUDA(stack_forward(T, SP, QB, R, all_greedy));
   } else {
     // the pass's shape and every layer's slicing name the graph; `graphs` is keyed by the order in which they were first seen
-    std::vector<uint64_t> shape{(uint64_t)T | ((uint64_t)stack_lat_split << 16) | ((uint64_t)(stack_lat_keys / 32) << 24) | (all_greedy ? 1ull << 60 : 0ull)};
+    std::vector<uint64_t> shape{(uint64_t)T | (all_greedy ? 1ull << 60 : 0ull)};
     for (auto &pl : stack_att_plan) shape.push_back((uint64_t)pl.first | ((uint64_t)pl.second << 8));
     const uint64_t key = stack_graph_ids.emplace(shape, (uint64_t)stack_graph_ids.size()).first->second;
     auto it = graphs.find(key);
@@ -1067,6 +1176,8 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
   StackModel &M = *stack;
   StepMeta &mt = meta_pre;
   const int W = M.c.width, taps = M.c.canon_taps;
+  const float res_mult = M.c.residual_mult;
+  const float *vfirst = nullptr;  // values of the pass's first value-mixing layer, once it has run
   const float eps = M.c.norm_eps;
   const bool f32 = M.f32;
   StackSpans sp{mt.d<uint32_t>(mt.o_tokens), mt.d<int>(mt.o_pos), mt.d<int>(mt.o_ptrow), mt.d<int>(mt.o_span),
@@ -1142,7 +1253,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       kl++;
       const float *src = pend_y ? (pend_parts > 1 || pend_bias ? pend_src : pend_y) : nullptr;
       const cudaError_t e = launch_stack_boundary_hc(M.x, n_streams, src, pend_parts, pend_stride, pend_bias, pend_hc, next_hc, pre, M.hc, f32, T,
-                                                     W, eps, stream);
+                                                     W, eps, res_mult, stream);
       pend_y = nullptr; pend_parts = 1; pend_bias = nullptr; pend_hc = nullptr;
       return e;
     }
@@ -1183,37 +1294,41 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     kl++;
     return launch_stack_copy_act(M.hn, M.hc, f32, (long long)T * W, stream);
   };
-  const int lat_split = stack_lat_split, lat_keys = stack_lat_keys;
   const bool later = single || ln;  // the boundary kernel of the next sublayer sums a product's slices and adds its bias
   auto norm_w = [&](StackLayer &L, int k) { return ln ? reinterpret_cast<const float *>(L.ln_w[k].ptr) : L.g4 + k; };
   auto norm_b = [&](StackLayer &L, int k) { return ln ? reinterpret_cast<const float *>(L.ln_b[k].ptr) : nullptr; };
   int max_span = 0;
   for (auto &sh : stack_spans_h) max_span = std::max(max_span, sh.len);
+  // bf16, a unit without biases (gelu_tanh or SiLU gate), prompt-sized passes: gate and up run as one tensor-core product with
+  // two accumulators whose epilogue writes act(gate) * up (the product the Llama path uses with SiLU).  Decode-sized passes
+  // keep the split-K product below, whose slices the gated unit sums: at these widths a single pass over K leaves each CTA a
+  // long thin loop (measured: 0.337 against 0.320 ms per step of four layers at width 1024).
+  auto glu_fused_ok = [&](const StackTensor &w_gu, const StackTensor &b_gu, int act_kind) {
+    return stack_tc && !f32 && (act_kind == DIS_ACT_GELU_TANH || act_kind == DIS_ACT_SILU) && !b_gu.ptr && W % 8 == 0 && !w_gu.f32 &&
+           gemm_token_tile(T) >= 128;
+  };
+  auto glu_product = [&](const StackTensor &w_gu, int ff, int act_kind, void *act, int ld_act) -> cudaError_t {
+    const int tc_act = act_kind == DIS_ACT_GELU_TANH ? 1 : 0;
+    kl++;
+    if (stack_persist && gemm_use_persist(T, ff, true)) {  // paired gate / up tiles on the persistent kernel
+      const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, 256);
+      const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, 64);
+      if (!xm || !wm) return cudaErrorInvalidValue;
+      return launch_gemm_persist_glu(*wm, *xm, reinterpret_cast<uint16_t *>(act), T, ff, W, 0, tc_act, cur_st, ld_act);
+    }
+    const int tr = 128;
+    const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, (uint32_t)gemm_token_tile(T));
+    const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, (uint32_t)tr);
+    if (!xm || !wm) return cudaErrorInvalidValue;
+    return launch_gemm_glu(*wm, *xm, reinterpret_cast<uint16_t *>(act), T, ff, W, 0, tr, tc_act, cur_st, ld_act);
+  };
   // A dense gated unit out = W_down act(W_gate h, W_up h) on the sublayer input M.hc.  later: the slices of the down projection
   // may stay unsummed for the next boundary kernel (out is then M.y, as the caller expects).
   auto dense_ff = [&](const StackTensor &w_gu, const StackTensor &b_gu, const StackTensor &w_down, const StackTensor &b_down, int ff,
                       int act_kind, float limit, float *out, bool later_ok) -> cudaError_t {
     const int gu_rows = act_kind == DIS_ACT_RELU2 ? 1 : 2;  // an ungated unit has no gate rows
-    // bf16, a unit without biases (gelu_tanh or SiLU gate), prompt-sized passes: gate and up run as one tensor-core product with
-    // two accumulators whose epilogue writes act(gate) * up (the product the Llama path uses with SiLU).  Decode-sized passes
-    // keep the split-K product below, whose slices the gated unit sums: at these widths a single pass over K leaves each CTA a
-    // long thin loop (measured: 0.337 against 0.320 ms per step of four layers at width 1024).
-    if (stack_tc && !f32 && (act_kind == DIS_ACT_GELU_TANH || act_kind == DIS_ACT_SILU) && !b_gu.ptr && W % 8 == 0 && !w_gu.f32 &&
-        gemm_token_tile(T) >= 128) {
-      const int tc_act = act_kind == DIS_ACT_GELU_TANH ? 1 : 0;
-      if (stack_persist && gemm_use_persist(T, ff, true)) {  // paired gate / up tiles on the persistent kernel
-        const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, 256);
-        const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, 64);
-        if (!xm || !wm) return cudaErrorInvalidValue;
-        RET_CUDA(launch_gemm_persist_glu(*wm, *xm, reinterpret_cast<uint16_t *>(cur_act), T, ff, W, 0, tc_act, cur_st));
-      } else {
-        const int tr = 128;
-        const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, (uint32_t)gemm_token_tile(T));
-        const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, (uint32_t)tr);
-        if (!xm || !wm) return cudaErrorInvalidValue;
-        RET_CUDA(launch_gemm_glu(*wm, *xm, reinterpret_cast<uint16_t *>(cur_act), T, ff, W, 0, tr, tc_act, cur_st));
-      }
-      kl++;
+    if (glu_fused_ok(w_gu, b_gu, act_kind)) {
+      RET_CUDA(glu_product(w_gu, ff, act_kind, cur_act, ff));
       return gemm(cur_act, f32, ff, w_down, 0, nullptr, out, T, W, ff, cap_tokens, nullptr, later_ok);
     }
     // an ungated unit in prompt-sized bf16 passes: the persistent product's epilogue squares the relu and writes bf16
@@ -1248,11 +1363,18 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     }
     next_hc = reinterpret_cast<const float *>(L.hc[0].ptr);
     RET_CUDA(sublayer_in(norm_w(L, 0), norm_b(L, 0), L.canon1, Rn.cstate1));
-    const int N = L.n_in;
+    // Parallel layers: the feed-forward reads the same h.  Its gate and up rows follow the mixer's in the input projection, so a
+    // decode-sized pass runs them as one product; a prompt-sized pass keeps the product whose epilogue is the gated unit.  Either way
+    // the unit's output goes to the columns behind the mixer's in M.act, and one product with [mixer.o | down] ends the layer.
+    const int par_ff = L.par_ff;
+    const bool split_in = par_ff > 0 && glu_fused_ok(L.w_gu, StackTensor(), lc.mlp_act);
+    const int N = split_in ? L.n_in : L.n_rows;
+    void *ff_act = f32 ? (void *)(reinterpret_cast<float *>(M.act) + L.n_act) : (void *)(reinterpret_cast<uint16_t *>(M.act) + L.n_act);
     const float *in_bias = nullptr;  // minGRU adds its projections' biases itself when the product left them out
     const bool is_attn = lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL;
-    // a plain attention mixer's preparation kernel sums the slices of a split-K input projection itself
-    const bool prep_sums = lc.mixer == DIS_MIX_ATTENTION;
+    // the preparation kernels of attention (alone), latent attention and retention sum the slices of a split-K input projection themselves
+    const bool prep_sums = lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_LATENT || lc.mixer == DIS_MIX_RETENTION;
+    if (split_in) RET_CUDA(glu_product(L.w_gu, par_ff, lc.mlp_act, ff_act, L.ld_act));
     RET_CUDA(gemm(M.hc, f32, W, L.w_in, 0, L.b_in.ptr ? reinterpret_cast<const float *>(L.b_in.ptr) : nullptr, M.proj, T, N, W, cap_tokens,
                   lc.mixer == DIS_MIX_MINGRU || is_attn ? &in_bias : nullptr, prep_sums));
     const float *in_src = M.proj;
@@ -1260,6 +1382,10 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     long long in_stride = 0;
     if (prep_sums && (pend_parts > 1 || pend_bias)) { in_src = pend_src; in_parts = pend_parts; in_stride = pend_stride; in_bias = pend_bias; }
     pend_parts = 1; pend_bias = nullptr;
+    if (par_ff > 0 && !split_in) {
+      RET_CUDA(launch_stack_glu(in_src + L.n_in, in_parts, in_stride, nullptr, ff_act, f32, nullptr, T, par_ff, lc.limit, lc.mlp_act, stream, N, L.ld_act));
+      kl++;
+    }
     int n_mix = 0;
     const float *o_bias = nullptr;
     if (lc.mixer == DIS_MIX_LIGHTNING) {
@@ -1273,6 +1399,16 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       RET_CUDA(launch_stack_norm_gate(M.mix, reinterpret_cast<const float *>(L.norm_w.ptr), M.proj + L.g_off, N, M.act, f32, T, H * dv, eps, stream));
       kl += 2;
       n_mix = H * dv;
+    } else if (lc.mixer == DIS_MIX_RETENTION) {
+      const int H = lc.heads, d = lc.dim, dv = lc.vdim, nb = stack_retention_blocks(d, dv);
+      RET_CUDA(launch_stack_retention_prep(in_src, N, in_parts, in_stride, L.n_in, M.proj, N, 0, L.k_off, H, d, L.freq, lc.rot_dims,
+                                           1.f / std::sqrt((float)d), sp, stream));
+      const bool segments = M.light_seg && d <= 128 && stack_lightning_segmented(sp.n_spans, T, H * nb, max_span);
+      RET_CUDA(launch_stack_retention(M.proj, N, 0, L.k_off, L.v_off, reinterpret_cast<const float *>(L.decay_d.ptr), Rn.state, sp, M.mix, H, d, dv,
+                                      segments ? M.light_seg : nullptr, max_span, stream));
+      RET_CUDA(launch_stack_headnorm_silu(M.mix, nullptr, M.proj + L.g_off, N, M.act, L.ld_act, 0, 1.f, f32, T, H, dv, eps, stream));
+      kl += segments ? 5 : 3;
+      n_mix = L.ld_act;
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, Ns = lc.ssm_state, G = lc.ssm_groups, C = L.conv_ch, inner = H * P;
       const long long ld_b = C;  // x | B | C
@@ -1297,7 +1433,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     } else if (is_attn) {
       const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
       const bool par = lc.mixer == DIS_MIX_PARALLEL;
-      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, eps, lc.mask_chunk, lc.mask_window, lc.score_softcap};
+      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, eps, lc.mask_chunk, lc.mask_window, lc.score_softcap, lc.mask_keep};
       const float *qkn = reinterpret_cast<const float *>(L.qk_norm.ptr), *tpb = reinterpret_cast<const float *>(L.temp_pb.ptr);
       // the gains of the key norm follow those of the query norm: [H*d] then [G*d] (whole projection), or [d] then [d] (per head)
       const float *kn = qkn ? qkn + ((lc.attn_flags & DIS_ATTN_QK_NORM_HEAD) ? (size_t)d : (size_t)H * d) : nullptr;
@@ -1305,14 +1441,20 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       StackRun &KV = M.runs[(size_t)Rn.kv_run];
       // the gate logits are read by the attention kernel from M.proj: when the projection came as slices the preparation writes
       // their sums there
-      const bool gated = (lc.attn_flags & DIS_ATTN_GATE) != 0;
-      RET_CUDA(launch_stack_attn_prep(in_src, N, in_parts, in_stride, N, L.g_off, gated && in_src != M.proj ? M.proj + L.g_off : nullptr, N, L.q_off,
+      const bool gated = (lc.attn_flags & (DIS_ATTN_GATE | DIS_ATTN_GATE_FULL)) != 0;
+      StackVMix vm;
+      if (lc.attn_flags & DIS_ATTN_V_MIX) {
+        if (!vfirst) vm.save = M.vfirst;
+        else { vm.first = vfirst; vm.lam = reinterpret_cast<const float *>(L.vmix.ptr); }
+        vfirst = M.vfirst;
+      }
+      RET_CUDA(launch_stack_attn_prep(in_src, N, in_parts, in_stride, L.n_in, L.g_off, gated && in_src != M.proj ? M.proj + L.g_off : nullptr, N, L.q_off,
                                       L.k_off, L.v_off, in_bias, qkn, kn, L.freq, L.vfreq, sa, sp, M.qf, own ? Rn.kpool : nullptr,
-                                      own ? Rn.vpool : nullptr, M.vrot, f32, d_page_table, max_pages, page_size, stream));
+                                      own ? Rn.vpool : nullptr, M.vrot, f32, d_page_table, max_pages, page_size, vm, stream));
       const std::pair<int, int> slices = stack_att_plan[(size_t)Rn.layer];
       RET_CUDA(launch_stack_attn(M.qf, KV.kpool, KV.vpool, f32, tpb, tpb ? tpb + H : nullptr, reinterpret_cast<const float *>(L.sink.ptr), sa, sp,
                                  mt.d<int>(mt.o_kb_tok0), mt.d<int>(mt.o_kb_len), stack_kb, single ? 1 : stack_abq, d_page_table, max_pages,
-                                 page_size, M.act, L.n_act, 0, par ? lc.mix_scale : 1.f, M.vrot, M.proj + L.g_off, N, slices.first,
+                                 page_size, M.act, L.ld_act, 0, par ? lc.mix_scale : 1.f, M.vrot, M.proj + L.g_off, N, slices.first,
                                  slices.second, M.attn_part, stream));
       kl += slices.first > 1 ? 3 : 2;
       if (par) {
@@ -1322,24 +1464,50 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         const bool segments = M.light_seg && M.light_seg_a && stack_lightning_segmented(sp.n_spans, T, Hr, max_span);
         RET_CUDA(launch_stack_gla(M.proj, N, L.gq_off, L.gk_off, L.gv_off, M.dec, Rn.state, sp, M.mix, Hr, dr, dvr,
                                   segments ? M.light_seg : nullptr, segments ? M.light_seg_a : nullptr, max_span, stream));
-        RET_CUDA(launch_stack_headnorm_silu(M.mix, reinterpret_cast<const float *>(L.gla_norm.ptr), M.proj + L.gg_off, N, M.act, L.n_act,
+        RET_CUDA(launch_stack_headnorm_silu(M.mix, reinterpret_cast<const float *>(L.gla_norm.ptr), M.proj + L.gg_off, N, M.act, L.ld_act,
                                             H * dv, lc.gla_scale, f32, T, Hr, dvr, eps, stream));
         kl += segments ? 5 : 3;
       }
       o_bias = reinterpret_cast<const float *>(L.b_o.ptr);
-      n_mix = L.n_act;
+      n_mix = L.ld_act;
     } else {
       const int H = lc.heads, d = lc.dim, dr = lc.rot_dim, dv = lc.vdim, r = lc.kv_rank, D = r + dr;
-      StackLatent sl{H, d, dr, dv, r, lc.rot_dims, lc.rot_base, lc.scale, eps};
+      const StackLatent sl = stack_latent_shape(lc, eps);
+      const std::pair<int, int> slices = stack_att_plan[(size_t)Rn.layer];
+      const bool gated = !(lc.latent_flags & DIS_LATENT_NO_GATE);
+      const float *gate = gated ? M.proj + L.g_off : nullptr;
       StackRun &KV = M.runs[(size_t)Rn.kv_run];
-      RET_CUDA(launch_stack_latent_prep(M.proj, N, L.q_off, L.dkv_off, lc.kv_from < 0 ? reinterpret_cast<const float *>(L.norm_w.ptr) : nullptr, sl, sp,
-                                        M.qf, lc.kv_from < 0 ? Rn.pool : nullptr, f32, d_page_table, max_pages, page_size, stream));
+      const float *qsrc = in_src;  // the queries [T][q_ld]: columns L.q_off + h * (d + dr)
+      long long q_ld = N;
+      {
+        StackLatentPrep a;
+        a.proj = in_src; a.ld = N; a.n_part = in_parts; a.stride = in_stride; a.n_cols = L.n_in; a.freq = L.freq;
+        a.q_off = L.q_off; a.dkv_off = L.dkv_off;
+        if (lc.kv_from < 0) { a.dkv_norm = reinterpret_cast<const float *>(L.norm_w.ptr); a.pool = Rn.pool; }
+        if (lc.q_rank > 0) { a.dq_off = 0; a.dq_norm = reinterpret_cast<const float *>(L.q_norm.ptr); a.cq = M.cq; }
+        else a.qf = M.qf;
+        if (in_parts > 1) {  // sliced projection: the columns that later kernels read go to M.proj
+          a.keep = M.proj; a.ld_keep = N;
+          if (lc.q_rank > 0) { a.keep = gated ? M.proj + L.g_off : nullptr; a.keep_off = L.g_off; a.keep_n = L.n_in - L.g_off; }
+          else { a.keep_off = 0; a.keep_n = L.n_in; }
+          qsrc = M.proj;
+        }
+        RET_CUDA(launch_stack_latent_prep(a, sl, sp, f32, d_page_table, max_pages, page_size, stream));
+      }
+      if (lc.q_rank > 0) {  // queries from their latent, then their rotation
+        RET_CUDA(gemm(M.cq, f32, lc.q_rank, L.w_uq, 0, nullptr, M.ql, T, H * (d + dr), lc.q_rank, cap_tokens));
+        qsrc = M.ql; q_ld = (long long)H * (d + dr);
+        StackLatentPrep a;
+        a.proj = M.ql; a.ld = q_ld; a.n_cols = H * (d + dr); a.freq = L.freq; a.qf = M.qf;
+        RET_CUDA(launch_stack_latent_prep(a, sl, sp, f32, d_page_table, max_pages, page_size, stream));
+        kl++;
+      }
       // absorbed queries: qf[t][h][0..r) = sum_a q[t][h][a] * uk[h*d + a][.]  (one batch entry per head).  Large bf16 passes:
       // one tensor-core product per head over the head's queries packed contiguously; else the batched fp32-FMA product.
       const bool head_tc = M.lat_gemm && T >= 256 && !L.ukT.f32 && !L.uv.f32 && d % 8 == 0 && ((size_t)r * d * 2) % 16 == 0 &&
                            ((size_t)dv * r * 2) % 16 == 0 && ((size_t)T * d * 2) % 16 == 0 && ((size_t)T * r * 2) % 16 == 0;
       if (head_tc) {
-        RET_CUDA(launch_stack_heads_pack(M.proj, N, L.q_off, d + dr, d, T, H, M.lat_qb, stream));
+        RET_CUDA(launch_stack_heads_pack(qsrc, q_ld, L.q_off, d + dr, d, T, H, M.lat_qb, stream));
         for (int h = 0; h < H; h++) {
           TmaMap xm;
           RET_CUDA(make_tma_map_2d(&xm, M.lat_qb + (size_t)h * T * d, (uint64_t)T, (uint64_t)d, (uint32_t)gemm_token_tile(T)));
@@ -1351,36 +1519,37 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         kl += H + 1;
       } else {
         StackGemm g;
-        g.A = M.proj + L.q_off; g.a_f32 = true; g.lda = N; g.a_bs = d + dr;
+        g.A = qsrc + L.q_off; g.a_f32 = true; g.lda = q_ld; g.a_bs = d + dr;
         g.W = L.ukT.ptr; g.w_f32 = L.ukT.f32; g.ldw = d; g.w_bs = (long long)r * d;
         g.out = M.qf; g.ldo = (long long)H * D; g.o_bs = D;
         g.M = T; g.N = r; g.K = d; g.batch = H;
         RET_CUDA(launch_stack_gemm(g, stream));
       }
       RET_CUDA(launch_stack_latent_attn(M.qf, KV.pool, f32, reinterpret_cast<const float *>(L.sink.ptr), sl, sp, mt.d<int>(mt.o_ab_tok0),
-                                        mt.d<int>(mt.o_ab_len), n_qb, d_page_table, max_pages, page_size, M.mix, lat_split, lat_keys,
+                                        mt.d<int>(mt.o_ab_len), n_qb, d_page_table, max_pages, page_size, M.mix, slices.first, slices.second,
                                         M.lat_part, stream));
-      if (lat_split > 1) kl++;
+      if (slices.first > 1) kl++;
       bool any_products = false;
       for (auto &sh : stack_spans_h) any_products = any_products || sh.products;
       if (any_products) {
         RET_CUDA(launch_stack_copy_act(M.qf, M.lat_qb, false, (long long)T * H * D, stream)); kl++;
         for (auto &sh : stack_spans_h) {
           if (!sh.products) continue;
-          const int ctx = sh.pos0 + sh.len, ctx8 = (ctx + 7) / 8 * 8;
+          const int first = stack_latent_row_lo(sl, sh.pos0) / 8 * 8;  // with a window: the first key any of the span's tokens sees, rounded down
+          const int pos0 = sh.pos0 - first, ctx = pos0 + sh.len, ctx8 = (ctx + 7) / 8 * 8;  // positions from there on
           RET_CUDA(launch_stack_latent_gather(KV.pool, d_page_table + (size_t)sh.slot * max_pages, page_size, D, r, ctx, ctx8, M.lat_cg,
-                                              M.lat_cgt, stream));
+                                              M.lat_cgt, first, stream));
           kl++;
           const int max_nq = (int)std::min<size_t>(M.lat_s_elems / ((size_t)H * ctx8), 4096);
           for (int j = 0; j < sh.len; j += max_nq) {
             const int nq = std::min(max_nq, sh.len - j), rows = nq * H;
-            const int nkeys = (sh.pos0 + j + nq + 7) / 8 * 8;  // keys the block's last query sees, rounded up (the rest are masked)
+            const int nkeys = (pos0 + j + nq + 7) / 8 * 8;  // keys the block's last query sees, rounded up (the rest are masked)
             TmaMap qm, cm, pm, ctm;
             RET_CUDA(make_tma_map_2d(&qm, M.lat_qb + (size_t)(sh.tok0 + j) * H * D, (uint64_t)rows, (uint64_t)D, (uint32_t)gemm_token_tile(rows)));
             RET_CUDA(make_tma_map_2d(&cm, M.lat_cg, (uint64_t)nkeys, (uint64_t)D, 128));
             RET_CUDA(launch_gemm_partial(cm, qm, M.lat_s, rows, nkeys, D, 0, 1, stream));
-            RET_CUDA(launch_stack_latent_softmax(M.lat_s, rows, nkeys, reinterpret_cast<const float *>(L.sink.ptr), H, sh.pos0 + j, sl.scale,
-                                                 M.lat_p, stream));
+            RET_CUDA(launch_stack_latent_softmax(M.lat_s, rows, nkeys, reinterpret_cast<const float *>(L.sink.ptr), H, pos0 + j, sl.scale,
+                                                 M.lat_p, sl.window, stream));
             RET_CUDA(make_tma_map_2d(&pm, M.lat_p, (uint64_t)rows, (uint64_t)nkeys, (uint32_t)gemm_token_tile(rows)));
             RET_CUDA(make_tma_map_2d(&ctm, M.lat_cgt, (uint64_t)r, (uint64_t)ctx8, 128));
             RET_CUDA(launch_gemm_partial(ctm, pm, M.mix + (size_t)(sh.tok0 + j) * H * r, rows, r, nkeys, 0, 1, stream));
@@ -1398,7 +1567,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
           if (!wm) return cudaErrorInvalidValue;
           RET_CUDA(launch_gemm_partial(*wm, xm, M.mix2 + (size_t)h * T * dv, T, dv, r, 0, 1, stream));
         }
-        RET_CUDA(launch_stack_gate(M.mix2, M.proj + L.g_off, N, M.act, f32, T, H * dv, H, stream));
+        RET_CUDA(launch_stack_gate(M.mix2, gate, N, M.act, f32, T, H * dv, H, stream, L.ld_act));
         kl += H;
       } else {
         StackGemm v;
@@ -1407,14 +1576,14 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         v.out = M.mix2; v.ldo = (long long)H * dv; v.o_bs = dv;
         v.M = T; v.N = dv; v.K = r; v.batch = H;
         RET_CUDA(launch_stack_gemm(v, stream));
-        RET_CUDA(launch_stack_gate(M.mix2, M.proj + L.g_off, N, M.act, f32, T, H * dv, 0, stream));
+        RET_CUDA(launch_stack_gate(M.mix2, gate, N, M.act, f32, T, H * dv, 0, stream, L.ld_act));
       }
       kl += 5;
-      n_mix = H * dv;
+      n_mix = L.ld_act;
     }
     RET_CUDA(gemm(M.act, f32, n_mix, L.w_o, 0, o_bias, M.y, T, W, n_mix, cap_tokens, nullptr, later));
     pend_y = M.y; pend_post = norm_w(L, 1); pend_post_b = norm_b(L, 1); pend_hc = reinterpret_cast<const float *>(L.hc[0].ptr);
-    if (lc.mlp == DIS_MLP_NONE) continue;
+    if (lc.mlp == DIS_MLP_NONE || par_ff > 0) continue;  // (a parallel layer's feed-forward is in the product above)
     next_hc = reinterpret_cast<const float *>(L.hc[1].ptr);
     RET_CUDA(sublayer_in(norm_w(L, 2), norm_b(L, 2), L.canon2, Rn.cstate2));
     if (lc.mlp == DIS_MLP_DENSE) {

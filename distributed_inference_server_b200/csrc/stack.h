@@ -57,7 +57,7 @@ cudaError_t launch_stack_embed(const void *embed, bool f32, const uint32_t *toke
 // u = sum_s next[s] x_s (null: x_0) is RMS-normed with the gain vector pre_w into hc (pre_w null: only the streams move on).
 cudaError_t launch_stack_boundary_hc(float *xs, int streams, const float *y, int n_part, long long stride, const float *bias,
                                      const float *prev, const float *next, const float *pre_w, void *hc, bool f32, int T, int W, float eps,
-                                     cudaStream_t st);
+                                     float mult, cudaStream_t st);  // mult: factor on y
 // x += unit_rms(y) * post (when y), then hn = unit_rms(x) * pre (when hn).  post / pre: device scalars.
 cudaError_t launch_stack_resid_norm(float *x, const float *y, const float *post, const float *pre, float *hn, int T, int W,
                                     float eps, cudaStream_t st);
@@ -104,6 +104,15 @@ size_t stack_lightning_seg_decay_floats(int cap_tokens, int max_spans, int H, in
 cudaError_t launch_stack_gla(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *dec, float *state,
                              const StackSpans &sp, float *o, int H, int d, int dv, float *seg, float *seg_a, int max_len,
                              cudaStream_t st);
+// Retention (DIS_MIX_RETENTION): rotation of q and k and the factor kscale on k, one block per token.  src: the token's row of n_cols
+// columns as n_part slices (one slice: it may be dst itself); every column lands in dst.  freq [rot_dims/2].
+cudaError_t launch_stack_retention_prep(const float *src, long long ld_src, int n_part, long long stride, int n_cols, float *dst,
+                                        long long ld_dst, int q_off, int k_off, int H, int d, const double *freq, int rot_dims, float kscale,
+                                        const StackSpans &sp, cudaStream_t st);
+// S = decay S + k v^T, o = S^T q over rows of proj as prepared; decay [H * stack_retention_blocks()], each head's value repeated per block
+int stack_retention_blocks(int d, int dv);
+cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *decay, float *state,
+                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, cudaStream_t st);
 // State-space mixer (DIS_MIX_SSM), three steps around the recurrence kernel of gated linear attention.
 // 1. proj [T][ld] holds z | x | B | C | dt as projected.  The C = inner + 2 G N channels from x_off on pass a causal depthwise
 //    convolution over time (cw [C][taps], last tap = the current token; the taps - 1 inputs before a span come from cstate
@@ -122,7 +131,7 @@ cudaError_t launch_stack_ssd(const float *buf, long long ld_b, int c_off, int b_
 //    the compute type.  x: buf column 0 on (row stride ld_b), z: proj column 0 on (row stride ld).
 cudaError_t launch_stack_ssm_out(const float *o, const float *buf, long long ld_b, const float *z, long long ld, const float *D,
                                  const float *w, int parts, void *out, bool f32, int T, int H, int P, float eps, cudaStream_t st);
-// out[t][off + h*dv + j] = scale * unit_rms_over_head(o[t][h])[j] * w[j] * silu(gate[t][h*dv + j]); out [T][ldo] compute type
+// out[t][off + h*dv + j] = scale * unit_rms_over_head(o[t][h])[j] * w[j] * silu(gate[t][h*dv + j]); out [T][ldo] compute type; w null: ones
 cudaError_t launch_stack_headnorm_silu(const float *o, const float *w, const float *gate, long long ldg, void *out, long long ldo,
                                        int off, float scale, bool f32, int T, int H, int dv, float eps, cudaStream_t st);
 // Attention over paged keys and values (k_stack_attn.cu).
@@ -133,7 +142,10 @@ struct StackAttn {
   int chunk;       // > 0: position i sees only keys from floor(i / chunk) * chunk on
   int window = 0;  // > 0: position i sees only the keys j with i - j < window
   float softcap = 0.f;  // > 0: score <- softcap * tanh(score / softcap), after the factor `scale` (softmax weights only)
+  int keep = 0;    // keys below it stay visible to every later position
 };
+// DIS_ATTN_DISTANCE: 2^(-8 (h + 1) / H)
+__host__ __device__ inline float stack_attn_slope(int h, int H) { return exp2f(-8.f * (float)(h + 1) / (float)H); }
 // first key position the query at position `pos` may see (both masks are monotone in pos, so a block of consecutive queries
 // starts its walk at the bound of its first token)
 __host__ __device__ inline int stack_attn_row_lo(const StackAttn &c, int pos) {
@@ -147,20 +159,26 @@ __host__ __device__ inline int stack_attn_row_lo(const StackAttn &c, int pos) {
 // unrotated keys; rotated by pos * vfreq[m] over pairs m, m + dv/2 with DIS_ATTN_ROT_V) to the token's row of the pools
 // ([pages*page_size][G*d] and [..][G*dv]); vrot [T][dv] receives cos | sin of the value angles for the output's rotation back.
 // kpool == null: the layer reads another layer's cache -- only the queries are prepared.
+// mix: value mixing (DIS_ATTN_V_MIX).
 // n_part > 1: proj holds split-K slices (slice stride `stride`) of n_cols columns, summed here with the bias.  gate_out (or
-// null): [T][ld_gate] receives columns gate_off .. + H of every row (the logits of the output gates).
+// null): [T][ld_gate] receives columns gate_off .. of every row, H or H*dv of them (the logits of the output gates).
+struct StackVMix {
+  float *save = nullptr;         // [T][G*dv] fp32: the layer is the first of its kind and leaves its values here
+  const float *first = nullptr;  // [T][G*dv]: v <- (1 - lam[0]) v + lam[0] first
+  const float *lam = nullptr;
+};
 cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, long long stride, int n_cols, int gate_off, float *gate_out,
                                    long long ld_gate, int q_off, int k_off, int v_off, const float *bias, const float *qn,
                                    const float *kn, const double *freq, const double *vfreq, const StackAttn &c, const StackSpans &sp,
                                    float *qf, void *kpool, void *vpool, float *vrot, bool f32, const int *page_table, int max_pages,
-                                   int page_size, cudaStream_t st);
+                                   int page_size, const StackVMix &mix, cudaStream_t st);
 // query blocks hold at most stack_attn_block_tokens() tokens of one span (bq: the most tokens a block of this pass holds); n_split > 1: slices of keys_per_split keys (a multiple
 // of 32), records of dv + 2 floats per (slice, token, head) in `part`, merged by a second kernel.  The result, times out_scale
 // and rotated back when values were rotated, lands in out [T][ld_out] (compute type) at columns out_off + h * dv.
 // bf16 with dim % 8 == 0, vdim % 16 == 0, both <= 128 and at most 64 query heads per key/value head: the mma.sync kernel (blocks
 // of 64 (token, head) rows); otherwise the fp32-arithmetic kernel.
 // sink [H] (DIS_ATTN_SINK): per-head logit in the softmax denominator.  gate [T][ld_gate] (DIS_ATTN_GATE): head h's output is
-// multiplied by sigmoid(gate[t][h]).  With c.chunk > 0 a block's history starts at the chunk of its first token, and the slices
+// multiplied by sigmoid(gate[t][h]); with DIS_ATTN_GATE_FULL its coordinate j by sigmoid(gate[t][h*dv + j]).  With c.chunk > 0 a block's history starts at the chunk of its first token, and the slices
 // are counted from there.
 int stack_attn_block_tokens(const StackAttn &c, bool f32);
 cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vpool, bool f32, const float *temp, const float *pb,
@@ -171,9 +189,9 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
 // out = unit_rms(o) * w * sigmoid(gate) per token over n = H*dv coordinates; gate [T][ldg]
 cudaError_t launch_stack_norm_gate(const float *o, const float *w, const float *gate, long long ldg, void *out, bool f32, int T,
                                    int n, float eps, cudaStream_t st);
-// out = o * sigmoid(gate); heads > 0: o is [heads][T][n / heads] instead of [T][n]
+// out = o * sigmoid(gate) (gate null: o), rows of out ldo apart (0: n); heads > 0: o is [heads][T][n / heads] instead of [T][n]
 cudaError_t launch_stack_gate(const float *o, const float *gate, long long ldg, void *out, bool f32, int T, int n, int heads,
-                              cudaStream_t st);
+                              cudaStream_t st, long long ldo = 0);
 // head h of src [T][ld] (columns off + h * hs .. + wd) -> dst bf16 [H][T][wd], and fp32 [H][T][wd] back into such columns
 cudaError_t launch_stack_heads_pack(const float *src, long long ld, int off, int hs, int wd, int T, int H, uint16_t *dst, cudaStream_t st);
 cudaError_t launch_stack_heads_unpack(const float *src, int wd, int T, int H, float *dst, long long ld, int off, int hs, cudaStream_t st);
@@ -186,18 +204,40 @@ cudaError_t launch_stack_mingru(const float *proj, long long ld, const float *bi
 // the normed latent and the rotated shared key part go to the token's row of the page pool ([pages*page_size][r+dr]).
 struct StackLatent {
   int H, d, dr, dv, r, rot_dims;
-  float rot_base, scale, eps;
+  float scale, eps;
+  int window = 0;     // > 0: position i sees only the keys j with i - j < window
+  int rot_pairs = 0;  // rotation turns coordinates 2i, 2i + 1 together instead of i, i + rot_dims/2
+  int q_rank = 0;     // size of the query latent (0: queries come from the input projection)
 };
-cudaError_t launch_stack_latent_prep(const float *proj, long long ld, int q_off, int dkv_off, const float *dkv_norm,
-                                     const StackLatent &c, const StackSpans &sp, float *qf, void *pool, bool f32,
-                                     const int *page_table, int max_pages, int page_size, cudaStream_t st);
-// step 2: scores of qf against the pool rows of the sequence (causal, softmax with a per-head sink in the denominator),
+__host__ __device__ inline int stack_latent_row_lo(const StackLatent &c, int pos) {
+  return c.window > 0 && pos - c.window + 1 > 0 ? pos - c.window + 1 : 0;
+}
+struct StackLatentPrep {
+  const float *proj = nullptr;  // [T][ld], or n_part slices of n_cols columns, `stride` apart
+  long long ld = 0, stride = 0;
+  int n_part = 1, n_cols = 0;
+  int q_off = 0;                // queries [H][d + dr]: their rotated parts go to qf (when given)
+  float *qf = nullptr;
+  int dkv_off = 0;              // latent and rotated key part: to the pool (when given)
+  const float *dkv_norm = nullptr;
+  void *pool = nullptr;
+  int dq_off = 0;               // query latent, RMS-normed with dq_norm: to cq [T][q_rank] in the compute type (when given)
+  const float *dq_norm = nullptr;
+  void *cq = nullptr;
+  float *keep = nullptr;        // receives columns keep_off .. + keep_n of the summed row (when given)
+  long long ld_keep = 0;
+  int keep_off = 0, keep_n = 0;
+  const double *freq = nullptr; // [rot_dims/2]
+};
+cudaError_t launch_stack_latent_prep(const StackLatentPrep &a, const StackLatent &c, const StackSpans &sp, bool f32, const int *page_table,
+                                     int max_pages, int page_size, cudaStream_t st);
+// step 2: scores of qf against the pool rows of the sequence (causal, softmax; sink or null: a per-head sink in the denominator),
 // output the weighted sum of the latents: ol [T][H][r] fp32.  qb_tok0 / qb_len: query blocks (tokens of one span).
 // n_split > 1: the history is cut into slices of keys_per_split keys (a multiple of 32), one CTA per (block, slice), whose
 // records ([n_split][T*H][r+2] floats in `part`) a second kernel merges -- few query blocks then still fill the GPU.
 int stack_latent_block_tokens(const StackLatent &c);
-// the mma.sync form of the kernel applies (bf16, kv_rank % 8 == 0, (kv_rank + rot_dim) % 16 == 0, heads <= 16): query blocks
-// then hold at most 16 (token, head) pairs
+// the mma.sync form of the kernel applies (bf16, kv_rank % 8 == 0, (kv_rank + rot_dim) % 16 == 0, kv_rank <= 1024): query blocks
+// then hold at most 16 (token, head) pairs, or one token when there are more heads
 bool stack_latent_mma_ok(const StackLatent &c, bool f32);
 cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32, const float *sink, const StackLatent &c,
                                      const StackSpans &sp, const int *qb_tok0, const int *qb_len, int n_qb,
@@ -206,15 +246,15 @@ cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32
 // Long prompt portions in bf16: latents of one sequence out of their pages into cg [ctx8][D] and cgt [r][ctx8] (rows / columns
 // from ctx to ctx8 zero), and softmax weights (bf16) from a block of raw score rows; the products between run on tcgen05.
 cudaError_t launch_stack_latent_gather(const void *pool, const int *pt_row, int page_size, int D, int r, int ctx, int ctx8,
-                                       uint16_t *cg, uint16_t *cgt, cudaStream_t st);
+                                       uint16_t *cg, uint16_t *cgt, int first, cudaStream_t st);  // first: position of row 0
 cudaError_t launch_stack_latent_softmax(const float *S, int rows, int ld, const float *sink, int H, int pos_first, float scale,
-                                        uint16_t *P, cudaStream_t st);
+                                        uint16_t *P, int window, cudaStream_t st);
 // kind DIS_ACT_CLAMPED: act = g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit);
 // DIS_ACT_GELU_TANH: act = gelu_tanh(g) u; DIS_ACT_SILU: act = g sigmoid(g) u.  gu [M][2*ff] (gate | up)
 // gu may come as n_part split-K slices (slice stride `stride`), summed here; bias (or null): [2*ff], added here when the product
-// that made gu left it out
+// that made gu left it out.  ld_gu / ld_act: row strides (0: contiguous rows)
 cudaError_t launch_stack_glu(const float *gu, int n_part, long long stride, const float *bias, void *act, bool f32, const int *rows_ptr,
-                             int M, int ff, float limit, int kind, cudaStream_t st);
+                             int M, int ff, float limit, int kind, cudaStream_t st, long long ld_gu = 0, long long ld_act = 0);
 // Router: logits in fp32 from hc and the fp32 router matrix; `top` experts by value (lowest index wins a tie).
 // kind DIS_ROUTE_SOFTMAX_TOP: by logit, weights = softmax over the chosen.  DIS_ROUTE_SIGMOID_GROUPS: by c = sigmoid(logit) +
 // correction[e], restricted to the `keep` best of `groups` contiguous runs of experts (a run ranks by the sum of its top two c;
@@ -270,7 +310,12 @@ struct StackLayer {
   StackTensor temp_pb;   // [2H] fp32: per-head factor on the score, then per-head bias under the sigmoid
   StackTensor b_o;       // [W] fp32: bias of the output projection
   double *freq = nullptr, *vfreq = nullptr;  // device: rotary frequencies [rot_dims/2] (scaled) and value frequencies [vdim/2]
-  int n_act = 0;         // columns of the output projection's input: H*vdim (+ gla_heads*gla_vdim behind them)
+  int n_act = 0;         // columns the mixer adds to the output projection's input: H*vdim (+ gla_heads*gla_vdim behind them)
+  int par_ff = 0;        // parallel frame: hidden size of the feed-forward whose rows and columns follow the mixer's (0: none)
+  int n_rows = 0;        // rows of w_in: n_in, then the parallel feed-forward's gate | up
+  int ld_act = 0;        // columns of w_o: n_act, then the parallel feed-forward's par_ff
+  StackTensor vmix;      // attention with DIS_ATTN_V_MIX: the scalar weight of the first layer's values
+  StackTensor w_uq, q_norm;  // latent with a query latent: [H*(d+dr)][q_rank] compute type, gain of its norm [q_rank] fp32
   // gated linear attention (second half of a parallel mixer): w_in rows q | k | v | g | bottleneck behind the attention's
   int gq_off = 0, gk_off = 0, gv_off = 0, gg_off = 0, ga_off = 0;
   StackTensor a2, a2_b, gla_norm;  // [Hd][rank] compute type, [Hd] fp32, [gla_vdim] fp32
@@ -315,6 +360,10 @@ struct StackModel {
   float *x0 = nullptr;             // the scaled embedding rows of the pass (input of every loop pass)
   void *xcat = nullptr;            // [x ; x0] in the compute type
   float *dec = nullptr;            // gated linear attention: the decays of the pass [T][H*d]
+  void *cq = nullptr;              // latent attention: the normed query latents of the pass [T][q_rank], compute type
+  float *ql = nullptr;             // and the queries made from them [T][H*(d+dr)]
+  int vmix_cols = 0;               // value mixing: kv_heads * vdim of the layers that take part (0: none)
+  float *vfirst = nullptr;         // and the first such layer's values of the pass [T][vmix_cols]
   float *vrot = nullptr;           // attention with rotated values: cos | sin of every token's value angles [T][vdim]
   float *attn_part = nullptr;      // attention: slice records
   size_t attn_part_elems = 0;

@@ -17,6 +17,14 @@ __device__ __forceinline__ void st_el(void *p, long long i, float v) {
 __device__ __forceinline__ float sigmoidf_(float v) { return 1.f / (1.f + __expf(-v)); }
 __device__ __forceinline__ float sigmoid_precise(float v) { return 1.f / (1.f + expf(-v)); }
 
+// sine and cosine of the rotary angle pos * f: formed and brought into [-pi, pi] in double (position 100000 is then as exact as
+// position 5), the functions of the reduced angle in float
+__device__ __forceinline__ void angle_sincos(int p, double f, float *sn_out, float *cs_out) {
+  const double a = (double)p * f;
+  const double r = a - 6.283185307179586476925 * rint(a * 0.15915494309189533577);
+  sincosf((float)r, sn_out, cs_out);
+}
+
 __device__ __forceinline__ float block_sum(float v, float *sh) {  // sh: 32 floats; every thread gets the total
   v = warp_sum(v);
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;

@@ -30,6 +30,13 @@ engine's description of the model and names every tensor.  Two families exist:
             tanh soft cap on the scores, a sliding window, and a softmax whose denominator carries one extra 1) and `mamba2`
             (selective state space with a short causal convolution, gated and group-normalised); feed-forward of ungated
             squared-ReLU units, dense or as a mixture chosen by a softmax router, with an optional always-on shared unit.
+  Nifulix   a layer-list decoder of the same engine whose layers are parallel: one RMS norm (its vector stored around zero) feeds
+            the mixer and a SiLU-gated feed-forward, and their sum, times a constant, joins the residual; mixers `retention`
+            (linear attention with a fixed per-head decay, rotated queries and keys, per-head output norm without a gain, SiLU
+            gate), `latent_attention` (queries through a latent of their own, neighbouring-pair rotation, sliding window, plain
+            softmax, no gate) and `attention` (grouped-query softmax attention without rotation: tanh soft cap and a per-head
+            distance term on the scores, a sliding window beside which the first positions stay visible, values blended with
+            those of the first such layer, an element-wise sigmoid output gate).
 
 The reference has no model loading at all (crates/inference/src/worker.rs:1 is empty).
 """
@@ -47,7 +54,7 @@ import numpy as np
 from . import binding as B
 
 _MIXERS = {"lightning": B.MIX_LIGHTNING, "mingru": B.MIX_MINGRU, "latent_attention": B.MIX_LATENT,
-           "attention": B.MIX_ATTENTION, "parallel": B.MIX_PARALLEL, "ssm": B.MIX_SSM}
+           "attention": B.MIX_ATTENTION, "parallel": B.MIX_PARALLEL, "ssm": B.MIX_SSM, "retention": B.MIX_RETENTION}
 _ACTS = {"clamped": B.ACT_CLAMPED, "gelu_tanh": B.ACT_GELU_TANH, "silu": B.ACT_SILU, "relu2": B.ACT_RELU2}
 _ROUTES = {"softmax_top": B.ROUTE_SOFTMAX_TOP, "sigmoid_groups": B.ROUTE_SIGMOID_GROUPS, "softmax_all": B.ROUTE_SOFTMAX_ALL}
 
@@ -98,6 +105,9 @@ class LayerSpec:
     conv_taps: int = 0
     ssm_norm_groups: int = 1
     shared_plain: bool = False  # the shared expert joins the sum without a gate
+    mask_keep: int = 0  # attention: first positions that stay visible beside the window
+    q_rank: int = 0  # latent attention: size of the query latent (0 = queries straight from the input)
+    latent_flags: int = 0
 
     @property
     def gated(self) -> bool:
@@ -113,7 +123,7 @@ class StackSpec:
     layers: List[LayerSpec]
     canon_taps: int = 0
     norm_eps: float = 1e-5
-    norm_kind: str = "rms_scalar"  # rms_scalar | layer | rms
+    norm_kind: str = "rms_scalar"  # rms_scalar | layer | rms | rms_one (gain vectors stored as their distance from one)
     embed_scale: float = 1.0
     logit_scale: float = 1.0
     loop: Tuple[int, int, int] = (0, 0, 0)  # start, stop, times (times 0 = no loop)
@@ -124,6 +134,8 @@ class StackSpec:
     pos_base: float = 10000.0
     loop_plain: bool = False  # the loop's passes follow each other without an input projection
     tied_head: bool = False  # logits from the embedding table: the file has no "head"
+    parallel: bool = False  # mixer and feed-forward read one norm and are added together; needs pre_norm
+    residual_mult: float = 1.0  # factor on what a layer adds to the residual; needs pre_norm
 
     def layer_runs(self) -> List[int]:
         """Layer index of every layer run of one forward pass, the looped stretch repeated."""
@@ -137,7 +149,7 @@ class StackSpec:
         W, out = self.width, {"embed": (self.vocab, self.width), "head": (self.vocab, self.width)}
         if self.tied_head:
             del out["head"]
-        vec = self.norm_kind in ("layer", "rms")
+        vec = self.norm_kind in ("layer", "rms", "rms_one")
         post = not self.pre_norm
 
         def norm(name):
@@ -157,7 +169,10 @@ class StackSpec:
                 out.update({f"{p}hc{q}.in": (self.streams,), f"{p}hc{q}.out": (self.streams,), f"{p}hc{q}.mix": (self.streams, self.streams)})
             if self.canon_taps >= 1:
                 out[p + "canon1"] = (W, self.canon_taps)
-            if L.mixer == "lightning":
+            if L.mixer == "retention":
+                out.update({p + "mix.q": (L.heads * L.dim, W), p + "mix.k": (L.heads * L.dim, W), p + "mix.v": (L.heads * L.vdim, W),
+                            p + "mix.g": (L.heads * L.vdim, W), p + "mix.o": (W, L.heads * L.vdim)})
+            elif L.mixer == "lightning":
                 out.update({p + "mix.q": (L.heads * L.dim, W), p + "mix.k": (L.heads * L.dim, W), p + "mix.v": (L.heads * L.vdim, W),
                             p + "mix.g": (L.heads * L.vdim, W), p + "mix.o": (W, L.heads * L.vdim), p + "mix.norm": (L.heads * L.vdim,)})
             elif L.mixer == "mingru":
@@ -192,6 +207,10 @@ class StackSpec:
                     out[a + "sink"] = (L.heads,)
                 if L.attn_flags & B.ATTN_GATE:
                     out[a + "g"] = (L.heads, W)
+                if L.attn_flags & B.ATTN_GATE_FULL:
+                    out[a + "g"] = (L.heads * L.vdim, W)
+                if L.attn_flags & B.ATTN_V_MIX:
+                    out[a + "vmix"] = ()
                 if L.attn_flags & B.ATTN_SIGMOID:
                     out.update({a + "temp": (L.heads,), a + "pb": (L.heads,)})
                 if L.mixer == "parallel":
@@ -199,15 +218,24 @@ class StackSpec:
                     out.update({r + "q": (n, W), r + "k": (n, W), r + "v": (nv, W), r + "g": (nv, W), r + "o": (W, nv),
                                 r + "norm": (L.gla_vdim,), r + "a1": (L.gla_rank, W), r + "a2": (n, L.gla_rank), r + "a2.b": (n,)})
             else:
-                out[p + "mix.q"] = (L.heads * (L.dim + L.rot_dim), W)
+                if L.q_rank > 0:
+                    out.update({p + "mix.dq": (L.q_rank, W), p + "mix.dq.norm": (L.q_rank,),
+                                p + "mix.uq": (L.heads * (L.dim + L.rot_dim), L.q_rank)})
+                else:
+                    out[p + "mix.q"] = (L.heads * (L.dim + L.rot_dim), W)
                 if L.kv_from < 0:
                     out[p + "mix.dkv"] = (L.kv_rank + L.rot_dim, W)
                     out[p + "mix.dkv.norm"] = (L.kv_rank,)
                 out.update({p + "mix.uk": (L.heads * L.dim, L.kv_rank), p + "mix.uv": (L.heads * L.vdim, L.kv_rank),
-                            p + "mix.sink": (L.heads,), p + "mix.g": (L.heads * L.vdim, W), p + "mix.o": (W, L.heads * L.vdim)})
+                            p + "mix.o": (W, L.heads * L.vdim)})
+                if not L.latent_flags & B.LATENT_NO_SINK:
+                    out[p + "mix.sink"] = (L.heads,)
+                if not L.latent_flags & B.LATENT_NO_GATE:
+                    out[p + "mix.g"] = (L.heads * L.vdim, W)
             if L.mlp == "none":
                 continue
-            norm(p + "norm2")
+            if not self.parallel:
+                norm(p + "norm2")
             if post:
                 norm(p + "norm2b")
             if self.canon_taps >= 1:
@@ -268,13 +296,15 @@ class StackSpec:
             c.mask_window, c.score_softcap = L.mask_window, L.score_softcap
             c.ssm_state, c.ssm_groups, c.conv_taps, c.ssm_norm_groups = L.ssm_state, L.ssm_groups, L.conv_taps, L.ssm_norm_groups
             c.mlp_flags = B.MLP_SHARED_PLAIN if L.shared_plain else 0
+            c.mask_keep, c.q_rank, c.latent_flags = L.mask_keep, L.q_rank, L.latent_flags
         sc = B.StackConfig(self.vocab, self.width, len(self.layers), self.canon_taps, max_ctx, max_logit_rows,
                            B.F32 if f32 else B.BF16, self.norm_eps, arr,
-                           {"rms_scalar": B.NORM_RMS_SCALAR, "layer": B.NORM_LAYER, "rms": B.NORM_RMS}[self.norm_kind],
+                           {"rms_scalar": B.NORM_RMS_SCALAR, "layer": B.NORM_LAYER, "rms": B.NORM_RMS, "rms_one": B.NORM_RMS_ONE}[self.norm_kind],
                            self.embed_scale, self.logit_scale, *self.loop, self.logit_softcap,
                            (B.FRAME_PRE_NORM if self.pre_norm else 0) | (B.FRAME_POS_SINUS if self.pos_sinus else 0) |
-                           (B.FRAME_LOOP_PLAIN if self.loop_plain else 0) | (B.FRAME_TIED_HEAD if self.tied_head else 0),
-                           self.streams, self.pos_base)
+                           (B.FRAME_LOOP_PLAIN if self.loop_plain else 0) | (B.FRAME_TIED_HEAD if self.tied_head else 0) |
+                           (B.FRAME_PARALLEL if self.parallel else 0),
+                           self.streams, self.pos_base, self.residual_mult)
         return sc, keep
 
 
@@ -467,6 +497,49 @@ def goperax_spec(cfg: dict) -> StackSpec:
                      streams=int(cfg.get("streams") or 0), pos_sinus=True, pos_base=10000.0, loop_plain=True, tied_head=True)
 
 
+def nifulix_spec(cfg: dict) -> StackSpec:
+    """Nifulix's config.json -> StackSpec: every size and constant from the file.  A part the file leaves out is off: no `mask` =
+    the whole past, no `keep_first` = none, no `softcap` = none, no `v_mix` = the layer's own values, no `rot` = no rotation, no
+    `q_rank` = queries straight from the input, `mlp` null = the mixer alone."""
+    layers = []
+    for i, ly in enumerate(cfg["layers"]):
+        kind, mx = ly["type"], ly["mixer"]
+        if kind not in ("retention", "latent_attention", "attention"):
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        L = LayerSpec(kind)
+        L.heads, L.dim, L.vdim = int(mx["heads"]), int(mx["dim"]), int(mx["vdim"])
+        rot, mask = mx.get("rot") or {}, mx.get("mask") or {}
+        if kind != "attention":
+            L.rot_dims, L.rot_base = int(rot.get("dims", 0)), float(rot.get("base", 10000.0))
+        if kind == "retention":
+            L.decay = [float(a) for a in mx["decay"]]
+            if len(L.decay) != L.heads:
+                raise ValueError(f"layer {i}: decay must list one value per head")
+            if L.rot_dims > L.dim or L.rot_dims % 2:
+                raise ValueError(f"layer {i}: rot.dims must be even and at most dim")
+        elif kind == "latent_attention":
+            L.kv_rank, L.rot_dim, L.q_rank = int(mx["kv_rank"]), int(mx["rot_dim"]), int(mx.get("q_rank") or 0)
+            if L.rot_dims > L.rot_dim or L.rot_dims % 2:
+                raise ValueError(f"layer {i}: rot.dims must be even and at most rot_dim")
+            L.scale, L.mask_window = float(mx["scale"]), int(mask.get("size") or 0)
+            L.latent_flags = B.LATENT_NO_SINK | B.LATENT_NO_GATE | B.LATENT_ROT_PAIRS
+        else:
+            L.kv_heads, L.scale = int(mx["kv_heads"]), float(mx["scale"])
+            if L.kv_heads < 1 or L.heads % L.kv_heads:
+                raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
+            L.mask_window, L.mask_keep = int(mask.get("size") or 0), int(mask.get("keep_first") or 0)
+            L.score_softcap = float(mx.get("softcap") or 0.0)
+            L.attn_flags = B.ATTN_GATE_FULL | B.ATTN_DISTANCE | (B.ATTN_V_MIX if mx.get("v_mix") else 0)
+        ml = ly.get("mlp")
+        if ml is not None:
+            if ml.get("kind") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {ml.get('kind')!r}")
+            L.mlp, L.ff, L.mlp_act = "dense", int(ml["ff"]), "silu"
+        layers.append(L)
+    return StackSpec("Nifulix", int(cfg["vocab"]), int(cfg["width"]), layers, 0, float((cfg.get("norm") or {}).get("eps", 1e-5)), "rms_one",
+                     pre_norm=True, parallel=True, residual_mult=float(cfg.get("residual_mult", 1.0)))
+
+
 def llama_shape(cfg: dict):
     """A Hugging Face style Llama config.json -> ModelShape."""
     from .worker import ModelShape
@@ -483,6 +556,7 @@ ARCHITECTURES: Dict[str, Tuple[str, Callable[..., object]]] = {
     "Motolix": ("stack", motolix_spec),
     "Fakonex": ("stack", fakonex_spec),
     "Goperax": ("stack", goperax_spec),
+    "Nifulix": ("stack", nifulix_spec),
     "LlamaForCausalLM": ("llama", llama_shape),
     "llama": ("llama", llama_shape),
 }
@@ -605,7 +679,9 @@ def random_tensors(spec: StackSpec, seed: int = 0, scale: float = 1.0) -> Dict[s
     for name, shape in spec.tensor_shapes().items():
         leaf = name.rsplit(".", 1)[-1]
         if shape == ():
-            a = np.asarray(rng.uniform(0.5, 1.5), np.float32)
+            a = np.asarray(rng.uniform(0.2, 0.8) if leaf == "vmix" else rng.uniform(0.5, 1.5), np.float32)
+        elif spec.norm_kind == "rms_one" and (leaf == "norm1" or name == "final.norm"):
+            a = rng.normal(0.0, 0.2, shape).astype(np.float32)
         elif leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm" or name.endswith(("q.norm", "k.norm")):
             a = rng.uniform(0.5, 1.5, shape).astype(np.float32)
         elif leaf == "temp":

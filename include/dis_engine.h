@@ -430,12 +430,15 @@ typedef enum dis_mixer_kind {
                             is chosen by attn_flags */
   DIS_MIX_PARALLEL = 4,  /* two mixers read the same input: DIS_MIX_ATTENTION (the fields above) and gated linear attention
                             (the gla_* fields); their outputs are added with the weights mix_scale / gla_scale */
-  DIS_MIX_SSM = 5        /* selective state-space mixer (state-space duality form): one projection "in" gives z | x | B | C | dt;
+  DIS_MIX_SSM = 5,       /* selective state-space mixer (state-space duality form): one projection "in" gives z | x | B | C | dt;
                             x, B, C pass a causal depthwise convolution ("conv" [channels][conv_taps], last tap = current token, bias
                             "conv.b") and SiLU; dt = softplus(dt + "dt_bias"); per head (heads, value size vdim, state size ssm_state; head
                             h reads B, C of group h / (heads / ssm_groups)) S = exp(-exp("A_log"[h]) dt) S + dt B x^T, y = S^T C + "D"[h] x;
                             y silu(z) is RMS-normed in ssm_norm_groups equal parts, times "norm", then projected by "o".  Sequence state:
                             S (fp32) and the convolution's last conv_taps - 1 inputs */
+  DIS_MIX_RETENTION = 6  /* linear attention, fixed decay per head, no activation: q and k are rotated (rot_dims, rot_base: coordinate i turns
+                            with i + rot_dims/2), k is then multiplied by dim^(-1/2); S = decay S + k v^T, o = S^T q; each head's o is
+                            divided by its root mean square (no gain), multiplied by silu("g" u) and projected */
 } dis_mixer_kind;
 typedef enum dis_mlp_kind { DIS_MLP_NONE = 0, DIS_MLP_DENSE = 1, DIS_MLP_MOE = 2 } dis_mlp_kind;
 /* Feed-forward unit.  CLAMPED: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, +-limit), biases on every
@@ -444,7 +447,8 @@ typedef enum dis_mlp_act { DIS_ACT_CLAMPED = 0, DIS_ACT_GELU_TANH = 1, DIS_ACT_S
 /* RELU2 is an ungated unit: "down" (relu("up" h))^2 -- there is no "gate" matrix, in dense layers, experts and shared experts alike. */
 /* Norms around the sublayers.  RMS_SCALAR: x / rms(x) times one scalar gain (tensor of shape []).  LAYER: (x - mean) / sqrt(var +
  * eps) * w + b with vectors w ("<name>") and b ("<name>.b").  RMS: x / rms(x) * w with a gain vector w ("<name>"), no bias. */
-typedef enum dis_norm_kind { DIS_NORM_RMS_SCALAR = 0, DIS_NORM_LAYER = 1, DIS_NORM_RMS = 2 } dis_norm_kind;
+/* RMS_ONE: the RMS form whose stored vector is the gain's distance from one, x / rms(x) * (1 + w). */
+typedef enum dis_norm_kind { DIS_NORM_RMS_SCALAR = 0, DIS_NORM_LAYER = 1, DIS_NORM_RMS = 2, DIS_NORM_RMS_ONE = 3 } dis_norm_kind;
 /* How a mixture of experts picks and weighs its experts from the fp32 router logits z.
  * SOFTMAX_TOP: the `top` largest z; weights = softmax over the chosen z.
  * SIGMOID_GROUPS: s = sigmoid(z) and c = s + "correction" (a vector per layer).  The expert indices are cut into route_groups
@@ -473,6 +477,15 @@ typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUP
                                    and "g" a [heads][width] matrix: a scalar gate per (token, head) */
 #define DIS_ATTN_SINK_UNIT 512u /* softmax only: one more term of logit 0 in the denominator, exp(score_j) / (1 + sum_j exp(score_j)); no
                                    tensor */
+#define DIS_ATTN_GATE_FULL 1024u /* out <- out * sigmoid("g" u) element by element, "g" a [heads * vdim][width] matrix (in place of DIS_ATTN_GATE) */
+#define DIS_ATTN_DISTANCE 2048u /* softmax only: score <- score - slope_h (i - j) after the soft cap, slope_h = 2^(-8 (h + 1) / heads) */
+#define DIS_ATTN_V_MIX  4096u /* values v <- (1 - l) v + l v', v' the values of the same token in the first such layer of the pass and l the
+                                   scalar tensor "vmix" (that first layer keeps its own values); the mixed values are cached.  All such
+                                   layers have the same kv_heads * vdim */
+/* dis_layer_config.latent_flags */
+#define DIS_LATENT_NO_SINK   1u /* no "sink": a plain softmax over the visible keys */
+#define DIS_LATENT_NO_GATE   2u /* no output gate: no "g" */
+#define DIS_LATENT_ROT_PAIRS 4u /* rotation turns coordinates 2i and 2i + 1 together instead of i and i + rot_dims/2 */
 /* dis_layer_config.mlp_flags */
 #define DIS_MLP_SHARED_PLAIN 1u /* the shared expert's output joins the experts' sum as it is: there is no "shared.sg" gate */
 /* dis_stack_config.frame_flags */
@@ -481,6 +494,8 @@ typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUP
                                    sin(p pos_base^(-2i/width)), entry 2i+1 = cos of the same angle, p the position in the sequence */
 #define DIS_FRAME_LOOP_PLAIN 4u /* passes of the loop follow each other directly: no "loop.in" / "loop.step" */
 #define DIS_FRAME_TIED_HEAD  8u /* the logits are products with the embedding table itself (without embed_scale): no "head" tensor */
+#define DIS_FRAME_PARALLEL  16u /* (with DIS_FRAME_PRE_NORM, one residual) a layer is x += residual_mult (mixer(h) + ff(h)) with the one norm
+                                   h = norm1(x): no "norm2".  Mixers attention, parallel, latent, retention; dense feed-forwards without biases */
 
 typedef struct dis_layer_config {
   int32_t mixer;                 /* dis_mixer_kind */
@@ -523,6 +538,10 @@ typedef struct dis_layer_config {
   int32_t conv_taps;             /* DIS_MIX_SSM: taps of the convolution over x | B | C (1 .. 16) */
   int32_t ssm_norm_groups;       /* DIS_MIX_SSM: equal parts of heads * vdim that are normalised separately (0 is read as 1) */
   uint32_t mlp_flags;            /* DIS_MLP_* */
+  int32_t mask_keep;             /* attention: positions j < mask_keep stay visible to every later position, whatever mask_chunk and
+                                    mask_window say; 0: none.  (mask_window applies to latent attention too, mask_chunk and mask_keep do not) */
+  int32_t q_rank;                /* latent: q > 0: queries go through a latent of this size, q = "uq" (rms_norm("dq" u) * "dq.norm"); 0: q = "q" u */
+  uint32_t latent_flags;         /* DIS_LATENT_* */
 } dis_layer_config;
 
 typedef struct dis_stack_config {
@@ -548,6 +567,7 @@ typedef struct dis_stack_config {
    * final norm reads the sum of the streams.  0: one residual, x += y. */
   int32_t streams;
   float pos_base;                /* DIS_FRAME_POS_SINUS: base of the position vector's frequencies (0 is read as 10000) */
+  float residual_mult;           /* pre-norm frame: factor on what a layer adds to the residual (0 is read as 1) */
 } dis_stack_config;
 
 /* cfg->model is ignored (model_info reports vocab, width, layers and max_ctx of the stack); tensor parallelism and the
