@@ -1148,6 +1148,111 @@ def run_goperax(args):
     return 0
 
 
+def run_nifulix(args):
+    """Prefill and decode throughput of Nifulix (parallel layers under one norm; retention, latent attention with a query latent
+    and a window, soft-capped attention with a distance term, a window with kept first positions, value mixing and an
+    element-wise gate; SiLU-gated units) next to the closest existing models at equal width, depth, vocabulary and head geometry:
+    Kidolorn's lightning and latent layers (the same recurrence and latent kernels), Goperax's windowed attention and Motolix's
+    attention (the same attention kernels; Motolix with a gated unit of the same size) and the Llama decoder; random weights, one
+    GPU: one pass over `batch` prompts of `prompt_len` tokens, then K decode steps of the batch, timed by the engine's CUDA events
+    around each pass (metadata upload and token read-back included).  Weights exceed L2 at every size."""
+    from distributed_inference_server_b200 import Engine, InferenceParams, ModelShape, WorkerConfig, models
+    from distributed_inference_server_b200.binding import FLAG_NO_GRAPH as B_FLAG_NO_GRAPH
+    sizes = {"w1024": (1024, 4096), "w2048": (2048, 8192)}
+    want = [k for k in (args.sizes.split(",") if args.sizes else sizes) if k in sizes]
+    batch, plen, vocab = args.batch or 8, args.prompt_len, 32000
+    rng = np.random.default_rng(0)
+    out = []
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.mark_start()
+    for key in want:
+        W, ff = sizes[key]
+        H = W // 128
+        G = max(1, H // 4)
+        window = max(64, plen // 2)
+        att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                                              "v_mix": True, "mask": {"size": window, "keep_first": 4}}}
+        ret = {"type": "retention", "mixer": {"heads": H, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128},
+                                              "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * h / max(1, H - 1)) for h in range(H)]}}
+        lat_sizes = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5}
+        lat = {"type": "latent_attention", "mixer": dict(lat_sizes, q_rank=768, mask={"size": window})}
+        dense = {"kind": "dense", "ff": ff}
+        kinds = {"attention": att, "retention": ret, "latent": lat}
+        variants = {"mixed": ["attention", "retention", "latent", "attention"]}
+        if args.per_mixer:
+            variants.update({k: [k] * 4 for k in kinds})
+        if args.variant:
+            variants = {k: v for k, v in variants.items() if k in args.variant.split(",")}
+        rec = {"size": key, "width": W, "layers": 4, "dense_ff": ff, "vocab": vocab, "batch": batch, "prompt_len": plen, "window": window}
+        prompts = [rng.integers(0, vocab, plen).tolist() for _ in range(batch)]
+        P = InferenceParams(max_tokens=1 << 20, temperature=0.0)
+        ctx = plen + args.steps + args.warmup + 64
+
+        def measure(eng):
+            slots = [eng.seq_add(p, P) for p in prompts]
+            t_pre = []
+            for it in range(1 + max(1, args.ttft_runs)):
+                if it:
+                    for sl in slots:
+                        eng.seq_remove(sl)
+                    slots = [eng.seq_add(p, P) for p in prompts]
+                eng.step(slots, batch * plen)
+                t_pre.append(eng.status().last_step_ms)
+            for _ in range(args.warmup):
+                eng.decode(slots)
+            k0 = eng.status().kernel_launches
+            ms = 0.0
+            for _ in range(args.steps):
+                eng.decode(slots)
+                ms += eng.status().last_step_ms
+            launches = eng.status().kernel_launches - k0
+            for sl in slots:
+                eng.seq_remove(sl)
+            eng.close()
+            pre = min(t_pre[1:])
+            return {"prefill_ms": round(pre, 3), "prefill_tokens_per_s": round(batch * plen / pre * 1e3, 1),
+                    "decode_ms_per_step": round(ms / args.steps, 4), "decode_tokens_per_s": round(batch * args.steps / ms * 1e3, 1),
+                    "launches_per_decode_step": launches // max(1, args.steps)}
+
+        def stack_engine(spec):
+            eng = Engine(WorkerConfig(None, max_batch=batch, max_step_tokens=batch * plen, page_size=64, kv_pages=(batch * ctx + 63) // 64,
+                                      stack=spec, context_size=ctx, compute_dtype="bfloat16", flags=B_FLAG_NO_GRAPH if args.no_graph else 0))
+            for name, a in models.random_tensors(spec, seed=1).items():
+                eng.load_named(name, a)
+            eng.finalize()
+            return eng
+
+        def cfg_of(arch, layers, **extra):
+            return dict({"architecture": arch, "vocab": vocab, "width": W, "norm": {"eps": 1e-5},
+                         "layers": [dict(json.loads(json.dumps(m)), mlp=json.loads(json.dumps(f))) for m, f in layers]}, **extra)
+        for vname, names in variants.items():
+            cfg = cfg_of("Nifulix", [(kinds[n], dense) for n in names], residual_mult=0.5)
+            rec["nifulix_" + vname] = measure(stack_engine(models.nifulix_spec(cfg)))
+        if not args.nifulix_only:
+            clamped = {"kind": "dense", "ff": ff, "limit": 7.0}
+            k_light = {"type": "lightning", "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": ret["mixer"]["decay"]}}
+            for nm, mx in (("kidolorn_lightning", k_light), ("kidolorn_latent", {"type": "latent_attention", "mixer": lat_sizes})):
+                rec[nm] = measure(stack_engine(models.kidolorn_spec(cfg_of("Kidolorn", [(mx, clamped)] * 4, canon={"taps": 4}))))
+            g_att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+                                                    "mask": {"size": window}}}
+            rec["goperax_attention"] = measure(stack_engine(models.goperax_spec(cfg_of("Goperax", [(g_att, dense)] * 4, embedding={"scale": float(W) ** 0.5}))))
+            m_att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 1000000.0, "dims": 64}}}
+            rec["motolix_attention"] = measure(stack_engine(models.motolix_spec(cfg_of("Motolix", [(m_att, dense)] * 4, embedding={"scale": float(W) ** 0.5}))))
+            shape = ModelShape(vocab, W, 4, H, G, 128, ff, ctx)
+            eng = Engine(WorkerConfig(shape, max_batch=batch, max_step_tokens=batch * plen, page_size=64, kv_pages=(batch * ctx + 63) // 64 + batch))
+            eng.load_synthetic(1)
+            eng.finalize()
+            rec["llama"] = measure(eng)
+        out.append(rec)
+    clocks.mark_end()
+    line = {"metric": "nifulix_vs_closest_models_equal_size", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "dtype": "bf16", "data": "synthetic (random weights, uniform random tokens)", "higher_is_better": True, "sizes": out,
+            "clocks": clocks.stop()}
+    print(json.dumps(line))
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1166,10 +1271,12 @@ def main():
     ap.add_argument("--nccl-allreduce", action="store_true", help="TP: use NCCL instead of the fused peer-memory exchange (A/B)")
     ap.add_argument("--tp-exchange", choices=["auto", "oneshot", "twoshot", "ll", "wide"], default="auto",
                     help="TP: peer-memory exchange kernel (auto = ll, the flag-in-data row kernel, up to hidden 4096; wide, the same protocol on a (row, column block) grid, above)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "prefix", "kidolorn", "motolix", "fakonex", "goperax"], help="serving = BASELINE configs[4]; prefix = TTFT with prefix KV reuse (row f2); kidolorn / motolix / fakonex / goperax = that layer-list design beside Llama (and its closest layer-list relatives) at equal size")
-    ap.add_argument("--sizes", default="", help="kidolorn, motolix, fakonex, goperax: comma list out of w1024,w2048 (default both)")
-    ap.add_argument("--per-mixer", action="store_true", help="kidolorn, motolix, fakonex, goperax: also four layers of each mixer (fakonex: of each cache / mask arrangement) alone")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "prefix", "kidolorn", "motolix", "fakonex", "goperax", "nifulix"], help="serving = BASELINE configs[4]; prefix = TTFT with prefix KV reuse (row f2); kidolorn / motolix / fakonex / goperax / nifulix = that layer-list design beside Llama (and its closest layer-list relatives) at equal size")
+    ap.add_argument("--sizes", default="", help="kidolorn, motolix, fakonex, goperax, nifulix: comma list out of w1024,w2048 (default both)")
+    ap.add_argument("--per-mixer", action="store_true", help="kidolorn, motolix, fakonex, goperax, nifulix: also four layers of each mixer (fakonex: of each cache / mask arrangement) alone")
     ap.add_argument("--goperax-only", action="store_true", help="goperax: skip the other models' rows (profiling under ncu)")
+    ap.add_argument("--nifulix-only", action="store_true", help="nifulix: skip the other models' rows (profiling under ncu)")
+    ap.add_argument("--variant", default="", help="nifulix: comma list out of mixed,attention,retention,latent (default all that are asked for)")
     ap.add_argument("--model", default="8b", choices=["8b", "70b"], help="70b = BASELINE configs[3] (TP=8, batch 32)")
     ap.add_argument("--requests", type=int, default=256)
     ap.add_argument("--prefill-budget", type=int, default=0, help="serving: prompt tokens read per scheduler step (0 = library default)")
@@ -1195,6 +1302,8 @@ def main():
         return run_fakonex(args)
     if args.workload == "goperax":
         return run_goperax(args)
+    if args.workload == "nifulix":
+        return run_nifulix(args)
     return run_ours(args)
 
 

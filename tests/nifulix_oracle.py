@@ -70,8 +70,8 @@ def distance_slope(h, heads):
 
 
 def score(q, k, scale, cap, slope, dist):
-    """Scaled product, squeezed by the cap, then lowered in proportion to the distance."""
-    s = float(q @ k) * scale
+    """Scaled product, squeezed by the cap, then lowered in proportion to the distance.  k: one key or a row per key."""
+    s = k @ q * scale
     if cap:
         s = cap * np.tanh(s / cap)
     return s - slope * dist
@@ -89,18 +89,19 @@ def attention(mx, P, p, h, shared):
     window, keep, cap = int(mask.get("size", 0)), int(mask.get("keep_first", 0)), float(mx.get("softcap") or 0.0)
     q = (h @ P[p + "q"].T).reshape(T, H, d)
     k = (h @ P[p + "k"].T).reshape(T, G, d)
-    v = (h @ P[p + "v"].T).reshape(T, G, dv)
+    v = h @ P[p + "v"].T
     if mx.get("v_mix"):
         if "first" in shared:
             v = mixed_values(v, shared["first"], float(P[p + "vmix"]))
         else:
             shared["first"] = v
+    v = v.reshape(T, G, dv)
     out = np.zeros((T, H, dv))
     for i in range(T):
         seen = [j for j in range(i + 1) if in_window(i, j, window, keep)]
         for hd in range(H):
             g = hd // (H // G)
-            wts = softmax([score(q[i, hd], k[j, g], mx["scale"], cap, distance_slope(hd, H), i - j) for j in seen])
+            wts = softmax(score(q[i, hd], k[seen, g], mx["scale"], cap, distance_slope(hd, H), i - np.array(seen)))
             out[i, hd] = wts @ v[seen, g]
     return (out.reshape(T, -1) * sigmoid(h @ P[p + "g"].T)) @ P[p + "o"].T
 
@@ -135,8 +136,11 @@ def latent_attention(mx, P, p, h, eps):
     H, d, dr, dv, r = mx["heads"], mx["dim"], mx["rot_dim"], mx["vdim"], mx["kv_rank"]
     dims, base = int(mx["rot"]["dims"]), float(mx["rot"]["base"])
     window = int((mx.get("mask") or {}).get("size", 0))
-    cq = rms_norm_plain(h @ P[p + "dq"].T, P[p + "dq.norm"], eps)
-    q = (cq @ P[p + "uq"].T).reshape(T, H, d + dr)
+    if mx.get("q_rank"):
+        q = rms_norm_plain(h @ P[p + "dq"].T, P[p + "dq.norm"], eps) @ P[p + "uq"].T
+    else:
+        q = h @ P[p + "q"].T
+    q = q.reshape(T, H, d + dr)
     both = h @ P[p + "dkv"].T
     c = rms_norm_plain(both[:, :r], P[p + "dkv.norm"], eps)
     kr = np.stack([rotate_neighbours(both[t, r:], t, dims, base) for t in range(T)])
@@ -147,7 +151,7 @@ def latent_attention(mx, P, p, h, eps):
         seen = [j for j in range(i + 1) if in_window(i, j, window)]
         for hd in range(H):
             qr = rotate_neighbours(q[i, hd, d:], i, dims, base)
-            wts = softmax([(q[i, hd, :d] @ k[j, hd] + qr @ kr[j]) * mx["scale"] for j in seen])
+            wts = softmax((k[seen, hd] @ q[i, hd, :d] + kr[seen] @ qr) * mx["scale"])
             out[i, hd] = wts @ v[seen, hd]
     return out.reshape(T, -1) @ P[p + "o"].T
 

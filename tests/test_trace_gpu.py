@@ -51,6 +51,17 @@ def test_trace_replay_of_a_goperax_model(tmp_path, dtype, tol):
     _replay(tmp_path, dtype, tol, cfg, G.weights(cfg, seed=3), G.oracle_logits)
 
 
+@pytest.mark.parametrize("dtype,tol", [("float32", 2e-4), ("bfloat16", None)])
+def test_trace_replay_of_a_nifulix_model(tmp_path, dtype, tol):
+    """The same schedule through a Nifulix model: windows of 24, 50 and 100 positions against pages of 64, kept first positions,
+    values carried between layers, recurrent state handed on from request to request."""
+    from tests import _nifulix_util as N
+    cfg = N.config([(N.attention(dim=16, window=24), N.dense()), (N.retention(), N.dense()), (N.latent(window=50), None),
+                    (N.attention(heads=6, kv_heads=2, dim=6, vdim=16, window=100, keep=9), N.dense()), (N.latent(heads=4, dim=16, rot_dim=16, vdim=16, kv_rank=32), None)],
+                   vocab=90, width=40)
+    _replay(tmp_path, dtype, tol, cfg, N.weights(cfg, seed=3), N.oracle_logits)
+
+
 def _replay(tmp_path, dtype, tol, cfg, W, oracle_logits):
     model = tmp_path / "model"
     model.mkdir()
