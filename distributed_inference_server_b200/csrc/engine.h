@@ -60,6 +60,7 @@ struct StepMeta {
   size_t o_tokens, o_pos, o_ptrow, o_ctx, o_rowmap, o_temp, o_topp, o_seed, o_step;
   size_t o_qb_tok0, o_qb_len, o_qb_pos0, o_qb_ptrow;  // prefill query blocks
   size_t o_arstep;                                     // forward-pass counter (epoch of the peer-memory exchange)
+  size_t o_lb_tok0 = 0, o_lb_len = 0, o_ls = 0, o_lin = 0;  // latent attention of prompt portions: query blocks, spans, per (latent layer, slot) row of position 0
   size_t o_span = 0, o_ab_tok0 = 0, o_ab_len = 0, o_kb_tok0 = 0, o_kb_len = 0;       // layer-list family: span of each token; attention query blocks
   template <class T_> T_ *h(size_t off) { return reinterpret_cast<T_ *>(host + off); }
   template <class T_> T_ *d(size_t off) { return reinterpret_cast<T_ *>(dev + off); }
@@ -169,7 +170,10 @@ struct Engine {
   std::map<std::string, StackTarget> stack_names;
   int stack_bq = 8;
   bool stack_capturing = false;  // a decode pass is being captured: nothing in it may wait for the device
-  struct StackSpanH { int tok0, len, pos0, slot; bool products; };
+  struct StackSpanH { int tok0, len, pos0, slot; bool products; int lb0 = 0, n_lb = 0, ls = 0; };  // lb0, n_lb: its query blocks; ls: its place among the long spans
+  // consecutive long spans whose per-head keys and values of one latent layer are made together
+  struct StackLatGroup { int ls0, n, rows, max_keys, lb0, n_lb; };
+  std::vector<std::vector<StackLatGroup>> stack_lat_groups;  // per latent layer
   std::vector<StackSpanH> stack_spans_h;  // spans of the pass being built; products: its latent attention runs as matrix products
   int stack_abq = 0;          // tokens per query block of paged attention (0: the model has none); smallest over its layers
   int stack_kb = 0;           // its query blocks in the pass being built

@@ -156,7 +156,12 @@ gemm_persist_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
           }
         } else {
           tmem_ld_wait();
-          if (n < N && out_act) {  // ungated unit: the square of relu, rounded to bf16 for the product that follows
+          if (n < N && out_act && !kDual && up_row_off < 0) {  // the sums themselves, rounded to bf16
+            uint16_t *o = out_act + (size_t)(t0 + c) * N + n;
+#pragma unroll
+            for (int jj = 0; jj < 32; jj++)
+              if (t0 + c + jj < T) o[(size_t)jj * N] = float_to_bf16_bits(__uint_as_float(g[jj]));
+          } else if (n < N && out_act) {  // ungated unit: the square of relu, rounded to bf16 for the product that follows
             uint16_t *o = out_act + (size_t)(t0 + c) * N + n;
 #pragma unroll
             for (int jj = 0; jj < 32; jj++)
@@ -381,6 +386,14 @@ cudaError_t launch_gemm_persist_relu2(const TmaMap &w_map, const TmaMap &x_map25
   if (T <= 0) return cudaSuccess;
   if (!act) return cudaErrorInvalidValue;
   return persist_launch<256, false>(w_map, x_map256, nullptr, act, T, N, K, w_row0, 0, st);
+}
+
+// The same product, its sums rounded to bf16 by the epilogue.
+cudaError_t launch_gemm_persist_bf16(const TmaMap &w_map, const TmaMap &x_map256, uint16_t *out, int T, int N, int K, int w_row0,
+                                     cudaStream_t st) {
+  if (T <= 0) return cudaSuccess;
+  if (!out) return cudaErrorInvalidValue;
+  return persist_launch<256, false>(w_map, x_map256, nullptr, out, T, N, K, w_row0, -1, st);  // up_off < 0: plain bf16 result
 }
 
 // w_map64: 64-row boxes over the fused [2I][K] weight (gate rows, then up rows); x_map256: 256-row boxes.

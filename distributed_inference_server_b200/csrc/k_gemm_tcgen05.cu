@@ -179,7 +179,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
         }
       } else {
         tmem_ld_wait();
-        if (n < N) {
+        if (n < N && out_act) {  // one slice, the sums rounded to bf16
+          uint16_t *o = out_act + (size_t)(t0 + c) * N + n;
+#pragma unroll
+          for (int jj = 0; jj < 32; jj++)
+            if (t0 + c + jj < T) o[(size_t)jj * N] = float_to_bf16_bits(__uint_as_float(g[jj]));
+        } else if (n < N) {
           float *o = out_partial + ((size_t)blockIdx.z * T + t0 + c) * N + n;
 #pragma unroll
           for (int jj = 0; jj < 32; jj++)
@@ -295,6 +300,17 @@ cudaError_t launch_gemm_partial(const TmaMap &w_map, const TmaMap &x_map, float 
     case 64: return gemm_launch<64, false>(w_map, x_map, out, nullptr, T, N, K, w_row0, 0, split_k, kBM, st);
     case 128: return gemm_launch<128, false>(w_map, x_map, out, nullptr, T, N, K, w_row0, 0, split_k, kBM, st);
     default: return gemm_launch<256, false>(w_map, x_map, out, nullptr, T, N, K, w_row0, 0, split_k, kBM, st);
+  }
+}
+
+cudaError_t launch_gemm_bf16(const TmaMap &w_map, const TmaMap &x_map, uint16_t *out, int T, int N, int K, int w_row0, cudaStream_t st) {
+  if (T <= 0) return cudaSuccess;
+  if (!out) return cudaErrorInvalidValue;
+  switch (gemm_token_tile(T)) {
+    case 32: return gemm_launch<32, false>(w_map, x_map, nullptr, out, T, N, K, w_row0, 0, 1, kBM, st);
+    case 64: return gemm_launch<64, false>(w_map, x_map, nullptr, out, T, N, K, w_row0, 0, 1, kBM, st);
+    case 128: return gemm_launch<128, false>(w_map, x_map, nullptr, out, T, N, K, w_row0, 0, 1, kBM, st);
+    default: return gemm_launch<256, false>(w_map, x_map, nullptr, out, T, N, K, w_row0, 0, 1, kBM, st);
   }
 }
 

@@ -426,16 +426,24 @@ bool stack_attn_mma_ok(const StackAttn &c, bool f32) {
 }
 int stack_attn_mma_block_tokens(const StackAttn &c) { return std::max(1, kMmRows / (c.H / c.G)); }
 
-template <int DMAX, bool SIG, bool DIST>
-__global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const float *__restrict__ qf, const uint16_t *__restrict__ kpool,
-                                                                       const uint16_t *__restrict__ vpool, const float *temp,
+// Where the keys and values of a head lie: row r of position p is lin[slot] + p (gathered rows) or, lin null, the row of p's page.  A
+// key is its first dk coordinates at k + r * k_ld + head * k_hs, then (k2, shared by the heads) the rest at k2 + r * k2_ld.
+struct AttnKV {
+  const uint16_t *k, *k2, *v;
+  long long k_ld, k2_ld, v_ld;
+  int k_hs, dk, v_hs;
+  const int *lin;
+};
+// DQ, DV: compiled sizes of a query / key and of a value (the layer's are at most these).
+template <int DQ, int DV, bool SIG, bool DIST>
+__global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mma_kernel(const float *__restrict__ qf, long long ldq, AttnKV kv, const float *temp,
                                                                        const float *pb, const float *sink, StackAttn c, StackSpans sp, const int *qb_tok0,
                                                                        const int *qb_len, const int *page_table, int max_pages,
                                                                        int page_size, AttnOut o, int keys_per_split, float *part) {
-  constexpr int PITCH = DMAX + 8;  // elements per shared row: 16-byte rows land in distinct bank groups
+  constexpr int KP = DQ + 8, VP = DV + 8;  // elements per shared row: 16-byte rows land in distinct bank groups
   extern __shared__ __align__(16) uint16_t smem[];
-  uint16_t *Ks = smem;                                  // [2][64][PITCH]
-  uint16_t *Vs = smem + 2 * kMmKeys * PITCH;            // [2][64][PITCH]
+  uint16_t *Ks = smem;                               // [2][64][KP]
+  uint16_t *Vs = smem + 2 * kMmKeys * KP;            // [2][64][VP]
   const int d = c.d, dv = c.dv, R = c.H / c.G, kvh = blockIdx.y;
   // the blocks of a span come in ascending position, and the later ones walk a longer history: taking the grid backwards starts
   // the long ones first, so the last CTAs to start are short
@@ -452,11 +460,11 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
   const int nk16 = (d + 15) >> 4, nv8 = dv >> 3, dc = d >> 3, vc = dv >> 3;  // k-steps of Q K^T, n-tiles of P V, 16-byte chunks per row
   // columns d .. 16 nk16 of the K stages are read by the last k-step: zero them once (cp.async never touches them)
   if (d & 15)
-    for (int i = threadIdx.x; i < 2 * kMmKeys * 8; i += blockDim.x) Ks[(i >> 3) * PITCH + d + (i & 7)] = 0;
+    for (int i = threadIdx.x; i < 2 * kMmKeys * 8; i += blockDim.x) Ks[(i >> 3) * KP + d + (i & 7)] = 0;
   // ---- this thread's rows: r0 = 16 warp + gid and r0 + 8
   int r_tok[2], r_head[2], r_pos[2], r_lo[2];
   bool r_ok[2];
-  uint32_t qa[DMAX / 16][4];
+  uint32_t qa[DQ / 16][4];
 #pragma unroll
   for (int e = 0; e < 2; e++) {
     const int r = warp * 16 + gid + e * 8;
@@ -467,10 +475,10 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
     r_lo[e] = r_ok[e] ? stack_attn_row_lo(c, r_pos[e]) : 0;
   }
 #pragma unroll
-  for (int ks = 0; ks < DMAX / 16; ks++) {
+  for (int ks = 0; ks < DQ / 16; ks++) {
 #pragma unroll
     for (int e = 0; e < 2; e++) {
-      const float *qr = qf + ((long long)r_tok[e] * c.H + r_head[e]) * d;
+      const float *qr = qf + (long long)r_tok[e] * ldq + (long long)r_head[e] * d;
 #pragma unroll
       for (int hf = 0; hf < 2; hf++) {
         const int col = ks * 16 + hf * 8 + qd * 2;
@@ -483,9 +491,9 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
       }
     }
   }
-  float oacc[DMAX / 8][4];
+  float oacc[DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < DMAX / 8; j++) { oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f; }
+  for (int j = 0; j < DV / 8; j++) { oacc[j][0] = oacc[j][1] = oacc[j][2] = oacc[j][3] = 0.f; }
   float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};
   if (!SIG && sink && blockIdx.z == 0) {  // the sink term of the denominator enters as the initial state of the first slice (one lane of the four holds its 1)
 #pragma unroll
@@ -509,23 +517,29 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
   const int warp_first_pos = pos_first + (warp * 16) / R;
   const int warp_lo = stack_attn_row_lo(c, warp_first_pos);        // first key any row of the warp sees
   const int warp_lo_max = stack_attn_row_lo(c, warp_last_pos);     // first key every row of the warp sees
-  const long long krow = (long long)c.G * d, vrow = (long long)c.G * dv;
+  const uint16_t *kh = kv.k + (long long)kvh * kv.k_hs, *vh = kv.v + (long long)kvh * kv.v_hs;
+  const int dk8 = kv.dk >> 3;
+  const long long lin0 = kv.lin ? kv.lin[slot] : 0;
   const uint32_t ks_base = (uint32_t)__cvta_generic_to_shared(Ks), vs_base = (uint32_t)__cvta_generic_to_shared(Vs);
   // two threads per key row: one page-table read per thread and tile, then the row's 16-byte chunks alternate between the two
   const int ld_row = threadIdx.x >> 1, ld_part = threadIdx.x & 1;
   const int pshift = 31 - __clz(page_size);  // page_size is a power of two
   // the page of this thread's row is read one tile ahead of the copy that needs it
-  auto page_of = [&](int k0) { const int v = k0 + ld_row; return v < k_end ? pt[wk.key(v) >> pshift] : 0; };
+  auto page_of = [&](int k0) { const int v = k0 + ld_row; return v < k_end && !kv.lin ? pt[wk.key(v) >> pshift] : 0; };
   int page_next = page_of(k_begin);
   auto load_tile = [&](int k0, int stage) {
     const int kp = wk.key(k0 + ld_row);
     const bool ok = k0 + ld_row < k_end;
-    const long long prow = ok ? (long long)page_next * page_size + (kp & (page_size - 1)) : 0;
+    const long long prow = !ok ? 0 : kv.lin ? lin0 + kp : (long long)page_next * page_size + (kp & (page_size - 1));
     page_next = page_of(k0 + kMmKeys);
-    const uint16_t *ksrc = kpool + prow * krow + (long long)kvh * d, *vsrc = vpool + prow * vrow + (long long)kvh * dv;
-    const uint32_t kdst = ks_base + (uint32_t)(((stage * kMmKeys + ld_row) * PITCH) * 2), vdst = vs_base + (uint32_t)(((stage * kMmKeys + ld_row) * PITCH) * 2);
+    const uint16_t *ksrc = kh + prow * kv.k_ld, *vsrc = vh + prow * kv.v_ld;
+    const uint32_t kdst = ks_base + (uint32_t)(((stage * kMmKeys + ld_row) * KP) * 2), vdst = vs_base + (uint32_t)(((stage * kMmKeys + ld_row) * VP) * 2);
 #pragma unroll 4
-    for (int ch = ld_part; ch < dc; ch += 2) cp_async16(kdst + ch * 16, ksrc + ch * 8, ok ? 16 : 0);
+    for (int ch = ld_part; ch < dk8; ch += 2) cp_async16(kdst + ch * 16, ksrc + ch * 8, ok ? 16 : 0);
+    if (dk8 < dc) {  // the shared part of the key
+      const uint16_t *k2 = kv.k2 + prow * kv.k2_ld;
+      for (int ch = dk8 + ld_part; ch < dc; ch += 2) cp_async16(kdst + ch * 16, k2 + (ch - dk8) * 8, ok ? 16 : 0);
+    }
 #pragma unroll 4
     for (int ch = ld_part; ch < vc; ch += 2) cp_async16(vdst + ch * 16, vsrc + ch * 8, ok ? 16 : 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -545,17 +559,17 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
     if (warp_live && key_a <= warp_last_pos && (key_z >= warp_lo || key_a < c.keep)) {
       // S = Q K^T: k-steps outside, key tiles inside, so that consecutive products go to different accumulators; one ldmatrix
       // brings the fragments of two key tiles (lane l: matrix l / 8 = (tile, column half), row l % 8)
-      const uint32_t kt = ks_base + (uint32_t)(stage * kMmKeys * PITCH * 2);
+      const uint32_t kt = ks_base + (uint32_t)(stage * kMmKeys * KP * 2);
       float sacc[kMmKeys / 8][4];
 #pragma unroll
       for (int j = 0; j < kMmKeys / 8; j++) { sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f; }
 #pragma unroll
-      for (int ks = 0; ks < DMAX / 16; ks++) {
+      for (int ks = 0; ks < DQ / 16; ks++) {
         if (ks < nk16) {
 #pragma unroll
           for (int j = 0; j < kMmKeys / 8; j += 2) {
             uint32_t b0, b1, b2, b3;
-            ldsm_x4(kt + (uint32_t)((((j + (lane >> 4)) * 8 + (lane & 7)) * PITCH + ks * 16 + ((lane >> 3) & 1) * 8) * 2), b0, b1, b2, b3);
+            ldsm_x4(kt + (uint32_t)((((j + (lane >> 4)) * 8 + (lane & 7)) * KP + ks * 16 + ((lane >> 3) & 1) * 8) * 2), b0, b1, b2, b3);
             mma_bf16_16816(sacc[j], qa[ks], b0, b1);
             mma_bf16_16816(sacc[j + 1], qa[ks], b2, b3);
           }
@@ -588,10 +602,10 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
             lrow[e] += pv;
           }
 #pragma unroll
-        for (int j = 0; j < DMAX / 8; j++) { oacc[j][0] *= corr[0]; oacc[j][1] *= corr[0]; oacc[j][2] *= corr[1]; oacc[j][3] *= corr[1]; }
+        for (int j = 0; j < DV / 8; j++) { oacc[j][0] *= corr[0]; oacc[j][1] *= corr[0]; oacc[j][2] *= corr[1]; oacc[j][3] *= corr[1]; }
       }
       // ---- O += P V
-      const uint32_t vt = vs_base + (uint32_t)(stage * kMmKeys * PITCH * 2);
+      const uint32_t vt = vs_base + (uint32_t)(stage * kMmKeys * VP * 2);
 #pragma unroll
       for (int kk = 0; kk < kMmKeys / 16; kk++) {
         uint32_t pa[4];
@@ -600,11 +614,11 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
         pa[2] = pack_bf16(sacc[2 * kk + 1][0], sacc[2 * kk + 1][1]);
         pa[3] = pack_bf16(sacc[2 * kk + 1][2], sacc[2 * kk + 1][3]);
 #pragma unroll
-        for (int j = 0; j < DMAX / 8; j += 2) {
+        for (int j = 0; j < DV / 8; j += 2) {
           if (j < nv8) {
             // lanes 0-15: keys 16 kk + lane of columns 8 j; lanes 16-31: the same keys of columns 8 (j + 1)
             uint32_t b0, b1, b2, b3;
-            ldsm_x4_trans(vt + (uint32_t)(((kk * 16 + (lane & 15)) * PITCH + (j + (lane >> 4)) * 8) * 2), b0, b1, b2, b3);
+            ldsm_x4_trans(vt + (uint32_t)(((kk * 16 + (lane & 15)) * VP + (j + (lane >> 4)) * 8) * 2), b0, b1, b2, b3);
             mma_bf16_16816(oacc[j], pa, b0, b1);
             mma_bf16_16816(oacc[j + 1], pa, b2, b3);
           }
@@ -628,7 +642,7 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
 #pragma unroll
     for (int e = 0; e < 2; e++) {
 #pragma unroll
-      for (int j = 0; j < DMAX / 8; j++)
+      for (int j = 0; j < DV / 8; j++)
         if (j < nv8) { ot[(gid + e * 8) * (dv + 1) + j * 8 + qd * 2] = oacc[j][e * 2]; ot[(gid + e * 8) * (dv + 1) + j * 8 + qd * 2 + 1] = oacc[j][e * 2 + 1]; }
       if (qd == 0) ot[(gid + e * 8) * (dv + 1) + dv] = attn_out_factor(o, r_tok[e], r_head[e]) * (SIG ? 1.f : 1.f / lrow[e]);
     }
@@ -657,7 +671,7 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
     if (part) {
       float *rec = part + (((long long)blockIdx.z * sp.T + r_tok[e]) * c.H + r_head[e]) * (dv + 2);
 #pragma unroll
-      for (int j = 0; j < DMAX / 8; j++)
+      for (int j = 0; j < DV / 8; j++)
         if (j < nv8) { rec[j * 8 + qd * 2] = oacc[j][e * 2]; rec[j * 8 + qd * 2 + 1] = oacc[j][e * 2 + 1]; }
       if (qd == 0) { rec[dv] = SIG ? 0.f : mrow[e] * kLn2; rec[dv + 1] = lrow[e]; }  // the maximum back in natural units
       continue;
@@ -666,13 +680,65 @@ __global__ void __launch_bounds__(kMmWarps * 32, 3) stack_attn_mma_kernel(const 
     uint16_t *orow = reinterpret_cast<uint16_t *>(o.out) + (long long)r_tok[e] * o.ld + o.off + (long long)r_head[e] * dv;
     const float *gr = o.gate_full ? o.gate_full + (long long)r_tok[e] * o.ldg + (long long)r_head[e] * dv + qd * 2 : nullptr;
 #pragma unroll
-    for (int j = 0; j < DMAX / 8; j++)
+    for (int j = 0; j < DV / 8; j++)
       if (j < nv8) {
         float a0 = oacc[j][e * 2] * inv, a1 = oacc[j][e * 2 + 1] * inv;
         if (gr) { a0 *= sigmoid_precise(gr[j * 8]); a1 *= sigmoid_precise(gr[j * 8 + 1]); }
         *reinterpret_cast<uint32_t *>(orow + j * 8 + qd * 2) = pack_bf16(a0, a1);
       }
   }
+}
+
+static cudaError_t attn_mma_go(const float *qf, long long ldq, const AttnKV &kv, const float *temp, const float *pb, const float *sink,
+                               const StackAttn &c, const StackSpans &sp, const int *qb_tok0, const int *qb_len, dim3 grid, const int *page_table,
+                               int max_pages, int page_size, const AttnOut &o, int keys_per_split, float *part, cudaStream_t st) {
+  static DeviceOnce once;
+  DIS_CUDA_TRY(once.run([&] {
+    cudaError_t e = cudaSuccess;
+    auto allow = [&](auto kern) { if (e == cudaSuccess) e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); };
+    allow(stack_attn_mma_kernel<64, 64, true, false>);
+    allow(stack_attn_mma_kernel<64, 64, false, false>);
+    allow(stack_attn_mma_kernel<64, 64, false, true>);
+    allow(stack_attn_mma_kernel<128, 128, true, false>);
+    allow(stack_attn_mma_kernel<128, 128, false, false>);
+    allow(stack_attn_mma_kernel<128, 128, false, true>);
+    allow(stack_attn_mma_kernel<192, 128, false, false>);
+    return e;
+  }));
+  const bool sig = (c.flags & DIS_ATTN_SIGMOID) != 0, dist = (c.flags & DIS_ATTN_DISTANCE) != 0;
+  const bool small = c.d <= 64 && c.dv <= 64;
+  const int dq = small ? 64 : c.d <= 128 ? 128 : 192, dvp = small ? 64 : 128;
+  if (c.d > dq || c.dv > dvp || (dq == 192 && (sig || dist))) return cudaErrorInvalidValue;
+  const size_t shm = (size_t)2 * kMmKeys * (dq + dvp + 16) * sizeof(uint16_t);
+#define DIS_ATTN_MMA(Q, V, S, B) \
+  stack_attn_mma_kernel<Q, V, S, B><<<grid, kMmWarps * 32, shm, st>>>(qf, ldq, kv, temp, pb, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, o, keys_per_split, part)
+  if (dq == 192) DIS_ATTN_MMA(192, 128, false, false);
+  else if (small && sig) DIS_ATTN_MMA(64, 64, true, false);
+  else if (small && dist) DIS_ATTN_MMA(64, 64, false, true);
+  else if (small) DIS_ATTN_MMA(64, 64, false, false);
+  else if (sig) DIS_ATTN_MMA(128, 128, true, false);
+  else if (dist) DIS_ATTN_MMA(128, 128, false, true);
+  else DIS_ATTN_MMA(128, 128, false, false);
+#undef DIS_ATTN_MMA
+  return cudaGetLastError();
+}
+
+// Latent attention of prompt portions on the same kernel: every head has keys and values of its own, made from the gathered latents
+// (kv [rows][H*(d + dv)]: all heads' unrotated key parts, then all heads' values), and the rotated key part krot [rows][dr] is shared.
+// Position p of the sequence in slot s is row lin[s] + p.
+bool stack_latent_flash_ok(const StackLatent &c, bool f32) {
+  return !f32 && c.r % 8 == 0 && c.d % 8 == 0 && c.dr % 8 == 0 && c.dv % 16 == 0 && c.d + c.dr <= 192 && c.dv <= 128;
+}
+int stack_latent_flash_tokens() { return kMmRows; }
+cudaError_t launch_stack_latent_flash(const float *q, long long ldq, const uint16_t *kv, const uint16_t *krot, const int *lin, const float *sink,
+                                      const StackLatent &c, const StackSpans &sp, const int *qb_tok0, const int *qb_len, int n_qb, void *out,
+                                      long long ld_out, const float *gate, long long ld_gate, cudaStream_t st) {
+  if (n_qb <= 0) return cudaSuccess;
+  const StackAttn a{c.H, c.H, c.d + c.dr, c.dv, 0, 0u, c.scale, c.eps, 0, c.window};
+  const long long ld = (long long)c.H * (c.d + c.dv);
+  const AttnKV src{kv, krot, kv + (long long)c.H * c.d, ld, (long long)c.dr, ld, c.d, c.d, c.dv, lin};
+  const AttnOut o{out, ld_out, 0, 1.f, nullptr, nullptr, ld_gate, gate};
+  return attn_mma_go(q, ldq, src, nullptr, nullptr, sink, a, sp, qb_tok0, qb_len, dim3(n_qb, c.H, 1), nullptr, 0, 1, o, 0, nullptr, st);
 }
 
 cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vpool, bool f32, const float *temp, const float *pb,
@@ -702,31 +768,9 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
   if (use_mma < 0) { const char *e = getenv("DIS_STACK_ATTN_MMA"); use_mma = (e && atoi(e) == 0) ? 0 : 1; }
   // the output's 4-byte stores want even columns; bq is the block size the pass was planned with
   if (use_mma && stack_attn_mma_ok(c, f32) && bq <= stack_attn_mma_block_tokens(c) && ld_out % 2 == 0 && out_off % 2 == 0) {
-    static DeviceOnce once_mma;
-    DIS_CUDA_TRY(once_mma.run([&] {
-      cudaError_t e = cudaSuccess;
-      auto allow = [&](auto kern) { if (e == cudaSuccess) e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); };
-      allow(stack_attn_mma_kernel<64, true, false>);
-      allow(stack_attn_mma_kernel<64, false, false>);
-      allow(stack_attn_mma_kernel<64, false, true>);
-      allow(stack_attn_mma_kernel<128, true, false>);
-      allow(stack_attn_mma_kernel<128, false, false>);
-      allow(stack_attn_mma_kernel<128, false, true>);
-      return e;
-    }));
-    const bool small = c.d <= 64 && c.dv <= 64;
-    const size_t shm = (size_t)4 * kMmKeys * ((small ? 64 : 128) + 8) * sizeof(uint16_t);
     const uint16_t *kp = reinterpret_cast<const uint16_t *>(kpool), *vp = reinterpret_cast<const uint16_t *>(vpool);
-    const bool dist = (c.flags & DIS_ATTN_DISTANCE) != 0;
-#define DIS_ATTN_MMA(D, S, B) \
-  stack_attn_mma_kernel<D, S, B><<<grid, kMmWarps * 32, shm, st>>>(qf, kp, vp, temp, pb, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, o, keys_per_split, part)
-    if (small && sig) DIS_ATTN_MMA(64, true, false);
-    else if (small && dist) DIS_ATTN_MMA(64, false, true);
-    else if (small) DIS_ATTN_MMA(64, false, false);
-    else if (sig) DIS_ATTN_MMA(128, true, false);
-    else if (dist) DIS_ATTN_MMA(128, false, true);
-    else DIS_ATTN_MMA(128, false, false);
-#undef DIS_ATTN_MMA
+    const AttnKV kv{kp, nullptr, vp, (long long)c.G * c.d, 0, (long long)c.G * c.dv, c.d, c.d, c.dv, nullptr};
+    DIS_CUDA_TRY(attn_mma_go(qf, (long long)c.H * c.d, kv, temp, pb, sink, c, sp, qb_tok0, qb_len, grid, page_table, max_pages, page_size, o, keys_per_split, part, st));
     if (part) {
       const size_t msh = (size_t)(c.dv + n_split) * sizeof(float);
       if (sig) stack_attn_merge_kernel<false, true><<<sp.T * c.H, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);

@@ -1008,12 +1008,14 @@ __device__ __forceinline__ float latent_rotated(const float *v, int i, const Sta
 // Columns of the row: queries (rotated parts go to qf) at q_off when qf is given; latent and rotated key part at dkv_off when pool is
 // given; the query latent at dq_off when cq is given (RMS-normed with the gain dq_norm into cq [T][q_rank], compute type).  The row may
 // come as n_part slices of n_cols columns; columns keep_off .. keep_off + keep_n of their sum then go to keep [T][ld_keep] as well.
+// qx (or null): the rotated query parts are also written where the queries lie, [T][ld_qx] from the first head's column on (the row
+// itself, or its copy in keep).
 template <bool F32>
 __global__ void __launch_bounds__(256) stack_latent_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
                                                                 int q_off, int dkv_off, const float *dkv_norm, int dq_off,
                                                                 const float *dq_norm, void *cq, float *keep, long long ld_keep,
                                                                 int keep_off, int keep_n, const double *__restrict__ freq,
-                                                                StackLatent c, StackSpans sp, float *qf, void *pool,
+                                                                StackLatent c, StackSpans sp, float *qf, float *qx, long long ld_qx, void *pool,
                                                                 const int *page_table, int max_pages, int page_size) {
   extern __shared__ __align__(16) float lsh[];  // cos [half], sin [half], then (n_part > 1) the summed row
   __shared__ float sh[32];
@@ -1046,11 +1048,23 @@ __global__ void __launch_bounds__(256) stack_latent_prep_kernel(const float *pro
   __syncthreads();
   if (keep)
     for (int i = threadIdx.x; i < keep_n; i += blockDim.x) keep[(long long)t * ld_keep + i] = row[keep_off + i];
-  if (qf)
-    for (int i = threadIdx.x; i < c.H * c.dr; i += blockDim.x) {
-      const int h = i / c.dr, k = i % c.dr;
-      qf[((long long)t * c.H + h) * D + c.r + k] = latent_rotated(row + q_off + (long long)h * (c.d + c.dr) + c.d, k, c, cs, sn);
+  if (qf || qx) {
+    if (keep && qx) __syncthreads();  // the copy's unrotated parts land first
+    const int per = half + (c.dr - c.rot_dims);  // a head's pairs, then its coordinates that stay
+    for (int i = threadIdx.x; i < c.H * per; i += blockDim.x) {
+      const int h = i / per, p = i - h * per, col = h * (c.d + c.dr) + c.d;
+      float *qo = qf ? qf + ((long long)t * c.H + h) * D + c.r : nullptr;
+      const float *v = row + q_off + col;
+      if (p >= half) {
+        if (qo) qo[p + half] = v[p + half];
+        continue;
+      }
+      const int a = c.rot_pairs ? 2 * p : p, b = c.rot_pairs ? 2 * p + 1 : p + half;
+      const float x = v[a], y = v[b], ra = x * cs[p] - y * sn[p], rb = y * cs[p] + x * sn[p];
+      if (qo) { qo[a] = ra; qo[b] = rb; }
+      if (qx) { qx[(long long)t * ld_qx + col + a] = ra; qx[(long long)t * ld_qx + col + b] = rb; }
     }
+  }
   if (cq) {
     const float *dq = row + dq_off;
     float s = 0.f;
@@ -1082,7 +1096,7 @@ cudaError_t launch_stack_latent_prep(const StackLatentPrep &a, const StackLatent
   }));
 #define DIS_LAT_PREP(F)                                                                                                                      \
   stack_latent_prep_kernel<F><<<sp.T, 256, sh, st>>>(a.proj, a.ld, n_part, a.stride, a.n_cols, a.q_off, a.dkv_off, a.dkv_norm, a.dq_off, a.dq_norm, \
-                                                     a.cq, a.keep, a.ld_keep, a.keep_off, a.keep_n, a.freq, c, sp, a.qf, a.pool, page_table, max_pages, page_size)
+                                                     a.cq, a.keep, a.ld_keep, a.keep_off, a.keep_n, a.freq, c, sp, a.qf, a.qx, a.ld_qx, a.pool, page_table, max_pages, page_size)
   if (f32) DIS_LAT_PREP(true);
   else DIS_LAT_PREP(false);
 #undef DIS_LAT_PREP
@@ -1414,6 +1428,34 @@ __global__ void stack_latent_merge_kernel(const float *part, const float *sink, 
     for (int s = 0; s < n_split; s++) v = fmaf(part[((long long)s * pairs_total + p) * (r + 2) + j], ws[s], v);
     ol[(long long)p * r + j] = v * inv_den;
   }
+}
+
+// Latents of prompt portions out of their pages, for the keys and values made from them: grid (8 keys, span of the list `ls`), a warp
+// per key; position p of the span's sequence goes to row lin[slot] + p, latent to cg [rows][r], rotated key part to krot [rows][dr].
+__global__ void __launch_bounds__(256) stack_latent_rows_kernel(const uint16_t *__restrict__ pool, StackLatent c, StackSpans sp,
+                                                                const int *__restrict__ ls, const int *__restrict__ lin,
+                                                                const int *__restrict__ page_table, int max_pages, int page_size,
+                                                                uint16_t *__restrict__ cg, uint16_t *__restrict__ krot) {
+  const int s = ls[blockIdx.y], pos0 = sp.sp_pos0[s], slot = sp.sp_slot[s], D = c.r + c.dr, l = threadIdx.x & 31;
+  const int key = stack_latent_row_lo(c, pos0) + blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (key >= pos0 + sp.sp_len[s]) return;
+  const long long row = (long long)lin[slot] + key;
+  const long long prow = (long long)page_table[(long long)slot * max_pages + key / page_size] * page_size + key % page_size;
+  const uint4 *src = reinterpret_cast<const uint4 *>(pool + prow * D);
+  uint4 *d1 = reinterpret_cast<uint4 *>(cg + row * c.r), *d2 = reinterpret_cast<uint4 *>(krot + row * c.dr);
+  for (int i = l; i < D >> 3; i += 32) {
+    if (i < c.r >> 3) d1[i] = src[i];
+    else d2[i - (c.r >> 3)] = src[i];
+  }
+}
+cudaError_t launch_stack_latent_rows(const void *pool, const StackLatent &c, const StackSpans &sp, const int *ls, int n_ls, int max_keys,
+                                     const int *lin, const int *page_table, int max_pages, int page_size, uint16_t *cg, uint16_t *krot,
+                                     cudaStream_t st) {
+  if (n_ls <= 0 || max_keys <= 0) return cudaSuccess;
+  if (c.r % 8 || c.dr % 8) return cudaErrorInvalidValue;
+  stack_latent_rows_kernel<<<dim3((max_keys + 7) / 8, n_ls), 256, 0, st>>>(reinterpret_cast<const uint16_t *>(pool), c, sp, ls, lin, page_table,
+                                                                          max_pages, page_size, cg, krot);
+  return cudaGetLastError();
 }
 
 // ---- latent attention of long prompt portions as matrix products (bf16 operands, fp32 accumulation): the sequence's latents

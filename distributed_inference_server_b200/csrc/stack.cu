@@ -77,6 +77,8 @@ cudaError_t Engine::stack_meta(StepMeta &s, int cap_t, int cap_rows) {
   s.o_rowmap = sec(cr * 4); s.o_temp = sec(cr * 4); s.o_topp = sec(cr * 4); s.o_seed = sec(cr * 8); s.o_step = sec(cr * 8);
   s.o_qb_tok0 = sec(ct * 4); s.o_qb_len = sec(ct * 4); s.o_qb_pos0 = sec(ct * 4); s.o_qb_ptrow = sec(ct * 4);
   s.o_ab_tok0 = sec(ct * 4); s.o_ab_len = sec(ct * 4);
+  s.o_lb_tok0 = sec(ct * 4); s.o_lb_len = sec(ct * 4); s.o_ls = sec((size_t)max_batch * 4);
+  s.o_lin = sec((size_t)std::max(1, stack->n_lat) * max_batch * 4);
   s.o_kb_tok0 = sec(ct * 4); s.o_kb_len = sec(ct * 4);
   s.o_arstep = sec(16);
   s.bytes = o;
@@ -107,6 +109,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   if ((page_size & (page_size - 1)) || page_size < 8) return fail(DIS_ERR_INVALID_ARGUMENT, "page_size must be a power of two >= 8");
   max_pages = (m.max_ctx + page_size - 1) / page_size;
 
+  if (const char *g = getenv("DIS_STACK_TC")) stack_tc = atoi(g) != 0;
   stack = new StackModel();
   StackModel &M = *stack;
   M.c = *sc;
@@ -151,6 +154,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       L.g_off = L.dkv_off + (lc.kv_from < 0 ? lc.kv_rank + lc.rot_dim : 0);
       L.n_in = L.g_off + ((lc.latent_flags & DIS_LATENT_NO_GATE) ? 0 : lc.heads * lc.vdim);
       L.n_act = lc.heads * lc.vdim;
+      L.lat_ix = M.n_lat++;
       if (lc.mask_window < 0 || lc.mask_chunk != 0 || lc.mask_keep != 0 || lc.q_rank < 0)
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "latent attention: mask_window and q_rank must not be negative; it has no chunked mask and no kept positions");
       const StackLatent sl = stack_latent_shape(lc, sc->norm_eps);
@@ -360,7 +364,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   static StackTensor dummy;  // scalars are written through their own small tensors below
   (void)dummy;
-  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0;
+  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0, lat_row = 0, lat_w[3] = {0, 0, 0};
   int max_top = 0, max_e = 0;
   bool any_shared = false;
   size_t max_sff = 0;
@@ -582,7 +586,17 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       if (!(lc.latent_flags & DIS_LATENT_NO_GATE)) name(pre + "mix.g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
       ENG_CUDA(tensor(L.ukT, (size_t)H * r * d, M.f32));
       name(pre + "mix.uk", &L.ukT, 0, {H * d, r}, i, /*transpose each head's [d][r] block*/ 1);
-      ENG_CUDA(tensor(L.uv, (size_t)H * dv * r, M.f32));
+      {
+        const char *fl = getenv("DIS_STACK_LATENT_FLASH");  // 0: long portions as products over the latents (A/B runs)
+        L.flash = !(fl && atoi(fl) == 0) && stack_tc && stack_latent_flash_ok(stack_latent_shape(lc, sc->norm_eps), M.f32);
+      }
+      if (L.flash) {
+        ENG_CUDA(tensor(L.ukv, (size_t)H * (d + dv) * r, false));
+        L.uv.n = (size_t)H * dv * r; L.uv.f32 = false;
+        L.uv.ptr = reinterpret_cast<uint16_t *>(L.ukv.ptr) + (size_t)H * d * r;
+        lat_row = std::max(lat_row, (size_t)H * (d + dv) + r + dr);
+        lat_w[0] = std::max(lat_w[0], (size_t)r); lat_w[1] = std::max(lat_w[1], (size_t)dr); lat_w[2] = std::max(lat_w[2], (size_t)H * (d + dv));
+      } else ENG_CUDA(tensor(L.uv, (size_t)H * dv * r, M.f32));
       name(pre + "mix.uv", &L.uv, 0, {H * dv, r}, i);
       if (!(lc.latent_flags & DIS_LATENT_NO_SINK)) {
         ENG_CUDA(tensor(L.sink, (size_t)H, true));
@@ -756,6 +770,15 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_cgt), (size_t)M.lat_ctx_cap * max_r * 2));
       ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_s), M.lat_s_elems * 4));
       ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_p), M.lat_s_elems * 2));
+      if (lat_row) {  // rows for two passes' worth of tokens or one whole history, within 1 GiB; what does not fit runs as products
+        size_t rows = std::min((size_t)max_batch * M.lat_ctx_cap, std::max((size_t)2 * cap_tokens, (size_t)M.lat_ctx_cap));
+        rows = std::min(rows, ((size_t)1 << 30) / (lat_row * 2)) / 8 * 8;
+        if (const char *g = getenv("DIS_STACK_LATENT_ROWS")) rows = std::min(rows, (size_t)std::max(8, atoi(g)) / 8 * 8);  // (tests)
+        M.lat_rows = (int)rows;
+        ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_rc), rows * lat_w[0] * 2));
+        ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_rk), rows * std::max((size_t)8, lat_w[1]) * 2));
+        ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_kv), rows * lat_w[2] * 2));
+      }
     }
   }
   {
@@ -783,7 +806,6 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     M.lat_part_elems = (size_t)2048 * stack_lat_rec;  // (tokens x slices) of one pass
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.lat_part), M.lat_part_elems * 4));
   }
-  if (const char *g = getenv("DIS_STACK_TC")) stack_tc = atoi(g) != 0;
   if (const char *g = getenv("DIS_STACK_PERSIST")) stack_persist = atoi(g) != 0;
   if (!M.f32 && stack_tc) {
     M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), (size_t)W);
@@ -891,7 +913,12 @@ int Engine::load_named(const char *nm, const void *host, int dtype, const int64_
   if (dtype == DIS_F32) memcpy(f.data(), host, n * 4);
   else for (size_t i = 0; i < n; i++) f[i] = bf16_bits_to_float(reinterpret_cast<const uint16_t *>(host)[i]);
   if (t.transform == 3) for (float &v : f) v += 1.f;  // a gain stored as its distance from one
-  if (t.transform == 1) {  // [H*d][r] -> per head [r][d]
+  if (t.transform == 1) {  // [H*d][r] -> per head [r][d]; as it is in front of ukv where the layer has that
+    if (stack->layers[(size_t)t.layer].flash) {
+      std::vector<uint16_t> b(n);
+      for (size_t i = 0; i < n; i++) b[i] = float_to_bf16_bits(f[i]);
+      ENG_CUDA(cudaMemcpy(stack->layers[(size_t)t.layer].ukv.ptr, b.data(), n * 2, cudaMemcpyHostToDevice));
+    }
     const dis_layer_config &lc = stack->layers[(size_t)t.layer].c;
     const size_t H = (size_t)lc.heads, d = (size_t)lc.dim, r = (size_t)lc.kv_rank;
     std::vector<float> g(n);
@@ -982,7 +1009,7 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
   std::vector<int> take(idx.size());
   plan_mixed_step((int)idx.size(), rem.data(), max_prefill_tokens > 0 ? max_prefill_tokens : cap_tokens, cap_tokens, take.data());
   StepMeta &mt = meta_pre;
-  int T = 0, R = 0, SP = 0, QB = 0, KB = 0;
+  int T = 0, R = 0, SP = 0, QB = 0, KB = 0, LB = 0, LS = 0;
   stack_max_ctx = 0;
   stack_spans_h.clear();
   bool all_greedy = true;
@@ -1020,7 +1047,19 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
     SP++;
     // long portions: latent attention as matrix products; short ones and decode rows: query blocks of the paged kernel
     const bool products = M.lat_gemm && tk >= 32 && (size_t)stack_lat_heads * ((p0 + tk + 7) / 8 * 8) <= M.lat_s_elems;
-    stack_spans_h.push_back({T, tk, p0, slots[i], products});
+    StackSpanH shn{T, tk, p0, slots[i], products};
+    if (products) {
+      const int fb = stack_latent_flash_tokens();
+      shn.lb0 = LB; shn.ls = LS;
+      for (int j = 0; j < tk; j += fb) {
+        mt.h<int>(mt.o_lb_tok0)[LB] = T + j;
+        mt.h<int>(mt.o_lb_len)[LB] = std::min(fb, tk - j);
+        LB++;
+      }
+      shn.n_lb = LB - shn.lb0;
+      mt.h<int>(mt.o_ls)[LS++] = SP - 1;
+    }
+    stack_spans_h.push_back(shn);
     for (int j = 0; j < tk && !products; j += stack_bq) {
       mt.h<int>(mt.o_ab_tok0)[QB] = T + j;
       mt.h<int>(mt.o_ab_len)[QB] = std::min(stack_bq, tk - j);
@@ -1048,6 +1087,25 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
     T += tk;
   }
   if (T == 0) { last_rows = 0; return DIS_OK; }
+  // latent layers that make per-head keys and values for the long spans: rows are given out span by span, a group ends where they
+  // run out; a span that alone has more keys than there are rows stays out (it runs as products)
+  stack_lat_groups.assign((size_t)M.n_lat, {});
+  for (size_t li = 0; li < M.layers.size() && LS > 0 && M.lat_rows > 0; li++) {
+    const StackLayer &L = M.layers[li];
+    if (!L.flash) continue;
+    const StackLatent sl = stack_latent_shape(L.c, m.rms_eps);
+    auto &groups = stack_lat_groups[(size_t)L.lat_ix];
+    bool open = false;
+    for (auto &sh : stack_spans_h) {
+      if (!sh.products) continue;
+      const int first = stack_latent_row_lo(sl, sh.pos0), keys = sh.pos0 + sh.len - first;
+      if (keys > M.lat_rows) { open = false; continue; }
+      if (!open || groups.back().rows + keys > M.lat_rows) { groups.push_back({sh.ls, 0, 0, 0, sh.lb0, 0}); open = true; }
+      StackLatGroup &g = groups.back();
+      mt.h<int>(mt.o_lin)[(size_t)L.lat_ix * max_batch + sh.slot] = g.rows - first;
+      g.n++; g.rows += keys; g.max_keys = std::max(g.max_keys, keys); g.n_lb += sh.n_lb;
+    }
+  }
   if (pt_dirty) {
     ENG_CUDA(cudaMemcpyAsync(d_page_table, h_page_table, (size_t)max_batch * max_pages * sizeof(int), cudaMemcpyHostToDevice, stream));
     pt_dirty = false;
@@ -1477,6 +1535,21 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       const bool gated = !(lc.latent_flags & DIS_LATENT_NO_GATE);
       const float *gate = gated ? M.proj + L.g_off : nullptr;
       StackRun &KV = M.runs[(size_t)Rn.kv_run];
+      // Long spans of a flash layer make their own keys and values per head; the other tokens keep to the latents: their runs
+      const std::vector<StackLatGroup> &groups = stack_lat_groups[(size_t)L.lat_ix];
+      auto in_flash = [&](const StackSpanH &sh) {
+        if (!sh.products) return false;
+        for (auto &g : groups) if (sh.ls >= g.ls0 && sh.ls < g.ls0 + g.n) return true;
+        return false;
+      };
+      std::vector<std::pair<int, int>> runs;  // (first token, tokens)
+      bool any_products = false;
+      for (auto &sh : stack_spans_h) {
+        if (in_flash(sh)) continue;
+        any_products = any_products || sh.products;
+        if (!runs.empty() && runs.back().first + runs.back().second == sh.tok0) runs.back().second += sh.len;
+        else runs.push_back({sh.tok0, sh.len});
+      }
       const float *qsrc = in_src;  // the queries [T][q_ld]: columns L.q_off + h * (d + dr)
       long long q_ld = N;
       {
@@ -1485,7 +1558,10 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         a.q_off = L.q_off; a.dkv_off = L.dkv_off;
         if (lc.kv_from < 0) { a.dkv_norm = reinterpret_cast<const float *>(L.norm_w.ptr); a.pool = Rn.pool; }
         if (lc.q_rank > 0) { a.dq_off = 0; a.dq_norm = reinterpret_cast<const float *>(L.q_norm.ptr); a.cq = M.cq; }
-        else a.qf = M.qf;
+        else {
+          if (!runs.empty()) a.qf = M.qf;
+          if (!groups.empty()) { a.qx = M.proj + L.q_off; a.ld_qx = N; }
+        }
         if (in_parts > 1) {  // sliced projection: the columns that later kernels read go to M.proj
           a.keep = M.proj; a.ld_keep = N;
           if (lc.q_rank > 0) { a.keep = gated ? M.proj + L.g_off : nullptr; a.keep_off = L.g_off; a.keep_n = L.n_in - L.g_off; }
@@ -1493,48 +1569,62 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
           qsrc = M.proj;
         }
         RET_CUDA(launch_stack_latent_prep(a, sl, sp, f32, d_page_table, max_pages, page_size, stream));
+        kl++;
       }
       if (lc.q_rank > 0) {  // queries from their latent, then their rotation
-        RET_CUDA(gemm(M.cq, f32, lc.q_rank, L.w_uq, 0, nullptr, M.ql, T, H * (d + dr), lc.q_rank, cap_tokens));
-        qsrc = M.ql; q_ld = (long long)H * (d + dr);
+        const int nq = H * (d + dr);
+        RET_CUDA(gemm(M.cq, f32, lc.q_rank, L.w_uq, 0, nullptr, M.ql, T, nq, lc.q_rank, cap_tokens, nullptr, true));
+        qsrc = M.ql; q_ld = nq;
         StackLatentPrep a;
-        a.proj = M.ql; a.ld = q_ld; a.n_cols = H * (d + dr); a.freq = L.freq; a.qf = M.qf;
+        a.proj = M.ql; a.ld = q_ld; a.n_cols = nq; a.freq = L.freq;
+        if (pend_parts > 1) { a.proj = pend_src; a.n_part = pend_parts; a.stride = pend_stride; a.keep = M.ql; a.ld_keep = q_ld; a.keep_n = nq; }
+        pend_parts = 1; pend_bias = nullptr;
+        if (!runs.empty()) a.qf = M.qf;
+        if (!groups.empty()) { a.qx = M.ql; a.ld_qx = q_ld; }
         RET_CUDA(launch_stack_latent_prep(a, sl, sp, f32, d_page_table, max_pages, page_size, stream));
         kl++;
       }
-      // absorbed queries: qf[t][h][0..r) = sum_a q[t][h][a] * uk[h*d + a][.]  (one batch entry per head).  Large bf16 passes:
-      // one tensor-core product per head over the head's queries packed contiguously; else the batched fp32-FMA product.
-      const bool head_tc = M.lat_gemm && T >= 256 && !L.ukT.f32 && !L.uv.f32 && d % 8 == 0 && ((size_t)r * d * 2) % 16 == 0 &&
-                           ((size_t)dv * r * 2) % 16 == 0 && ((size_t)T * d * 2) % 16 == 0 && ((size_t)T * r * 2) % 16 == 0;
-      if (head_tc) {
-        RET_CUDA(launch_stack_heads_pack(qsrc, q_ld, L.q_off, d + dr, d, T, H, M.lat_qb, stream));
-        for (int h = 0; h < H; h++) {
-          TmaMap xm;
-          RET_CUDA(make_tma_map_2d(&xm, M.lat_qb + (size_t)h * T * d, (uint64_t)T, (uint64_t)d, (uint32_t)gemm_token_tile(T)));
-          const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.ukT.ptr) + (size_t)h * r * d, (uint64_t)r, (uint64_t)d, 128);
-          if (!wm) return cudaErrorInvalidValue;
-          RET_CUDA(launch_gemm_partial(*wm, xm, M.mix2 + (size_t)h * T * r, T, r, d, 0, 1, stream));
+      // large runs of bf16 tokens: one tensor-core product per head over the head's rows packed contiguously; else the batched product
+      auto head_tc = [&](int n) {
+        return M.lat_gemm && n >= 256 && !L.ukT.f32 && !L.uv.f32 && d % 8 == 0 && ((size_t)r * d * 2) % 16 == 0 && ((size_t)dv * r * 2) % 16 == 0 &&
+               ((size_t)n * d * 2) % 16 == 0 && ((size_t)n * r * 2) % 16 == 0;
+      };
+      // absorbed queries: qf[t][h][0..r) = sum_a q[t][h][a] * uk[h*d + a][.]  (one batch entry per head)
+      for (auto &run : runs) {
+        const int t0 = run.first, n = run.second;
+        const float *qr = qsrc + (size_t)t0 * q_ld;
+        float *qo = M.qf + (size_t)t0 * H * D;
+        if (head_tc(n)) {
+          RET_CUDA(launch_stack_heads_pack(qr, q_ld, L.q_off, d + dr, d, n, H, M.lat_qb, stream));
+          for (int h = 0; h < H; h++) {
+            TmaMap xm;
+            RET_CUDA(make_tma_map_2d(&xm, M.lat_qb + (size_t)h * n * d, (uint64_t)n, (uint64_t)d, (uint32_t)gemm_token_tile(n)));
+            const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.ukT.ptr) + (size_t)h * r * d, (uint64_t)r, (uint64_t)d, 128);
+            if (!wm) return cudaErrorInvalidValue;
+            RET_CUDA(launch_gemm_partial(*wm, xm, M.mix2 + (size_t)h * n * r, n, r, d, 0, 1, stream));
+          }
+          RET_CUDA(launch_stack_heads_unpack(M.mix2, r, n, H, qo, (long long)H * D, 0, D, stream));
+          kl += H + 2;
+        } else {
+          StackGemm g;
+          g.A = qr + L.q_off; g.a_f32 = true; g.lda = q_ld; g.a_bs = d + dr;
+          g.W = L.ukT.ptr; g.w_f32 = L.ukT.f32; g.ldw = d; g.w_bs = (long long)r * d;
+          g.out = qo; g.ldo = (long long)H * D; g.o_bs = D;
+          g.M = n; g.N = r; g.K = d; g.batch = H;
+          RET_CUDA(launch_stack_gemm(g, stream));
+          kl++;
         }
-        RET_CUDA(launch_stack_heads_unpack(M.mix2, r, T, H, M.qf, (long long)H * D, 0, D, stream));
-        kl += H + 1;
-      } else {
-        StackGemm g;
-        g.A = qsrc + L.q_off; g.a_f32 = true; g.lda = q_ld; g.a_bs = d + dr;
-        g.W = L.ukT.ptr; g.w_f32 = L.ukT.f32; g.ldw = d; g.w_bs = (long long)r * d;
-        g.out = M.qf; g.ldo = (long long)H * D; g.o_bs = D;
-        g.M = T; g.N = r; g.K = d; g.batch = H;
-        RET_CUDA(launch_stack_gemm(g, stream));
       }
-      RET_CUDA(launch_stack_latent_attn(M.qf, KV.pool, f32, reinterpret_cast<const float *>(L.sink.ptr), sl, sp, mt.d<int>(mt.o_ab_tok0),
-                                        mt.d<int>(mt.o_ab_len), n_qb, d_page_table, max_pages, page_size, M.mix, slices.first, slices.second,
-                                        M.lat_part, stream));
-      if (slices.first > 1) kl++;
-      bool any_products = false;
-      for (auto &sh : stack_spans_h) any_products = any_products || sh.products;
+      if (n_qb > 0) {
+        RET_CUDA(launch_stack_latent_attn(M.qf, KV.pool, f32, reinterpret_cast<const float *>(L.sink.ptr), sl, sp, mt.d<int>(mt.o_ab_tok0),
+                                          mt.d<int>(mt.o_ab_len), n_qb, d_page_table, max_pages, page_size, M.mix, slices.first, slices.second,
+                                          M.lat_part, stream));
+        kl += slices.first > 1 ? 2 : 1;
+      }
       if (any_products) {
         RET_CUDA(launch_stack_copy_act(M.qf, M.lat_qb, false, (long long)T * H * D, stream)); kl++;
         for (auto &sh : stack_spans_h) {
-          if (!sh.products) continue;
+          if (!sh.products || in_flash(sh)) continue;
           const int first = stack_latent_row_lo(sl, sh.pos0) / 8 * 8;  // with a window: the first key any of the span's tokens sees, rounded down
           const int pos0 = sh.pos0 - first, ctx = pos0 + sh.len, ctx8 = (ctx + 7) / 8 * 8;  // positions from there on
           RET_CUDA(launch_stack_latent_gather(KV.pool, d_page_table + (size_t)sh.slot * max_pages, page_size, D, r, ctx, ctx8, M.lat_cg,
@@ -1558,27 +1648,48 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         }
       }
       // values: mix2[t][h][0..dv) = sum_b ol[t][h][b] * uv[h*dv + .][b]
-      if (head_tc) {
-        RET_CUDA(launch_stack_heads_pack(M.mix, (long long)H * r, 0, r, r, T, H, M.lat_qb, stream));
-        for (int h = 0; h < H; h++) {
-          TmaMap xm;
-          RET_CUDA(make_tma_map_2d(&xm, M.lat_qb + (size_t)h * T * r, (uint64_t)T, (uint64_t)r, (uint32_t)gemm_token_tile(T)));
-          const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.uv.ptr) + (size_t)h * dv * r, (uint64_t)dv, (uint64_t)r, 128);
-          if (!wm) return cudaErrorInvalidValue;
-          RET_CUDA(launch_gemm_partial(*wm, xm, M.mix2 + (size_t)h * T * dv, T, dv, r, 0, 1, stream));
+      for (auto &run : runs) {
+        const int t0 = run.first, n = run.second;
+        const float *ol = M.mix + (size_t)t0 * H * r, *gt = gate ? gate + (size_t)t0 * N : nullptr;
+        void *ao = f32 ? (void *)(reinterpret_cast<float *>(M.act) + (size_t)t0 * L.ld_act) : (void *)(reinterpret_cast<uint16_t *>(M.act) + (size_t)t0 * L.ld_act);
+        if (head_tc(n)) {
+          RET_CUDA(launch_stack_heads_pack(ol, (long long)H * r, 0, r, r, n, H, M.lat_qb, stream));
+          for (int h = 0; h < H; h++) {
+            TmaMap xm;
+            RET_CUDA(make_tma_map_2d(&xm, M.lat_qb + (size_t)h * n * r, (uint64_t)n, (uint64_t)r, (uint32_t)gemm_token_tile(n)));
+            const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.uv.ptr) + (size_t)h * dv * r, (uint64_t)dv, (uint64_t)r, 128);
+            if (!wm) return cudaErrorInvalidValue;
+            RET_CUDA(launch_gemm_partial(*wm, xm, M.mix2 + (size_t)h * n * dv, n, dv, r, 0, 1, stream));
+          }
+          RET_CUDA(launch_stack_gate(M.mix2, gt, N, ao, f32, n, H * dv, H, stream, L.ld_act));
+          kl += H + 2;
+        } else {
+          StackGemm v;
+          v.A = ol; v.a_f32 = true; v.lda = (long long)H * r; v.a_bs = r;
+          v.W = L.uv.ptr; v.w_f32 = L.uv.f32; v.ldw = r; v.w_bs = (long long)dv * r;
+          v.out = M.mix2; v.ldo = (long long)H * dv; v.o_bs = dv;
+          v.M = n; v.N = dv; v.K = r; v.batch = H;
+          RET_CUDA(launch_stack_gemm(v, stream));
+          RET_CUDA(launch_stack_gate(M.mix2, gt, N, ao, f32, n, H * dv, 0, stream, L.ld_act));
+          kl += 2;
         }
-        RET_CUDA(launch_stack_gate(M.mix2, gate, N, M.act, f32, T, H * dv, H, stream, L.ld_act));
-        kl += H;
-      } else {
-        StackGemm v;
-        v.A = M.mix; v.a_f32 = true; v.lda = (long long)H * r; v.a_bs = r;
-        v.W = L.uv.ptr; v.w_f32 = L.uv.f32; v.ldw = r; v.w_bs = (long long)dv * r;
-        v.out = M.mix2; v.ldo = (long long)H * dv; v.o_bs = dv;
-        v.M = T; v.N = dv; v.K = r; v.batch = H;
-        RET_CUDA(launch_stack_gemm(v, stream));
-        RET_CUDA(launch_stack_gate(M.mix2, gate, N, M.act, f32, T, H * dv, 0, stream, L.ld_act));
       }
-      kl += 5;
+      // long spans: gathered latents -> per-head keys and values (one product with [uk ; uv]) -> the tensor-core attention kernel
+      for (auto &g : groups) {
+        const int *lin = mt.d<int>(mt.o_lin) + (size_t)L.lat_ix * max_batch;
+        const int nkv = H * (d + dv);
+        RET_CUDA(launch_stack_latent_rows(KV.pool, sl, sp, mt.d<int>(mt.o_ls) + g.ls0, g.n, g.max_keys, lin, d_page_table, max_pages, page_size,
+                                          M.lat_rc, M.lat_rk, stream));
+        const bool persist = stack_persist && gemm_use_persist(g.rows, nkv, false);
+        const TmaMap *xm = stack_map(M.lat_rc, (uint64_t)M.lat_rows, (uint64_t)r, persist ? 256u : (uint32_t)gemm_token_tile(g.rows));
+        const TmaMap *wm = stack_map(L.ukv.ptr, (uint64_t)nkv, (uint64_t)r, 128);
+        if (!xm || !wm) return cudaErrorInvalidValue;
+        if (persist) RET_CUDA(launch_gemm_persist_bf16(*wm, *xm, M.lat_kv, g.rows, nkv, r, 0, stream));
+        else RET_CUDA(launch_gemm_bf16(*wm, *xm, M.lat_kv, g.rows, nkv, r, 0, stream));
+        RET_CUDA(launch_stack_latent_flash(qsrc + L.q_off, q_ld, M.lat_kv, M.lat_rk, lin, reinterpret_cast<const float *>(L.sink.ptr), sl, sp,
+                                           mt.d<int>(mt.o_lb_tok0) + g.lb0, mt.d<int>(mt.o_lb_len) + g.lb0, g.n_lb, M.act, L.ld_act, gate, N, stream));
+        kl += 3;
+      }
       n_mix = L.ld_act;
     }
     RET_CUDA(gemm(M.act, f32, n_mix, L.w_o, 0, o_bias, M.y, T, W, n_mix, cap_tokens, nullptr, later));

@@ -218,6 +218,8 @@ struct StackLatentPrep {
   int n_part = 1, n_cols = 0;
   int q_off = 0;                // queries [H][d + dr]: their rotated parts go to qf (when given)
   float *qf = nullptr;
+  float *qx = nullptr;          // and back where the queries lie (when given): [T][ld_qx], first head's column
+  long long ld_qx = 0;
   int dkv_off = 0;              // latent and rotated key part: to the pool (when given)
   const float *dkv_norm = nullptr;
   void *pool = nullptr;
@@ -243,7 +245,19 @@ cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32
                                      const StackSpans &sp, const int *qb_tok0, const int *qb_len, int n_qb,
                                      const int *page_table, int max_pages, int page_size, float *ol, int n_split,
                                      int keys_per_split, float *part, cudaStream_t st);
-// Long prompt portions in bf16: latents of one sequence out of their pages into cg [ctx8][D] and cgt [r][ctx8] (rows / columns
+// Prompt portions in bf16, sizes within the tensor-core attention kernel's (stack_latent_flash_ok): per-head keys and values are made
+// from the gathered latents by one product with [uk ; uv], and that kernel runs over them -- its work is bounded by the window and its
+// rows are 64 tokens of one head.  Blocks: stack_latent_flash_tokens() tokens.  lin [slots]: row of position 0 of the slot's sequence.
+bool stack_latent_flash_ok(const StackLatent &c, bool f32);
+int stack_latent_flash_tokens();
+cudaError_t launch_stack_latent_rows(const void *pool, const StackLatent &c, const StackSpans &sp, const int *ls, int n_ls, int max_keys,
+                                     const int *lin, const int *page_table, int max_pages, int page_size, uint16_t *cg, uint16_t *krot,
+                                     cudaStream_t st);
+// q [T][ldq], head h at columns h * (d + dr); result (times sigmoid(gate [T][ld_gate]) element by element when given) to out [T][ld_out]
+cudaError_t launch_stack_latent_flash(const float *q, long long ldq, const uint16_t *kv, const uint16_t *krot, const int *lin, const float *sink,
+                                      const StackLatent &c, const StackSpans &sp, const int *qb_tok0, const int *qb_len, int n_qb, void *out,
+                                      long long ld_out, const float *gate, long long ld_gate, cudaStream_t st);
+// Otherwise: latents of one sequence out of their pages into cg [ctx8][D] and cgt [r][ctx8] (rows / columns
 // from ctx to ctx8 zero), and softmax weights (bf16) from a block of raw score rows; the products between run on tcgen05.
 cudaError_t launch_stack_latent_gather(const void *pool, const int *pt_row, int page_size, int D, int r, int ctx, int ctx8,
                                        uint16_t *cg, uint16_t *cgt, int first, cudaStream_t st);  // first: position of row 0
@@ -297,7 +311,8 @@ struct StackLayer {
   StackTensor w_o;      // output projection
   StackTensor norm_w;   // lightning: gain of the head norm; latent: gain of the latent norm (fp32)
   StackTensor ukT;      // latent: per head [r][d] = transpose of the head's block of the key up-projection
-  StackTensor uv;       // latent: [H*dv][r]
+  StackTensor uv;       // latent: [H*dv][r] (the second part of ukv when the layer has that)
+  StackTensor ukv;      // latent in bf16 with tensor-core sizes: [H*d + H*dv][r], the two up-projections as loaded
   StackTensor sink;     // latent, attention with DIS_ATTN_SINK: [H] fp32
   StackTensor decay_d;  // lightning: [H] fp32
   int n_in = 0, q_off = 0, dkv_off = 0, g_off = 0;
@@ -315,6 +330,8 @@ struct StackLayer {
   int n_rows = 0;        // rows of w_in: n_in, then the parallel feed-forward's gate | up
   int ld_act = 0;        // columns of w_o: n_act, then the parallel feed-forward's par_ff
   StackTensor vmix;      // attention with DIS_ATTN_V_MIX: the scalar weight of the first layer's values
+  int lat_ix = -1;       // latent: index among the latent layers
+  bool flash = false;    // latent: prompt portions run on per-head keys and values
   StackTensor w_uq, q_norm;  // latent with a query latent: [H*(d+dr)][q_rank] compute type, gain of its norm [q_rank] fp32
   // gated linear attention (second half of a parallel mixer): w_in rows q | k | v | g | bottleneck behind the attention's
   int gq_off = 0, gk_off = 0, gv_off = 0, gg_off = 0, ga_off = 0;
@@ -374,7 +391,10 @@ struct StackModel {
   float *x = nullptr, *y = nullptr, *hn = nullptr, *proj = nullptr, *mix = nullptr, *mix2 = nullptr, *qf = nullptr, *logits = nullptr;
   void *hc = nullptr, *act = nullptr, *xr = nullptr;
   // latent attention of long portions as matrix products: bf16 queries, gathered latents and their transpose, score block, weights
-  bool lat_gemm = false;
+  bool lat_gemm = false;  // long portions leave the blocks of the paged latent kernel
+  // latents gathered for the per-head keys and values of prompt portions, and those: lat_rows rows
+  int lat_rows = 0, n_lat = 0;     // n_lat: latent layers
+  uint16_t *lat_rc = nullptr, *lat_rk = nullptr, *lat_kv = nullptr;
   int lat_ctx_cap = 0;
   size_t lat_s_elems = 0;
   uint16_t *lat_qb = nullptr, *lat_cg = nullptr, *lat_cgt = nullptr, *lat_p = nullptr;

@@ -129,6 +129,35 @@ def test_tensor_core_shapes(name):
         assert float(np.quantile(e16, 0.8)) < 3e-2 and float(e16.max()) < 0.3, cuts
 
 
+LATENT_ROUTES = {  # how prompt portions of latent layers run in bfloat16: per-head keys and values; products over the latents; both in one pass
+    "per_head": {}, "products": {"DIS_STACK_LATENT_FLASH": "0"}, "rows_for_one_span": {"DIS_STACK_LATENT_ROWS": "152"}, "rows_for_short_spans_only": {"DIS_STACK_LATENT_ROWS": "104"},
+    "fp32_products": {"DIS_STACK_TC": "0"},
+}
+
+
+@pytest.mark.parametrize("route", sorted(LATENT_ROUTES))
+def test_prompt_portions_of_latent_layers(route, monkeypatch):
+    """Four sequences' portions beside a decoded token in one pass, with histories: all through per-head keys and values in one
+    group or a group per span, through the products over the latents, or span by span either way (a span with more keys than rows)."""
+    for k, v in LATENT_ROUTES[route].items():
+        monkeypatch.setenv(k, v)
+    cfg = U.config([(U.latent(heads=4, dim=16, rot_dim=16, vdim=16, kv_rank=32, q_rank=24, window=0), U.dense(24)), (U.latent(heads=3, dim=24, rot_dim=8, vdim=32, kv_rank=40, q_rank=16, window=70), None),
+                    (U.latent(heads=2, dim=8, rot_dim=8, vdim=16, kv_rank=24, q_rank=0, window=50), U.dense(24))], width=40)
+    W = U.weights(cfg, seed=22)
+    seqs = {k: toks(n, seed=60 + k) for k, n in enumerate((150, 140, 100, 90, 60))}
+    want = {k: U.oracle_logits(cfg, W, v) for k, v in seqs.items()}
+    e = U.engine(cfg, W, "bfloat16", max_batch=5, pool_tokens=640, page_size=16, max_step_tokens=300)
+    f = U.Feeder(e)
+    f.step([(0, seqs[0], 100), (1, seqs[1], 33), (4, seqs[4], 31)])
+    f.step([(1, seqs[1], 70), (0, seqs[0], 1), (2, seqs[2], 64), (4, seqs[4], 1), (3, seqs[3], 40)])
+    f.step([(0, seqs[0], 49), (4, seqs[4], 1), (1, seqs[1], 37), (2, seqs[2], 36), (3, seqs[3], 50)])
+    f.step([(4, seqs[4], 27)])
+    for k in seqs:
+        e16 = U.row_errs(f.end(k), want[k])
+        assert float(e16.max()) < 3e-2, (route, k, int(e16.argmax()))
+    e.close()
+
+
 def test_attention_over_slices_of_the_history():
     """A single decoding sequence with a long visible history has its keys cut into slices that a second kernel merges.  A layer
     without a window slices the whole history, one with a long window its window and the kept positions, one with a short window
