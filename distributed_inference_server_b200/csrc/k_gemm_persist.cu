@@ -150,7 +150,7 @@ gemm_persist_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
               const int t = t0 + c + jj;
               if (t < T) {
                 const float gv = __uint_as_float(g[jj]), uv = __uint_as_float(u[jj]);
-                out_act[(size_t)t * N + n] = float_to_bf16_bits((gv / (1.0f + expf(-gv))) * uv);
+                out_act[(size_t)t * N + n] = float_to_bf16_bits(gate_act_fast(0, gv) * uv);
               }
             }
           }
@@ -325,8 +325,7 @@ gemm_persist_pair_kernel(const __grid_constant__ CUtensorMap w_map64, const __gr
               const float other = take[jj * 32 + lane], mine = __uint_as_float(kv[jj]);
               const float gv = is_up ? other : mine, uv = is_up ? mine : other;
               // act_kind 0: silu(gate) * up; 1: gelu_tanh(gate) * up
-              const float av = act_kind == 1 ? 0.5f * gv * (1.f + tanhf(0.7978845608028654f * (gv + 0.044715f * gv * gv * gv)))
-                                             : gv / (1.0f + expf(-gv));
+              const float av = gate_act_fast(act_kind, gv);
               out_act[(size_t)t * ld_act + n] = float_to_bf16_bits(av * uv);
             }
           }

@@ -171,8 +171,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
             if (t < T) {
               const float gv = __uint_as_float(g[jj]), uv = __uint_as_float(u[jj]);
               // act_kind 0: silu(gate) * up; 1: gelu_tanh(gate) * up
-              const float av = act_kind == 1 ? 0.5f * gv * (1.f + tanhf(0.7978845608028654f * (gv + 0.044715f * gv * gv * gv)))
-                                             : gv / (1.0f + expf(-gv));
+              const float av = gate_act_fast(act_kind, gv);
               out_act[(size_t)t * ld_act + n] = float_to_bf16_bits(av * uv);
             }
           }

@@ -18,7 +18,7 @@ namespace dis {
 // (DIS_ATTN_GATE_FULL) H*dv of them (the logits of the output gates, which the attention kernel reads from memory).
 // mix: DIS_ATTN_V_MIX -- the first such layer of a pass leaves its values in mix.save, the later ones blend theirs with them.
 template <bool F32>
-__global__ void __launch_bounds__(128) stack_attn_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
+__global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
                                                               int gate_off, float *gate_out, long long ld_gate, int q_off, int k_off, int v_off,
                                                               const float *bias, const float *qn, const float *kn, const double *freq,
                                                               const double *vfreq, StackAttn c, StackSpans sp, float *qf, void *kpool,
@@ -137,8 +137,9 @@ cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, 
     cudaError_t e = cudaFuncSetAttribute(stack_attn_prep_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_attn_prep_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   }));
-  if (f32) stack_attn_prep_kernel<true><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
-  else stack_attn_prep_kernel<false><<<sp.T, 128, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
+  const int th = sp.T <= 148 ? 512 : 128;  // few tokens: a block per token leaves the GPU empty, so the blocks are large
+  if (f32) stack_attn_prep_kernel<true><<<sp.T, th, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
+  else stack_attn_prep_kernel<false><<<sp.T, th, sh, st>>>(proj, ld, n_part, stride, n_cols, gate_off, gate_out, ld_gate, q_off, k_off, v_off, bias, qn, kn, freq, vfreq, c, sp, qf, kpool, vpool, vrot, page_table, max_pages, page_size, mix);
   return cudaGetLastError();
 }
 

@@ -89,12 +89,21 @@ __global__ void __launch_bounds__(256) stack_lightning_kernel(const float *proj,
 // GATE 3 (retention): one decay per head as in GATE 0, but q, k and v enter as they are.
 // Rows and columns beyond d and dv: shared memory starts as zeros and nobody writes those entries, so their k, q and decays are
 // zero and their part of S stays zero; the inner loop needs no bounds checks.
+// Retention's outputs can leave the kernel finished (fin.act): each token's o of the head is divided by its root mean square, times
+// silu(gate), and stored in the compute type at act [T][ld], columns h * dv + j -- eight tokens of a group, one per warp.
+struct LightFin {
+  void *act = nullptr;
+  long long ld = 0, ldg = 0;
+  const float *gate = nullptr;  // [T][ldg], columns h * dv + j
+  float eps = 0.f;
+  int f32 = 0;
+};
 constexpr int kLightTok = 8, kLightSeg = 64;
 template <int RI, int RJ, int MODE, int GATE>
 __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float *__restrict__ proj, long long ld, LightCols col,
                                                                      const float *decay, const float *__restrict__ dec, float qscale,
                                                                      float *state, StackSpans sp, float *__restrict__ o, int H, int d,
-                                                                     int dv, float *seg, float *seg_a, int max_seg) {
+                                                                     int dv, float *seg, float *seg_a, int max_seg, LightFin fin) {
   extern __shared__ __align__(16) float shm[];
   constexpr int DP = RI * 8, DVP = RJ * 32;
   constexpr bool DEC = GATE == 1 || GATE == 2;  // decays come per token
@@ -215,7 +224,31 @@ __global__ void __launch_bounds__(256, 2) stack_lightning_reg_kernel(const float
         for (int jj = 0; jj < RJ; jj++) part[(t * 8 + w) * DVP + l + jj * 32] = acc[jj];
       }
     }
-    if (MODE != 1) {
+    if (GATE == 3 && MODE != 1 && fin.act) {  // warp w finishes token w of the group
+      __syncthreads();
+      if (w < ct) {
+        float ov[RJ], ss = 0.f;
+#pragma unroll
+        for (int jj = 0; jj < RJ; jj++) {
+          float acc = 0.f;
+#pragma unroll
+          for (int k = 0; k < 8; k++) acc += part[(w * 8 + k) * DVP + l + jj * 32];
+          ov[jj] = acc;  // columns beyond dv are zero
+          ss += acc * acc;
+        }
+        const float r = rsqrtf(warp_sum(ss) / (float)dv + fin.eps);
+        const long long t = first + t0 + w;
+#pragma unroll
+        for (int jj = 0; jj < RJ; jj++) {
+          const int j = l + jj * 32;
+          if (j < dv) {
+            const float v = ov[jj] * r * silu_(fin.gate[t * fin.ldg + (long long)h * dv + j]);
+            if (fin.f32) st_el<true>(fin.act, t * fin.ld + (long long)h * dv + j, v);
+            else st_el<false>(fin.act, t * fin.ld + (long long)h * dv + j, v);
+          }
+        }
+      }
+    } else if (MODE != 1) {
       __syncthreads();
       for (int e = threadIdx.x; e < ct * dv; e += blockDim.x) {
         const int t = e / dv, j = e - t * dv;
@@ -320,7 +353,7 @@ size_t stack_lightning_seg_decay_floats(int cap_tokens, int max_spans, int H, in
 template <int RI, int RJ, int GATE>
 static cudaError_t lightning_reg(const float *proj, long long ld, LightCols col, const float *decay, const float *dec, float qscale,
                                  float *state, const StackSpans &sp, float *o, int H, int d, int dv, float *seg, float *seg_a,
-                                 int max_len, cudaStream_t st) {
+                                 int max_len, cudaStream_t st, const LightFin &fin = LightFin()) {
   constexpr bool DEC = GATE == 1 || GATE == 2;
   const size_t sh = (size_t)kLightTok * ((DEC ? 3 : 2) * RI * 8 + RJ * 32 + 8 * RJ * 32) * sizeof(float);
   static DeviceOnce once;
@@ -330,13 +363,13 @@ static cudaError_t lightning_reg(const float *proj, long long ld, LightCols col,
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_lightning_reg_kernel<RI, RJ, 2, GATE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
   }));
   if (!seg || (DEC && !seg_a) || max_len <= kLightSeg) {
-    stack_lightning_reg_kernel<RI, RJ, 0, GATE><<<sp.n_spans * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, nullptr, nullptr, 1);
+    stack_lightning_reg_kernel<RI, RJ, 0, GATE><<<sp.n_spans * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, nullptr, nullptr, 1, fin);
     return cudaGetLastError();
   }
   const int max_seg = (max_len + kLightSeg - 1) / kLightSeg;
-  stack_lightning_reg_kernel<RI, RJ, 1, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg);
+  stack_lightning_reg_kernel<RI, RJ, 1, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg, fin);
   stack_lightning_carry_kernel<<<sp.n_spans * H * ((d * dv + 255) / 256), 256, 0, st>>>(decay, DEC ? seg_a : nullptr, state, sp, seg, H, d, dv);
-  stack_lightning_reg_kernel<RI, RJ, 2, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg);
+  stack_lightning_reg_kernel<RI, RJ, 2, GATE><<<sp.n_spans * max_seg * H, 256, sh, st>>>(proj, ld, col, decay, dec, qscale, state, sp, o, H, d, dv, seg, seg_a, max_seg, fin);
   return cudaGetLastError();
 }
 
@@ -358,7 +391,7 @@ cudaError_t launch_stack_lightning(const float *proj, long long ld, const float 
 // In front of the recurrence, one block per token: q and k [H][d] of the token's row are rotated over the first rot_dims
 // coordinates of every head (pairs i, i + rot_dims/2, angle pos * freq[i]), k is multiplied by kscale.  The row comes as n_part
 // slices of n_cols columns (n_part 1: it may be dst itself); every column lands in dst.  Cosine and sine are formed once per token.
-__global__ void __launch_bounds__(256) stack_retention_prep_kernel(const float *src, long long ld_src, int n_part, long long stride,
+__global__ void __launch_bounds__(512) stack_retention_prep_kernel(const float *src, long long ld_src, int n_part, long long stride,
                                                                    int n_cols, float *dst, long long ld_dst, int q_off, int k_off, int H,
                                                                    int d, const double *__restrict__ freq, int rot_dims, float kscale,
                                                                    const int *__restrict__ pos) {
@@ -416,7 +449,7 @@ cudaError_t launch_stack_retention_prep(const float *src, long long ld_src, int 
   if (sh > 200 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_retention_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); }));
-  stack_retention_prep_kernel<<<sp.T, 256, sh, st>>>(src, ld_src, n_part, stride, n_cols, dst, ld_dst, q_off, k_off, H, d, freq, rot_dims, kscale, sp.pos);
+  stack_retention_prep_kernel<<<sp.T, sp.T <= 148 ? 512 : 256, sh, st>>>(src, ld_src, n_part, stride, n_cols, dst, ld_dst, q_off, k_off, H, d, freq, rot_dims, kscale, sp.pos);
   return cudaGetLastError();
 }
 
@@ -429,22 +462,33 @@ int stack_retention_blocks(int d, int dv) {
   return nb;
 }
 cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *decay, float *state,
-                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, cudaStream_t st) {
+                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, const float *gate,
+                                   long long ldg, void *act, long long ld_act, bool f32, float eps, cudaStream_t st) {
   const int nb = stack_retention_blocks(d, dv);
   LightCols col{q_off, k_off, v_off};
   col.hpg = nb;
+  const int H0 = H, dv0 = dv;
   H *= nb; dv /= nb;
-  if (d <= 32 && dv <= 64) return lightning_reg<4, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
-  if (d <= 64 && dv <= 64) return lightning_reg<8, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
-  if (d <= 128 && dv <= 64) return lightning_reg<16, 2, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
-  if (d <= 128 && dv <= 128) return lightning_reg<16, 4, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st);
+  LightFin fin;
+  if (nb == 1) fin = {act, ld_act, ldg, gate, eps, f32 ? 1 : 0};  // (a head in several blocks is normalised by a second kernel)
+#define DIS_RET(RI, RJ)                                                                                                                        \
+  do {                                                                                                                                        \
+    DIS_CUDA_TRY((lightning_reg<RI, RJ, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st, fin)));          \
+    return fin.act ? cudaSuccess : launch_stack_headnorm_silu(o, nullptr, gate, ldg, act, ld_act, 0, 1.f, f32, sp.T, H0, dv0, eps, st);            \
+  } while (0)
+  if (d <= 32 && dv <= 64) DIS_RET(4, 2);
+  if (d <= 64 && dv <= 64) DIS_RET(8, 2);
+  if (d <= 128 && dv <= 64) DIS_RET(16, 2);
+  if (d <= 128 && dv <= 128) DIS_RET(16, 4);
+#undef DIS_RET
   const int threads = 256;
   const size_t sh = ((size_t)d * dv + 2 * d + dv + (size_t)(threads / 32) * dv) * sizeof(float);
   if (sh > 220 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_lightning_kernel<3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); }));
   stack_lightning_kernel<3><<<dim3(sp.n_spans, H), threads, sh, st>>>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv);
-  return cudaGetLastError();
+  DIS_CUDA_TRY(cudaGetLastError());
+  return launch_stack_headnorm_silu(o, nullptr, gate, ldg, act, ld_act, 0, 1.f, f32, sp.T, H0, dv0, eps, st);
 }
 
 // ------------------------------------------------------------------------------------------------ gated linear attention
@@ -1011,7 +1055,7 @@ __device__ __forceinline__ float latent_rotated(const float *v, int i, const Sta
 // qx (or null): the rotated query parts are also written where the queries lie, [T][ld_qx] from the first head's column on (the row
 // itself, or its copy in keep).
 template <bool F32>
-__global__ void __launch_bounds__(256) stack_latent_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
+__global__ void __launch_bounds__(512) stack_latent_prep_kernel(const float *proj, long long ld, int n_part, long long stride, int n_cols,
                                                                 int q_off, int dkv_off, const float *dkv_norm, int dq_off,
                                                                 const float *dq_norm, void *cq, float *keep, long long ld_keep,
                                                                 int keep_off, int keep_n, const double *__restrict__ freq,
@@ -1095,7 +1139,7 @@ cudaError_t launch_stack_latent_prep(const StackLatentPrep &a, const StackLatent
     return e != cudaSuccess ? e : cudaFuncSetAttribute(stack_latent_prep_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
   }));
 #define DIS_LAT_PREP(F)                                                                                                                      \
-  stack_latent_prep_kernel<F><<<sp.T, 256, sh, st>>>(a.proj, a.ld, n_part, a.stride, a.n_cols, a.q_off, a.dkv_off, a.dkv_norm, a.dq_off, a.dq_norm, \
+  stack_latent_prep_kernel<F><<<sp.T, sp.T <= 148 ? 512 : 256, sh, st>>>(a.proj, a.ld, n_part, a.stride, a.n_cols, a.q_off, a.dkv_off, a.dkv_norm, a.dq_off, a.dq_norm, \
                                                      a.cq, a.keep, a.ld_keep, a.keep_off, a.keep_n, a.freq, c, sp, a.qf, a.qx, a.ld_qx, a.pool, page_table, max_pages, page_size)
   if (f32) DIS_LAT_PREP(true);
   else DIS_LAT_PREP(false);

@@ -139,4 +139,12 @@ cudaError_t launch_k(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem,
   return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
 }
 
+// Gate activation of the products' epilogues, whose result is rounded to bf16 at once: kind 0 = silu(g) = g sigmoid(g), kind 1 =
+// gelu_tanh(g) = 0.5 g (1 + tanh y) = g sigmoid(2 y) with y = sqrt(2/pi) (g + 0.044715 g^3).  The approximate exponential and
+// division are good to a few parts in 10^6 and keep the epilogue warp free of the exact division's branches.
+__device__ __forceinline__ float gate_act_fast(int kind, float g) {
+  const float z = kind == 1 ? 1.5957691216057308f * fmaf(0.044715f * g * g, g, g) : g;
+  return __fdividef(g, 1.f + __expf(-z));
+}
+
 }  // namespace dis

@@ -1463,9 +1463,8 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
                                            1.f / std::sqrt((float)d), sp, stream));
       const bool segments = M.light_seg && d <= 128 && stack_lightning_segmented(sp.n_spans, T, H * nb, max_span);
       RET_CUDA(launch_stack_retention(M.proj, N, 0, L.k_off, L.v_off, reinterpret_cast<const float *>(L.decay_d.ptr), Rn.state, sp, M.mix, H, d, dv,
-                                      segments ? M.light_seg : nullptr, max_span, stream));
-      RET_CUDA(launch_stack_headnorm_silu(M.mix, nullptr, M.proj + L.g_off, N, M.act, L.ld_act, 0, 1.f, f32, T, H, dv, eps, stream));
-      kl += segments ? 5 : 3;
+                                      segments ? M.light_seg : nullptr, max_span, M.proj + L.g_off, N, M.act, L.ld_act, f32, eps, stream));
+      kl += (segments ? 4 : 2) + (nb > 1 || d > 128 || dv > 128 ? 1 : 0);
       n_mix = L.ld_act;
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, Ns = lc.ssm_state, G = lc.ssm_groups, C = L.conv_ch, inner = H * P;

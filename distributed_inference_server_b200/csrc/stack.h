@@ -109,10 +109,13 @@ cudaError_t launch_stack_gla(const float *proj, long long ld, int q_off, int k_o
 cudaError_t launch_stack_retention_prep(const float *src, long long ld_src, int n_part, long long stride, int n_cols, float *dst,
                                         long long ld_dst, int q_off, int k_off, int H, int d, const double *freq, int rot_dims, float kscale,
                                         const StackSpans &sp, cudaStream_t st);
-// S = decay S + k v^T, o = S^T q over rows of proj as prepared; decay [H * stack_retention_blocks()], each head's value repeated per block
+// S = decay S + k v^T, o = S^T q over rows of proj as prepared; decay [H * stack_retention_blocks()], each head's value repeated per block.
+// Each head's o, divided by its root mean square and times silu(gate [T][ldg]), lands in act [T][ld_act] (compute type): inside the
+// recurrence kernel, or (values in several blocks, sizes beyond the register kernel) through o [T][H*dv] and a second kernel.
 int stack_retention_blocks(int d, int dv);
 cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *decay, float *state,
-                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, cudaStream_t st);
+                                   const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, const float *gate,
+                                   long long ldg, void *act, long long ld_act, bool f32, float eps, cudaStream_t st);
 // State-space mixer (DIS_MIX_SSM), three steps around the recurrence kernel of gated linear attention.
 // 1. proj [T][ld] holds z | x | B | C | dt as projected.  The C = inner + 2 G N channels from x_off on pass a causal depthwise
 //    convolution over time (cw [C][taps], last tap = the current token; the taps - 1 inputs before a span come from cstate
