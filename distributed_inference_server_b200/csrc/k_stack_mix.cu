@@ -470,7 +470,9 @@ cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, i
   const int H0 = H, dv0 = dv;
   H *= nb; dv /= nb;
   LightFin fin;
-  if (nb == 1) fin = {act, ld_act, ldg, gate, eps, f32 ? 1 : 0};  // (a head in several blocks is normalised by a second kernel)
+  // finished inside the kernel, unless a head's values are in several blocks or spans are cut into segments (whose output kernel has
+  // no warps to spare for it)
+  if (nb == 1 && !(seg && max_len > kLightSeg)) fin = {act, ld_act, ldg, gate, eps, f32 ? 1 : 0};
 #define DIS_RET(RI, RJ)                                                                                                                        \
   do {                                                                                                                                        \
     DIS_CUDA_TRY((lightning_reg<RI, RJ, 3>(proj, ld, col, decay, nullptr, 1.f, state, sp, o, H, d, dv, seg, nullptr, max_len, st, fin)));          \

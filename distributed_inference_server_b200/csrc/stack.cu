@@ -1113,11 +1113,14 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
   ENG_CUDA(cudaMemcpyAsync(mt.dev, mt.host, mt.bytes, cudaMemcpyHostToDevice, stream));
   // latent attention: with few query blocks the history is cut into slices so that about two CTAs per SM run
   // (a windowed layer walks at most its window plus the block's own tokens)
+  // keys of a slice: whole tiles of the kernel, as few as `want` slices (at most 64) of them need
+  auto slice_keys = [](int ctx, int tile, int want) {
+    const int tiles = (ctx + tile - 1) / tile, n = std::max(1, std::min(std::min(want, 64), tiles));
+    return (tiles + n - 1) / n * tile;
+  };
   auto lat_slices = [&](int ctx) -> std::pair<int, int> {
     if (!(QB > 0 && QB < kNumSMs && ctx >= 256 && stack_lat_rec)) return {1, 0};
-    int sp = std::min(std::min((2 * kNumSMs + QB - 1) / QB, ctx / (stack_lat_mma ? 64 : 32)), 64);  // a slice holds at least one tile of keys
-    const int keys = ((ctx + sp - 1) / sp + 31) / 32 * 32;
-    sp = (ctx + keys - 1) / keys;
+    const int keys = slice_keys(ctx, stack_lat_mma ? 64 : 32, (2 * kNumSMs + QB - 1) / QB), sp = (ctx + keys - 1) / keys;
     if (sp > 1 && (size_t)sp * T * stack_lat_rec <= M.lat_part_elems) return {sp, keys};
     return {1, 0};
   };
@@ -1126,10 +1129,7 @@ int Engine::stack_step(int n, const int *slots, int max_prefill_tokens, uint32_t
   stack_kb = KB;
   auto att_slices = [&](int ctx) -> std::pair<int, int> {
     if (!(KB > 0 && KB * stack_att_groups < kNumSMs && ctx >= 256 && stack_att_rec)) return {1, 0};
-    int sp = std::min(std::min((2 * kNumSMs + KB * stack_att_groups - 1) / (KB * stack_att_groups), ctx / 64), 64);
-    if (sp <= 1) return {1, 0};
-    const int keys = ((ctx + sp - 1) / sp + 31) / 32 * 32;
-    sp = (ctx + keys - 1) / keys;
+    const int keys = slice_keys(ctx, 64, (2 * kNumSMs + KB * stack_att_groups - 1) / (KB * stack_att_groups)), sp = (ctx + keys - 1) / keys;
     if (sp > 1 && (size_t)sp * T * stack_att_rec <= M.attn_part_elems) return {sp, keys};
     return {1, 0};
   };
@@ -1464,7 +1464,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       const bool segments = M.light_seg && d <= 128 && stack_lightning_segmented(sp.n_spans, T, H * nb, max_span);
       RET_CUDA(launch_stack_retention(M.proj, N, 0, L.k_off, L.v_off, reinterpret_cast<const float *>(L.decay_d.ptr), Rn.state, sp, M.mix, H, d, dv,
                                       segments ? M.light_seg : nullptr, max_span, M.proj + L.g_off, N, M.act, L.ld_act, f32, eps, stream));
-      kl += (segments ? 4 : 2) + (nb > 1 || d > 128 || dv > 128 ? 1 : 0);
+      kl += segments ? 5 : nb > 1 || d > 128 || dv > 128 ? 3 : 2;
       n_mix = L.ld_act;
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, Ns = lc.ssm_state, G = lc.ssm_groups, C = L.conv_ch, inner = H * P;

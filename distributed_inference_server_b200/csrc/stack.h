@@ -111,7 +111,7 @@ cudaError_t launch_stack_retention_prep(const float *src, long long ld_src, int 
                                         const StackSpans &sp, cudaStream_t st);
 // S = decay S + k v^T, o = S^T q over rows of proj as prepared; decay [H * stack_retention_blocks()], each head's value repeated per block.
 // Each head's o, divided by its root mean square and times silu(gate [T][ldg]), lands in act [T][ld_act] (compute type): inside the
-// recurrence kernel, or (values in several blocks, sizes beyond the register kernel) through o [T][H*dv] and a second kernel.
+// recurrence kernel, or (segments, values in several blocks, sizes beyond the register kernel) through o [T][H*dv] and a second kernel.
 int stack_retention_blocks(int d, int dv);
 cudaError_t launch_stack_retention(const float *proj, long long ld, int q_off, int k_off, int v_off, const float *decay, float *state,
                                    const StackSpans &sp, float *o, int H, int d, int dv, float *seg, int max_len, const float *gate,
