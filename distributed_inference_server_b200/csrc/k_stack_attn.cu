@@ -323,23 +323,31 @@ __global__ void stack_attn_merge_kernel(const float *part, int n_split, int T, i
   const int p = blockIdx.x, tok = p / H, h = p - tok * H;
   const long long stride = (long long)T * H * (dv + 2);
   const float *rec = part + (long long)p * (dv + 2);
-  if (!SIG) {
-    float M = -INFINITY;
-    for (int s = 0; s < n_split; s++) M = fmaxf(M, rec[s * stride + dv]);
-    for (int s = threadIdx.x; s < n_split; s += blockDim.x) {
-      const float m = rec[s * stride + dv];
-      ws[s] = m == -INFINITY ? 0.f : expf(m - M);
+  if (!SIG && threadIdx.x < 32) {  // a lane per slice (at most 64): every slice's maximum and denominator are fetched at once
+    const int l = threadIdx.x;
+    float m[2], d[2], M = -INFINITY, den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      const int s = l + 32 * u;
+      m[u] = s < n_split ? rec[s * stride + dv] : -INFINITY;
+      d[u] = s < n_split ? rec[s * stride + dv + 1] : 0.f;
+      M = fmaxf(M, m[u]);
     }
-    __syncthreads();
-    if (threadIdx.x == 0) {
-      float den = 0.f;
-      for (int s = 0; s < n_split; s++) den += rec[s * stride + dv + 1] * ws[s];
-      inv_den = 1.f / den;
+    M = warp_max(M);
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      const int s = l + 32 * u;
+      const float w = m[u] == -INFINITY ? 0.f : expf(m[u] - M);
+      if (s < n_split) ws[s] = w;
+      den = fmaf(d[u], w, den);
     }
+    den = warp_sum(den);
+    if (l == 0) inv_den = 1.f / den;
   }
   __syncthreads();
   for (int j = threadIdx.x; j < dv; j += blockDim.x) {
     float v = 0.f;
+#pragma unroll 8
     for (int s = 0; s < n_split; s++) v = SIG ? v + rec[s * stride + j] : fmaf(rec[s * stride + j], ws[s], v);
     a[j] = v;
   }
@@ -774,8 +782,8 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
     DIS_CUDA_TRY(attn_mma_go(qf, (long long)c.H * c.d, kv, temp, pb, sink, c, sp, qb_tok0, qb_len, grid, page_table, max_pages, page_size, o, keys_per_split, part, st));
     if (part) {
       const size_t msh = (size_t)(c.dv + n_split) * sizeof(float);
-      if (sig) stack_attn_merge_kernel<false, true><<<sp.T * c.H, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
-      else stack_attn_merge_kernel<false, false><<<sp.T * c.H, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
+      if (sig) stack_attn_merge_kernel<false, true><<<sp.T * c.H, 128, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
+      else stack_attn_merge_kernel<false, false><<<sp.T * c.H, 128, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
     }
     return cudaGetLastError();
   }

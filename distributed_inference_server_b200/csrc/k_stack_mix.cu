@@ -1,5 +1,5 @@
-// k_stack_mix.cu -- the token mixers of the layer-list decoders: the decayed linear-attention scan, the minimal gated recurrence,
-// and latent attention (query absorption happens in a batched matrix product in stack.cu; here: rotary + cache write, and the
+// k_stack_mix.cu -- the token mixers of the layer-list decoders: the decayed linear-attention scan (also as retention), the minimal
+// gated recurrence, the state-space mixer, and latent attention (query absorption happens in a batched matrix product in stack.cu; here: rotary + cache write, and the
 // attention itself over the paged latents).  States and scores are fp32.
 #include <cstdlib>
 #include "stack_dev.cuh"
@@ -1456,21 +1456,32 @@ __global__ void stack_latent_merge_kernel(const float *part, const float *sink, 
   __shared__ float inv_den;
   const int p = blockIdx.x;
   const float sk = sink ? sink[p % H] : -INFINITY;
-  float M = sk;
-  for (int s = 0; s < n_split; s++) M = fmaxf(M, part[((long long)s * pairs_total + p) * (r + 2) + r]);
-  for (int s = threadIdx.x; s < n_split; s += blockDim.x) {
-    const float m = part[((long long)s * pairs_total + p) * (r + 2) + r];
-    ws[s] = m == -INFINITY ? 0.f : expf(m - M);
-  }
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    float den = sink ? expf(sk - M) : 0.f;
-    for (int s = 0; s < n_split; s++) den += part[((long long)s * pairs_total + p) * (r + 2) + r + 1] * ws[s];
-    inv_den = 1.f / den;
+  if (threadIdx.x < 32) {  // a lane per slice (at most 64): every slice's maximum and denominator are fetched at once
+    const int l = threadIdx.x;
+    float m[2], d[2], M = sk, den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      const int s = l + 32 * u;
+      const float *rec = part + ((long long)s * pairs_total + p) * (r + 2) + r;
+      m[u] = s < n_split ? rec[0] : -INFINITY;
+      d[u] = s < n_split ? rec[1] : 0.f;
+      M = fmaxf(M, m[u]);
+    }
+    M = warp_max(M);
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      const int s = l + 32 * u;
+      const float w = m[u] == -INFINITY ? 0.f : expf(m[u] - M);
+      if (s < n_split) ws[s] = w;
+      den = fmaf(d[u], w, den);
+    }
+    den = warp_sum(den);
+    if (l == 0) inv_den = 1.f / (den + (sink ? expf(sk - M) : 0.f));
   }
   __syncthreads();
   for (int j = threadIdx.x; j < r; j += blockDim.x) {
     float v = 0.f;
+#pragma unroll 8
     for (int s = 0; s < n_split; s++) v = fmaf(part[((long long)s * pairs_total + p) * (r + 2) + j], ws[s], v);
     ol[(long long)p * r + j] = v * inv_den;
   }
@@ -1577,7 +1588,7 @@ cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32
     const uint16_t *pl = reinterpret_cast<const uint16_t *>(pool);
     if (c.r <= 512) stack_latent_attn_mma_kernel<8><<<grid, 256, shm, st>>>(qf, pl, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);
     else stack_latent_attn_mma_kernel<16><<<grid, 256, shm, st>>>(qf, pl, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);
-    if (part) stack_latent_merge_kernel<<<sp.T * c.H, 128, 0, st>>>(part, sink, n_split, sp.T * c.H, c.H, c.r, ol);
+    if (part) stack_latent_merge_kernel<<<sp.T * c.H, c.r > 256 ? 512 : 128, 0, st>>>(part, sink, n_split, sp.T * c.H, c.H, c.r, ol);
     return cudaGetLastError();
   }
   const int D = c.r + c.dr, bq = stack_latent_block_tokens(c);
@@ -1591,7 +1602,7 @@ cudaError_t launch_stack_latent_attn(const float *qf, const void *pool, bool f32
   const dim3 grid(n_qb, n_split);
   if (f32) stack_latent_attn_kernel<true><<<grid, kLatWarps * 32, sh, st>>>(qf, pool, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);
   else stack_latent_attn_kernel<false><<<grid, kLatWarps * 32, sh, st>>>(qf, pool, sink, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, ol, keys_per_split, part);
-  if (part) stack_latent_merge_kernel<<<sp.T * c.H, 128, 0, st>>>(part, sink, n_split, sp.T * c.H, c.H, c.r, ol);
+  if (part) stack_latent_merge_kernel<<<sp.T * c.H, c.r > 256 ? 512 : 128, 0, st>>>(part, sink, n_split, sp.T * c.H, c.H, c.r, ol);
   return cudaGetLastError();
 }
 

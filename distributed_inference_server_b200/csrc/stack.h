@@ -1,6 +1,7 @@
 // stack.h -- layer-list decoders: a model given as a list of layers, each with one token mixer (linear attention with a
-// fixed decay, a minimal gated recurrence, or latent attention over a compressed KV cache) and an optional
-// feed-forward (dense or mixture of experts).  The engine's sequences, page allocator, step planner, sampler and C ABI
+// fixed decay, a minimal gated recurrence, latent attention over a compressed KV cache, grouped-query attention, gated linear
+// attention beside it, a state-space mixer, or retention) and an optional feed-forward (dense or mixture of experts), behind or
+// beside the mixer.  The engine's sequences, page allocator, step planner, sampler and C ABI
 // are shared with the Llama path; this header holds what differs: the per-layer weights, the per-slot recurrent state,
 // the latent page pools and the launchers of k_stack.cu.
 #pragma once

@@ -31,9 +31,11 @@ extern "C" {
 #endif
 
 #define DIS_API __attribute__((visibility("default")))
-#define DIS_ABI_VERSION 5 /* 2: 16-byte request ids, logprob on token events / callback, dis_serving_cancel; 3: dis_layer_config and dis_stack_config grew (attention and parallel mixers, layer norms, layer loops); 4: they grew again (chunked mask, sink, per-head query/key norm and output gate of attention, shared key/value cache, grouped sigmoid router, shared expert, RMS norms with gain vectors, logit soft cap); 5: and again (state-space mixer, sliding window, score soft cap and unit sink of
+#define DIS_ABI_VERSION 6 /* 2: 16-byte request ids, logprob on token events / callback, dis_serving_cancel; 3: dis_layer_config and dis_stack_config grew (attention and parallel mixers, layer norms, layer loops); 4: they grew again (chunked mask, sink, per-head query/key norm and output gate of attention, shared key/value cache, grouped sigmoid router, shared expert, RMS norms with gain vectors, logit soft cap); 5: and again (state-space mixer, sliding window, score soft cap and unit sink of
                              attention, ungated squared-ReLU units, softmax-over-all router, ungated shared expert, residual streams, pre-norm frame,
-                             sinusoidal positions, loops without an input projection, head tied to the embedding) */
+                             sinusoidal positions, loops without an input projection, head tied to the embedding); 6: and again (retention, query latent and window of latent
+                             attention, kept first positions, distance term, value mixing and full output gate of attention, parallel layers, gains stored around
+                             zero, residual multiplier) */
 
 /* ---- status codes: WorkerError, crates/core/src/error.rs:115-128 ------------------------------ */
 typedef enum dis_status {
