@@ -34,17 +34,19 @@ class EngineConfig(C.Structure):
                 ("eos_token", C.c_int32), ("stream", C.c_void_p), ("nccl_id", C.c_uint8 * 128)]
 
 
-MIX_LIGHTNING, MIX_MINGRU, MIX_LATENT, MIX_ATTENTION, MIX_PARALLEL, MIX_SSM, MIX_RETENTION = range(7)
+MIX_LIGHTNING, MIX_MINGRU, MIX_LATENT, MIX_ATTENTION, MIX_PARALLEL, MIX_SSM, MIX_RETENTION, MIX_CHANNEL_DELTA = range(8)
 MLP_NONE, MLP_DENSE, MLP_MOE = range(3)
 ACT_CLAMPED, ACT_GELU_TANH, ACT_SILU, ACT_RELU2 = range(4)
 NORM_RMS_SCALAR, NORM_LAYER, NORM_RMS, NORM_RMS_ONE = range(4)
-ROUTE_SOFTMAX_TOP, ROUTE_SIGMOID_GROUPS, ROUTE_SOFTMAX_ALL = range(3)
+ROUTE_SOFTMAX_TOP, ROUTE_SIGMOID_GROUPS, ROUTE_SOFTMAX_ALL, ROUTE_SOFTMAX_GROUPS = range(4)
 ATTN_SIGMOID, ATTN_QK_NORM, ATTN_V_IS_K, ATTN_ROT_V, ATTN_BIAS = 1, 2, 4, 8, 16
 ATTN_BIAS_QKV, ATTN_QK_NORM_HEAD, ATTN_SINK, ATTN_GATE, ATTN_SINK_UNIT = 32, 64, 128, 256, 512
 ATTN_GATE_FULL, ATTN_DISTANCE, ATTN_V_MIX = 1024, 2048, 4096
+ATTN_DIFF, ATTN_ROT_PAIRS, ATTN_ROT_LINEAR = 8192, 16384, 32768
 LATENT_NO_SINK, LATENT_NO_GATE, LATENT_ROT_PAIRS = 1, 2, 4
 MLP_SHARED_PLAIN = 1
 FRAME_PRE_NORM, FRAME_POS_SINUS, FRAME_LOOP_PLAIN, FRAME_TIED_HEAD, FRAME_PARALLEL = 1, 2, 4, 8, 16
+FRAME_TWO_NORMS, FRAME_LAYER_SCALE, FRAME_LOOP_EMBED = 32, 64, 128
 
 
 class LayerConfig(C.Structure):
@@ -58,7 +60,8 @@ class LayerConfig(C.Structure):
                [(n, C.c_int32) for n in ("mask_chunk", "route_kind", "route_groups", "route_keep", "shared_ff", "mask_window")] + \
                [("score_softcap", C.c_float)] + \
                [(n, C.c_int32) for n in ("ssm_state", "ssm_groups", "conv_taps", "ssm_norm_groups")] + [("mlp_flags", C.c_uint32)] + \
-               [("mask_keep", C.c_int32), ("q_rank", C.c_int32), ("latent_flags", C.c_uint32)]
+               [("mask_keep", C.c_int32), ("q_rank", C.c_int32), ("latent_flags", C.c_uint32)] + \
+               [("attn_diff", C.c_float), ("decay_rank", C.c_int32), ("gate_rank", C.c_int32)]
 
 
 class StackConfig(C.Structure):

@@ -486,6 +486,10 @@ int Engine::finalize() {
   if (stack)
     for (auto &kv : stack_names)
       if (!kv.second.loaded) return fail(DIS_ERR_MODEL_NOT_LOADED, "finalize: tensor '" + kv.first + "' was not loaded");
+  if (stack) {
+    const int rc = stack_finalize();
+    if (rc != DIS_OK) return rc;
+  }
   loaded = true;
   return DIS_OK;
 }

@@ -197,6 +197,7 @@ struct Engine {
   int seq_probe(int slot, const int *pos, int n);
   cudaError_t stack_forward(int T, int n_spans, int n_qb, int R, bool all_greedy);
   cudaError_t stack_meta(StepMeta &s, int cap_t, int cap_rows);
+  int stack_finalize();  // numbers made from loaded tensors
   void free_stack();
 
   ~Engine();

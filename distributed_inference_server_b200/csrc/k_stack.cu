@@ -660,6 +660,129 @@ cudaError_t launch_stack_boundary_hc(float *xs, int streams, const float *y, int
 #undef DIS_HC
 }
 
+// Boundary of parallel layers with two norms (StackParBoundary): one block per token, the row in shared memory.
+// VEC: W is a multiple of 4 and every pointer 16-byte aligned.
+template <bool F32, bool VEC>
+__global__ void __launch_bounds__(256) stack_boundary_par_kernel(float *x, StackParBoundary b, float mult, const float *__restrict__ w1, void *h1,
+                                                                 const float *__restrict__ w2, void *h2, int W, float eps) {
+  extern __shared__ __align__(16) float row[];  // [W]
+  __shared__ float sh[32], wts[32];
+  __shared__ long long at[32];  // offsets of the experts' rows
+  constexpr int V = VEC ? 4 : 1;
+  const long long t = blockIdx.x;
+  if (b.rows && threadIdx.x < b.top) {
+    wts[threadIdx.x] = b.wt[t * b.top + threadIdx.x];
+    at[threadIdx.x] = (long long)b.where[t * b.top + threadIdx.x] * W;
+  }
+  __syncthreads();
+  const float g2 = b.y2_gate ? sigmoid_precise(b.y2_gate[t]) : 1.f;
+  auto ld = [](const float *p, float (&o)[V]) {
+    if (VEC) { const float4 v = *reinterpret_cast<const float4 *>(p); o[0] = v.x; o[V > 1 ? 1 : 0] = v.y; o[V > 2 ? 2 : 0] = v.z; o[V > 3 ? 3 : 0] = v.w; }
+    else o[0] = p[0];
+  };
+  auto st = [](float *p, const float (&o)[V]) {
+    if (VEC) *reinterpret_cast<float4 *>(p) = make_float4(o[0], o[V > 1 ? 1 : 0], o[V > 2 ? 2 : 0], o[V > 3 ? 3 : 0]);
+    else p[0] = o[0];
+  };
+  auto slices = [&](const float *y, int n, long long stride, const float *bias, int i, float (&o)[V]) {
+    if (bias) ld(bias + i, o);
+    else {
+#pragma unroll
+      for (int e = 0; e < V; e++) o[e] = 0.f;
+    }
+#pragma unroll 4
+    for (int k = 0; k < n; k++) {
+      float p[V];
+      ld(y + (long long)k * stride + t * W + i, p);
+#pragma unroll
+      for (int e = 0; e < V; e++) o[e] += p[e];
+    }
+  };
+  float q = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    float v[V], m[V], f[V], u[V];
+    ld(x + t * W + i, v);
+    if (b.y1) {
+      slices(b.y1, b.n1, b.s1, b.b1, i, m);
+      if (b.ls1) {
+        ld(b.ls1 + i, u);
+#pragma unroll
+        for (int e = 0; e < V; e++) m[e] *= u[e];
+      }
+#pragma unroll
+      for (int e = 0; e < V; e++) f[e] = 0.f;
+      if (b.y2) {
+        slices(b.y2, b.n2, b.s2, b.b2, i, f);
+#pragma unroll
+        for (int e = 0; e < V; e++) f[e] *= g2;
+      }
+      if (b.rows)
+#pragma unroll 4
+        for (int k = 0; k < b.top; k++) {
+          ld(b.rows + at[k] + i, u);
+#pragma unroll
+          for (int e = 0; e < V; e++) f[e] = fmaf(wts[k], u[e], f[e]);
+        }
+      if (b.ls2 && (b.y2 || b.rows)) {
+        ld(b.ls2 + i, u);
+#pragma unroll
+        for (int e = 0; e < V; e++) f[e] *= u[e];
+      }
+#pragma unroll
+      for (int e = 0; e < V; e++) v[e] = fmaf(mult, m[e] + f[e], v[e]);
+    }
+    if (b.add) {
+      ld(b.add + t * W + i, u);
+#pragma unroll
+      for (int e = 0; e < V; e++) v[e] += u[e];
+    }
+    if (b.y1 || b.add) st(x + t * W + i, v);
+    st(row + i, v);
+#pragma unroll
+    for (int e = 0; e < V; e++) q += v[e] * v[e];
+  }
+  if (!w1) return;
+  const float r = rsqrtf(block_sum(q, sh) / (float)W + eps);
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {  // each thread re-reads what it wrote itself
+    float v[V], g[V], o[V];
+    ld(row + i, v);
+    for (int k = 0; k < 2; k++) {
+      void *h = k ? h2 : h1;
+      if (k && !w2) break;
+      ld((k ? w2 : w1) + i, g);
+#pragma unroll
+      for (int e = 0; e < V; e++) o[e] = v[e] * r * g[e];
+      if (VEC && !F32) {
+        uint2 p;
+        p.x = (uint32_t)float_to_bf16_bits(o[0]) | ((uint32_t)float_to_bf16_bits(o[V > 1 ? 1 : 0]) << 16);
+        p.y = (uint32_t)float_to_bf16_bits(o[V > 2 ? 2 : 0]) | ((uint32_t)float_to_bf16_bits(o[V > 3 ? 3 : 0]) << 16);
+        *reinterpret_cast<uint2 *>(reinterpret_cast<uint16_t *>(h) + t * W + i) = p;
+      } else if (VEC) st(reinterpret_cast<float *>(h) + t * W + i, o);
+      else st_el<F32>(h, t * W + i, o[0]);
+    }
+  }
+}
+cudaError_t launch_stack_boundary_par(float *x, const StackParBoundary &b, float mult, const float *w1, void *h1, const float *w2, void *h2, bool f32,
+                                      int T, int W, float eps, cudaStream_t st) {
+  if ((size_t)W * 4 > 160 * 1024 || (b.rows && b.top > 32)) return cudaErrorInvalidValue;
+  if (T <= 0) return cudaSuccess;
+  auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool vec = W % 4 == 0 && b.s1 % 4 == 0 && b.s2 % 4 == 0 && al(x) && al(b.y1) && al(b.b1) && al(b.ls1) && al(b.ls2) && al(b.rows) && al(b.y2) && al(b.b2) &&
+                   al(b.add) && al(w1) && al(w2) && al(h1) && al(h2);
+#define DIS_PAR(F, VV)                                                                                                                                   \
+  do {                                                                                                                                                  \
+    static DeviceOnce once;                                                                                                                             \
+    DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_boundary_par_kernel<F, VV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); })); \
+    stack_boundary_par_kernel<F, VV><<<T, 256, (size_t)W * 4, st>>>(x, b, mult, w1, h1, w2, h2, W, eps);                                               \
+  } while (0)
+  if (f32 && vec) DIS_PAR(true, true);
+  else if (f32) DIS_PAR(true, false);
+  else if (vec) DIS_PAR(false, true);
+  else DIS_PAR(false, false);
+#undef DIS_PAR
+  return cudaGetLastError();
+}
+
 __global__ void stack_scale_kernel(float *v, long long n, float s) {
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) v[i] *= s;
 }
@@ -894,6 +1017,7 @@ cudaError_t launch_stack_glu(const float *gu, int n_part, long long stride, cons
 // DIS_ROUTE_SIGMOID_GROUPS: s = sigmoid(z), c = s + correction; with groups > 1 the expert indices are cut into `groups`
 // contiguous runs, a run is ranked by the sum of its top two c, and experts of runs ranked below `keep` get c = -inf; `top`
 // rounds of arg-max over c; weight of a chosen expert = its s over the chosen experts' sum of s (+ 1e-20).
+// DIS_ROUTE_SOFTMAX_GROUPS: s = softmax(z) over all experts; the rest as with the sigmoid, but a run is ranked by its largest c.
 // extra (or null): one more fp32 row [W] whose product with the token lands in extra_out[t] (the logit of a per-token gate).
 constexpr int kRouteWarps = 8;
 template <bool F32>
@@ -979,10 +1103,15 @@ __global__ void __launch_bounds__(kRouteWarps * 32) stack_route_kernel(const voi
     if (j >= nt) return;
     const int t = t0 + j;
     float *z = zs + j * per_tok, *c = z + E, *gs = c + E;
-    const bool sig = kind == DIS_ROUTE_SIGMOID_GROUPS;
+    const bool all = kind == DIS_ROUTE_SOFTMAX_GROUPS, sig = kind == DIS_ROUTE_SIGMOID_GROUPS || all;  // scores plus correction, groups
     if (sig) {
+      float zm = -INFINITY, zsum = 0.f;
+      if (all) {
+        for (int e = 0; e < E; e++) zm = fmaxf(zm, z[e]);
+        for (int e = 0; e < E; e++) { z[e] = expf(z[e] - zm); zsum += z[e]; }
+      }
       for (int e = 0; e < E; e++) {
-        const float sv = sigmoid_precise(z[e]);
+        const float sv = all ? z[e] / zsum : sigmoid_precise(z[e]);
         z[e] = sv;
         c[e] = sv + corr_s[e];
       }
@@ -995,7 +1124,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) stack_route_kernel(const voi
             if (v > a) { b = a; a = v; }
             else if (v > b) b = v;
           }
-          gs[g] = per > 1 ? a + b : a;
+          gs[g] = per > 1 && !all ? a + b : a;
         }
         unsigned kept = 0;  // groups <= E <= 32
         for (int k = 0; k < keep; k++) {
@@ -1031,10 +1160,17 @@ __global__ void __launch_bounds__(kRouteWarps * 32) stack_route_kernel(const voi
   for (int j = w; j < nt; j += kRouteWarps) {
     const int t = t0 + j;
     float *z = zs + j * per_tok, *c = z + E, *gs = c + E;
-    const bool sig = kind == DIS_ROUTE_SIGMOID_GROUPS;
+    const bool all = kind == DIS_ROUTE_SOFTMAX_GROUPS, sig = kind == DIS_ROUTE_SIGMOID_GROUPS || all;
     if (sig) {
+      float zm = -INFINITY, zsum = 0.f;
+      if (all) {
+        for (int e = l; e < E; e += 32) zm = fmaxf(zm, z[e]);
+        zm = warp_max(zm);
+        for (int e = l; e < E; e += 32) { z[e] = expf(z[e] - zm); zsum += z[e]; }
+        zsum = warp_sum(zsum);
+      }
       for (int e = l; e < E; e += 32) {
-        const float sv = sigmoid_precise(z[e]);
+        const float sv = all ? z[e] / zsum : sigmoid_precise(z[e]);
         z[e] = sv;
         c[e] = sv + corr_s[e];
       }
@@ -1049,7 +1185,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) stack_route_kernel(const voi
             if (v > a) { b = a; a = v; }
             else if (v > b) b = v;
           }
-          gs[g] = per > 1 ? a + b : a;
+          gs[g] = per > 1 && !all ? a + b : a;
           kept[g] = 0;
         }
         __syncwarp();
@@ -1107,7 +1243,7 @@ cudaError_t launch_stack_route(const void *hc, bool f32, const float *router, in
   // softmax over all experts, then the chosen scores over their sum: the softmax's common factor cancels, and its 1e-20 guard
   // lies below the last bit of a sum that is at least 1 / E -- the weights are the softmax over the chosen logits
   if (kind == DIS_ROUTE_SOFTMAX_ALL) kind = DIS_ROUTE_SOFTMAX_TOP;
-  if (kind == DIS_ROUTE_SIGMOID_GROUPS && (!correction || groups < 0 || (groups > 1 && (E % groups || keep < 1)))) return cudaErrorInvalidValue;
+  if ((kind == DIS_ROUTE_SIGMOID_GROUPS || kind == DIS_ROUTE_SOFTMAX_GROUPS) && (!correction || groups < 0 || (groups > 1 && (E % groups || keep < 1)))) return cudaErrorInvalidValue;
   if (T <= 0) return cudaSuccess;
   // prompt-sized passes: eight tokens share every fetch of a router row; small passes keep a block per token (more blocks)
   const int per_tok = 2 * E + 2 * std::max(groups, 1);

@@ -25,7 +25,8 @@ __global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj,
                                                               void *vpool, float *vrot, const int *page_table, int max_pages,
                                                               int page_size, StackVMix mix) {
   extern __shared__ __align__(16) float tab[];  // cos [half], sin [half], value cos [dv/2], value sin [dv/2], per-head factors [H + G], summed row
-  const int srow_off = (c.rot_dims + c.dv + c.H + c.G + 3) & ~3;  // the summed row starts on a 16-byte boundary
+  const int HM = c.H * c.maps, GM = c.G * c.maps;  // heads of queries and keys, each map a head of its own here
+  const int srow_off = (c.rot_dims + c.dv + HM + GM + 3) & ~3;  // the summed row starts on a 16-byte boundary
   __shared__ float sh[32];
   const int t = blockIdx.x;
   const float *row = proj + (long long)t * ld;
@@ -66,7 +67,7 @@ __global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj,
       vrot[(long long)t * c.dv + i] = c_;
       vrot[(long long)t * c.dv + vhalf + i] = s_;
     }
-  const int nq = c.H * c.d, nk = c.G * c.d;
+  const int nq = HM * c.d, nk = GM * c.d;
   const float *qb = bias ? bias + q_off : nullptr, *kb = bias ? bias + k_off : nullptr, *vb = bias ? bias + v_off : nullptr;
   const bool head_norm = (c.flags & DIS_ATTN_QK_NORM_HEAD) != 0;
   float rq = 1.f, rk = 1.f;
@@ -79,10 +80,10 @@ __global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj,
     rk = rsqrtf(block_sum(s, sh) / (float)nk + c.eps);
   } else if (head_norm) {  // one factor per head: a warp per head at a time, query heads then key heads
     const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
-    for (int h = w; h < c.H + (own ? c.G : 0); h += (int)(blockDim.x >> 5)) {
-      const bool isq = h < c.H;
-      const int off = isq ? q_off + h * c.d : k_off + (h - c.H) * c.d;
-      const float *b = isq ? (qb ? qb + h * c.d : nullptr) : (kb ? kb + (h - c.H) * c.d : nullptr);
+    for (int h = w; h < HM + (own ? GM : 0); h += (int)(blockDim.x >> 5)) {
+      const bool isq = h < HM;
+      const int off = isq ? q_off + h * c.d : k_off + (h - HM) * c.d;
+      const float *b = isq ? (qb ? qb + h * c.d : nullptr) : (kb ? kb + (h - HM) * c.d : nullptr);
       float s = 0.f;
       for (int i = l; i < c.d; i += 32) { const float v = row[off + i] + (b ? b[i] : 0.f); s += v * v; }
       s = warp_sum(s);
@@ -99,6 +100,10 @@ __global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj,
   auto rotated = [&](int off, const float *b, const float *g, float r, const float *rh, int i) {
     const int e = i % c.d;
     if (e >= c.rot_dims) return val(off, b, g, r, rh, i);
+    if (c.flags & DIS_ATTN_ROT_PAIRS) {
+      const int p = e >> 1;
+      return e & 1 ? val(off, b, g, r, rh, i) * cs[p] + val(off, b, g, r, rh, i - 1) * sn[p] : val(off, b, g, r, rh, i) * cs[p] - val(off, b, g, r, rh, i + 1) * sn[p];
+    }
     if (e < half) return val(off, b, g, r, rh, i) * cs[e] - val(off, b, g, r, rh, i + half) * sn[e];
     return val(off, b, g, r, rh, i) * cs[e - half] + val(off, b, g, r, rh, i - half) * sn[e - half];
   };
@@ -107,7 +112,7 @@ __global__ void __launch_bounds__(512) stack_attn_prep_kernel(const float *proj,
   for (int i = threadIdx.x; i < nq; i += blockDim.x) qf[(long long)t * nq + i] = rotated(q_off, qb, qg, rq, hr, i);
   if (!own) return;
   const long long prow = (long long)page_table[(long long)slot * max_pages + pos / page_size] * page_size + pos % page_size;
-  for (int i = threadIdx.x; i < nk; i += blockDim.x) st_el<F32>(kpool, prow * nk + i, rotated(k_off, kb, kg, rk, hr + c.H, i));
+  for (int i = threadIdx.x; i < nk; i += blockDim.x) st_el<F32>(kpool, prow * nk + i, rotated(k_off, kb, kg, rk, hr + HM, i));
   const int nv = c.G * c.dv;
   for (int i = threadIdx.x; i < nv; i += blockDim.x) {
     float v;
@@ -130,7 +135,7 @@ cudaError_t launch_stack_attn_prep(const float *proj, long long ld, int n_part, 
                                    int page_size, const StackVMix &mix, cudaStream_t st) {
   if (sp.T <= 0) return cudaSuccess;
   if (n_part < 1) n_part = 1;
-  const size_t sh = (size_t)(((c.rot_dims + c.dv + c.H + c.G + 3) & ~3) + (n_part > 1 ? n_cols : 0)) * sizeof(float);
+  const size_t sh = (size_t)(((c.rot_dims + c.dv + (c.H + c.G) * c.maps + 3) & ~3) + (n_part > 1 ? n_cols : 0)) * sizeof(float);
   if (sh > 200 * 1024) return cudaErrorInvalidValue;
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] {
@@ -191,14 +196,14 @@ __device__ __forceinline__ void attn_store(const AttnOut &o, const float *a, flo
 
 int stack_attn_block_tokens(const StackAttn &c, bool f32) {
   if (stack_attn_mma_ok(c, f32)) return stack_attn_mma_block_tokens(c);
-  const int R = c.H / c.G;
+  const int R = c.H / c.G * c.maps;
   int bq = std::max(1, 32 / R);
-  while (bq > 1 && ((size_t)kAtTile * (c.d + c.dv + 2 + kAtWarps) + (size_t)bq * R * (c.d + c.dv + 2)) * 4 > 200 * 1024) bq >>= 1;
+  while (bq > 1 && ((size_t)kAtTile * (c.d * c.maps + c.dv + 2 + kAtWarps) + (size_t)bq * R * (c.d + c.dv + 2)) * 4 > 200 * 1024) bq >>= 1;
   return bq;
 }
 static size_t attn_smem(const StackAttn &c, int bq) {
-  const int R = c.H / c.G;
-  return ((size_t)kAtTile * (c.d + c.dv + 2 + kAtWarps) + (size_t)bq * R * (c.d + c.dv + 2)) * sizeof(float);
+  const int R = c.H / c.G * c.maps;
+  return ((size_t)kAtTile * (c.d * c.maps + c.dv + 2 + kAtWarps) + (size_t)bq * R * (c.d + c.dv + 2)) * sizeof(float);
 }
 
 template <bool F32, bool SIG>
@@ -207,7 +212,8 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
                                                                    const int *qb_len, const int *page_table, int max_pages,
                                                                    int page_size, AttnOut o, int keys_per_split, float *part) {
   extern __shared__ float shm[];
-  const int d = c.d, dv = c.dv, DP = d + 1, VP = dv + 1, R = c.H / c.G, g = blockIdx.y;
+  // with two maps a head counts twice: pair p = ((token * heads of the group) + head) * maps + map, a key row holds both maps
+  const int maps = c.maps, d = c.d, dk = d * maps, dv = c.dv, DP = dk + 1, VP = dv + 1, R = c.H / c.G * maps, g = blockIdx.y;
   const int tok0 = qb_tok0[blockIdx.x], nq = qb_len[blockIdx.x];
   const int pairs = nq * R;
   float *kt = shm;                               // [32][DP]
@@ -222,7 +228,7 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
   const int last_pos = sp.pos[tok0 + nq - 1];
   for (int i = threadIdx.x; i < pairs * d; i += blockDim.x) {
     const int p = i / d, e = i - p * d;
-    qs[i] = qf[((long long)(tok0 + p / R) * c.H + g * R + p % R) * d + e];
+    qs[i] = qf[((long long)(tok0 + p / R) * c.H * maps + g * R + p % R) * d + e];
   }
   for (int i = threadIdx.x; i < pairs * dv; i += blockDim.x) acc[i] = 0.f;
   const bool with_sink = !SIG && sink && blockIdx.z == 0;
@@ -232,16 +238,16 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
   const AttnWalk wk(c, k_lo);
   const int k_begin = part ? (int)blockIdx.z * keys_per_split : 0;  // indices of the walk
   const int k_end = part ? min(wk.total(last_pos), k_begin + keys_per_split) : wk.total(last_pos);
-  const long long krow = (long long)c.G * d, vrow = (long long)c.G * dv;
+  const long long krow = (long long)c.G * dk, vrow = (long long)c.G * dv;
   const bool dist = !SIG && (c.flags & DIS_ATTN_DISTANCE);
   const float inv_cap = c.softcap > 0.f ? 1.f / c.softcap : 0.f;
   for (int k0 = k_begin; k0 < k_end; k0 += kAtTile) {
     const int nk = min(kAtTile, k_end - k0);
     __syncthreads();
-    for (int i = threadIdx.x; i < nk * d; i += blockDim.x) {
-      const int kk = i / d, cc = i - kk * d, kp = wk.key(k0 + kk);
+    for (int i = threadIdx.x; i < nk * dk; i += blockDim.x) {
+      const int kk = i / dk, cc = i - kk * dk, kp = wk.key(k0 + kk);
       const long long prow = (long long)pt[kp / page_size] * page_size + kp % page_size;
-      kt[(size_t)kk * DP + cc] = ld_el<F32>(kpool, prow * krow + (long long)g * d + cc);
+      kt[(size_t)kk * DP + cc] = ld_el<F32>(kpool, prow * krow + (long long)g * dk + cc);
     }
     for (int i = threadIdx.x; i < nk * dv; i += blockDim.x) {
       const int kk = i / dv, cc = i - kk * dv, kp = wk.key(k0 + kk);
@@ -256,7 +262,7 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
       float sc = -INFINITY;
       const int kp = wk.key(k0 + l);
       if (l < nk && kp <= qpos && (kp >= qlo || kp < c.keep)) {
-        const float *kr = kt + (size_t)l * DP;
+        const float *kr = kt + (size_t)l * DP + (maps > 1 ? (p & 1) * d : 0);
         float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;  // four chains, added at the end: the sum's order is fixed by d alone
         int i = 0;
         for (; i + 3 < d; i += 4) {
@@ -298,6 +304,18 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
     }
   }
   __syncthreads();
+  if (!part && maps > 1) {  // a warp joins the two maps of a (token, head)
+    for (int p = 2 * w; p < pairs; p += 2 * kAtWarps) {
+      const float *a1 = acc + (size_t)p * dv, *a2 = a1 + dv;
+      const float f1 = 1.f / dn[p], f2 = c.diff_lambda / dn[p + 1];
+      float ss = 0.f;
+      for (int j = l; j < dv; j += 32) { const float v = a1[j] * f1 - a2[j] * f2; ss = fmaf(v, v, ss); }
+      const float k = rsqrtf(warp_sum(ss) / (float)dv + c.eps) * c.diff_out * o.scale;
+      const int tok = tok0 + p / R, h = (g * R + p % R) >> 1;
+      for (int j = l; j < dv; j += 32) st_el<F32>(o.out, (long long)tok * o.ld + o.off + (long long)h * dv + j, (a1[j] * f1 - a2[j] * f2) * k);
+    }
+    return;
+  }
   if (!part) {
     for (int i = threadIdx.x; i < pairs * dv; i += blockDim.x) {
       const int p = i / dv, j = i - p * dv;
@@ -308,7 +326,7 @@ __global__ void __launch_bounds__(kAtWarps * 32) stack_attn_kernel(const float *
   // slice record per (token, head): dv unnormalised sums, then the slice's maximum and denominator
   for (int i = threadIdx.x; i < pairs * (dv + 2); i += blockDim.x) {
     const int p = i / (dv + 2), j = i - p * (dv + 2);
-    float *rec = part + (((long long)blockIdx.z * sp.T + tok0 + p / R) * c.H + g * R + p % R) * (dv + 2);
+    float *rec = part + (((long long)blockIdx.z * sp.T + tok0 + p / R) * c.H * maps + g * R + p % R) * (dv + 2);
     rec[j] = j < dv ? acc[(size_t)p * dv + j] : j == dv ? mx[p] : dn[p];
   }
 }
@@ -353,6 +371,54 @@ __global__ void stack_attn_merge_kernel(const float *part, int n_split, int T, i
   }
   __syncthreads();
   for (int j = threadIdx.x; j < dv; j += blockDim.x) attn_store<F32>(o, a, SIG ? 1.f : inv_den, tok, h, dv, j);
+}
+
+// Merge with two maps: one block per (token, head), a warp forms each map's factors; records of the head's maps lie next to each other.
+template <bool F32>
+__global__ void __launch_bounds__(128) stack_attn_merge_maps_kernel(const float *part, int n_split, int T, int H, int dv, AttnOut o, float lambda,
+                                                                    float diff_out, float eps) {
+  extern __shared__ float msh[];  // [dv] joined sums, [2][n_split] factors
+  float *a = msh, *ws = msh + dv;
+  __shared__ float sh[32];
+  const int p = blockIdx.x, tok = p / H, h = p - tok * H;
+  const long long stride = (long long)T * H * 2 * (dv + 2);
+  const float *rec = part + (long long)p * 2 * (dv + 2);
+  if (threadIdx.x < 64) {  // factor of a slice: its weight over the map's denominator, the second map's times -lambda
+    const int m = threadIdx.x >> 5, l = threadIdx.x & 31;
+    const float *rm = rec + m * (dv + 2);
+    float mx[2], d[2], M = -INFINITY, den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      const int s = l + 32 * u;
+      mx[u] = s < n_split ? rm[s * stride + dv] : -INFINITY;
+      d[u] = s < n_split ? rm[s * stride + dv + 1] : 0.f;
+      M = fmaxf(M, mx[u]);
+    }
+    M = warp_max(M);
+#pragma unroll
+    for (int u = 0; u < 2; u++) {
+      mx[u] = mx[u] == -INFINITY ? 0.f : expf(mx[u] - M);
+      den = fmaf(d[u], mx[u], den);
+    }
+    const float f = (m ? -lambda : 1.f) / warp_sum(den);
+#pragma unroll
+    for (int u = 0; u < 2; u++)
+      if (l + 32 * u < n_split) ws[m * n_split + l + 32 * u] = mx[u] * f;
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int j = threadIdx.x; j < dv; j += blockDim.x) {
+    float v1 = 0.f, v2 = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < n_split; s++) {
+      v1 = fmaf(rec[s * stride + j], ws[s], v1);
+      v2 = fmaf(rec[s * stride + dv + 2 + j], ws[n_split + s], v2);
+    }
+    a[j] = v1 + v2;
+    ss = fmaf(a[j], a[j], ss);
+  }
+  const float k = rsqrtf(block_sum(ss, sh) / (float)dv + eps) * diff_out * o.scale;
+  for (int j = threadIdx.x; j < dv; j += blockDim.x) st_el<F32>(o.out, (long long)tok * o.ld + o.off + (long long)h * dv + j, a[j] * k);
 }
 
 // ------------------------------------------------------------------------------------------------ attention on mma.sync
@@ -443,13 +509,16 @@ struct AttnKV {
   int k_hs, dk, v_hs;
   const int *lin;
 };
-// DQ, DV: compiled sizes of a query / key and of a value (the layer's are at most these).
-template <int DQ, int DV, bool SIG, bool DIST>
-__global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mma_kernel(const float *__restrict__ qf, long long ldq, AttnKV kv, const float *temp,
+// DQ, DV: compiled sizes of a query / key (of one map) and of a value (the layer's are at most these).
+// DIFF: two maps per head (StackAttn::maps).  Twice the warps: warp w and warp w + kMmWarps own the same rows, the first with map 1, the
+// second with map 2; a key row in shared memory holds both maps, the value rows are shared.  At the end the second map's outputs go
+// through shared memory to the warps of the first, which join, norm and store.  Slice records: maps of a head next to each other.
+template <int DQ, int DV, bool SIG, bool DIST, bool DIFF = false>
+__global__ void __launch_bounds__(kMmWarps * 32 * (DIFF ? 2 : 1), DIFF ? (DQ > 64 ? 1 : 2) : DQ > 128 ? 2 : 3) stack_attn_mma_kernel(const float *__restrict__ qf, long long ldq, AttnKV kv, const float *temp,
                                                                        const float *pb, const float *sink, StackAttn c, StackSpans sp, const int *qb_tok0,
                                                                        const int *qb_len, const int *page_table, int max_pages,
                                                                        int page_size, AttnOut o, int keys_per_split, float *part) {
-  constexpr int KP = DQ + 8, VP = DV + 8;  // elements per shared row: 16-byte rows land in distinct bank groups
+  constexpr int KP = DQ * (DIFF ? 2 : 1) + 8, VP = DV + 8;  // elements per shared row: 16-byte rows land in distinct bank groups
   extern __shared__ __align__(16) uint16_t smem[];
   uint16_t *Ks = smem;                               // [2][64][KP]
   uint16_t *Vs = smem + 2 * kMmKeys * KP;            // [2][64][VP]
@@ -466,17 +535,20 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
   const AttnWalk wk(c, k_lo);
   const int k_begin = part ? (int)blockIdx.z * keys_per_split : 0;  // indices of the walk
   const int k_end = part ? min(wk.total(last_pos), k_begin + keys_per_split) : wk.total(last_pos);
-  const int nk16 = (d + 15) >> 4, nv8 = dv >> 3, dc = d >> 3, vc = dv >> 3;  // k-steps of Q K^T, n-tiles of P V, 16-byte chunks per row
+  constexpr int NTR = DIFF ? 4 : 2;  // threads that copy a key row
+  const int krow_d = DIFF ? 2 * d : d;
+  const int nk16 = (d + 15) >> 4, nv8 = dv >> 3, dc = krow_d >> 3, vc = dv >> 3;  // k-steps of Q K^T, n-tiles of P V, 16-byte chunks per row
   // columns d .. 16 nk16 of the K stages are read by the last k-step: zero them once (cp.async never touches them)
   if (d & 15)
-    for (int i = threadIdx.x; i < 2 * kMmKeys * 8; i += blockDim.x) Ks[(i >> 3) * KP + d + (i & 7)] = 0;
-  // ---- this thread's rows: r0 = 16 warp + gid and r0 + 8
+    for (int i = threadIdx.x; i < 2 * kMmKeys * 8; i += blockDim.x) Ks[(i >> 3) * KP + krow_d + (i & 7)] = 0;
+  const int rwarp = DIFF ? warp & (kMmWarps - 1) : warp, map = DIFF ? warp / kMmWarps : 0;
+  // ---- this thread's rows: r0 = 16 rwarp + gid and r0 + 8
   int r_tok[2], r_head[2], r_pos[2], r_lo[2];
   bool r_ok[2];
   uint32_t qa[DQ / 16][4];
 #pragma unroll
   for (int e = 0; e < 2; e++) {
-    const int r = warp * 16 + gid + e * 8;
+    const int r = rwarp * 16 + gid + e * 8;
     r_ok[e] = r < rows;
     r_tok[e] = tok0 + (r_ok[e] ? r / R : 0);
     r_head[e] = kvh * R + (r_ok[e] ? r % R : 0);
@@ -487,7 +559,7 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
   for (int ks = 0; ks < DQ / 16; ks++) {
 #pragma unroll
     for (int e = 0; e < 2; e++) {
-      const float *qr = qf + (long long)r_tok[e] * ldq + (long long)r_head[e] * d;
+      const float *qr = qf + (long long)r_tok[e] * ldq + (long long)(DIFF ? 2 * r_head[e] + map : r_head[e]) * d;
 #pragma unroll
       for (int hf = 0; hf < 2; hf++) {
         const int col = ks * 16 + hf * 8 + qd * 2;
@@ -521,17 +593,17 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
   // with a soft cap the scores are first brought to units of the cap (scale / cap), and the capped score to units of log 2
   const float cap2 = !SIG && c.softcap > 0.f ? c.softcap * kLog2e : 0.f;
   const float scale2 = cap2 > 0.f ? c.scale / c.softcap : c.scale * kLog2e;
-  const bool warp_live = warp * 16 < rows;
-  const int warp_last_pos = pos_first + min(rows - 1, warp * 16 + 15) / R;
-  const int warp_first_pos = pos_first + (warp * 16) / R;
+  const bool warp_live = rwarp * 16 < rows;
+  const int warp_last_pos = pos_first + min(rows - 1, rwarp * 16 + 15) / R;
+  const int warp_first_pos = pos_first + (rwarp * 16) / R;
   const int warp_lo = stack_attn_row_lo(c, warp_first_pos);        // first key any row of the warp sees
   const int warp_lo_max = stack_attn_row_lo(c, warp_last_pos);     // first key every row of the warp sees
   const uint16_t *kh = kv.k + (long long)kvh * kv.k_hs, *vh = kv.v + (long long)kvh * kv.v_hs;
   const int dk8 = kv.dk >> 3;
   const long long lin0 = kv.lin ? kv.lin[slot] : 0;
   const uint32_t ks_base = (uint32_t)__cvta_generic_to_shared(Ks), vs_base = (uint32_t)__cvta_generic_to_shared(Vs);
-  // two threads per key row: one page-table read per thread and tile, then the row's 16-byte chunks alternate between the two
-  const int ld_row = threadIdx.x >> 1, ld_part = threadIdx.x & 1;
+  // NTR threads per key row: one page-table read per thread and tile, then the row's 16-byte chunks alternate between them
+  const int ld_row = threadIdx.x / NTR, ld_part = threadIdx.x % NTR;
   const int pshift = 31 - __clz(page_size);  // page_size is a power of two
   // the page of this thread's row is read one tile ahead of the copy that needs it
   auto page_of = [&](int k0) { const int v = k0 + ld_row; return v < k_end && !kv.lin ? pt[wk.key(v) >> pshift] : 0; };
@@ -544,13 +616,13 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
     const uint16_t *ksrc = kh + prow * kv.k_ld, *vsrc = vh + prow * kv.v_ld;
     const uint32_t kdst = ks_base + (uint32_t)(((stage * kMmKeys + ld_row) * KP) * 2), vdst = vs_base + (uint32_t)(((stage * kMmKeys + ld_row) * VP) * 2);
 #pragma unroll 4
-    for (int ch = ld_part; ch < dk8; ch += 2) cp_async16(kdst + ch * 16, ksrc + ch * 8, ok ? 16 : 0);
+    for (int ch = ld_part; ch < dk8; ch += NTR) cp_async16(kdst + ch * 16, ksrc + ch * 8, ok ? 16 : 0);
     if (dk8 < dc) {  // the shared part of the key
       const uint16_t *k2 = kv.k2 + prow * kv.k2_ld;
-      for (int ch = dk8 + ld_part; ch < dc; ch += 2) cp_async16(kdst + ch * 16, k2 + (ch - dk8) * 8, ok ? 16 : 0);
+      for (int ch = dk8 + ld_part; ch < dc; ch += NTR) cp_async16(kdst + ch * 16, k2 + (ch - dk8) * 8, ok ? 16 : 0);
     }
 #pragma unroll 4
-    for (int ch = ld_part; ch < vc; ch += 2) cp_async16(vdst + ch * 16, vsrc + ch * 8, ok ? 16 : 0);
+    for (int ch = ld_part; ch < vc; ch += NTR) cp_async16(vdst + ch * 16, vsrc + ch * 8, ok ? 16 : 0);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   const int n_tiles = k_end > k_begin ? (k_end - k_begin + kMmKeys - 1) / kMmKeys : 0;
@@ -568,7 +640,7 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
     if (warp_live && key_a <= warp_last_pos && (key_z >= warp_lo || key_a < c.keep)) {
       // S = Q K^T: k-steps outside, key tiles inside, so that consecutive products go to different accumulators; one ldmatrix
       // brings the fragments of two key tiles (lane l: matrix l / 8 = (tile, column half), row l % 8)
-      const uint32_t kt = ks_base + (uint32_t)(stage * kMmKeys * KP * 2);
+      const uint32_t kt = ks_base + (uint32_t)((stage * kMmKeys * KP + (DIFF ? map * d : 0)) * 2);
       float sacc[kMmKeys / 8][4];
 #pragma unroll
       for (int j = 0; j < kMmKeys / 8; j++) { sacc[j][0] = sacc[j][1] = sacc[j][2] = sacc[j][3] = 0.f; }
@@ -643,6 +715,44 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
       lrow[e] += __shfl_xor_sync(0xffffffffu, lrow[e], 2);
     }
   }
+  if (DIFF && !part) {  // (the last tile's barrier has passed: the stages are free)
+    float *o2 = reinterpret_cast<float *>(smem);  // [64 rows][DV + 4]: the second map's normalised outputs
+    if (map == 1 && warp_live) {
+#pragma unroll
+      for (int e = 0; e < 2; e++) {
+        const float inv = 1.f / lrow[e];
+        float *orow = o2 + (size_t)(rwarp * 16 + gid + e * 8) * (DV + 4) + qd * 2;
+#pragma unroll
+        for (int j = 0; j < DV / 8; j++)
+          if (j < nv8) *reinterpret_cast<float2 *>(orow + j * 8) = make_float2(oacc[j][e * 2] * inv, oacc[j][e * 2 + 1] * inv);
+      }
+    }
+    __syncthreads();
+    if (map == 1) return;
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const float inv = 1.f / lrow[e];
+      const float *orow = o2 + (size_t)(rwarp * 16 + gid + e * 8) * (DV + 4) + qd * 2;
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < DV / 8; j++)
+        if (j < nv8) {
+          const float2 v = *reinterpret_cast<const float2 *>(orow + j * 8);
+          oacc[j][e * 2] = fmaf(-c.diff_lambda, v.x, oacc[j][e * 2] * inv);
+          oacc[j][e * 2 + 1] = fmaf(-c.diff_lambda, v.y, oacc[j][e * 2 + 1] * inv);
+          ss = fmaf(oacc[j][e * 2], oacc[j][e * 2], fmaf(oacc[j][e * 2 + 1], oacc[j][e * 2 + 1], ss));
+        }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const float k = rsqrtf(ss / (float)dv + c.eps) * c.diff_out * o.scale;
+      if (!r_ok[e]) continue;
+      uint16_t *out = reinterpret_cast<uint16_t *>(o.out) + (long long)r_tok[e] * o.ld + o.off + (long long)r_head[e] * dv + qd * 2;
+#pragma unroll
+      for (int j = 0; j < DV / 8; j++)
+        if (j < nv8) *reinterpret_cast<uint32_t *>(out + j * 8) = pack_bf16(oacc[j][e * 2] * k, oacc[j][e * 2 + 1] * k);
+    }
+    return;
+  }
   // ---- results: thread holds, for row e, columns 8 j + 2 qd + {0, 1} of every n-tile j
   if (!part && o.vrot) {
     // rotation back by the query's position pairs column m with m + dv/2: the warp's 16 x dv tile goes through shared memory
@@ -678,7 +788,7 @@ __global__ void __launch_bounds__(kMmWarps * 32, DQ > 128 ? 2 : 3) stack_attn_mm
   for (int e = 0; e < 2; e++) {
     if (!r_ok[e]) continue;
     if (part) {
-      float *rec = part + (((long long)blockIdx.z * sp.T + r_tok[e]) * c.H + r_head[e]) * (dv + 2);
+      float *rec = part + (((long long)blockIdx.z * sp.T + r_tok[e]) * c.H + r_head[e]) * (dv + 2) * (DIFF ? 2 : 1) + (DIFF ? map * (dv + 2) : 0);
 #pragma unroll
       for (int j = 0; j < DV / 8; j++)
         if (j < nv8) { rec[j * 8 + qd * 2] = oacc[j][e * 2]; rec[j * 8 + qd * 2 + 1] = oacc[j][e * 2 + 1]; }
@@ -712,11 +822,26 @@ static cudaError_t attn_mma_go(const float *qf, long long ldq, const AttnKV &kv,
     allow(stack_attn_mma_kernel<128, 128, false, false>);
     allow(stack_attn_mma_kernel<128, 128, false, true>);
     allow(stack_attn_mma_kernel<192, 128, false, false>);
+    allow(stack_attn_mma_kernel<64, 64, false, false, true>);
+    allow(stack_attn_mma_kernel<64, 128, false, false, true>);
+    allow(stack_attn_mma_kernel<128, 128, false, false, true>);
     return e;
   }));
   const bool sig = (c.flags & DIS_ATTN_SIGMOID) != 0, dist = (c.flags & DIS_ATTN_DISTANCE) != 0;
   const bool small = c.d <= 64 && c.dv <= 64;
   const int dq = small ? 64 : c.d <= 128 ? 128 : 192, dvp = small ? 64 : 128;
+  if (c.maps > 1) {
+    if (sig || dist || c.d > 128 || c.dv > 128) return cudaErrorInvalidValue;
+    const int dqm = c.d <= 64 ? 64 : 128, dvm = small ? 64 : 128;
+    const size_t shd = std::max((size_t)2 * kMmKeys * (2 * dqm + dvm + 16) * sizeof(uint16_t), (size_t)kMmRows * (dvm + 4) * sizeof(float));
+#define DIS_ATTN_DIFF_MMA(Q, V) \
+  stack_attn_mma_kernel<Q, V, false, false, true><<<grid, kMmWarps * 64, shd, st>>>(qf, ldq, kv, temp, pb, nullptr, c, sp, qb_tok0, qb_len, page_table, max_pages, page_size, o, keys_per_split, part)
+    if (dqm == 64 && dvm == 64) DIS_ATTN_DIFF_MMA(64, 64);
+    else if (dqm == 64) DIS_ATTN_DIFF_MMA(64, 128);
+    else DIS_ATTN_DIFF_MMA(128, 128);
+#undef DIS_ATTN_DIFF_MMA
+    return cudaGetLastError();
+  }
   if (c.d > dq || c.dv > dvp || (dq == 192 && (sig || dist))) return cudaErrorInvalidValue;
   const size_t shm = (size_t)2 * kMmKeys * (dq + dvp + 16) * sizeof(uint16_t);
 #define DIS_ATTN_MMA(Q, V, S, B) \
@@ -778,11 +903,14 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
   // the output's 4-byte stores want even columns; bq is the block size the pass was planned with
   if (use_mma && stack_attn_mma_ok(c, f32) && bq <= stack_attn_mma_block_tokens(c) && ld_out % 2 == 0 && out_off % 2 == 0) {
     const uint16_t *kp = reinterpret_cast<const uint16_t *>(kpool), *vp = reinterpret_cast<const uint16_t *>(vpool);
-    const AttnKV kv{kp, nullptr, vp, (long long)c.G * c.d, 0, (long long)c.G * c.dv, c.d, c.d, c.dv, nullptr};
-    DIS_CUDA_TRY(attn_mma_go(qf, (long long)c.H * c.d, kv, temp, pb, sink, c, sp, qb_tok0, qb_len, grid, page_table, max_pages, page_size, o, keys_per_split, part, st));
+    const int dk = c.d * c.maps;
+    const AttnKV kv{kp, nullptr, vp, (long long)c.G * dk, 0, (long long)c.G * c.dv, dk, dk, c.dv, nullptr};
+    DIS_CUDA_TRY(attn_mma_go(qf, (long long)c.H * dk, kv, temp, pb, sink, c, sp, qb_tok0, qb_len, grid, page_table, max_pages, page_size, o, keys_per_split, part, st));
     if (part) {
       const size_t msh = (size_t)(c.dv + n_split) * sizeof(float);
-      if (sig) stack_attn_merge_kernel<false, true><<<sp.T * c.H, 128, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
+      if (c.maps > 1)
+        stack_attn_merge_maps_kernel<false><<<sp.T * c.H, 128, msh + n_split * sizeof(float), st>>>(part, n_split, sp.T, c.H, c.dv, o, c.diff_lambda, c.diff_out, c.eps);
+      else if (sig) stack_attn_merge_kernel<false, true><<<sp.T * c.H, 128, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
       else stack_attn_merge_kernel<false, false><<<sp.T * c.H, 128, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
     }
     return cudaGetLastError();
@@ -798,7 +926,10 @@ cudaError_t launch_stack_attn(const float *qf, const void *kpool, const void *vp
   if (part) {
     const size_t msh = (size_t)(c.dv + n_split) * sizeof(float);
     const int rows = sp.T * c.H;
-    if (f32 && sig) stack_attn_merge_kernel<true, true><<<rows, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
+    if (c.maps > 1) {
+      if (f32) stack_attn_merge_maps_kernel<true><<<rows, 128, msh + n_split * sizeof(float), st>>>(part, n_split, sp.T, c.H, c.dv, o, c.diff_lambda, c.diff_out, c.eps);
+      else stack_attn_merge_maps_kernel<false><<<rows, 128, msh + n_split * sizeof(float), st>>>(part, n_split, sp.T, c.H, c.dv, o, c.diff_lambda, c.diff_out, c.eps);
+    } else if (f32 && sig) stack_attn_merge_kernel<true, true><<<rows, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
     else if (f32) stack_attn_merge_kernel<true, false><<<rows, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
     else if (sig) stack_attn_merge_kernel<false, true><<<rows, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);
     else stack_attn_merge_kernel<false, false><<<rows, 64, msh, st>>>(part, n_split, sp.T, c.H, c.dv, o);

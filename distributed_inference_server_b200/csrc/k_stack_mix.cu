@@ -708,8 +708,8 @@ __global__ void __launch_bounds__(256) stack_ssm_conv_tile_kernel(const float *_
   }
 }
 // The tail moves on to the span's last taps - 1 inputs (a span shorter than that keeps the end of the old tail in front).
-__global__ void stack_ssm_tail_kernel(const float *__restrict__ proj, long long ld, int x_off, float *cstate, StackSpans sp, int C,
-                                      int taps) {
+__global__ void stack_ssm_tail_kernel(const float *__restrict__ proj, long long ld, int n_part, long long stride, int x_off, float *cstate,
+                                      StackSpans sp, int C, int taps) {
   const int s = blockIdx.x;
   const int tok0 = sp.sp_tok0[s], len = sp.sp_len[s], pos0 = sp.sp_pos0[s], slot = sp.sp_slot[s];
   float *tail = cstate + (long long)slot * (taps - 1) * C;
@@ -718,11 +718,21 @@ __global__ void stack_ssm_tail_kernel(const float *__restrict__ proj, long long 
     float nv[kConvMaxTaps];
     for (int k = 0; k < n; k++) {
       const int rel = len - n + k;  // index relative to the span's first token of the position tail'[k] holds
-      if (rel >= 0) nv[k] = proj[(long long)(tok0 + rel) * ld + x_off + c];
-      else nv[k] = (pos0 + rel >= 0) ? tail[(long long)(n + rel) * C + c] : 0.f;
+      if (rel >= 0) {
+        const float *p = proj + (long long)(tok0 + rel) * ld + x_off + c;
+        nv[k] = p[0];
+        for (int s2 = 1; s2 < n_part; s2++) nv[k] += p[(long long)s2 * stride];
+      } else nv[k] = (pos0 + rel >= 0) ? tail[(long long)(n + rel) * C + c] : 0.f;
     }
     for (int k = 0; k < n; k++) tail[(long long)k * C + c] = nv[k];
   }
+}
+cudaError_t launch_stack_conv_tail(const float *proj, long long ld, int n_part, long long stride, int x_off, float *cstate, const StackSpans &sp,
+                                   int C, int taps, cudaStream_t st) {
+  if (taps < 1 || taps > kConvMaxTaps) return cudaErrorInvalidValue;
+  if (taps == 1) return cudaSuccess;
+  stack_ssm_tail_kernel<<<dim3(sp.n_spans, (C + 1023) / 1024), 256, 0, st>>>(proj, ld, n_part, stride, x_off, cstate, sp, C, taps);
+  return cudaGetLastError();
 }
 cudaError_t launch_stack_ssm_conv(const float *proj, long long ld, int x_off, int dt_off, int C, int H, int taps, const float *cw,
                                   const float *cb, const float *vec, float *cstate, const StackSpans &sp, float *buf, long long ld_b,
@@ -744,8 +754,8 @@ cudaError_t launch_stack_ssm_conv(const float *proj, long long ld, int x_off, in
   else { if (v4) DIS_CONV(true, false); else DIS_CONV(false, false); }
 #undef DIS_CONV_TILE
 #undef DIS_CONV
-  if (taps > 1 && !single) stack_ssm_tail_kernel<<<dim3(sp.n_spans, (C + 1023) / 1024), 256, 0, st>>>(proj, ld, x_off, cstate, sp, C, taps);
-  return cudaGetLastError();
+  DIS_CUDA_TRY(cudaGetLastError());
+  return single ? cudaSuccess : launch_stack_conv_tail(proj, ld, 1, 0, x_off, cstate, sp, C, taps, st);
 }
 
 // y = (o + D[h] x) silu(z), then each of `parts` equal stretches of the row is divided by its own root mean square, times w.
@@ -841,7 +851,7 @@ cudaError_t launch_stack_ssm_out(const float *o, const float *buf, long long ld_
 // outputs, its gain vector (null: ones) is shared by the heads.  One warp per (token, head).
 template <bool F32>
 __global__ void __launch_bounds__(256) stack_headnorm_silu_kernel(const float *o, const float *w, const float *gate, long long ldg, void *out,
-                                                                  long long ldo, int off, float scale, int rows, int H, int dv, float eps) {
+                                                                  long long ldo, int off, float scale, int rows, int H, int dv, float eps, int sig) {
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), l = threadIdx.x & 31;
   if (row >= rows) return;
   const int t = row / H, h = row - t * H;
@@ -852,15 +862,15 @@ __global__ void __launch_bounds__(256) stack_headnorm_silu_kernel(const float *o
   const float k = rsqrtf(s / (float)dv + eps) * scale;
   for (int j = l; j < dv; j += 32) {
     const float g = gate[(long long)t * ldg + (long long)h * dv + j];
-    st_el<F32>(out, (long long)t * ldo + off + (long long)h * dv + j, r[j] * k * (w ? w[j] : 1.f) * silu_(g));
+    st_el<F32>(out, (long long)t * ldo + off + (long long)h * dv + j, r[j] * k * (w ? w[j] : 1.f) * (sig ? sigmoid_precise(g) : silu_(g)));
   }
 }
 cudaError_t launch_stack_headnorm_silu(const float *o, const float *w, const float *gate, long long ldg, void *out, long long ldo,
-                                       int off, float scale, bool f32, int T, int H, int dv, float eps, cudaStream_t st) {
+                                       int off, float scale, bool f32, int T, int H, int dv, float eps, cudaStream_t st, bool sig) {
   const int rows = T * H;
   if (rows <= 0) return cudaSuccess;
-  if (f32) stack_headnorm_silu_kernel<true><<<(rows + 7) / 8, 256, 0, st>>>(o, w, gate, ldg, out, ldo, off, scale, rows, H, dv, eps);
-  else stack_headnorm_silu_kernel<false><<<(rows + 7) / 8, 256, 0, st>>>(o, w, gate, ldg, out, ldo, off, scale, rows, H, dv, eps);
+  if (f32) stack_headnorm_silu_kernel<true><<<(rows + 7) / 8, 256, 0, st>>>(o, w, gate, ldg, out, ldo, off, scale, rows, H, dv, eps, sig ? 1 : 0);
+  else stack_headnorm_silu_kernel<false><<<(rows + 7) / 8, 256, 0, st>>>(o, w, gate, ldg, out, ldo, off, scale, rows, H, dv, eps, sig ? 1 : 0);
   return cudaGetLastError();
 }
 

@@ -36,6 +36,18 @@ static StackLatent stack_latent_shape(const dis_layer_config &lc, float eps) {
   return c;
 }
 
+static StackAttn stack_attn_shape(const StackLayer &L, float eps) {
+  const dis_layer_config &lc = L.c;
+  StackAttn c{lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.rot_dims, lc.attn_flags, lc.scale, eps, lc.mask_chunk, lc.mask_window, lc.score_softcap, lc.mask_keep};
+  if (lc.attn_flags & DIS_ATTN_DIFF) { c.maps = 2; c.diff_lambda = L.diff_lambda; c.diff_out = 1.f - lc.attn_diff; }
+  return c;
+}
+
+static StackDelta stack_delta_shape(const StackLayer &L, float eps) {
+  const dis_layer_config &lc = L.c;
+  return StackDelta{lc.heads, lc.kv_heads, lc.dim, lc.vdim, lc.conv_taps, lc.decay_rank, lc.gate_rank, L.conv_ch, L.a_off, L.g_off, L.b_off, eps};
+}
+
 static size_t align_up16(size_t v) { return (v + 15) / 16 * 16; }
 
 void Engine::free_stack() {
@@ -50,6 +62,9 @@ void Engine::free_stack() {
     }
     if (stack->ev_fork) cudaEventDestroy(stack->ev_fork);
     if (stack->sh_stream) cudaStreamDestroy(stack->sh_stream);
+    if (stack->ff_stream) cudaStreamDestroy(stack->ff_stream);
+    if (stack->ev_ff_fork) cudaEventDestroy(stack->ev_ff_fork);
+    if (stack->ev_ff_join) cudaEventDestroy(stack->ev_ff_join);
     if (stack->ev_sh_fork) cudaEventDestroy(stack->ev_sh_fork);
     if (stack->ev_sh_join) cudaEventDestroy(stack->ev_sh_join);
     for (StackTensor *v : stack->views) delete v;
@@ -117,7 +132,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   const bool gain_from_one = sc->norm_kind == DIS_NORM_RMS_ONE;  // stored norm vectors get 1 added as they are loaded; the kernels see plain gains
   if (gain_from_one) M.c.norm_kind = DIS_NORM_RMS;
   if (M.c.residual_mult == 0.f) M.c.residual_mult = 1.f;
-  const bool par_frame = (sc->frame_flags & DIS_FRAME_PARALLEL) != 0;
+  const bool par_frame = (sc->frame_flags & DIS_FRAME_PARALLEL) != 0, two_norms = (sc->frame_flags & DIS_FRAME_TWO_NORMS) != 0;
   M.max_rows = std::max(sc->max_logit_rows > 0 ? sc->max_logit_rows : max_batch, max_batch);
   M.layers.resize((size_t)sc->n_layers);
   const int W = sc->width, taps = sc->canon_taps;
@@ -171,7 +186,8 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "attention needs heads (a multiple of kv_heads), dim, vdim and an even rot_dims <= dim");
       if ((lc.attn_flags & DIS_ATTN_V_IS_K) && lc.vdim != lc.dim) return fail(DIS_ERR_INVALID_ARGUMENT, at + "values that are the keys need vdim == dim");
       if ((lc.attn_flags & DIS_ATTN_ROT_V) && (lc.vdim & 1)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "rotated values need an even vdim");
-      if (lc.rot_factor != 0.f && (lc.rot_high == lc.rot_low || lc.rot_original <= 0 || lc.rot_low <= 0.f || lc.rot_high <= 0.f))
+      if ((lc.attn_flags & DIS_ATTN_ROT_LINEAR) && !(lc.rot_factor > 0.f)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "linear rotary scaling needs a positive factor");
+      if (lc.rot_factor != 0.f && !(lc.attn_flags & DIS_ATTN_ROT_LINEAR) && (lc.rot_high == lc.rot_low || lc.rot_original <= 0 || lc.rot_low <= 0.f || lc.rot_high <= 0.f))
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "rotary scaling needs original > 0 and 0 < low != high");
       const unsigned fl = lc.attn_flags;
       if ((fl & DIS_ATTN_SINK) && (fl & DIS_ATTN_SIGMOID)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "a sink belongs to softmax weights");
@@ -187,6 +203,8 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         if (M.vmix_cols && M.vmix_cols != n) return fail(DIS_ERR_INVALID_ARGUMENT, at + "layers that mix values must agree in kv_heads * vdim");
         M.vmix_cols = n;
       }
+      if ((fl & DIS_ATTN_DIFF) && ((fl & ~(DIS_ATTN_DIFF | DIS_ATTN_ROT_PAIRS | DIS_ATTN_ROT_LINEAR | DIS_ATTN_BIAS_QKV)) || lc.kv_from >= 0 || lc.mixer != DIS_MIX_ATTENTION))
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "differential attention takes plain softmax weights and keys and values of its own");
       if (!(lc.score_softcap >= 0.f)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "score_softcap must not be negative");
       if ((fl & DIS_ATTN_SIGMOID) && (lc.score_softcap > 0.f || (fl & DIS_ATTN_SINK_UNIT))) return fail(DIS_ERR_INVALID_ARGUMENT, at + "a score soft cap and a sink belong to softmax weights");
       if ((fl & DIS_ATTN_SINK) && (fl & DIS_ATTN_SINK_UNIT)) return fail(DIS_ERR_INVALID_ARGUMENT, at + "sink: a learned logit per head or the unit term, not both");
@@ -198,16 +216,16 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
             ((src.attn_flags ^ fl) & DIS_ATTN_ROT_V))
           return fail(DIS_ERR_INVALID_ARGUMENT, at + "kv_from must name an attention layer with a cache of its own and the same kv_heads, dim, vdim and rotation");
       }
-      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
-      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, sc->norm_eps, lc.mask_chunk, lc.mask_window, lc.score_softcap, lc.mask_keep};
+      const StackAttn sa = stack_attn_shape(L, sc->norm_eps);
+      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim, dm = d * sa.maps;
       const int bq = stack_attn_block_tokens(sa, sc->compute_dtype == DIS_F32);
-      if (((size_t)32 * (d + dv + 10) + (size_t)(H / G) * (d + dv + 2)) * 4 > 200 * 1024) return fail(DIS_ERR_INVALID_ARGUMENT, at + "dim + vdim does not fit shared memory");
+      if (((size_t)32 * (dm + dv + 10) + (size_t)(H / G) * sa.maps * (d + dv + 2)) * 4 > 200 * 1024) return fail(DIS_ERR_INVALID_ARGUMENT, at + "dim + vdim does not fit shared memory");
       stack_abq = stack_abq ? std::min(stack_abq, bq) : bq;
       stack_att_heads = std::max(stack_att_heads, H);
       stack_att_groups = stack_att_groups ? std::min(stack_att_groups, G) : G;
-      stack_att_rec = std::max(stack_att_rec, (size_t)H * (dv + 2));
+      stack_att_rec = std::max(stack_att_rec, (size_t)H * sa.maps * (dv + 2));
       // rows of the input projection: q | k | v (a layer with a cache of its own) | one gate row per head
-      L.q_off = 0; L.k_off = H * d; L.v_off = L.k_off + G * d;
+      L.q_off = 0; L.k_off = H * dm; L.v_off = L.k_off + G * dm;
       L.n_in = lc.kv_from >= 0 ? H * d : L.v_off + ((lc.attn_flags & DIS_ATTN_V_IS_K) ? 0 : G * dv);
       if (lc.kv_from >= 0) L.k_off = L.v_off = 0;
       if (fl & DIS_ATTN_GATE) { L.g_off = L.n_in; L.n_in += H; }
@@ -247,6 +265,17 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       L.k_off = H * lc.dim; L.v_off = 2 * H * lc.dim; L.g_off = L.v_off + H * lc.vdim;
       L.n_in = L.g_off + H * lc.vdim;
       L.n_act = H * lc.vdim;
+    } else if (lc.mixer == DIS_MIX_CHANNEL_DELTA) {
+      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
+      if (H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || lc.conv_taps < 1 || lc.conv_taps > 16 || lc.decay_rank <= 0 || lc.gate_rank <= 0)
+        return fail(DIS_ERR_INVALID_ARGUMENT, at + "the gated delta rule needs heads (a multiple of kv_heads), dim, vdim, conv_taps 1..16, decay_rank and gate_rank");
+      if (d > 256 || std::max(lc.decay_rank, lc.gate_rank) > 2048) return fail(DIS_ERR_INVALID_ARGUMENT, at + "the gated delta rule takes dim up to 256 and bottlenecks up to 2048");
+      // rows of the input projection: q | k | v | decay bottleneck | gate bottleneck | step sizes; the convolution runs over q | k | v
+      L.k_off = G * d; L.v_off = 2 * G * d;
+      L.conv_ch = 2 * G * d + H * dv;
+      L.a_off = L.conv_ch; L.g_off = L.a_off + lc.decay_rank; L.b_off = L.g_off + lc.gate_rank;
+      L.n_in = L.b_off + H;
+      L.n_act = H * dv;
     } else return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown mixer");
     if (lc.mlp_act != DIS_ACT_CLAMPED && lc.mlp_act != DIS_ACT_GELU_TANH && lc.mlp_act != DIS_ACT_SILU && lc.mlp_act != DIS_ACT_RELU2) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown feed-forward activation");
     L.gu_rows = lc.mlp_act == DIS_ACT_RELU2 ? 1 : 2;
@@ -254,15 +283,20 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     else if (lc.mlp == DIS_MLP_MOE) {
       if (lc.ff <= 0 || lc.experts <= 0 || lc.top <= 0 || lc.top > lc.experts || lc.top > 32 || lc.experts > 1024)
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "experts: 1 <= top <= min(experts, 32), experts <= 1024");
-      if (lc.route_kind != DIS_ROUTE_SOFTMAX_TOP && lc.route_kind != DIS_ROUTE_SIGMOID_GROUPS && lc.route_kind != DIS_ROUTE_SOFTMAX_ALL) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown router kind");
+      if (lc.route_kind != DIS_ROUTE_SOFTMAX_TOP && lc.route_kind != DIS_ROUTE_SIGMOID_GROUPS && lc.route_kind != DIS_ROUTE_SOFTMAX_ALL &&
+          lc.route_kind != DIS_ROUTE_SOFTMAX_GROUPS) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown router kind");
       if (lc.route_groups > 1) {
-        if (lc.route_kind != DIS_ROUTE_SIGMOID_GROUPS || lc.experts % lc.route_groups || lc.route_keep < 1 || lc.route_keep > lc.route_groups ||
+        if ((lc.route_kind != DIS_ROUTE_SIGMOID_GROUPS && lc.route_kind != DIS_ROUTE_SOFTMAX_GROUPS) || lc.experts % lc.route_groups || lc.route_keep < 1 || lc.route_keep > lc.route_groups ||
             lc.route_keep * (lc.experts / lc.route_groups) < lc.top)
           return fail(DIS_ERR_INVALID_ARGUMENT, at + "expert groups: a divisor of experts, 1 <= keep <= groups, and the kept groups must hold at least top experts");
       }
       if (lc.shared_ff < 0) return fail(DIS_ERR_INVALID_ARGUMENT, at + "shared_ff");
     } else if (lc.mlp != DIS_MLP_NONE) return fail(DIS_ERR_INVALID_ARGUMENT, at + "unknown feed-forward kind");
-    if (par_frame) {  // the feed-forward's rows follow the mixer's in both projections
+    if (lc.mixer == DIS_MIX_CHANNEL_DELTA && !two_norms) return fail(DIS_ERR_INVALID_ARGUMENT, at + "the gated delta rule needs parallel layers with two norms");
+    if (two_norms && lc.mixer != DIS_MIX_ATTENTION && lc.mixer != DIS_MIX_PARALLEL && lc.mixer != DIS_MIX_LATENT && lc.mixer != DIS_MIX_RETENTION && lc.mixer != DIS_MIX_CHANNEL_DELTA)
+      return fail(DIS_ERR_INVALID_ARGUMENT, at + "parallel layers with two norms take the mixers attention, parallel, latent, retention and the gated delta rule");
+    if (two_norms && lc.mlp == DIS_MLP_DENSE && lc.mlp_act == DIS_ACT_CLAMPED) return fail(DIS_ERR_INVALID_ARGUMENT, at + "parallel layers with two norms take feed-forwards without biases");
+    if (par_frame && !two_norms) {  // the feed-forward's rows follow the mixer's in both projections
       if (lc.mixer != DIS_MIX_ATTENTION && lc.mixer != DIS_MIX_PARALLEL && lc.mixer != DIS_MIX_LATENT && lc.mixer != DIS_MIX_RETENTION)
         return fail(DIS_ERR_INVALID_ARGUMENT, at + "the parallel frame takes the mixers attention, parallel, latent and retention");
       if (lc.mlp == DIS_MLP_MOE || (lc.mlp == DIS_MLP_DENSE && lc.mlp_act == DIS_ACT_CLAMPED))
@@ -282,7 +316,12 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   if (!pre_frame && (M.c.residual_mult != 1.f || par_frame || gain_from_one))
     return fail(DIS_ERR_INVALID_ARGUMENT, "stack: residual_mult, the parallel frame and gains stored around zero need the pre-norm frame");
   if (par_frame && sc->streams > 0) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: the parallel frame has one residual");
+  if ((sc->frame_flags & (DIS_FRAME_TWO_NORMS | DIS_FRAME_LAYER_SCALE | DIS_FRAME_LOOP_EMBED)) && !(par_frame && two_norms))
+    return fail(DIS_ERR_INVALID_ARGUMENT, "stack: two norms need the parallel frame, layer scales and the embedding in front of loop passes need the two norms");
+  const bool loop_embed = sc->loop_times > 1 && (sc->frame_flags & DIS_FRAME_LOOP_EMBED);
+  if (loop_embed && !(sc->frame_flags & DIS_FRAME_LOOP_PLAIN)) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: the embedding in front of loop passes takes the place of the input projection");
   const bool loop_proj = sc->loop_times > 0 && !(sc->frame_flags & DIS_FRAME_LOOP_PLAIN);
+  if (loop_proj && two_norms) return fail(DIS_ERR_INVALID_ARGUMENT, "stack: parallel layers with two norms have no input projection in front of loop passes");
   const int n_streams = std::max(1, sc->streams);
   if (sc->loop_times < 0 || (sc->loop_times > 0 && !(0 <= sc->loop_start && sc->loop_start < sc->loop_stop && sc->loop_stop <= sc->n_layers)))
     return fail(DIS_ERR_INVALID_ARGUMENT, "stack: a loop needs 0 <= loop_start < loop_stop <= n_layers");
@@ -364,10 +403,10 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   static StackTensor dummy;  // scalars are written through their own small tensors below
   (void)dummy;
-  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0, lat_row = 0, lat_w[3] = {0, 0, 0};
+  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0, lat_row = 0, lat_w[3] = {0, 0, 0}, max_gz = 0, max_bn[2] = {0, 0};
   int max_top = 0, max_e = 0;
   bool any_shared = false;
-  size_t max_sff = 0;
+  size_t max_sff = 0, max_moe[2] = {0, 0};
   const size_t slots = (size_t)max_batch;
   std::vector<StackTensor *> scalars;
   for (int i = 0; i < sc->n_layers; i++) {
@@ -384,13 +423,17 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       for (int k = 0; k < 4; k++) {
         if (k >= 2 && lc.mlp == DIS_MLP_NONE) continue;
         if (pre_frame && (k & 1)) continue;  // no norms behind the sublayers
-        if (par_frame && k >= 2) continue;   // one norm for both
+        if (par_frame && !two_norms && k >= 2) continue;  // one norm for both
         ENG_CUDA(tensor(L.ln_w[k], (size_t)W, true));
         name(pre + gn[k], &L.ln_w[k], 0, {W}, i, gain_tr);
         if (!ln_bias) continue;
         ENG_CUDA(tensor(L.ln_b[k], (size_t)W, true));
         name(pre + gn[k] + ".b", &L.ln_b[k], 0, {W}, i);
       }
+    }
+    for (int q = 0; q < (lc.mlp == DIS_MLP_NONE ? 1 : 2) && (sc->frame_flags & DIS_FRAME_LAYER_SCALE); q++) {
+      ENG_CUDA(tensor(L.ls[q], (size_t)W, true));
+      name(pre + (q ? "ls2" : "ls1"), &L.ls[q], 0, {W}, i);
     }
     for (int q = 0; q < (lc.mlp == DIS_MLP_NONE ? 1 : 2) && sc->streams > 0; q++) {  // coefficients of the residual streams
       const int S = sc->streams;
@@ -431,11 +474,17 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       max_mix = std::max(max_mix, (size_t)H * dv);
       max_act = std::max(max_act, (size_t)H * dv);
     } else if (lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL) {
-      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
+      const bool diff = (lc.attn_flags & DIS_ATTN_DIFF) != 0;
+      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim, dm = diff ? 2 * d : d;
       const std::string a = pre + (lc.mixer == DIS_MIX_PARALLEL ? "mix.left." : "mix.");
       const bool own = lc.kv_from < 0;
-      name(a + "q", &L.w_in, 0, {H * d, W}, i);
-      if (own) name(a + "k", &L.w_in, (size_t)L.k_off * W, {G * d, W}, i);
+      name(a + "q", &L.w_in, 0, {H * dm, W}, i);
+      if (own) name(a + "k", &L.w_in, (size_t)L.k_off * W, {G * dm, W}, i);
+      if (diff) {
+        ENG_CUDA(tensor(L.diff_vec, (size_t)4 * d, true));
+        const char *dn[4] = {"lq1", "lk1", "lq2", "lk2"};
+        for (int k = 0; k < 4; k++) name(a + dn[k], &L.diff_vec, (size_t)k * d, {d}, i);
+      }
       if (own && !(lc.attn_flags & DIS_ATTN_V_IS_K)) name(a + "v", &L.w_in, (size_t)L.v_off * W, {G * dv, W}, i);
       if (lc.attn_flags & DIS_ATTN_GATE) name(a + "g", &L.w_in, (size_t)L.g_off * W, {H, W}, i);
       if (lc.attn_flags & DIS_ATTN_GATE_FULL) name(a + "g", &L.w_in, (size_t)L.g_off * W, {H * dv, W}, i);
@@ -454,9 +503,9 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       }
       if (lc.attn_flags & DIS_ATTN_BIAS_QKV) {
         ENG_CUDA(tensor(L.b_in, (size_t)L.n_rows, true));
-        name(a + "q.b", &L.b_in, 0, {H * d}, i);
+        name(a + "q.b", &L.b_in, 0, {H * dm}, i);
         if (own) {
-          name(a + "k.b", &L.b_in, (size_t)L.k_off, {G * d}, i);
+          name(a + "k.b", &L.b_in, (size_t)L.k_off, {G * dm}, i);
           name(a + "v.b", &L.b_in, (size_t)L.v_off, {G * dv}, i);
         }
       }
@@ -485,7 +534,8 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         const double kPi = 3.14159265358979323846;
         for (int k = 0; k < lc.rot_dims / 2; k++) {
           double v = std::pow((double)lc.rot_base, -2.0 * k / (double)lc.rot_dims);
-          if (lc.rot_factor != 0.f) {
+          if (lc.attn_flags & DIS_ATTN_ROT_LINEAR) v /= (double)lc.rot_factor;
+          else if (lc.rot_factor != 0.f) {
             const double wl = 2.0 * kPi / v, orig = (double)lc.rot_original;
             if (wl > orig / (double)lc.rot_low) v = v / (double)lc.rot_factor;
             else if (!(wl < orig / (double)lc.rot_high)) {
@@ -503,7 +553,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
           max_vrot = std::max(max_vrot, (size_t)dv);
         }
       }
-      max_qf = std::max(max_qf, (size_t)H * d);
+      max_qf = std::max(max_qf, (size_t)H * dm);
       if (lc.mixer == DIS_MIX_PARALLEL) {
         const int Hr = lc.gla_heads, dr = lc.gla_dim, dvr = lc.gla_vdim, rk = lc.gla_rank;
         const std::string r = pre + "mix.right.";
@@ -522,6 +572,34 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         max_mix = std::max(max_mix, (size_t)Hr * dvr);
         max_dec = std::max(max_dec, (size_t)Hr * dr);
       }
+    } else if (lc.mixer == DIS_MIX_CHANNEL_DELTA) {
+      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim, ra = lc.decay_rank, rg = lc.gate_rank, taps_d = lc.conv_taps;
+      const std::string m_ = pre + "mix.";
+      ENG_CUDA(tensor(L.conv_w, (size_t)L.conv_ch * taps_d, true));
+      const struct { const char *n; int off, rows; } proj[3] = {{"q", 0, G * d}, {"k", L.k_off, G * d}, {"v", L.v_off, H * dv}};
+      for (auto &p : proj) {
+        name(m_ + p.n, &L.w_in, (size_t)p.off * W, {p.rows, W}, i);
+        name(m_ + p.n + ".conv", &L.conv_w, (size_t)p.off * taps_d, {p.rows, taps_d}, i);
+      }
+      name(m_ + "a1", &L.w_in, (size_t)L.a_off * W, {ra, W}, i);
+      name(m_ + "g1", &L.w_in, (size_t)L.g_off * W, {rg, W}, i);
+      name(m_ + "b", &L.w_in, (size_t)L.b_off * W, {H, W}, i);
+      ENG_CUDA(tensor(L.a2, (size_t)H * d * ra, M.f32));
+      name(m_ + "a2", &L.a2, 0, {H * d, ra}, i);
+      ENG_CUDA(tensor(L.g2, (size_t)H * dv * rg, M.f32));
+      name(m_ + "g2", &L.g2, 0, {H * dv, rg}, i);
+      ENG_CUDA(tensor(L.ssm_vec, (size_t)H + (size_t)H * d, true));
+      name(m_ + "A_log", &L.ssm_vec, 0, {H}, i);
+      name(m_ + "dt_bias", &L.ssm_vec, (size_t)H, {H * d}, i);
+      ENG_CUDA(tensor(L.norm_w, (size_t)dv, true));
+      name(m_ + "norm", &L.norm_w, 0, {dv}, i);
+      ENG_CUDA(tensor(L.w_o, (size_t)W * L.ld_act, M.f32));
+      out_block(m_ + "o", 0, H * dv);
+      max_mix = std::max(max_mix, (size_t)H * dv);
+      max_dec = std::max(max_dec, (size_t)H * d);
+      max_ssm = std::max(max_ssm, ((size_t)L.conv_ch + G + H + 3) / 4 * 4);
+      max_gz = std::max(max_gz, (size_t)H * dv);
+      max_bn[0] = std::max(max_bn[0], (size_t)ra); max_bn[1] = std::max(max_bn[1], (size_t)rg);
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, C = L.conv_ch, inner = H * P;
       name(pre + "mix.in", &L.w_in, 0, {L.n_in, W}, i);
@@ -633,6 +711,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       }
       max_proj = std::max(max_proj, (size_t)gr * ff);
       max_act = std::max(max_act, (size_t)ff);
+      if (two_norms) { max_sff = std::max(max_sff, (size_t)ff); any_shared = true; }  // it runs in the lane of shared experts
     } else if (lc.mlp == DIS_MLP_MOE) {
       const int ff = lc.ff, E = lc.experts, gr = L.gu_rows;
       const bool shared_gate = lc.shared_ff > 0 && !(lc.mlp_flags & DIS_MLP_SHARED_PLAIN);
@@ -640,7 +719,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       ENG_CUDA(tensor(L.w_down, (size_t)E * W * ff, M.f32));
       ENG_CUDA(tensor(L.router, (size_t)(E + (shared_gate ? 1 : 0)) * W, true));
       name(pre + "mlp.router", &L.router, 0, {E, W}, i);
-      if (lc.route_kind == DIS_ROUTE_SIGMOID_GROUPS) {
+      if (lc.route_kind == DIS_ROUTE_SIGMOID_GROUPS || lc.route_kind == DIS_ROUTE_SOFTMAX_GROUPS) {
         ENG_CUDA(tensor(L.correction, (size_t)E, true));
         name(pre + "mlp.correction", &L.correction, 0, {E}, i);
       }
@@ -663,8 +742,11 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
         name(ep + "up", &L.w_gu, ((size_t)e * gr * ff + (size_t)(gr - 1) * ff) * W, {ff, W}, i);
         name(ep + "down", &L.w_down, (size_t)e * W * ff, {W, ff}, i);
       }
-      max_proj = std::max(max_proj, (size_t)lc.top * gr * ff);
-      max_act = std::max(max_act, (size_t)lc.top * ff);
+      if (two_norms) { max_moe[0] = std::max(max_moe[0], (size_t)lc.top * gr * ff); max_moe[1] = std::max(max_moe[1], (size_t)lc.top * ff); }
+      else {
+        max_proj = std::max(max_proj, (size_t)lc.top * gr * ff);
+        max_act = std::max(max_act, (size_t)lc.top * ff);
+      }
       max_top = std::max(max_top, lc.top);
       max_e = std::max(max_e, E);
     }
@@ -710,7 +792,10 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     }
     if (lc.mixer == DIS_MIX_LIGHTNING || lc.mixer == DIS_MIX_RETENTION) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.heads * lc.dim * lc.vdim * 4));
     else if (lc.mixer == DIS_MIX_MINGRU) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.width * 4));
-    else if (lc.mixer == DIS_MIX_PARALLEL) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.gla_heads * lc.gla_dim * lc.gla_vdim * 4));
+    else if (lc.mixer == DIS_MIX_CHANNEL_DELTA) {
+      ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.heads * lc.vdim * lc.dim * 4));
+      if (lc.conv_taps > 1) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.conv_state), slots * (lc.conv_taps - 1) * M.layers[(size_t)R.layer].conv_ch * 4));
+    } else if (lc.mixer == DIS_MIX_PARALLEL) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.gla_heads * lc.gla_dim * lc.gla_vdim * 4));
     else if (lc.mixer == DIS_MIX_SSM) {
       ENG_CUDA(alloc(reinterpret_cast<void **>(&R.state), slots * lc.heads * lc.ssm_state * lc.vdim * 4));
       if (lc.conv_taps > 1) ENG_CUDA(alloc(reinterpret_cast<void **>(&R.conv_state), slots * (lc.conv_taps - 1) * M.layers[(size_t)R.layer].conv_ch * 4));
@@ -737,8 +822,22 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   ENG_CUDA(alloc(reinterpret_cast<void **>(&M.qf), cap * max_qf * 4));
   ENG_CUDA(alloc(&M.act, cap * max_act * esz));
   ENG_CUDA(alloc(&M.xr, (size_t)M.max_rows * W * esz));
+  if (two_norms) {
+    ENG_CUDA(alloc(&M.hc2, cap * W * esz));
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.moe_proj), cap * max_moe[0] * 4));
+    ENG_CUDA(alloc(&M.moe_act, cap * max_moe[1] * esz));
+    ENG_CUDA(cudaStreamCreateWithFlags(&M.ff_stream, cudaStreamNonBlocking));
+    ENG_CUDA(cudaEventCreateWithFlags(&M.ev_ff_fork, cudaEventDisableTiming));
+    ENG_CUDA(cudaEventCreateWithFlags(&M.ev_ff_join, cudaEventDisableTiming));
+  }
+  if (max_gz) {
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.gz), cap * max_gz * 4));
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.dz), cap * max_dec * 4));
+    ENG_CUDA(alloc(&M.bn_a, cap * max_bn[0] * esz));
+    ENG_CUDA(alloc(&M.bn_g, cap * max_bn[1] * esz));
+  }
+  if (loop_proj || loop_embed) ENG_CUDA(alloc(reinterpret_cast<void **>(&M.x0), cap * W * 4));
   if (loop_proj) {
-    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.x0), cap * W * 4));
     ENG_CUDA(alloc(&M.xcat, cap * 2 * W * esz));
   }
   if (max_dec) ENG_CUDA(alloc(reinterpret_cast<void **>(&M.dec), cap * max_dec * 4));
@@ -808,11 +907,27 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   if (const char *g = getenv("DIS_STACK_PERSIST")) stack_persist = atoi(g) != 0;
   if (!M.f32 && stack_tc) {
-    M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), (size_t)W);
+    M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), std::max((size_t)W, std::max(max_gz, max_gz ? max_dec : 0)));
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.scratch), M.scratch_elems * 4));
   }
   ENG_CUDA(alloc(reinterpret_cast<void **>(&M.logits), (size_t)M.max_rows * sc->vocab * 4));
   logits = nullptr;  // the Llama buffer is not allocated; last_logits reads stack->logits
+  if (any_shared) {  // a shared expert, or the dense unit of a parallel layer with two norms
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.y2), cap * W * 4));
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.r_sg), cap * 4));
+    const char *lane = getenv("DIS_STACK_SHARED_LANE");  // 0: the shared expert runs in the pass's own stream (A/B runs)
+    if (two_norms || !(lane && atoi(lane) == 0)) {
+      ENG_CUDA(alloc(reinterpret_cast<void **>(&M.sh_proj), cap * 2 * max_sff * 4));
+      ENG_CUDA(alloc(&M.sh_act, cap * max_sff * esz));
+      if (!M.f32 && stack_tc) {
+        M.sh_scratch_elems = 2 * cap * std::max((size_t)2 * max_sff, (size_t)W);
+        ENG_CUDA(alloc(reinterpret_cast<void **>(&M.sh_scratch), M.sh_scratch_elems * 4));
+      }
+      ENG_CUDA(cudaStreamCreateWithFlags(&M.sh_stream, cudaStreamNonBlocking));
+      ENG_CUDA(cudaEventCreateWithFlags(&M.ev_sh_fork, cudaEventDisableTiming));
+      ENG_CUDA(cudaEventCreateWithFlags(&M.ev_sh_join, cudaEventDisableTiming));
+    }
+  }
   if (max_top > 0) {
     const size_t rows = cap * max_top;
     M.max_tiles = (int)((rows + kStackGemmTile - 1) / kStackGemmTile) + max_e;
@@ -823,22 +938,6 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.where), rows * 4));
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.tiles), (size_t)(1 + 3 * M.max_tiles) * 4));
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.rows_out), rows * W * 4));
-    if (any_shared) {
-      ENG_CUDA(alloc(reinterpret_cast<void **>(&M.y2), cap * W * 4));
-      ENG_CUDA(alloc(reinterpret_cast<void **>(&M.r_sg), cap * 4));
-      const char *lane = getenv("DIS_STACK_SHARED_LANE");  // 0: the shared expert runs in the pass's own stream (A/B runs)
-      if (!(lane && atoi(lane) == 0)) {
-        ENG_CUDA(alloc(reinterpret_cast<void **>(&M.sh_proj), cap * 2 * max_sff * 4));
-        ENG_CUDA(alloc(&M.sh_act, cap * max_sff * esz));
-        if (!M.f32 && stack_tc) {
-          M.sh_scratch_elems = 2 * cap * std::max((size_t)2 * max_sff, (size_t)W);
-          ENG_CUDA(alloc(reinterpret_cast<void **>(&M.sh_scratch), M.sh_scratch_elems * 4));
-        }
-        ENG_CUDA(cudaStreamCreateWithFlags(&M.sh_stream, cudaStreamNonBlocking));
-        ENG_CUDA(cudaEventCreateWithFlags(&M.ev_sh_fork, cudaEventDisableTiming));
-        ENG_CUDA(cudaEventCreateWithFlags(&M.ev_sh_join, cudaEventDisableTiming));
-      }
-    }
     if (!M.f32 && stack_tc) {
       ENG_CUDA(alloc(&M.moe_x, rows * W * 2));
       ENG_CUDA(cudaMallocHost(reinterpret_cast<void **>(&M.h_counts), (size_t)max_e * sizeof(int)));
@@ -856,11 +955,12 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   // ---- pages: one pool per latent layer that owns a cache (rows of kv_rank + rot_dim elements), a key and a value pool per
   // attention layer that owns one; a page id is valid in all
   {
+    auto key_dims = [](const dis_layer_config &lc) { return (lc.attn_flags & DIS_ATTN_DIFF) ? 2 * lc.dim : lc.dim; };  // of a key head
     size_t row_bytes = 0;
     for (auto &R : M.runs) {
       const dis_layer_config &lc = M.layers[(size_t)R.layer].c;
       if (lc.mixer == DIS_MIX_LATENT && lc.kv_from < 0) row_bytes += (size_t)(lc.kv_rank + lc.rot_dim) * esz;
-      if ((lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL) && lc.kv_from < 0) row_bytes += (size_t)lc.kv_heads * (lc.dim + lc.vdim) * esz;
+      if ((lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL) && lc.kv_from < 0) row_bytes += (size_t)lc.kv_heads * (key_dims(lc) + lc.vdim) * esz;
     }
     int64_t want = c->kv_pages;
     const int64_t useful = (int64_t)max_batch * max_pages;
@@ -878,7 +978,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       if (lc.mixer == DIS_MIX_LATENT && lc.kv_from < 0)
         ENG_CUDA(alloc(&R.pool, (size_t)n_pages * page_size * (lc.kv_rank + lc.rot_dim) * esz));
       if ((lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL) && lc.kv_from < 0) {
-        ENG_CUDA(alloc(&R.kpool, (size_t)n_pages * page_size * lc.kv_heads * lc.dim * esz));
+        ENG_CUDA(alloc(&R.kpool, (size_t)n_pages * page_size * lc.kv_heads * key_dims(lc) * esz));
         ENG_CUDA(alloc(&R.vpool, (size_t)n_pages * page_size * lc.kv_heads * lc.vdim * esz));
       }
     }
@@ -943,6 +1043,20 @@ int Engine::load_named(const char *nm, const void *host, int dtype, const int64_
     else ENG_CUDA(cudaMemcpy(dst, b.data(), n * 2, cudaMemcpyHostToDevice));
   }
   t.loaded = true;
+  return DIS_OK;
+}
+
+int Engine::stack_finalize() {
+  ENG_CUDA(cudaSetDevice(cfg.device));
+  for (StackLayer &L : stack->layers) {
+    if (L.c.mixer != DIS_MIX_ATTENTION || !(L.c.attn_flags & DIS_ATTN_DIFF)) continue;
+    const size_t d = (size_t)L.c.dim;  // the second map's factor: one number per layer
+    std::vector<float> v(4 * d);
+    ENG_CUDA(cudaMemcpy(v.data(), L.diff_vec.ptr, v.size() * 4, cudaMemcpyDeviceToHost));
+    double s1 = 0.0, s2 = 0.0;
+    for (size_t i = 0; i < d; i++) { s1 += (double)v[i] * v[d + i]; s2 += (double)v[2 * d + i] * v[3 * d + i]; }
+    L.diff_lambda = (float)(std::exp(s1) - std::exp(s2) + (double)L.c.attn_diff);
+  }
   return DIS_OK;
 }
 
@@ -1297,6 +1411,9 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     return launch_stack_gemm(g, cur_st);
   };
   const bool pre_frame = (M.c.frame_flags & DIS_FRAME_PRE_NORM) != 0;  // x += f(norm(x)), over residual streams where the model has them
+  const bool two_norms = (M.c.frame_flags & DIS_FRAME_TWO_NORMS) != 0;
+  const void *ff_in = two_norms ? M.hc2 : M.hc;  // the feed-forward's input
+  StackParBoundary pend_par;                      // parallel layers with two norms: what the next boundary joins
   const int n_streams = std::max(1, M.c.streams);
   RET_CUDA(launch_stack_embed(M.embed.ptr, f32, sp.tokens, sp.pos, M.pos_freq, M.x, M.x0, M.c.embed_scale, T, W, n_streams, stream)); kl++;
   const float *pend_y = nullptr, *pend_post = nullptr, *pend_post_b = nullptr;
@@ -1369,18 +1486,18 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     const int tc_act = act_kind == DIS_ACT_GELU_TANH ? 1 : 0;
     kl++;
     if (stack_persist && gemm_use_persist(T, ff, true)) {  // paired gate / up tiles on the persistent kernel
-      const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, 256);
+      const TmaMap *xm = stack_map(ff_in, (uint64_t)cap_tokens, (uint64_t)W, 256);
       const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, 64);
       if (!xm || !wm) return cudaErrorInvalidValue;
       return launch_gemm_persist_glu(*wm, *xm, reinterpret_cast<uint16_t *>(act), T, ff, W, 0, tc_act, cur_st, ld_act);
     }
     const int tr = 128;
-    const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, (uint32_t)gemm_token_tile(T));
+    const TmaMap *xm = stack_map(ff_in, (uint64_t)cap_tokens, (uint64_t)W, (uint32_t)gemm_token_tile(T));
     const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)2 * ff, (uint64_t)W, (uint32_t)tr);
     if (!xm || !wm) return cudaErrorInvalidValue;
     return launch_gemm_glu(*wm, *xm, reinterpret_cast<uint16_t *>(act), T, ff, W, 0, tr, tc_act, cur_st, ld_act);
   };
-  // A dense gated unit out = W_down act(W_gate h, W_up h) on the sublayer input M.hc.  later: the slices of the down projection
+  // A dense gated unit out = W_down act(W_gate h, W_up h) on the feed-forward's input.  later: the slices of the down projection
   // may stay unsummed for the next boundary kernel (out is then M.y, as the caller expects).
   auto dense_ff = [&](const StackTensor &w_gu, const StackTensor &b_gu, const StackTensor &w_down, const StackTensor &b_down, int ff,
                       int act_kind, float limit, float *out, bool later_ok) -> cudaError_t {
@@ -1391,7 +1508,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     }
     // an ungated unit in prompt-sized bf16 passes: the persistent product's epilogue squares the relu and writes bf16
     if (stack_tc && stack_persist && !f32 && act_kind == DIS_ACT_RELU2 && !b_gu.ptr && W % 8 == 0 && !w_gu.f32 && gemm_use_persist(T, ff, false)) {
-      const TmaMap *xm = stack_map(M.hc, (uint64_t)cap_tokens, (uint64_t)W, 256);
+      const TmaMap *xm = stack_map(ff_in, (uint64_t)cap_tokens, (uint64_t)W, 256);
       const TmaMap *wm = stack_map(w_gu.ptr, (uint64_t)ff, (uint64_t)W, 128);
       if (!xm || !wm) return cudaErrorInvalidValue;
       RET_CUDA(launch_gemm_persist_relu2(*wm, *xm, reinterpret_cast<uint16_t *>(cur_act), T, ff, W, 0, cur_st));
@@ -1400,13 +1517,122 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     }
     // the gated unit sums the slices of its input product itself and adds the bias the product left out
     const float *gu_bias = nullptr;
-    RET_CUDA(gemm(M.hc, f32, W, w_gu, 0, reinterpret_cast<const float *>(b_gu.ptr), cur_proj, T, gu_rows * ff, W, cap_tokens, &gu_bias, true));
+    RET_CUDA(gemm(ff_in, f32, W, w_gu, 0, reinterpret_cast<const float *>(b_gu.ptr), cur_proj, T, gu_rows * ff, W, cap_tokens, &gu_bias, true));
     const bool sliced = pend_parts > 1 || pend_bias;
     RET_CUDA(launch_stack_glu(sliced ? pend_src : cur_proj, sliced ? pend_parts : 1, pend_stride, sliced ? pend_bias : gu_bias, cur_act, f32, nullptr,
                               T, ff, limit, act_kind, cur_st));
     kl++;
     pend_parts = 1; pend_bias = nullptr;
     return gemm(cur_act, f32, ff, w_down, 0, reinterpret_cast<const float *>(b_down.ptr), out, T, W, ff, cap_tokens, nullptr, later_ok);
+  };
+  // A mixture of experts on the feed-forward's input, launched in stream st0 with room for the experts' rows in mproj and mact.  Its sum
+  // goes to M.y, or (out) is left to the boundary kernel that out describes.
+  auto moe_ff = [&](StackLayer &L, cudaStream_t st0, float *mproj, void *mact, StackParBoundary *out) -> cudaError_t {
+    const dis_layer_config &lc = L.c;
+    const int ff = lc.ff, E = lc.experts, top = lc.top, rows = T * top;
+    const int gc = L.gu_rows * ff;  // columns of an expert's first product: gate | up, or up alone
+    const bool shared_gate = lc.shared_ff > 0 && !(lc.mlp_flags & DIS_MLP_SHARED_PLAIN);
+    // the always-on unit beside the experts: its dense product first (it borrows the buffers the experts' rows use afterwards);
+    // the logit of its per-token gate is one more row of the router matrix, and the combine kernel adds it in
+    const bool shared = lc.shared_ff > 0;
+    const float *sh_src = M.y2;
+    int sh_parts = 1;
+    long long sh_stride = 0;
+    const bool sh_lane = shared && M.sh_stream != nullptr;
+    if (shared) {
+      if (sh_lane) {  // fork: the shared expert's launches go to its own stream and buffers
+        RET_CUDA(cudaEventRecord(M.ev_sh_fork, st0));
+        RET_CUDA(cudaStreamWaitEvent(M.sh_stream, M.ev_sh_fork, 0));
+        cur_st = M.sh_stream; cur_scratch = M.sh_scratch; cur_scratch_elems = M.sh_scratch_elems; cur_proj = M.sh_proj; cur_act = M.sh_act;
+      }
+      const cudaError_t se = dense_ff(L.w_sgu, StackTensor(), L.w_sdown, StackTensor(), lc.shared_ff, lc.mlp_act, lc.limit, M.y2, true);
+      cur_st = stream; cur_scratch = M.scratch; cur_scratch_elems = M.scratch_elems; cur_proj = M.proj; cur_act = M.act;
+      RET_CUDA(se);
+      if (pend_parts > 1) { sh_src = pend_src; sh_parts = pend_parts; sh_stride = pend_stride; }  // the combine kernel sums the slices
+      pend_parts = 1; pend_bias = nullptr;
+    }
+    auto combine = [&]() -> cudaError_t {
+      if (out) {
+        out->rows = M.rows_out; out->where = M.where; out->wt = M.r_wt; out->top = top;
+        if (shared) { out->y2 = sh_src; out->n2 = sh_parts; out->s2 = sh_stride; out->y2_gate = shared_gate ? M.r_sg : nullptr; }
+        kl--;
+        return cudaSuccess;
+      }
+      return launch_stack_moe_combine(M.rows_out, M.where, M.r_wt, shared ? sh_src : nullptr, sh_parts, sh_stride, shared_gate ? M.r_sg : nullptr, M.y, T, W, top, st0);
+    };
+    auto join_shared = [&]() -> cudaError_t {
+      if (!sh_lane) return cudaSuccess;
+      RET_CUDA(cudaEventRecord(M.ev_sh_join, M.sh_stream));
+      return cudaStreamWaitEvent(st0, M.ev_sh_join, 0);
+    };
+    const float *router = reinterpret_cast<const float *>(L.router.ptr);
+    RET_CUDA(launch_stack_route(ff_in, f32, router, T, W, E, top, lc.route_kind, reinterpret_cast<const float *>(L.correction.ptr), lc.route_groups,
+                                lc.route_keep, shared_gate ? router + (size_t)E * W : nullptr, M.r_sg, M.r_idx, M.r_wt, st0));
+    RET_CUDA(launch_stack_moe_plan(M.r_idx, T, top, E, kStackGemmTile, M.counts, M.perm_tok, M.where, M.tiles, M.max_tiles, st0));
+    // Large passes in bf16: one tensor-core product per expert over its rows.  The row counts come back to the host (one
+    // small copy and a wait), so this path is not taken while a decode pass is being captured into a graph.
+    if (M.moe_x && !stack_capturing && rows >= 64 * E && W % 8 == 0 && ff % 8 == 0) {
+      RET_CUDA(launch_stack_moe_gather(ff_in, M.perm_tok, M.moe_x, rows, W, st0));
+      RET_CUDA(cudaMemcpyAsync(M.h_counts, M.counts, (size_t)E * sizeof(int), cudaMemcpyDeviceToHost, st0));
+      RET_CUDA(cudaStreamSynchronize(st0));
+      kl += 4;
+      // An expert's rows are few against the GPU (its products fill a fraction of the SMs, or one wave and a bit), so the
+      // experts run side by side: the pass's stream forks into kSide more, expert e keeps to stream e mod (kSide + 1) with its
+      // gate | up product, its gated unit and its down product in order, and the streams join in front of the combine kernel.
+      const bool forked = M.side[0] && !getenv("DIS_STACK_MOE_SERIAL");
+      auto lane = [&](int e) { const int k = e % (StackModel::kSide + 1); return forked && k > 0 ? M.side[k - 1] : st0; };
+      if (forked) {
+        RET_CUDA(cudaEventRecord(M.ev_fork, st0));
+        for (int k = 0; k < StackModel::kSide; k++) RET_CUDA(cudaStreamWaitEvent(M.side[k], M.ev_fork, 0));
+      }
+      int off = 0;
+      for (int e = 0; e < E; e++) {
+        const int cnt = M.h_counts[e];
+        if (cnt <= 0) continue;
+        cudaStream_t es = lane(e);
+        TmaMap xm, am;
+        RET_CUDA(make_tma_map_2d(&xm, reinterpret_cast<uint16_t *>(M.moe_x) + (size_t)off * W, (uint64_t)cnt, (uint64_t)W, (uint32_t)gemm_token_tile(cnt)));
+        const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.w_gu.ptr) + (size_t)e * gc * W, (uint64_t)gc, (uint64_t)W, 128);
+        if (!wm) return cudaErrorInvalidValue;
+        RET_CUDA(launch_gemm_partial(*wm, xm, mproj + (size_t)off * gc, cnt, gc, W, 0, 1, es));
+        RET_CUDA(launch_stack_glu(mproj + (size_t)off * gc, 1, 0, nullptr, reinterpret_cast<uint16_t *>(mact) + (size_t)off * ff, f32, nullptr, cnt, ff,
+                                  lc.limit, lc.mlp_act, es));
+        RET_CUDA(make_tma_map_2d(&am, reinterpret_cast<uint16_t *>(mact) + (size_t)off * ff, (uint64_t)cnt, (uint64_t)ff, (uint32_t)gemm_token_tile(cnt)));
+        const TmaMap *dm = stack_map(reinterpret_cast<const uint16_t *>(L.w_down.ptr) + (size_t)e * W * ff, (uint64_t)W, (uint64_t)ff, 128);
+        if (!dm) return cudaErrorInvalidValue;
+        RET_CUDA(launch_gemm_partial(*dm, am, M.rows_out + (size_t)off * W, cnt, W, ff, 0, 1, es));
+        off += cnt; kl += 3;
+      }
+      kl--;  // (the count above included one gated-unit launch over all rows)
+      if (forked)
+        for (int k = 0; k < StackModel::kSide; k++) {
+          RET_CUDA(cudaEventRecord(M.ev_join[k], M.side[k]));
+          RET_CUDA(cudaStreamWaitEvent(st0, M.ev_join[k], 0));
+        }
+      RET_CUDA(join_shared());
+      return combine();
+    }
+    const int tiles_cap = std::min(M.max_tiles, (rows + kStackGemmTile - 1) / kStackGemmTile + E);
+    StackGemm g;
+    g.A = ff_in; g.a_f32 = f32; g.lda = W; g.a_gather = M.perm_tok;
+    g.W = L.w_gu.ptr; g.w_f32 = L.w_gu.f32; g.ldw = W; g.w_bs = (long long)gc * W;
+    g.out = mproj; g.ldo = gc; g.M = rows; g.N = gc; g.K = W;
+    g.tiles = M.tiles; g.max_tiles = tiles_cap;
+    RET_CUDA(launch_stack_gemm(g, st0));
+    StackGemm dn;
+    dn.A = mact; dn.a_f32 = f32; dn.lda = ff;
+    dn.W = L.w_down.ptr; dn.w_f32 = L.w_down.f32; dn.ldw = ff; dn.w_bs = (long long)W * ff;
+    dn.out = M.rows_out; dn.ldo = W; dn.M = rows; dn.N = W; dn.K = ff;
+    dn.tiles = M.tiles; dn.max_tiles = tiles_cap;
+    static const bool few_glu = getenv("DIS_STACK_FEW_GLU") && atoi(getenv("DIS_STACK_FEW_GLU")) != 0;  // opt-in: measured slower (0.547 against 0.534 ms per step)
+    if (few_glu && L.gu_rows == 2 && stack_gemm_few_rows(dn)) {  // a handful of rows: the down product's loader applies the gated unit to the gate | up rows
+      dn.A = mproj; dn.a_f32 = true; dn.lda = 2 * ff; dn.a_glu = lc.mlp_act + 1; dn.a_limit = lc.limit;
+      kl--;
+    } else RET_CUDA(launch_stack_glu(mproj, 1, 0, nullptr, mact, f32, nullptr, rows, ff, lc.limit, lc.mlp_act, st0));
+    RET_CUDA(launch_stack_gemm(dn, st0));
+    RET_CUDA(join_shared());
+    kl += 6;
+    return combine();
   };
   for (size_t ri = 0; ri < M.runs.size(); ri++) {
     StackRun &Rn = M.runs[ri];
@@ -1420,7 +1646,16 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
                     2 * W, cap_tokens));
     }
     next_hc = reinterpret_cast<const float *>(L.hc[0].ptr);
-    RET_CUDA(sublayer_in(norm_w(L, 0), norm_b(L, 0), L.canon1, Rn.cstate1));
+    if (two_norms) {
+      pend_par.add = Rn.loop_pass > 0 ? M.x0 : nullptr;  // (allocated when the model wants the embedding in front of loop passes)
+      RET_CUDA(launch_stack_boundary_par(M.x, pend_par, res_mult, norm_w(L, 0), M.hc, reinterpret_cast<const float *>(L.ln_w[2].ptr), M.hc2, f32, T, W, eps, stream));
+      kl++;
+      pend_par = StackParBoundary();
+      if (lc.mlp != DIS_MLP_NONE) {  // the feed-forward runs beside the mixer, in a lane that joins in front of the next boundary
+        RET_CUDA(cudaEventRecord(M.ev_ff_fork, stream));
+        RET_CUDA(cudaStreamWaitEvent(M.ff_stream, M.ev_ff_fork, 0));
+      }
+    } else RET_CUDA(sublayer_in(norm_w(L, 0), norm_b(L, 0), L.canon1, Rn.cstate1));
     // Parallel layers: the feed-forward reads the same h.  Its gate and up rows follow the mixer's in the input projection, so a
     // decode-sized pass runs them as one product; a prompt-sized pass keeps the product whose epilogue is the gated unit.  Either way
     // the unit's output goes to the columns behind the mixer's in M.act, and one product with [mixer.o | down] ends the layer.
@@ -1431,7 +1666,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     const float *in_bias = nullptr;  // minGRU adds its projections' biases itself when the product left them out
     const bool is_attn = lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_PARALLEL;
     // the preparation kernels of attention (alone), latent attention and retention sum the slices of a split-K input projection themselves
-    const bool prep_sums = lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_LATENT || lc.mixer == DIS_MIX_RETENTION;
+    const bool prep_sums = lc.mixer == DIS_MIX_ATTENTION || lc.mixer == DIS_MIX_LATENT || lc.mixer == DIS_MIX_RETENTION || lc.mixer == DIS_MIX_CHANNEL_DELTA;
     if (split_in) RET_CUDA(glu_product(L.w_gu, par_ff, lc.mlp_act, ff_act, L.ld_act));
     RET_CUDA(gemm(M.hc, f32, W, L.w_in, 0, L.b_in.ptr ? reinterpret_cast<const float *>(L.b_in.ptr) : nullptr, M.proj, T, N, W, cap_tokens,
                   lc.mixer == DIS_MIX_MINGRU || is_attn ? &in_bias : nullptr, prep_sums));
@@ -1466,6 +1701,29 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
                                       segments ? M.light_seg : nullptr, max_span, M.proj + L.g_off, N, M.act, L.ld_act, f32, eps, stream));
       kl += segments ? 5 : nb > 1 || d > 128 || dv > 128 ? 3 : 2;
       n_mix = L.ld_act;
+    } else if (lc.mixer == DIS_MIX_CHANNEL_DELTA) {
+      const StackDelta sd = stack_delta_shape(L, eps);
+      const int nz = sd.H * sd.d, ng = sd.H * sd.dv;
+      StackDeltaPrep a;
+      a.proj = in_src; a.ld = N; a.n_part = in_parts; a.stride = in_stride;
+      a.cw = reinterpret_cast<const float *>(L.conv_w.ptr); a.vec = reinterpret_cast<const float *>(L.ssm_vec.ptr); a.cstate = Rn.conv_state;
+      a.a2 = L.a2.ptr; a.g2 = L.g2.ptr;
+      a.buf = M.ssm; a.ld_b = ((long long)sd.C + sd.G + sd.H + 3) / 4 * 4; a.dec = M.dec; a.gz = M.gz;
+      if (T > 64) {  // more tokens than the preparation should multiply by itself: the bottlenecks' products as matrix products
+        RET_CUDA(launch_stack_delta_pack(sd, a, f32, T, M.bn_a, M.bn_g, stream));
+        kl++;
+        if (in_parts > 1) cur_scratch = nullptr, cur_scratch_elems = 0;  // the input projection's slices are still wanted: no slices beside them
+        const cudaError_t ez = gemm(M.bn_a, f32, sd.ra, L.a2, 0, nullptr, M.dz, T, nz, sd.ra, cap_tokens);
+        const cudaError_t eg = ez != cudaSuccess ? ez : gemm(M.bn_g, f32, sd.rg, L.g2, 0, nullptr, M.gz, T, ng, sd.rg, cap_tokens);
+        cur_scratch = M.scratch; cur_scratch_elems = M.scratch_elems;
+        RET_CUDA(eg);
+        a.z = M.dz;
+      }
+      RET_CUDA(launch_stack_delta_prep(sd, a, L.a2.f32, sp, stream));
+      RET_CUDA(launch_stack_delta(sd, M.ssm, a.ld_b, M.dec, Rn.state, sp, M.mix, max_span, reinterpret_cast<const float *>(L.norm_w.ptr), M.gz, M.act,
+                                  L.ld_act, f32, &kl, stream));
+      kl += sd.taps > 1 && !single ? 2 : 1;
+      n_mix = L.ld_act;
     } else if (lc.mixer == DIS_MIX_SSM) {
       const int H = lc.heads, P = lc.vdim, Ns = lc.ssm_state, G = lc.ssm_groups, C = L.conv_ch, inner = H * P;
       const long long ld_b = C;  // x | B | C
@@ -1488,9 +1746,9 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       RET_CUDA(launch_stack_mingru(M.proj, N, in_bias, Rn.state, sp, M.act, f32, lc.width, max_len, stream)); kl++;
       n_mix = lc.width;
     } else if (is_attn) {
-      const int H = lc.heads, G = lc.kv_heads, d = lc.dim, dv = lc.vdim;
+      const int H = lc.heads, d = lc.dim, dv = lc.vdim;
       const bool par = lc.mixer == DIS_MIX_PARALLEL;
-      StackAttn sa{H, G, d, dv, lc.rot_dims, lc.attn_flags, lc.scale, eps, lc.mask_chunk, lc.mask_window, lc.score_softcap, lc.mask_keep};
+      const StackAttn sa = stack_attn_shape(L, eps);
       const float *qkn = reinterpret_cast<const float *>(L.qk_norm.ptr), *tpb = reinterpret_cast<const float *>(L.temp_pb.ptr);
       // the gains of the key norm follow those of the query norm: [H*d] then [G*d] (whole projection), or [d] then [d] (per head)
       const float *kn = qkn ? qkn + ((lc.attn_flags & DIS_ATTN_QK_NORM_HEAD) ? (size_t)d : (size_t)H * d) : nullptr;
@@ -1692,6 +1950,25 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       n_mix = L.ld_act;
     }
     RET_CUDA(gemm(M.act, f32, n_mix, L.w_o, 0, o_bias, M.y, T, W, n_mix, cap_tokens, nullptr, later));
+    if (two_norms) {
+      const bool sliced = pend_parts > 1 || pend_bias;
+      pend_par.y1 = sliced ? pend_src : M.y; pend_par.n1 = pend_parts; pend_par.s1 = pend_stride; pend_par.b1 = pend_bias;
+      pend_par.ls1 = reinterpret_cast<const float *>(L.ls[0].ptr); pend_par.ls2 = reinterpret_cast<const float *>(L.ls[1].ptr);
+      pend_parts = 1; pend_bias = nullptr;
+      if (lc.mlp == DIS_MLP_DENSE) {
+        cur_st = M.ff_stream; cur_scratch = M.sh_scratch; cur_scratch_elems = M.sh_scratch_elems; cur_proj = M.sh_proj; cur_act = M.sh_act;
+        const cudaError_t e = dense_ff(L.w_gu, L.b_gu, L.w_down, L.b_down, lc.ff, lc.mlp_act, lc.limit, M.y2, true);
+        cur_st = stream; cur_scratch = M.scratch; cur_scratch_elems = M.scratch_elems; cur_proj = M.proj; cur_act = M.act;
+        RET_CUDA(e);
+        pend_par.y2 = pend_parts > 1 ? pend_src : M.y2; pend_par.n2 = pend_parts; pend_par.s2 = pend_stride;
+        pend_parts = 1; pend_bias = nullptr;
+      } else if (lc.mlp == DIS_MLP_MOE) RET_CUDA(moe_ff(L, M.ff_stream, M.moe_proj, M.moe_act, &pend_par));
+      if (lc.mlp != DIS_MLP_NONE) {
+        RET_CUDA(cudaEventRecord(M.ev_ff_join, M.ff_stream));
+        RET_CUDA(cudaStreamWaitEvent(stream, M.ev_ff_join, 0));
+      }
+      continue;
+    }
     pend_y = M.y; pend_post = norm_w(L, 1); pend_post_b = norm_b(L, 1); pend_hc = reinterpret_cast<const float *>(L.hc[0].ptr);
     if (lc.mlp == DIS_MLP_NONE || par_ff > 0) continue;  // (a parallel layer's feed-forward is in the product above)
     next_hc = reinterpret_cast<const float *>(L.hc[1].ptr);
@@ -1699,110 +1976,14 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
     if (lc.mlp == DIS_MLP_DENSE) {
       RET_CUDA(dense_ff(L.w_gu, L.b_gu, L.w_down, L.b_down, lc.ff, lc.mlp_act, lc.limit, M.y, later));
     } else {
-      const int ff = lc.ff, E = lc.experts, top = lc.top, rows = T * top;
-      const int gc = L.gu_rows * ff;  // columns of an expert's first product: gate | up, or up alone
-      const bool shared_gate = lc.shared_ff > 0 && !(lc.mlp_flags & DIS_MLP_SHARED_PLAIN);
-      // the always-on unit beside the experts: its dense product first (it borrows the buffers the experts' rows use afterwards);
-      // the logit of its per-token gate is one more row of the router matrix, and the combine kernel adds it in
-      const bool shared = lc.shared_ff > 0;
-      const float *sh_src = M.y2;
-      int sh_parts = 1;
-      long long sh_stride = 0;
-      const bool sh_lane = shared && M.sh_stream != nullptr;
-      if (shared) {
-        if (sh_lane) {  // fork: the shared expert's launches go to its own stream and buffers
-          RET_CUDA(cudaEventRecord(M.ev_sh_fork, stream));
-          RET_CUDA(cudaStreamWaitEvent(M.sh_stream, M.ev_sh_fork, 0));
-          cur_st = M.sh_stream; cur_scratch = M.sh_scratch; cur_scratch_elems = M.sh_scratch_elems; cur_proj = M.sh_proj; cur_act = M.sh_act;
-        }
-        const cudaError_t se = dense_ff(L.w_sgu, StackTensor(), L.w_sdown, StackTensor(), lc.shared_ff, lc.mlp_act, lc.limit, M.y2, true);
-        cur_st = stream; cur_scratch = M.scratch; cur_scratch_elems = M.scratch_elems; cur_proj = M.proj; cur_act = M.act;
-        RET_CUDA(se);
-        if (pend_parts > 1) { sh_src = pend_src; sh_parts = pend_parts; sh_stride = pend_stride; }  // the combine kernel sums the slices
-        pend_parts = 1; pend_bias = nullptr;
-      }
-      auto join_shared = [&]() -> cudaError_t {
-        if (!sh_lane) return cudaSuccess;
-        RET_CUDA(cudaEventRecord(M.ev_sh_join, M.sh_stream));
-        return cudaStreamWaitEvent(stream, M.ev_sh_join, 0);
-      };
-      const float *router = reinterpret_cast<const float *>(L.router.ptr);
-      RET_CUDA(launch_stack_route(M.hc, f32, router, T, W, E, top, lc.route_kind, reinterpret_cast<const float *>(L.correction.ptr), lc.route_groups,
-                                  lc.route_keep, shared_gate ? router + (size_t)E * W : nullptr, M.r_sg, M.r_idx, M.r_wt, stream));
-      RET_CUDA(launch_stack_moe_plan(M.r_idx, T, top, E, kStackGemmTile, M.counts, M.perm_tok, M.where, M.tiles, M.max_tiles, stream));
-      // Large passes in bf16: one tensor-core product per expert over its rows.  The row counts come back to the host (one
-      // small copy and a wait), so this path is not taken while a decode pass is being captured into a graph.
-      const float *sh_gate = shared_gate ? M.r_sg : nullptr;  // null: the shared unit joins the sum as it is
-      if (M.moe_x && !stack_capturing && rows >= 64 * E && W % 8 == 0 && ff % 8 == 0) {
-        RET_CUDA(launch_stack_moe_gather(M.hc, M.perm_tok, M.moe_x, rows, W, stream));
-        RET_CUDA(cudaMemcpyAsync(M.h_counts, M.counts, (size_t)E * sizeof(int), cudaMemcpyDeviceToHost, stream));
-        RET_CUDA(cudaStreamSynchronize(stream));
-        kl += 4;
-        // An expert's rows are few against the GPU (its products fill a fraction of the SMs, or one wave and a bit), so the
-        // experts run side by side: the pass's stream forks into kSide more, expert e keeps to stream e mod (kSide + 1) with its
-        // gate | up product, its gated unit and its down product in order, and the streams join in front of the combine kernel.
-        const bool forked = M.side[0] && !getenv("DIS_STACK_MOE_SERIAL");
-        auto lane = [&](int e) { const int k = e % (StackModel::kSide + 1); return forked && k > 0 ? M.side[k - 1] : stream; };
-        if (forked) {
-          RET_CUDA(cudaEventRecord(M.ev_fork, stream));
-          for (int k = 0; k < StackModel::kSide; k++) RET_CUDA(cudaStreamWaitEvent(M.side[k], M.ev_fork, 0));
-        }
-        int off = 0;
-        for (int e = 0; e < E; e++) {
-          const int cnt = M.h_counts[e];
-          if (cnt <= 0) continue;
-          cudaStream_t es = lane(e);
-          TmaMap xm, am;
-          RET_CUDA(make_tma_map_2d(&xm, reinterpret_cast<uint16_t *>(M.moe_x) + (size_t)off * W, (uint64_t)cnt, (uint64_t)W, (uint32_t)gemm_token_tile(cnt)));
-          const TmaMap *wm = stack_map(reinterpret_cast<const uint16_t *>(L.w_gu.ptr) + (size_t)e * gc * W, (uint64_t)gc, (uint64_t)W, 128);
-          if (!wm) return cudaErrorInvalidValue;
-          RET_CUDA(launch_gemm_partial(*wm, xm, M.proj + (size_t)off * gc, cnt, gc, W, 0, 1, es));
-          RET_CUDA(launch_stack_glu(M.proj + (size_t)off * gc, 1, 0, nullptr, reinterpret_cast<uint16_t *>(M.act) + (size_t)off * ff, f32, nullptr, cnt, ff,
-                                    lc.limit, lc.mlp_act, es));
-          RET_CUDA(make_tma_map_2d(&am, reinterpret_cast<uint16_t *>(M.act) + (size_t)off * ff, (uint64_t)cnt, (uint64_t)ff, (uint32_t)gemm_token_tile(cnt)));
-          const TmaMap *dm = stack_map(reinterpret_cast<const uint16_t *>(L.w_down.ptr) + (size_t)e * W * ff, (uint64_t)W, (uint64_t)ff, 128);
-          if (!dm) return cudaErrorInvalidValue;
-          RET_CUDA(launch_gemm_partial(*dm, am, M.rows_out + (size_t)off * W, cnt, W, ff, 0, 1, es));
-          off += cnt; kl += 3;
-        }
-        kl--;  // (the count above included one gated-unit launch over all rows)
-        if (forked)
-          for (int k = 0; k < StackModel::kSide; k++) {
-            RET_CUDA(cudaEventRecord(M.ev_join[k], M.side[k]));
-            RET_CUDA(cudaStreamWaitEvent(stream, M.ev_join[k], 0));
-          }
-        RET_CUDA(join_shared());
-        RET_CUDA(launch_stack_moe_combine(M.rows_out, M.where, M.r_wt, shared ? sh_src : nullptr, sh_parts, sh_stride, sh_gate, M.y, T, W, top, stream));
-        pend_y = M.y; pend_post = norm_w(L, 3); pend_post_b = norm_b(L, 3); pend_hc = reinterpret_cast<const float *>(L.hc[1].ptr);
-        continue;
-      }
-      const int tiles_cap = std::min(M.max_tiles, (rows + kStackGemmTile - 1) / kStackGemmTile + E);
-      StackGemm g;
-      g.A = M.hc; g.a_f32 = f32; g.lda = W; g.a_gather = M.perm_tok;
-      g.W = L.w_gu.ptr; g.w_f32 = L.w_gu.f32; g.ldw = W; g.w_bs = (long long)gc * W;
-      g.out = M.proj; g.ldo = gc; g.M = rows; g.N = gc; g.K = W;
-      g.tiles = M.tiles; g.max_tiles = tiles_cap;
-      RET_CUDA(launch_stack_gemm(g, stream));
-      StackGemm dn;
-      dn.A = M.act; dn.a_f32 = f32; dn.lda = ff;
-      dn.W = L.w_down.ptr; dn.w_f32 = L.w_down.f32; dn.ldw = ff; dn.w_bs = (long long)W * ff;
-      dn.out = M.rows_out; dn.ldo = W; dn.M = rows; dn.N = W; dn.K = ff;
-      dn.tiles = M.tiles; dn.max_tiles = tiles_cap;
-      static const bool few_glu = getenv("DIS_STACK_FEW_GLU") && atoi(getenv("DIS_STACK_FEW_GLU")) != 0;  // opt-in: measured slower (0.547 against 0.534 ms per step)
-      if (few_glu && L.gu_rows == 2 && stack_gemm_few_rows(dn)) {  // a handful of rows: the down product's loader applies the gated unit to the gate | up rows
-        dn.A = M.proj; dn.a_f32 = true; dn.lda = 2 * ff; dn.a_glu = lc.mlp_act + 1; dn.a_limit = lc.limit;
-        kl--;
-      } else RET_CUDA(launch_stack_glu(M.proj, 1, 0, nullptr, M.act, f32, nullptr, rows, ff, lc.limit, lc.mlp_act, stream));
-      RET_CUDA(launch_stack_gemm(dn, stream));
-      RET_CUDA(join_shared());
-      RET_CUDA(launch_stack_moe_combine(M.rows_out, M.where, M.r_wt, shared ? sh_src : nullptr, sh_parts, sh_stride, sh_gate, M.y, T, W, top, stream));
-      kl += 6;
+      RET_CUDA(moe_ff(L, stream, M.proj, M.act, nullptr));
     }
     pend_y = M.y; pend_post = norm_w(L, 3); pend_post_b = norm_b(L, 3); pend_hc = reinterpret_cast<const float *>(L.hc[1].ptr);
   }
   next_hc = nullptr;
   // the last sublayer's output joins the residual; rows that need logits get the final norm and the head
-  if (single || ln) RET_CUDA(sublayer_in(nullptr, nullptr, nullptr, nullptr));
+  if (two_norms) { RET_CUDA(launch_stack_boundary_par(M.x, pend_par, res_mult, nullptr, nullptr, nullptr, nullptr, f32, T, W, eps, stream)); kl++; }
+  else if (single || ln) RET_CUDA(sublayer_in(nullptr, nullptr, nullptr, nullptr));
   else { RET_CUDA(launch_stack_resid_norm(M.x, pend_y, pend_post, nullptr, nullptr, T, W, eps, stream)); kl++; }
   if (R <= 0) return cudaSuccess;
   if (ln) RET_CUDA(launch_stack_final_ln(M.x, mt.d<int>(mt.o_rowmap), reinterpret_cast<const float *>(M.final_w.ptr),

@@ -1,6 +1,6 @@
 // stack.h -- layer-list decoders: a model given as a list of layers, each with one token mixer (linear attention with a
 // fixed decay, a minimal gated recurrence, latent attention over a compressed KV cache, grouped-query attention, gated linear
-// attention beside it, a state-space mixer, or retention) and an optional feed-forward (dense or mixture of experts), behind or
+// attention beside it, a state-space mixer, retention, or a gated delta rule) and an optional feed-forward (dense or mixture of experts), behind or
 // beside the mixer.  The engine's sequences, page allocator, step planner, sampler and C ABI
 // are shared with the Llama path; this header holds what differs: the per-layer weights, the per-slot recurrent state,
 // the latent page pools and the launchers of k_stack.cu.
@@ -135,9 +135,40 @@ cudaError_t launch_stack_ssd(const float *buf, long long ld_b, int c_off, int b_
 //    the compute type.  x: buf column 0 on (row stride ld_b), z: proj column 0 on (row stride ld).
 cudaError_t launch_stack_ssm_out(const float *o, const float *buf, long long ld_b, const float *z, long long ld, const float *D,
                                  const float *w, int parts, void *out, bool f32, int T, int H, int P, float eps, cudaStream_t st);
-// out[t][off + h*dv + j] = scale * unit_rms_over_head(o[t][h])[j] * w[j] * silu(gate[t][h*dv + j]); out [T][ldo] compute type; w null: ones
+// the tail [slots][taps-1][C] of a convolution over columns x_off .. x_off + C of proj (n_part slices) moves on to the spans' last inputs
+cudaError_t launch_stack_conv_tail(const float *proj, long long ld, int n_part, long long stride, int x_off, float *cstate, const StackSpans &sp,
+                                   int C, int taps, cudaStream_t st);
+// Gated delta rule (DIS_MIX_CHANNEL_DELTA, k_stack_delta.cu).
+struct StackDelta {
+  int H, G, d, dv, taps, ra, rg;  // value heads, query/key heads, sizes, convolution taps, bottlenecks of decay and gate
+  int C;                          // convolved channels q | k | v = 2 G d + H dv: the first columns of the projection
+  int a_off, g_off, b_off;        // columns of the bottlenecks and of the step sizes' logits
+  float eps;
+};
+struct StackDeltaPrep {
+  const float *proj = nullptr;    // [T][ld], or n_part slices, `stride` apart
+  long long ld = 0, stride = 0;
+  int n_part = 1;
+  const float *cw = nullptr;      // [C][taps]
+  const float *vec = nullptr;     // A_log [H] | dt_bias [H*d]
+  float *cstate = nullptr;        // [slots][taps-1][C]
+  const void *a2 = nullptr, *g2 = nullptr;  // [H*d][ra], [H*dv][rg], compute type
+  const float *z = nullptr;       // [T][H*d]: the products with a2, when they (and the gate's) were made by matrix products; null: made here
+  float *buf = nullptr;           // [T][ld_b]: q | k | v as they enter the recurrence, k.q [G], beta [H]
+  long long ld_b = 0;
+  float *dec = nullptr;           // [T][H*d]
+  float *gz = nullptr;            // [T][H*dv]: the gate's logits (written here when z is null)
+};
+// q, k, v, step sizes and decays of the pass's tokens; the convolution's tail moves on
+cudaError_t launch_stack_delta_prep(const StackDelta &c, const StackDeltaPrep &a, bool w_f32, const StackSpans &sp, cudaStream_t st);
+cudaError_t launch_stack_delta_pack(const StackDelta &c, const StackDeltaPrep &a, bool f32, int T, void *ua, void *ug, cudaStream_t st);
+// the recurrence over state [slots][H][dv][d], head norm and gate behind it: act [T][ld_act] (compute type).  o [T][H*dv]: room.  d <= 256
+cudaError_t launch_stack_delta(const StackDelta &c, const float *buf, long long ld_b, const float *dec, float *state, const StackSpans &sp, float *o,
+                               int max_len, const float *norm, const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches, cudaStream_t st);
+// out[t][off + h*dv + j] = scale * unit_rms_over_head(o[t][h])[j] * w[j] * silu(gate[t][h*dv + j]); out [T][ldo] compute type; w null: ones.
+// sig: times sigmoid(gate) instead
 cudaError_t launch_stack_headnorm_silu(const float *o, const float *w, const float *gate, long long ldg, void *out, long long ldo,
-                                       int off, float scale, bool f32, int T, int H, int dv, float eps, cudaStream_t st);
+                                       int off, float scale, bool f32, int T, int H, int dv, float eps, cudaStream_t st, bool sig = false);
 // Attention over paged keys and values (k_stack_attn.cu).
 struct StackAttn {
   int H, G, d, dv, rot_dims;
@@ -147,6 +178,9 @@ struct StackAttn {
   int window = 0;  // > 0: position i sees only the keys j with i - j < window
   float softcap = 0.f;  // > 0: score <- softcap * tanh(score / softcap), after the factor `scale` (softmax weights only)
   int keep = 0;    // keys below it stay visible to every later position
+  int maps = 1;    // 2 (DIS_ATTN_DIFF): every query and key head has two maps of d coordinates, [map 1, map 2]; the softmax outputs a1, a2
+                   // over the same values are joined as u(a1 - diff_lambda a2) diff_out, u the division by the root mean square
+  float diff_lambda = 0.f, diff_out = 1.f;
 };
 // DIS_ATTN_DISTANCE: 2^(-8 (h + 1) / H)
 __host__ __device__ inline float stack_attn_slope(int h, int H) { return exp2f(-8.f * (float)(h + 1) / (float)H); }
@@ -274,6 +308,8 @@ cudaError_t launch_stack_latent_softmax(const float *S, int rows, int ld, const 
 cudaError_t launch_stack_glu(const float *gu, int n_part, long long stride, const float *bias, void *act, bool f32, const int *rows_ptr,
                              int M, int ff, float limit, int kind, cudaStream_t st, long long ld_gu = 0, long long ld_act = 0);
 // Router: logits in fp32 from hc and the fp32 router matrix; `top` experts by value (lowest index wins a tie).
+// kind DIS_ROUTE_SOFTMAX_GROUPS: c = softmax(logits)[e] + correction[e], a run ranks by its largest c, weights = the chosen softmax scores over
+// their sum (+ 1e-20).
 // kind DIS_ROUTE_SOFTMAX_TOP: by logit, weights = softmax over the chosen.  DIS_ROUTE_SIGMOID_GROUPS: by c = sigmoid(logit) +
 // correction[e], restricted to the `keep` best of `groups` contiguous runs of experts (a run ranks by the sum of its top two c;
 // groups <= 1: no restriction), weights = the chosen sigmoids over their sum (+ 1e-20).
@@ -290,6 +326,28 @@ cudaError_t launch_stack_moe_gather(const void *hc, const int *perm_tok, void *x
 // n_part split-K slices of stride `stride`, summed here)
 cudaError_t launch_stack_moe_combine(const float *rows, const int *where, const float *wt, const float *shared, int n_part,
                                      long long stride, const float *shared_gate, float *y, int T, int W, int top, cudaStream_t st);
+// Boundary of parallel layers with two norms, one kernel per layer: the mixer's product (n1 slices) and the feed-forward's result join the
+// residual, x += mult (ls1 * mixer + ls2 * ff) [+ add]; then both coming sublayers' inputs, x / rms(x) * w1 -> h1 and * w2 -> h2 (compute
+// type).  The feed-forward is sum_k wt[t][k] rows[where[t][k]] (top experts; rows null: none) plus the n2 slices of y2 (a shared
+// expert, times sigmoid(y2_gate[t]) when given, or a dense unit; null: none).  y1 null: nothing joins (but add).
+struct StackParBoundary {
+  const float *y1 = nullptr;
+  int n1 = 1;
+  long long s1 = 0;
+  const float *b1 = nullptr;       // bias of the mixer's product
+  const float *ls1 = nullptr, *ls2 = nullptr;
+  const float *rows = nullptr;
+  const int *where = nullptr;
+  const float *wt = nullptr;
+  int top = 0;
+  const float *y2 = nullptr;
+  int n2 = 1;
+  long long s2 = 0;
+  const float *b2 = nullptr, *y2_gate = nullptr;
+  const float *add = nullptr;      // [T][W]
+};
+cudaError_t launch_stack_boundary_par(float *x, const StackParBoundary &b, float mult, const float *w1, void *h1, const float *w2, void *h2, bool f32,
+                                      int T, int W, float eps, cudaStream_t st);
 cudaError_t launch_stack_final_norm(const float *x, const int *row_map, const float *g, void *out, bool f32, int R, int W, float eps,
                                     cudaStream_t st);
 // out[m][n] = bias[n] + sum_s part[s][m][n]: the split-K slices of a tensor-core product, with the projection's bias
@@ -351,6 +409,12 @@ struct StackLayer {
   // state-space mixer: w_in rows z | x | B | C | dt; norm_w = gain of the group norm [H*vdim]
   StackTensor conv_w, conv_b, ssm_vec;     // [C][taps], [C], dt_bias | A_log | D [3H], all fp32
   int x_off = 0, dt_off = 0, conv_ch = 0;
+  StackTensor ls[2];                       // layer scales of the mixer's and the feed-forward's result [W]
+  StackTensor diff_vec;                    // differential attention: lq1 | lk1 | lq2 | lk2 [4 dim] fp32
+  float diff_lambda = 0.f;                 // and the second map's factor made from them when loading ends
+  // gated delta rule: w_in rows q | k | v | a1 | g1 | b; conv_w [C][taps]; ssm_vec = A_log | dt_bias; norm_w [vdim]; a2; g2 [H*vdim][gate_rank]
+  StackTensor g2;
+  int a_off = 0, b_off = 0;
 };
 
 // One execution of a layer inside a forward pass.  Without a loop every layer runs once; a looped stretch contributes one
@@ -394,6 +458,14 @@ struct StackModel {
   // activations
   float *x = nullptr, *y = nullptr, *hn = nullptr, *proj = nullptr, *mix = nullptr, *mix2 = nullptr, *qf = nullptr, *logits = nullptr;
   void *hc = nullptr, *act = nullptr, *xr = nullptr;
+  // parallel layers with two norms: the feed-forward's input, and its lane beside the mixer's (stream, experts' buffers)
+  void *hc2 = nullptr, *moe_act = nullptr;
+  float *moe_proj = nullptr;
+  cudaStream_t ff_stream = nullptr;
+  cudaEvent_t ev_ff_fork = nullptr, ev_ff_join = nullptr;
+  // gated delta rule: bottleneck rows in the compute type, products with a2, logits of the output gate
+  void *bn_a = nullptr, *bn_g = nullptr;
+  float *dz = nullptr, *gz = nullptr;
   // latent attention of long portions as matrix products: bf16 queries, gathered latents and their transpose, score block, weights
   bool lat_gemm = false;  // long portions leave the blocks of the paged latent kernel
   // latents gathered for the per-head keys and values of prompt portions, and those: lat_rows rows

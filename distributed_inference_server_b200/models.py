@@ -37,6 +37,12 @@ engine's description of the model and names every tensor.  Two families exist:
             softmax, no gate) and `attention` (grouped-query softmax attention without rotation: tanh soft cap and a per-head
             distance term on the scores, a sliding window beside which the first positions stay visible, values blended with
             those of the first such layer, an element-wise sigmoid output gate).
+  Bunosun   a layer-list decoder of the same engine whose layers are parallel under two norms (vectors stored around zero), with a
+            scale vector on each sublayer's result; a stretch of layers runs several times, the embedding joining the residual in
+            front of every pass but the first; mixers `attention` (differential: two softmax maps per head over the same values,
+            subtracted and normed; partial neighbouring-pair rotation with linearly scaled frequencies, a sliding window) and
+            `channel_delta` (gated delta rule with a decay per key channel, behind short convolutions); the feed-forward is a
+            mixture of SiLU-gated experts chosen by softmax scores plus a correction inside the best groups, and a plain shared one.
 
 The reference has no model loading at all (crates/inference/src/worker.rs:1 is empty).
 """
@@ -54,9 +60,11 @@ import numpy as np
 from . import binding as B
 
 _MIXERS = {"lightning": B.MIX_LIGHTNING, "mingru": B.MIX_MINGRU, "latent_attention": B.MIX_LATENT,
-           "attention": B.MIX_ATTENTION, "parallel": B.MIX_PARALLEL, "ssm": B.MIX_SSM, "retention": B.MIX_RETENTION}
+           "attention": B.MIX_ATTENTION, "parallel": B.MIX_PARALLEL, "ssm": B.MIX_SSM, "retention": B.MIX_RETENTION,
+           "channel_delta": B.MIX_CHANNEL_DELTA}
 _ACTS = {"clamped": B.ACT_CLAMPED, "gelu_tanh": B.ACT_GELU_TANH, "silu": B.ACT_SILU, "relu2": B.ACT_RELU2}
-_ROUTES = {"softmax_top": B.ROUTE_SOFTMAX_TOP, "sigmoid_groups": B.ROUTE_SIGMOID_GROUPS, "softmax_all": B.ROUTE_SOFTMAX_ALL}
+_ROUTES = {"softmax_top": B.ROUTE_SOFTMAX_TOP, "sigmoid_groups": B.ROUTE_SIGMOID_GROUPS, "softmax_all": B.ROUTE_SOFTMAX_ALL,
+           "softmax_groups": B.ROUTE_SOFTMAX_GROUPS}
 
 
 @dataclass
@@ -108,6 +116,9 @@ class LayerSpec:
     mask_keep: int = 0  # attention: first positions that stay visible beside the window
     q_rank: int = 0  # latent attention: size of the query latent (0 = queries straight from the input)
     latent_flags: int = 0
+    attn_diff: float = 0.0  # differential attention: the constant of the second map's factor
+    decay_rank: int = 0  # channel_delta: bottlenecks of the decay and of the output gate
+    gate_rank: int = 0
 
     @property
     def gated(self) -> bool:
@@ -136,6 +147,10 @@ class StackSpec:
     tied_head: bool = False  # logits from the embedding table: the file has no "head"
     parallel: bool = False  # mixer and feed-forward read one norm and are added together; needs pre_norm
     residual_mult: float = 1.0  # factor on what a layer adds to the residual; needs pre_norm
+    two_norms: bool = False  # parallel layers: the feed-forward reads a norm of its own
+    layer_scale: bool = False  # parallel layers with two norms: a vector on each sublayer's result
+    loop_embed: bool = False  # the embedding row joins the residual in front of every loop pass but the first
+    unused: Tuple[str, ...] = ()  # names a model file may carry although nothing reads them
 
     def layer_runs(self) -> List[int]:
         """Layer index of every layer run of one forward pass, the looped stretch repeated."""
@@ -178,6 +193,13 @@ class StackSpec:
             elif L.mixer == "mingru":
                 out.update({p + "mix.z": (L.width, W), p + "mix.z.b": (L.width,), p + "mix.x": (L.width, W), p + "mix.x.b": (L.width,),
                             p + "mix.g": (L.width, W), p + "mix.o": (W, L.width)})
+            elif L.mixer == "channel_delta":
+                nq, nv = L.kv_heads * L.dim, L.heads * L.vdim
+                m = p + "mix."
+                out.update({m + "q": (nq, W), m + "q.conv": (nq, L.conv_taps), m + "k": (nq, W), m + "k.conv": (nq, L.conv_taps),
+                            m + "v": (nv, W), m + "v.conv": (nv, L.conv_taps), m + "b": (L.heads, W), m + "A_log": (L.heads,),
+                            m + "norm": (L.vdim,), m + "a1": (L.decay_rank, W), m + "a2": (L.heads * L.dim, L.decay_rank),
+                            m + "dt_bias": (L.heads * L.dim,), m + "g1": (L.gate_rank, W), m + "g2": (nv, L.gate_rank), m + "o": (W, nv)})
             elif L.mixer == "ssm":
                 inner, gn = L.heads * L.vdim, L.ssm_groups * L.ssm_state
                 out.update({p + "mix.in": (2 * inner + 2 * gn + L.heads, W), p + "mix.conv": (inner + 2 * gn, L.conv_taps),
@@ -186,9 +208,12 @@ class StackSpec:
             elif L.mixer in ("attention", "parallel"):
                 a = p + ("mix.left." if L.mixer == "parallel" else "mix.")
                 own = L.kv_from < 0  # a layer that reads another layer's cache has nothing of the keys and values
-                out.update({a + "q": (L.heads * L.dim, W), a + "o": (W, L.heads * L.vdim)})
+                maps = 2 if L.attn_flags & B.ATTN_DIFF else 1
+                out.update({a + "q": (L.heads * maps * L.dim, W), a + "o": (W, L.heads * L.vdim)})
                 if own:
-                    out[a + "k"] = (L.kv_heads * L.dim, W)
+                    out[a + "k"] = (L.kv_heads * maps * L.dim, W)
+                if maps == 2:
+                    out.update({a + n: (L.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
                 if own and not L.attn_flags & B.ATTN_V_IS_K:
                     out[a + "v"] = (L.kv_heads * L.vdim, W)
                 if L.attn_flags & B.ATTN_BIAS:
@@ -232,9 +257,11 @@ class StackSpec:
                     out[p + "mix.sink"] = (L.heads,)
                 if not L.latent_flags & B.LATENT_NO_GATE:
                     out[p + "mix.g"] = (L.heads * L.vdim, W)
+            if self.layer_scale:
+                out.update({p + "ls1": (W,)} if L.mlp == "none" else {p + "ls1": (W,), p + "ls2": (W,)})
             if L.mlp == "none":
                 continue
-            if not self.parallel:
+            if not self.parallel or self.two_norms:
                 norm(p + "norm2")
             if post:
                 norm(p + "norm2b")
@@ -260,7 +287,7 @@ class StackSpec:
                 out[p + "mlp.router"] = (L.experts, W)
                 for e in range(L.experts):
                     out.update({f"{p}mlp.e{e}.gate": (L.ff, W), f"{p}mlp.e{e}.up": (L.ff, W), f"{p}mlp.e{e}.down": (W, L.ff)})
-                if L.route == "sigmoid_groups":
+                if L.route in ("sigmoid_groups", "softmax_groups"):
                     out[p + "mlp.correction"] = (L.experts,)
                 if L.shared_ff > 0:
                     out.update({p + "mlp.shared.gate": (L.shared_ff, W), p + "mlp.shared.up": (L.shared_ff, W),
@@ -297,13 +324,15 @@ class StackSpec:
             c.ssm_state, c.ssm_groups, c.conv_taps, c.ssm_norm_groups = L.ssm_state, L.ssm_groups, L.conv_taps, L.ssm_norm_groups
             c.mlp_flags = B.MLP_SHARED_PLAIN if L.shared_plain else 0
             c.mask_keep, c.q_rank, c.latent_flags = L.mask_keep, L.q_rank, L.latent_flags
+            c.attn_diff, c.decay_rank, c.gate_rank = L.attn_diff, L.decay_rank, L.gate_rank
         sc = B.StackConfig(self.vocab, self.width, len(self.layers), self.canon_taps, max_ctx, max_logit_rows,
                            B.F32 if f32 else B.BF16, self.norm_eps, arr,
                            {"rms_scalar": B.NORM_RMS_SCALAR, "layer": B.NORM_LAYER, "rms": B.NORM_RMS, "rms_one": B.NORM_RMS_ONE}[self.norm_kind],
                            self.embed_scale, self.logit_scale, *self.loop, self.logit_softcap,
                            (B.FRAME_PRE_NORM if self.pre_norm else 0) | (B.FRAME_POS_SINUS if self.pos_sinus else 0) |
                            (B.FRAME_LOOP_PLAIN if self.loop_plain else 0) | (B.FRAME_TIED_HEAD if self.tied_head else 0) |
-                           (B.FRAME_PARALLEL if self.parallel else 0),
+                           (B.FRAME_PARALLEL if self.parallel else 0) | (B.FRAME_TWO_NORMS if self.two_norms else 0) |
+                           (B.FRAME_LAYER_SCALE if self.layer_scale else 0) | (B.FRAME_LOOP_EMBED if self.loop_embed else 0),
                            self.streams, self.pos_base, self.residual_mult)
         return sc, keep
 
@@ -540,6 +569,68 @@ def nifulix_spec(cfg: dict) -> StackSpec:
                      pre_norm=True, parallel=True, residual_mult=float(cfg.get("residual_mult", 1.0)))
 
 
+def bunosun_spec(cfg: dict, shapes: Optional[Dict[str, Tuple[int, ...]]] = None) -> StackSpec:
+    """Bunosun's config.json -> StackSpec: every size and constant from the file.  A part the file leaves out is off: no `mask` = the
+    whole past, no `rot` = no rotation, no `scaling` = plain frequencies, no `groups` = a choice among all experts, no `shared` = no
+    shared expert, `mlp` null = the mixer alone, no `loop` = every layer once.  The bottlenecks of the decay and of the output gate
+    are given by the shapes of the file's tensors, or by `decay_rank` / `gate_rank` beside the mixer's other sizes."""
+    layers, unused = [], []
+    for i, ly in enumerate(cfg["layers"]):
+        kind, mx = ly["type"], ly["mixer"]
+        if kind not in ("attention", "channel_delta"):
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        L = LayerSpec(kind)
+        L.heads, L.kv_heads, L.dim, L.vdim = int(mx["heads"]), int(mx["kv_heads"]), int(mx["dim"]), int(mx["vdim"])
+        if L.kv_heads < 1 or L.heads % L.kv_heads:
+            raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
+        if kind == "attention":
+            rot = mx.get("rot") or {}
+            L.rot_dims, L.rot_base = int(rot.get("dims", 0)), float(rot.get("base", 10000.0))
+            if L.rot_dims > L.dim or L.rot_dims % 2:
+                raise ValueError(f"layer {i}: rot.dims must be even and at most dim")
+            L.attn_flags = B.ATTN_DIFF | B.ATTN_ROT_PAIRS
+            sc = rot.get("scaling")
+            if sc:
+                L.rot_factor = float(sc["factor"])
+                L.attn_flags |= B.ATTN_ROT_LINEAR
+            L.scale, L.attn_diff = float(mx["scale"]), float(mx["diff"])
+            L.mask_window = int((mx.get("mask") or {}).get("size") or 0)
+        else:
+            L.conv_taps = int(mx["conv"])
+            for f, t in (("decay_rank", "a1"), ("gate_rank", "g1")):
+                shape = (shapes or {}).get(f"l{i}.mix.{t}")
+                if shape is None and f not in mx:
+                    raise ValueError(f"layer {i}: {f} is given by neither a tensor nor the configuration")
+                setattr(L, f, int(shape[0] if shape is not None else mx[f]))
+        ml = ly.get("mlp")
+        if ml is not None:
+            if ml.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {ml.get('kind')!r}")
+            r = ml["router"]
+            L.mlp, L.mlp_act, L.ff = "moe", "silu", int(ml["expert"]["ff"])
+            L.experts, L.top, L.route = int(r["experts"]), int(r["top"]), "softmax_groups"
+            gr = r.get("groups")
+            if gr:
+                L.route_groups, L.route_keep = int(gr["count"]), int(gr["keep"])
+                if L.route_groups < 1 or L.experts % L.route_groups or not 1 <= L.route_keep <= L.route_groups:
+                    raise ValueError(f"layer {i}: groups.count must divide experts and 1 <= groups.keep <= groups.count")
+                if L.route_keep * (L.experts // L.route_groups) < L.top:
+                    raise ValueError(f"layer {i}: the kept groups hold fewer experts than top")
+            sh = ml.get("shared")
+            if sh:
+                L.shared_ff, L.shared_plain = int(sh["ff"]), True
+        else:
+            unused += [f"l{i}.norm2", f"l{i}.ls2"]
+        layers.append(L)
+    lp = cfg.get("loop")
+    loop = (int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp and int(lp.get("times", 0)) > 0 else (0, 0, 0)
+    if loop[2] > 0 and not 0 <= loop[0] < loop[1] <= len(layers):
+        raise ValueError("loop: start < stop must lie inside the layer list")
+    return StackSpec("Bunosun", int(cfg["vocab"]), int(cfg["width"]), layers, 0, float((cfg.get("norm") or {}).get("eps", 1e-5)), "rms_one",
+                     embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)), loop=loop, pre_norm=True, loop_plain=True,
+                     parallel=True, two_norms=True, layer_scale=True, loop_embed=True, unused=tuple(unused))
+
+
 def llama_shape(cfg: dict):
     """A Hugging Face style Llama config.json -> ModelShape."""
     from .worker import ModelShape
@@ -557,6 +648,7 @@ ARCHITECTURES: Dict[str, Tuple[str, Callable[..., object]]] = {
     "Fakonex": ("stack", fakonex_spec),
     "Goperax": ("stack", goperax_spec),
     "Nifulix": ("stack", nifulix_spec),
+    "Bunosun": ("stack", bunosun_spec),
     "LlamaForCausalLM": ("llama", llama_shape),
     "llama": ("llama", llama_shape),
 }
@@ -573,7 +665,7 @@ def read_config(model_dir: str):
     """(family, description) of the model in `model_dir`."""
     cfg = json.load(open(os.path.join(model_dir, "config.json")))
     family, reader = ARCHITECTURES[architecture_of(cfg)]
-    if reader is motolix_spec:
+    if reader in (motolix_spec, bunosun_spec):  # sizes that only the tensors' shapes give
         st = os.path.join(model_dir, "model.safetensors")
         return family, reader(cfg, safetensors_shapes(st) if os.path.exists(st) else None)
     return family, reader(cfg)
@@ -636,6 +728,8 @@ def load_model(model_dir: str, dtype: str = "bfloat16", max_batch: int = 32, max
         want = desc.tensor_shapes()
         for name, arr, code, shape in read_safetensors(st):
             if name not in want:
+                if name in desc.unused:
+                    continue
                 raise ValueError(f"{st}: tensor {name!r} is not part of this configuration")
             if code is None:
                 raise ValueError(f"{st}: {name!r} is an integer table; this design has none")
@@ -680,10 +774,14 @@ def random_tensors(spec: StackSpec, seed: int = 0, scale: float = 1.0) -> Dict[s
         leaf = name.rsplit(".", 1)[-1]
         if shape == ():
             a = np.asarray(rng.uniform(0.2, 0.8) if leaf == "vmix" else rng.uniform(0.5, 1.5), np.float32)
-        elif spec.norm_kind == "rms_one" and (leaf == "norm1" or name == "final.norm"):
+        elif spec.norm_kind == "rms_one" and (leaf in ("norm1", "norm2") or name == "final.norm"):
             a = rng.normal(0.0, 0.2, shape).astype(np.float32)
         elif leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm" or name.endswith(("q.norm", "k.norm")):
             a = rng.uniform(0.5, 1.5, shape).astype(np.float32)
+        elif leaf in ("ls1", "ls2"):
+            a = rng.uniform(0.3, 1.0, shape).astype(np.float32)
+        elif leaf in ("lq1", "lk1", "lq2", "lk2"):
+            a = rng.normal(0, 0.1, shape).astype(np.float32)
         elif leaf == "temp":
             a = rng.uniform(0.5, 1.5, shape).astype(np.float32)
         elif leaf == "pb":
@@ -712,7 +810,7 @@ def random_tensors(spec: StackSpec, seed: int = 0, scale: float = 1.0) -> Dict[s
             a = rng.normal(1.0, 0.3, shape).astype(np.float32)
         elif leaf == "conv":
             a = rng.normal(0, 0.5, shape).astype(np.float32)
-        elif leaf == "b":
+        elif leaf == "b" and len(shape) == 1:
             a = rng.normal(0, 0.3, shape).astype(np.float32)
         elif name in ("embed",):
             a = rng.normal(0, 1.0, shape).astype(np.float32)

@@ -31,11 +31,12 @@ extern "C" {
 #endif
 
 #define DIS_API __attribute__((visibility("default")))
-#define DIS_ABI_VERSION 6 /* 2: 16-byte request ids, logprob on token events / callback, dis_serving_cancel; 3: dis_layer_config and dis_stack_config grew (attention and parallel mixers, layer norms, layer loops); 4: they grew again (chunked mask, sink, per-head query/key norm and output gate of attention, shared key/value cache, grouped sigmoid router, shared expert, RMS norms with gain vectors, logit soft cap); 5: and again (state-space mixer, sliding window, score soft cap and unit sink of
+#define DIS_ABI_VERSION 7 /* 2: 16-byte request ids, logprob on token events / callback, dis_serving_cancel; 3: dis_layer_config and dis_stack_config grew (attention and parallel mixers, layer norms, layer loops); 4: they grew again (chunked mask, sink, per-head query/key norm and output gate of attention, shared key/value cache, grouped sigmoid router, shared expert, RMS norms with gain vectors, logit soft cap); 5: and again (state-space mixer, sliding window, score soft cap and unit sink of
                              attention, ungated squared-ReLU units, softmax-over-all router, ungated shared expert, residual streams, pre-norm frame,
                              sinusoidal positions, loops without an input projection, head tied to the embedding); 6: and again (retention, query latent and window of latent
                              attention, kept first positions, distance term, value mixing and full output gate of attention, parallel layers, gains stored around
-                             zero, residual multiplier) */
+                             zero, residual multiplier); 7: and again (gated delta rule, differential attention, neighbouring-pair rotation and linear
+                             frequency scaling of attention, grouped softmax router, parallel layers with two norms and layer scales) */
 
 /* ---- status codes: WorkerError, crates/core/src/error.rs:115-128 ------------------------------ */
 typedef enum dis_status {
@@ -438,9 +439,17 @@ typedef enum dis_mixer_kind {
                             h reads B, C of group h / (heads / ssm_groups)) S = exp(-exp("A_log"[h]) dt) S + dt B x^T, y = S^T C + "D"[h] x;
                             y silu(z) is RMS-normed in ssm_norm_groups equal parts, times "norm", then projected by "o".  Sequence state:
                             S (fp32) and the convolution's last conv_taps - 1 inputs */
-  DIS_MIX_RETENTION = 6  /* linear attention, fixed decay per head, no activation: q and k are rotated (rot_dims, rot_base: coordinate i turns
+  DIS_MIX_RETENTION = 6, /* linear attention, fixed decay per head, no activation: q and k are rotated (rot_dims, rot_base: coordinate i turns
                             with i + rot_dims/2), k is then multiplied by dim^(-1/2); S = decay S + k v^T, o = S^T q; each head's o is
                             divided by its root mean square (no gain), multiplied by silu("g" u) and projected */
+  DIS_MIX_CHANNEL_DELTA = 7 /* gated delta rule with one decay per key channel.  q, k (kv_heads x dim) and v (heads x vdim) pass a causal
+                            depthwise convolution ("q.conv" .. [channels][conv_taps], last tap = current token, no bias) and SiLU; q and k
+                            are divided by their length, sqrt(sum of squares + 1e-6), per head, q also multiplied by dim^(-1/2); beta =
+                            sigmoid("b" u) per head; g = exp(-exp("A_log"[h]) softplus("a2" ("a1" u) + "dt_bias")) per head and key channel
+                            (bottleneck decay_rank).  Per head, reading q and k of head h / (heads / kv_heads): S = diag(g) S,
+                            w = beta (v - S^T k), S = S + k w^T, o = S^T q; each head's o is divided by its root mean square, times "norm"
+                            [vdim], times sigmoid("g2" ("g1" u)) (bottleneck gate_rank), then projected by "o".  Sequence state: S (fp32) and
+                            the convolution's last conv_taps - 1 inputs */
 } dis_mixer_kind;
 typedef enum dis_mlp_kind { DIS_MLP_NONE = 0, DIS_MLP_DENSE = 1, DIS_MLP_MOE = 2 } dis_mlp_kind;
 /* Feed-forward unit.  CLAMPED: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit), u' = clamp(u, +-limit), biases on every
@@ -460,7 +469,9 @@ typedef enum dis_norm_kind { DIS_NORM_RMS_SCALAR = 0, DIS_NORM_LAYER = 1, DIS_NO
 /* SOFTMAX_ALL: s = softmax(z) over all experts, the `top` largest s (ties: lowest index), weights s_e / (sum_{S} s + 1e-20).  The
  * common factor of the softmax cancels, so choice and weights are those of SOFTMAX_TOP; the kind exists so that a configuration can
  * say what its file says. */
-typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUPS = 1, DIS_ROUTE_SOFTMAX_ALL = 2 } dis_route_kind;
+/* SOFTMAX_GROUPS: s = softmax(z) over all experts and c = s + "correction"; groups as in SIGMOID_GROUPS, but a block ranks by its largest
+ * c alone; the `top` largest remaining c are chosen and weigh s_e / (sum_{S} s + 1e-20). */
+typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUPS = 1, DIS_ROUTE_SOFTMAX_ALL = 2, DIS_ROUTE_SOFTMAX_GROUPS = 3 } dis_route_kind;
 /* dis_layer_config.attn_flags */
 #define DIS_ATTN_SIGMOID   1u   /* weight of a visible key = sigmoid(score * temp[h] + pb[h]) (per-head tensors "temp", "pb"),
                                    not normalised over the keys; without the flag: softmax over the visible keys */
@@ -484,6 +495,12 @@ typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUP
 #define DIS_ATTN_V_MIX  4096u /* values v <- (1 - l) v + l v', v' the values of the same token in the first such layer of the pass and l the
                                    scalar tensor "vmix" (that first layer keeps its own values); the mixed values are cached.  All such
                                    layers have the same kv_heads * vdim */
+#define DIS_ATTN_DIFF   8192u /* differential attention: every query and key head has two maps of dim coordinates each (rows of "q" and "k": head by
+                                   head [map 1, map 2]), each an attention of its own over the head's values; with a1, a2 their outputs and
+                                   l = exp(sum "lq1" "lk1") - exp(sum "lq2" "lk2") + attn_diff (vectors of dim), o = a1 - l a2 is divided by its
+                                   root mean square over vdim and multiplied by 1 - attn_diff.  Plain softmax weights only */
+#define DIS_ATTN_ROT_PAIRS 16384u /* rotation turns coordinates 2i and 2i + 1 together instead of i and i + rot_dims/2 */
+#define DIS_ATTN_ROT_LINEAR 32768u /* every rotary frequency is divided by rot_factor (rot_low, rot_high, rot_original unused) */
 /* dis_layer_config.latent_flags */
 #define DIS_LATENT_NO_SINK   1u /* no "sink": a plain softmax over the visible keys */
 #define DIS_LATENT_NO_GATE   2u /* no output gate: no "g" */
@@ -498,6 +515,12 @@ typedef enum dis_route_kind { DIS_ROUTE_SOFTMAX_TOP = 0, DIS_ROUTE_SIGMOID_GROUP
 #define DIS_FRAME_TIED_HEAD  8u /* the logits are products with the embedding table itself (without embed_scale): no "head" tensor */
 #define DIS_FRAME_PARALLEL  16u /* (with DIS_FRAME_PRE_NORM, one residual) a layer is x += residual_mult (mixer(h) + ff(h)) with the one norm
                                    h = norm1(x): no "norm2".  Mixers attention, parallel, latent, retention; dense feed-forwards without biases */
+#define DIS_FRAME_TWO_NORMS 32u /* (with DIS_FRAME_PARALLEL) the feed-forward reads norm2(x) instead, and may be a mixture of experts:
+                                   x += residual_mult (mixer(norm1(x)) + ff(norm2(x))); the mixer may be DIS_MIX_CHANNEL_DELTA too */
+#define DIS_FRAME_LAYER_SCALE 64u /* (with DIS_FRAME_TWO_NORMS) the mixer's result is multiplied element by element by "ls1", the
+                                   feed-forward's by "ls2" (vectors of width) before the sum */
+#define DIS_FRAME_LOOP_EMBED 128u /* (with DIS_FRAME_LOOP_PLAIN and DIS_FRAME_TWO_NORMS) in front of every pass of the loop but the first the
+                                   scaled embedding row joins the residual once more */
 
 typedef struct dis_layer_config {
   int32_t mixer;                 /* dis_mixer_kind */
@@ -514,7 +537,7 @@ typedef struct dis_layer_config {
   int32_t experts, top;          /* mixture of experts: how many, how many per token */
   float limit;                   /* clamp of the gate (above) and up (both sides) branches */
   /* attention (DIS_MIX_ATTENTION, and the first half of DIS_MIX_PARALLEL): heads, dim, vdim, rot_dims, rot_base, scale above */
-  int32_t kv_heads;              /* key/value heads; query head h reads head h / (heads / kv_heads) */
+  int32_t kv_heads;              /* (also DIS_MIX_CHANNEL_DELTA: heads of q and k) key/value heads; query head h reads head h / (heads / kv_heads) */
   uint32_t attn_flags;           /* DIS_ATTN_* */
   float rot_factor, rot_low, rot_high; /* frequency scaling by wavelength l = 2 pi / f against rot_original: l < original/high
                                     keeps f, l > original/low uses f / factor, between them the blend (1 - s) f / factor + s f
@@ -537,13 +560,15 @@ typedef struct dis_layer_config {
   int32_t mask_window;           /* attention: w > 0: position i sees key j iff 0 <= i - j < w (on top of mask_chunk, if both are set); 0: none */
   float score_softcap;           /* attention: c > 0: score <- c tanh(score / c) after the factor `scale`; 0: none */
   int32_t ssm_state, ssm_groups; /* DIS_MIX_SSM (with heads, vdim above): state size per head; groups of heads that share B and C */
-  int32_t conv_taps;             /* DIS_MIX_SSM: taps of the convolution over x | B | C (1 .. 16) */
+  int32_t conv_taps;             /* DIS_MIX_SSM, DIS_MIX_CHANNEL_DELTA: taps of the convolution over x | B | C or q | k | v (1 .. 16) */
   int32_t ssm_norm_groups;       /* DIS_MIX_SSM: equal parts of heads * vdim that are normalised separately (0 is read as 1) */
   uint32_t mlp_flags;            /* DIS_MLP_* */
   int32_t mask_keep;             /* attention: positions j < mask_keep stay visible to every later position, whatever mask_chunk and
                                     mask_window say; 0: none.  (mask_window applies to latent attention too, mask_chunk and mask_keep do not) */
   int32_t q_rank;                /* latent: q > 0: queries go through a latent of this size, q = "uq" (rms_norm("dq" u) * "dq.norm"); 0: q = "q" u */
   uint32_t latent_flags;         /* DIS_LATENT_* */
+  float attn_diff;               /* DIS_ATTN_DIFF: the constant in the second map's factor and in the output's */
+  int32_t decay_rank, gate_rank; /* DIS_MIX_CHANNEL_DELTA: bottlenecks of the decay and of the output gate */
 } dis_layer_config;
 
 typedef struct dis_stack_config {
