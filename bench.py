@@ -1253,6 +1253,107 @@ def run_nifulix(args):
     return 0
 
 
+def run_bunosun(args):
+    """Prefill and decode throughput of Bunosun (parallel layers under two norms with layer scales; differential attention with a
+    window; a gated delta rule with a decay per key channel behind short convolutions; a mixture of SiLU-gated experts with a plain
+    shared one) next to the closest existing models at equal width, depth, vocabulary and head geometry: Fakonex (the same attention
+    kernels under a chunked mask of the window's length, the same mixture), Goperax's state-space layers (convolution and
+    recurrence, a mixture), Nifulix's retention layers (recurrence, parallel layers) and the Llama decoder; random weights, one
+    GPU: one pass over `batch` prompts of `prompt_len` tokens, then K decode steps of the batch, timed by the engine's CUDA events
+    around each pass (metadata upload and token read-back included).  Weights exceed L2 at every size."""
+    from distributed_inference_server_b200 import Engine, InferenceParams, ModelShape, WorkerConfig, models
+    from distributed_inference_server_b200.binding import FLAG_NO_GRAPH as B_FLAG_NO_GRAPH
+    sizes = {"w1024": 1024, "w2048": 2048}
+    want = [k for k in (args.sizes.split(",") if args.sizes else sizes) if k in sizes]
+    batch, plen, vocab = args.batch or 8, args.prompt_len, 32000
+    rng = np.random.default_rng(0)
+    out = []
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.mark_start()
+    for key in want:
+        W = sizes[key]
+        H = W // 128
+        G = max(1, H // 4)
+        window = max(64, plen // 2)
+        att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.5, "mask": {"size": window},
+                                              "rot": {"base": 500000.0, "dims": 32, "scaling": {"factor": 4.0}}}}
+        dlt = {"type": "channel_delta", "mixer": {"heads": H, "kv_heads": max(1, H // 2), "dim": 128, "vdim": 128, "conv": 4, "decay_rank": 128, "gate_rank": 128}}
+        moe = {"kind": "moe", "expert": {"ff": W}, "router": {"experts": 8, "top": 2, "groups": {"count": 4, "keep": 2}}, "shared": {"ff": W}}
+        kinds = {"attention": att, "delta": dlt}
+        variants = {"mixed": ["delta", "attention", "delta", "attention"]}
+        if args.per_mixer:
+            variants.update({k: [k] * 4 for k in kinds})
+            variants["delta_alone"] = ["delta"] * 4  # (no feed-forward)
+        if args.variant:
+            variants = {k: v for k, v in variants.items() if k in args.variant.split(",")}
+        rec = {"size": key, "width": W, "layers": 4, "expert_ff": W, "experts": 8, "top": 2, "vocab": vocab, "batch": batch, "prompt_len": plen, "window": window}
+        prompts = [rng.integers(0, vocab, plen).tolist() for _ in range(batch)]
+        P = InferenceParams(max_tokens=1 << 20, temperature=0.0)
+        ctx = plen + args.steps + args.warmup + 64
+
+        def measure(eng):
+            slots = [eng.seq_add(p, P) for p in prompts]
+            t_pre = []
+            for it in range(1 + max(1, args.ttft_runs)):
+                if it:
+                    for sl in slots:
+                        eng.seq_remove(sl)
+                    slots = [eng.seq_add(p, P) for p in prompts]
+                eng.step(slots, batch * plen)
+                t_pre.append(eng.status().last_step_ms)
+            for _ in range(args.warmup):
+                eng.decode(slots)
+            k0 = eng.status().kernel_launches
+            ms = 0.0
+            for _ in range(args.steps):
+                eng.decode(slots)
+                ms += eng.status().last_step_ms
+            launches = eng.status().kernel_launches - k0
+            eng.close()
+            pre = min(t_pre[1:])
+            return {"prefill_ms": round(pre, 3), "prefill_tokens_per_s": round(batch * plen / pre * 1e3, 1),
+                    "decode_ms_per_step": round(ms / args.steps, 4), "decode_tokens_per_s": round(batch * args.steps / ms * 1e3, 1),
+                    "launches_per_decode_step": launches // max(1, args.steps)}
+
+        def stack_engine(spec):
+            eng = Engine(WorkerConfig(None, max_batch=batch, max_step_tokens=batch * plen, page_size=64, kv_pages=(batch * ctx + 63) // 64,
+                                      stack=spec, context_size=ctx, compute_dtype="bfloat16", flags=B_FLAG_NO_GRAPH if args.no_graph else 0))
+            for name, a in models.random_tensors(spec, seed=1).items():
+                eng.load_named(name, a)
+            eng.finalize()
+            return eng
+
+        def cfg_of(arch, layers, **extra):
+            return dict({"architecture": arch, "vocab": vocab, "width": W, "norm": {"eps": 1e-5},
+                         "layers": [dict(json.loads(json.dumps(m)), mlp=json.loads(json.dumps(f))) for m, f in layers]}, **extra)
+        for vname, names in variants.items():
+            cfg = cfg_of("Bunosun", [(kinds[n], None if vname == "delta_alone" else moe) for n in names], embedding={"scale": 1.0})
+            rec["bunosun_" + vname] = measure(stack_engine(models.bunosun_spec(cfg)))
+        if not args.bunosun_only:
+            f_att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": window}}}
+            rec["fakonex_attention_moe"] = measure(stack_engine(models.fakonex_spec(cfg_of("Fakonex", [(f_att, moe)] * 4))))
+            ssm = {"type": "mamba2", "mixer": {"heads": 2 * W // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}}
+            g_moe = {"kind": "moe", "expert": {"ff": W}, "router": {"experts": 8, "top": 2}, "shared": {"ff": W}}
+            rec["goperax_ssm_moe"] = measure(stack_engine(models.goperax_spec(cfg_of("Goperax", [(ssm, g_moe)] * 4, embedding={"scale": float(W) ** 0.5}))))
+            ret = {"type": "retention", "mixer": {"heads": H, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128},
+                                                  "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * h / max(1, H - 1)) for h in range(H)]}}
+            for nm, ff in (("nifulix_retention", {"kind": "dense", "ff": 4 * W}), ("nifulix_retention_alone", None)):
+                rec[nm] = measure(stack_engine(models.nifulix_spec(cfg_of("Nifulix", [(ret, ff)] * 4, residual_mult=0.5))))
+            eng = Engine(WorkerConfig(ModelShape(vocab, W, 4, H, G, 128, 4 * W, ctx), max_batch=batch, max_step_tokens=batch * plen, page_size=64,
+                                      kv_pages=(batch * ctx + 63) // 64 + batch))
+            eng.load_synthetic(1)
+            eng.finalize()
+            rec["llama"] = measure(eng)
+        out.append(rec)
+    clocks.mark_end()
+    line = {"metric": "bunosun_vs_closest_models_equal_size", "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "dtype": "bf16", "data": "synthetic (random weights, uniform random tokens)", "higher_is_better": True, "sizes": out,
+            "clocks": clocks.stop()}
+    print(json.dumps(line))
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1271,12 +1372,13 @@ def main():
     ap.add_argument("--nccl-allreduce", action="store_true", help="TP: use NCCL instead of the fused peer-memory exchange (A/B)")
     ap.add_argument("--tp-exchange", choices=["auto", "oneshot", "twoshot", "ll", "wide"], default="auto",
                     help="TP: peer-memory exchange kernel (auto = ll, the flag-in-data row kernel, up to hidden 4096; wide, the same protocol on a (row, column block) grid, above)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "prefix", "kidolorn", "motolix", "fakonex", "goperax", "nifulix"], help="serving = BASELINE configs[4]; prefix = TTFT with prefix KV reuse (row f2); kidolorn / motolix / fakonex / goperax / nifulix = that layer-list design beside Llama (and its closest layer-list relatives) at equal size")
-    ap.add_argument("--sizes", default="", help="kidolorn, motolix, fakonex, goperax, nifulix: comma list out of w1024,w2048 (default both)")
-    ap.add_argument("--per-mixer", action="store_true", help="kidolorn, motolix, fakonex, goperax, nifulix: also four layers of each mixer (fakonex: of each cache / mask arrangement) alone")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "prefix", "kidolorn", "motolix", "fakonex", "goperax", "nifulix", "bunosun"], help="serving = BASELINE configs[4]; prefix = TTFT with prefix KV reuse (row f2); kidolorn / motolix / fakonex / goperax / nifulix / bunosun = that layer-list design beside Llama (and its closest layer-list relatives) at equal size")
+    ap.add_argument("--sizes", default="", help="kidolorn, motolix, fakonex, goperax, nifulix, bunosun: comma list out of w1024,w2048 (default both)")
+    ap.add_argument("--per-mixer", action="store_true", help="kidolorn, motolix, fakonex, goperax, nifulix, bunosun: also four layers of each mixer (fakonex: of each cache / mask arrangement) alone")
     ap.add_argument("--goperax-only", action="store_true", help="goperax: skip the other models' rows (profiling under ncu)")
     ap.add_argument("--nifulix-only", action="store_true", help="nifulix: skip the other models' rows (profiling under ncu)")
-    ap.add_argument("--variant", default="", help="nifulix: comma list out of mixed,attention,retention,latent (default all that are asked for)")
+    ap.add_argument("--bunosun-only", action="store_true", help="bunosun: skip the other models' rows (profiling under ncu)")
+    ap.add_argument("--variant", default="", help="nifulix: comma list out of mixed,attention,retention,latent; bunosun: out of mixed,attention,delta,delta_alone (default all that are asked for)")
     ap.add_argument("--model", default="8b", choices=["8b", "70b"], help="70b = BASELINE configs[3] (TP=8, batch 32)")
     ap.add_argument("--requests", type=int, default=256)
     ap.add_argument("--prefill-budget", type=int, default=0, help="serving: prompt tokens read per scheduler step (0 = library default)")
@@ -1304,6 +1406,8 @@ def main():
         return run_goperax(args)
     if args.workload == "nifulix":
         return run_nifulix(args)
+    if args.workload == "bunosun":
+        return run_bunosun(args)
     return run_ours(args)
 
 

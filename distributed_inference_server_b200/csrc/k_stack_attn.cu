@@ -383,6 +383,16 @@ __global__ void __launch_bounds__(128) stack_attn_merge_maps_kernel(const float 
   const int p = blockIdx.x, tok = p / H, h = p - tok * H;
   const long long stride = (long long)T * H * 2 * (dv + 2);
   const float *rec = part + (long long)p * 2 * (dv + 2);
+  // the sums of the first slices are requested beside the maxima and denominators
+  constexpr int U = 8;
+  const int j0 = threadIdx.x;
+  float r1[U], r2[U];
+#pragma unroll
+  for (int s = 0; s < U; s++) {
+    const bool on = s < n_split && j0 < dv;
+    r1[s] = on ? rec[s * stride + j0] : 0.f;
+    r2[s] = on ? rec[s * stride + dv + 2 + j0] : 0.f;
+  }
   if (threadIdx.x < 64) {  // factor of a slice: its weight over the map's denominator, the second map's times -lambda
     const int m = threadIdx.x >> 5, l = threadIdx.x & 31;
     const float *rm = rec + m * (dv + 2);
@@ -407,10 +417,15 @@ __global__ void __launch_bounds__(128) stack_attn_merge_maps_kernel(const float 
   }
   __syncthreads();
   float ss = 0.f;
-  for (int j = threadIdx.x; j < dv; j += blockDim.x) {
+  for (int j = j0; j < dv; j += blockDim.x) {
     float v1 = 0.f, v2 = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < n_split; s++) {
+    if (j == j0) {
+#pragma unroll
+      for (int s = 0; s < U; s++)
+        if (s < n_split) { v1 = fmaf(r1[s], ws[s], v1); v2 = fmaf(r2[s], ws[n_split + s], v2); }
+    }
+#pragma unroll 8
+    for (int s = j == j0 ? U : 0; s < n_split; s++) {
       v1 = fmaf(rec[s * stride + j], ws[s], v1);
       v2 = fmaf(rec[s * stride + dv + 2 + j], ws[n_split + s], v2);
     }
@@ -418,7 +433,7 @@ __global__ void __launch_bounds__(128) stack_attn_merge_maps_kernel(const float 
     ss = fmaf(a[j], a[j], ss);
   }
   const float k = rsqrtf(block_sum(ss, sh) / (float)dv + eps) * diff_out * o.scale;
-  for (int j = threadIdx.x; j < dv; j += blockDim.x) st_el<F32>(o.out, (long long)tok * o.ld + o.off + (long long)h * dv + j, a[j] * k);
+  for (int j = j0; j < dv; j += blockDim.x) st_el<F32>(o.out, (long long)tok * o.ld + o.off + (long long)h * dv + j, a[j] * k);
 }
 
 // ------------------------------------------------------------------------------------------------ attention on mma.sync

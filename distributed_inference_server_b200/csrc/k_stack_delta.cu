@@ -8,8 +8,7 @@ namespace dis {
 
 // ------------------------------------------------------------------------------------------------ preparation
 // One launch; blockIdx.x is a tile of tokens, blockIdx.y a role:
-//   [0, G)            queries and keys of one key head: convolution, SiLU, division by the length (queries also times d^(-1/2)),
-//                     and their inner product
+//   [0, G)            queries and keys of one key head: convolution, SiLU, division by the length (queries also times d^(-1/2))
 //   then nvb blocks   128 value channels each: convolution and SiLU (the first also forms the step sizes sigmoid(.))
 //   then ndb blocks   128 decays each: exp(-exp(A_log) softplus(z + dt_bias)), z from memory or as the product with the bottleneck
 //   then ngb blocks   128 logits of the output gate each, as products with their bottleneck (absent when z comes from memory)
@@ -128,13 +127,12 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
     const float qscale = rsqrtf((float)d);
     for (int t = t0 + w; t < t1; t += kDeltaTh / 32) {
       const float *q = qs + (t - t0) * d, *k = ks + (t - t0) * d;
-      float qq = 0.f, kk = 0.f, qk = 0.f;
-      for (int i = l; i < d; i += 32) { qq = fmaf(q[i], q[i], qq); kk = fmaf(k[i], k[i], kk); qk = fmaf(q[i], k[i], qk); }
-      qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+      float qq = 0.f, kk = 0.f;
+      for (int i = l; i < d; i += 32) { qq = fmaf(q[i], q[i], qq); kk = fmaf(k[i], k[i], kk); }
+      qq = warp_sum(qq); kk = warp_sum(kk);
       const float rq = rsqrtf(qq + 1e-6f) * qscale, rk = rsqrtf(kk + 1e-6f);
       float *row = a.buf + (long long)t * a.ld_b;
       for (int i = l; i < d; i += 32) { row[g * d + i] = q[i] * rq; row[(c.G + g) * d + i] = k[i] * rk; }
-      if (l == 0) row[C + g] = qk * rq * rk;
     }
     return;
   }
@@ -144,7 +142,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
     if (role == 0)
       for (int e = threadIdx.x; e < (t1 - t0) * c.H; e += kDeltaTh) {
         const int t = t0 + e / c.H, h = e % c.H;
-        a.buf[(long long)t * a.ld_b + C + c.G + h] = sigmoid_precise(in(t, c.b_off + h));
+        a.buf[(long long)t * a.ld_b + C + h] = sigmoid_precise(in(t, c.b_off + h));
       }
     if (ch < C) conv(ch, [&](int t, float v) { a.buf[(long long)t * a.ld_b + ch] = v; });
     return;
@@ -174,11 +172,134 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
     a.dec[(long long)t * n + i] = expf(-ea * spl);
   }
 }
+// The same for passes with prompts whose sizes let a lane take four neighbouring channels (d and dv multiples of 4, d <= 128, decay
+// logits from memory): a warp works on eight consecutive tokens and 128 channels by itself -- all their inputs are in flight together,
+// and a head's squares are added up across the warp.  Roles as above, without the gate's.
+constexpr int kDeltaWarpTok = 8, kDeltaVecTile = kDeltaWarpTok * kDeltaTh / 32;
+template <int TAPS>
+__global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_vec_kernel(StackDelta c, StackDeltaPrep a, StackSpans sp, int nvb) {
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, C = c.C;
+  const int t0 = blockIdx.x * kDeltaVecTile + w * kDeltaWarpTok, nt = min(kDeltaWarpTok, sp.T - t0);
+  if (nt <= 0) return;
+  auto f4 = [](const float *p) { return *reinterpret_cast<const float4 *>(p); };
+  auto in4 = [&](int t, int col) {
+    const float *p = a.proj + (long long)t * a.ld + col;
+    float4 v = f4(p);
+    for (int k = 1; k < a.n_part; k++) {
+      const float4 q = f4(p + (long long)k * a.stride);
+      v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+    }
+    return v;
+  };
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  // channels ch .. ch + 3 (on: they exist) over the warp's tokens; put is called by every lane
+  auto conv = [&](int ch, bool on, auto &&put) {
+    float wt[TAPS][4];
+    float4 cur[kDeltaWarpTok], win[TAPS > 1 ? TAPS - 1 : 1];
+#pragma unroll
+    for (int u = 0; u < kDeltaWarpTok; u++) cur[u] = on && u < nt ? in4(t0 + u, ch) : zero;
+#pragma unroll
+    for (int j = 0; j < TAPS; j++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) wt[j][e] = on ? a.cw[(long long)(ch + e) * TAPS + j] : 0.f;
+    int prev = -1;
+#pragma unroll
+    for (int u = 0; u < kDeltaWarpTok; u++) {
+      const int t = t0 + u;
+      if (u >= nt) break;
+      const int s = sp.span[t];
+      if (TAPS > 1 && s != prev) {
+        prev = s;
+        const int back_in_span = t - sp.sp_tok0[s], pos0 = sp.sp_pos0[s];
+        const float *tail = a.cstate + (long long)sp.sp_slot[s] * (TAPS - 1) * C + ch;
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; j++) {
+          const int back = TAPS - 1 - j;
+          win[j] = !on ? zero : back <= back_in_span ? in4(t - back, ch) : pos0 + back_in_span - back >= 0 ? f4(tail + (long long)((TAPS - 1) - (back - back_in_span)) * C) : zero;
+        }
+      }
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < TAPS; j++) {
+        const float4 v = j + 1 < TAPS ? win[TAPS > 1 && j + 1 < TAPS ? j : 0] : cur[u];
+        acc[0] = fmaf(wt[j][0], v.x, acc[0]); acc[1] = fmaf(wt[j][1], v.y, acc[1]); acc[2] = fmaf(wt[j][2], v.z, acc[2]); acc[3] = fmaf(wt[j][3], v.w, acc[3]);
+      }
+      if (TAPS > 1) {
+#pragma unroll
+        for (int j = 0; j + 2 < TAPS; j++) win[j] = win[j + 1];
+        win[TAPS > 1 ? TAPS - 2 : 0] = cur[u];
+      }
+      put(t, make_float4(delta_silu(acc[0]), delta_silu(acc[1]), delta_silu(acc[2]), delta_silu(acc[3])));
+    }
+  };
+  int role = blockIdx.y;
+  if (role < c.G) {
+    const bool on = 4 * l < c.d;
+    for (int k = 0; k < 2; k++) {  // query, then key
+      const int ch = (k * c.G + role) * c.d + 4 * l;
+      const float scale = k ? 1.f : rsqrtf((float)c.d);
+      conv(ch, on, [&](int t, float4 v) {
+        const float f = rsqrtf(warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)))) + 1e-6f) * scale;
+        if (on) *reinterpret_cast<float4 *>(a.buf + (long long)t * a.ld_b + ch) = make_float4(v.x * f, v.y * f, v.z * f, v.w * f);
+      });
+    }
+    return;
+  }
+  role -= c.G;
+  if (role < nvb) {
+    const int ch = 2 * c.G * c.d + role * kDeltaTh + 4 * l;
+    if (role == 0)
+      for (int e = l; e < nt * c.H; e += 32) {
+        const int t = t0 + e / c.H, h = e % c.H;
+        const float *p = a.proj + (long long)t * a.ld + c.b_off + h;
+        float v = p[0];
+        for (int k = 1; k < a.n_part; k++) v += p[(long long)k * a.stride];
+        a.buf[(long long)t * a.ld_b + C + h] = sigmoid_precise(v);
+      }
+    const bool on = ch < C;
+    conv(ch, on, [&](int t, float4 v) { if (on) *reinterpret_cast<float4 *>(a.buf + (long long)t * a.ld_b + ch) = v; });
+    return;
+  }
+  role -= nvb;
+  const int n = c.H * c.d, i = role * kDeltaTh + 4 * l;
+  if (i >= n) return;
+  const float ea = expf(a.vec[i / c.d]);
+  float bias[4];
+#pragma unroll
+  for (int e = 0; e < 4; e++) bias[e] = a.vec[c.H + i + e];
+  float4 z[kDeltaWarpTok];
+#pragma unroll
+  for (int u = 0; u < kDeltaWarpTok; u++) z[u] = u < nt ? f4(a.z + (long long)(t0 + u) * n + i) : zero;
+#pragma unroll
+  for (int u = 0; u < kDeltaWarpTok; u++) {
+    if (u >= nt) break;
+    float y[4] = {z[u].x, z[u].y, z[u].z, z[u].w};
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+      y[e] += bias[e];
+      y[e] = expf(-ea * (fmaxf(y[e], 0.f) + log1pf(expf(-fabsf(y[e])))));
+    }
+    *reinterpret_cast<float4 *>(a.dec + (long long)(t0 + u) * n + i) = make_float4(y[0], y[1], y[2], y[3]);
+  }
+}
 cudaError_t launch_stack_delta_prep(const StackDelta &c, const StackDeltaPrep &a, bool w_f32, const StackSpans &sp, cudaStream_t st) {
   if (sp.T <= 0) return cudaSuccess;
   if (c.taps < 1 || c.taps > kDeltaMaxTaps) return cudaErrorInvalidValue;
   const int single = sp.T == sp.n_spans ? 1 : 0, tile = single ? 1 : 16;
   const int nvb = (c.H * c.dv + kDeltaTh - 1) / kDeltaTh, ndb = (c.H * c.d + kDeltaTh - 1) / kDeltaTh, ngb = a.z ? 0 : (c.H * c.dv + kDeltaTh - 1) / kDeltaTh;
+  auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (!single && a.z && c.taps <= 4 && c.d <= 128 && c.d % 4 == 0 && c.dv % 4 == 0 && a.ld % 4 == 0 && a.stride % 4 == 0 && a.ld_b % 4 == 0 && al(a.proj) && al(a.buf) &&
+      al(a.z) && al(a.dec) && al(a.cstate)) {
+    const dim3 vgrid((sp.T + kDeltaVecTile - 1) / kDeltaVecTile, c.G + nvb + ndb);
+    switch (c.taps) {
+      case 1: stack_delta_prep_vec_kernel<1><<<vgrid, kDeltaTh, 0, st>>>(c, a, sp, nvb); break;
+      case 2: stack_delta_prep_vec_kernel<2><<<vgrid, kDeltaTh, 0, st>>>(c, a, sp, nvb); break;
+      case 3: stack_delta_prep_vec_kernel<3><<<vgrid, kDeltaTh, 0, st>>>(c, a, sp, nvb); break;
+      default: stack_delta_prep_vec_kernel<4><<<vgrid, kDeltaTh, 0, st>>>(c, a, sp, nvb);
+    }
+    DIS_CUDA_TRY(cudaGetLastError());
+    return c.taps > 1 ? launch_stack_conv_tail(a.proj, a.ld, a.n_part, a.stride, 0, a.cstate, sp, c.C, c.taps, st) : cudaSuccess;
+  }
   const int rank = std::max(c.ra, c.rg);
   const size_t shb = (size_t)tile * std::max(2 * c.d, a.z ? 0 : (rank + 3) & ~3) * sizeof(float);
   if (shb > 200 * 1024) return cudaErrorInvalidValue;
@@ -230,16 +351,23 @@ cudaError_t launch_stack_delta_pack(const StackDelta &c, const StackDeltaPrep &a
 
 // ------------------------------------------------------------------------------------------------ the recurrence
 // Per head, S [d][dv]:  S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
+// Four tokens at a time.  With S the state in front of them and G_t = g_1 .. g_t (products of the chunk's decays, per channel),
+//   u_t = beta_t (v_t - S^T (G_t k_t) - sum_{s<t} A_ts u_s),   A_ts = sum_i k_t (g_{s+1} .. g_t) k_s,
+//   o_t = S^T (G_t q_t) + sum_{s<=t} B_ts u_s,                 B_ts = sum_i q_t (g_{s+1} .. g_t) k_s,
+//   S  <- G_4 S + sum_s (g_{s+1} .. g_4) k_s u_s^T
+// -- no quotient of decays, so a factor may be zero.  The eight inner products over S do not wait for one another; what has to happen in
+// order is six multiplications of numbers per column.  G_t k_t, G_t q_t, the suffix products times k_s, A and B of the next four tokens
+// are made while the present ones are worked on (all warps of a CTA share them), and the tokens after those are on their way into
+// shared memory.
 // The columns of S do not touch each other, so a head is cut into blocks of columns that never exchange anything: a warp owns 2 CL
-// columns, its half-warps CL each, and the sixteen lanes of a half share the rows (RL each).  Both inner products run over the
-// decayed state before the write -- o = (gS)^T q + u (k.q) -- so a token costs one reduction over sixteen lanes: a butterfly that
-// halves the values a lane still carries at every step (products with k end in lanes 0-7, those with q in lanes 8-15), then u is
-// handed back to all lanes.  Rows are taken in pairs by packed fp32 operations.  q, k, g, v, beta and k.q of the next kDeltaTok
-// tokens are on their way into shared memory while the present ones are worked on; a CTA's warps share them.
+// columns, its half-warps CL each, and the sixteen lanes of a half share the rows (RL each, taken in pairs by packed fp32 operations).
+// The inner products are added up by a butterfly over the sixteen lanes that halves the values a lane still carries at every step:
+// lanes 0-7 end with a column's products with the k's and solve for u, lanes 8-15 with those with the q's and form o.
+// A chunk starts where its span does; tokens beyond the span's end enter as k = q = 0, beta = 0, g = 1.
 // State: [slots][H][dv][d], a column's rows next to each other.
 // fin.act: the CTA holds whole heads, and each token's o of the head is divided by its root mean square, times norm, times
 // sigmoid(gate), and stored in the compute type; else o goes to o [T][H*dv] as it is.
-constexpr int kDeltaTok = 8;
+constexpr int kDeltaTok = 4;
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack2(float lo, float hi) { f32x2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
 __device__ __forceinline__ void unpack2(f32x2 v, float &lo, float &hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
@@ -260,25 +388,34 @@ struct DeltaFin {
   float eps;
   int f32;
 };
+constexpr int kDeltaVec = 3 * kDeltaTok + 1;  // vectors of a chunk: G_t k_t, G_t q_t, suffix products times k_s, G_4
+template <int RL>
+constexpr int delta_smem_floats(int nw, int vc) {  // three chunks as they came, vectors and numbers of two, outputs of two
+  return 3 * kDeltaTok * (3 * 16 * RL + vc + 4) + 2 * kDeltaVec * 16 * RL + 2 * nw * 16 + nw * 16 + 2 * kDeltaTok * vc;
+}
 template <int RL, int CL>
 __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const float *__restrict__ buf, long long ld_b, const float *__restrict__ dec,
-                                                          float *state, StackSpans sp, float *__restrict__ o, int ncb, int vec, DeltaFin fin) {
+                                                             float *state, StackSpans sp, float *__restrict__ o, int ncb, int vec, DeltaFin fin) {
   extern __shared__ __align__(16) float sh[];
-  constexpr int DP = 16 * RL, V = RL < 4 ? RL : 4, NM = RL / V, NP = RL / 2, CW = 2 * CL;
+  constexpr int DP = 16 * RL, V = RL < 4 ? RL : 4, NM = RL / V, NP = RL / 2, CW = 2 * CL, CT = kDeltaTok;
   const int H = c.H, d = c.d, dv = c.dv;
   const int h = blockIdx.x % H, rest = blockIdx.x / H, cb = rest % ncb, s = rest / ncb;  // heads vary fastest: CTAs that run together read whole rows
   const int tok0 = sp.sp_tok0[s], n = sp.sp_len[s], pos0 = sp.sp_pos0[s], slot = sp.sp_slot[s];
   const int NW = blockDim.x >> 5, w = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 15, hf = lane >> 4;
   const int VC = NW * CW, col_cta = cb * VC, nv = min(VC, dv - col_cta);
-  const int PT = 3 * DP + VC + 4;  // a token's stage: q | k | g | v | beta, k.q
-  float *os = sh + 2 * kDeltaTok * PT;  // [kDeltaTok][VC] outputs of a group (fin)
-  for (int i = threadIdx.x; i < 2 * kDeltaTok * PT + (fin.act ? kDeltaTok * VC : 0); i += blockDim.x) sh[i] = 0.f;  // rows beyond d and columns beyond dv stay zero
+  const int PT = 3 * DP + VC + 4;  // a token as it comes: q | k | g | v | beta
+  float *vecs = sh + 3 * CT * PT;                // [2][kDeltaVec][DP]
+  float *part = vecs + 2 * kDeltaVec * DP;       // [2][NW][16]: A and B, a warp's share of the channels
+  float *sc = part + 2 * NW * 16 + w * 16;       // [16] A (2,1) (3,1) (3,2) (4,1) (4,2) (4,3), B (t, s) row by row
+  float *os = part + 3 * NW * 16;                // [2][CT][VC]
+  for (int i = threadIdx.x; i < delta_smem_floats<RL>(NW, VC); i += blockDim.x) sh[i] = 0.f;  // rows beyond d and columns beyond dv stay zero
   const int kvh = h / (H / c.G);
   const float *qsrc = buf + kvh * d, *ksrc = buf + (c.G + kvh) * d, *vsrc = buf + 2 * c.G * d + (long long)h * dv + col_cta;
-  const float *gsrc = dec + (long long)h * d, *bsrc = buf + c.C + c.G + h, *xsrc = buf + c.C + kvh;
-  auto fetch = [&](int i0, int stage) {
-    const int ct = min(kDeltaTok, n - i0);
-    float *dst0 = sh + stage * kDeltaTok * PT;
+  const float *gsrc = dec + (long long)h * d, *bsrc = buf + c.C + h;
+  const int nch = (n + CT - 1) / CT;
+  auto fetch = [&](int ch) {
+    const int i0 = ch * CT, ct = min(CT, n - i0);
+    float *dst0 = sh + (ch % 3) * CT * PT;
     const int per = vec ? 4 : 1, dq = d / per, nc = 3 * dq + nv / per;
     for (int i = threadIdx.x; i < ct * nc; i += blockDim.x) {
       const int tt = i / nc, e = i - tt * nc;
@@ -292,11 +429,56 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
       if (vec) delta_cp16(dst, src);
       else delta_cp4(dst, src);
     }
-    for (int i = threadIdx.x; i < 2 * ct; i += blockDim.x) {
-      const long long t = tok0 + i0 + (i >> 1);
-      delta_cp4(dst0 + (i >> 1) * PT + 3 * DP + VC + (i & 1), (i & 1 ? xsrc : bsrc) + t * ld_b);
-    }
+    for (int tt = threadIdx.x; tt < ct; tt += blockDim.x) delta_cp4(dst0 + tt * PT + 3 * DP + VC, bsrc + (long long)(tok0 + i0 + tt) * ld_b);
     asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // vectors and numbers of chunk ch, a thread per channel
+  auto prepare = [&](int ch) {
+    const int ct = min(CT, n - ch * CT);
+    const float *raw = sh + (ch % 3) * CT * PT;
+    float *vd = vecs + (ch & 1) * kDeltaVec * DP;
+    float acc[16];
+#pragma unroll
+    for (int j = 0; j < 16; j++) acc[j] = 0.f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+      float q[CT], k[CT], g[CT];
+#pragma unroll
+      for (int t = 0; t < CT; t++) {
+        const bool on = t < ct;
+        q[t] = on ? raw[t * PT + i] : 0.f; k[t] = on ? raw[t * PT + DP + i] : 0.f; g[t] = on ? raw[t * PT + 2 * DP + i] : 1.f;
+      }
+      float G = 1.f, suf = 1.f;
+#pragma unroll
+      for (int t = 0; t < CT; t++) {
+        G *= g[t];
+        vd[t * DP + i] = G * k[t];
+        vd[(CT + t) * DP + i] = G * q[t];
+      }
+      vd[3 * CT * DP + i] = G;
+#pragma unroll
+      for (int t = CT - 1; t >= 0; t--) { vd[(2 * CT + t) * DP + i] = suf * k[t]; suf *= g[t]; }
+#pragma unroll
+      for (int t2 = 0; t2 < CT; t2++) {
+        float x = k[t2];
+        acc[6 + t2 * (t2 + 1) / 2 + t2] = fmaf(q[t2], x, acc[6 + t2 * (t2 + 1) / 2 + t2]);
+#pragma unroll
+        for (int t = t2 + 1; t < CT; t++) {
+          x *= g[t];
+          acc[t * (t - 1) / 2 + t2] = fmaf(k[t], x, acc[t * (t - 1) / 2 + t2]);
+          acc[6 + t * (t + 1) / 2 + t2] = fmaf(q[t], x, acc[6 + t * (t + 1) / 2 + t2]);
+        }
+      }
+    }
+    const bool c4 = lane & 16, c3 = lane & 8, c2 = lane & 4, c1 = lane & 2;
+#pragma unroll
+    for (int j = 0; j < 8; j++) acc[j] = (c4 ? acc[j + 8] : acc[j]) + __shfl_xor_sync(0xffffffffu, c4 ? acc[j] : acc[j + 8], 16);
+#pragma unroll
+    for (int j = 0; j < 4; j++) acc[j] = (c3 ? acc[j + 4] : acc[j]) + __shfl_xor_sync(0xffffffffu, c3 ? acc[j] : acc[j + 4], 8);
+#pragma unroll
+    for (int j = 0; j < 2; j++) acc[j] = (c2 ? acc[j + 2] : acc[j]) + __shfl_xor_sync(0xffffffffu, c2 ? acc[j] : acc[j + 2], 4);
+    acc[0] = (c1 ? acc[1] : acc[0]) + __shfl_xor_sync(0xffffffffu, c1 ? acc[0] : acc[1], 2);
+    acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
+    if (!(lane & 1)) part[((ch & 1) * NW + w) * 16 + (lane >> 1)] = acc[0];
   };
   // ---- the state: columns col0 + cc, rows r V + 16 V m + e
   const int wc = w * CW + hf * CL, col0 = col_cta + wc;
@@ -321,71 +503,123 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
 #pragma unroll
     for (int q = 0; q < NP; q++) S[cc][q] = pack2(v[2 * q], v[2 * q + 1]);
   }
+  auto ld_vec = [&](const float *p, f32x2 (&x)[NP]) {  // this lane's rows of a vector
+#pragma unroll
+    for (int m = 0; m < NM; m++) {
+      if (V == 4) {
+        const ulonglong2 a = *reinterpret_cast<const ulonglong2 *>(p + r * V + 16 * V * m);
+        x[V == 4 ? 2 * m : 0] = a.x; x[V == 4 ? 2 * m + 1 : 0] = a.y;
+      } else x[m] = *reinterpret_cast<const f32x2 *>(p + r * V + 16 * V * m);
+    }
+  };
   __syncthreads();
-  fetch(0, 0);
+  fetch(0);
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  if (nch > 1) fetch(1);
+  prepare(0);
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
   const bool b3 = lane & 8, b2 = lane & 4, b1 = lane & 2, b0 = lane & 1;
   const int mycol = CL == 8 ? (lane & 7) : (lane & 7) >> 1;  // the column whose sums end in this lane
-  int stage = 0;
-  for (int i0 = 0; i0 < n; i0 += kDeltaTok, stage ^= 1) {
-    const int ct = min(kDeltaTok, n - i0);
-    if (i0 + kDeltaTok < n) {
-      fetch(i0 + kDeltaTok, stage ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    for (int tt = 0; tt < ct; tt++) {
-      const float *row = sh + (stage * kDeltaTok + tt) * PT;
-      f32x2 kp[NP], qp[NP], gp[NP];
+  for (int ch = 0; ch < nch; ch++) {
+    const int i0 = ch * CT, ct = min(CT, n - i0);
+    if (ch + 2 < nch) fetch(ch + 2);
+    if (ch + 1 < nch) prepare(ch + 1);
+    const float *raw = sh + (ch % 3) * CT * PT, *vd = vecs + (ch & 1) * kDeltaVec * DP;
+    if (lane < 16) {
+      float v = 0.f;
+      for (int k = 0; k < NW; k++) v += part[((ch & 1) * NW + k) * 16 + lane];
+      sc[lane] = v;
+    }
+    float x[CT][CL];
 #pragma unroll
-      for (int m = 0; m < NM; m++) {
-        const float *p = row + r * V + 16 * V * m;
-        if (V == 4) {
-          const ulonglong2 a = *reinterpret_cast<const ulonglong2 *>(p), b = *reinterpret_cast<const ulonglong2 *>(p + DP), g = *reinterpret_cast<const ulonglong2 *>(p + 2 * DP);
-          qp[2 * m] = a.x; qp[V == 4 ? 2 * m + 1 : 0] = a.y; kp[2 * m] = b.x; kp[V == 4 ? 2 * m + 1 : 0] = b.y; gp[2 * m] = g.x; gp[V == 4 ? 2 * m + 1 : 0] = g.y;
-        } else {
-          qp[m] = *reinterpret_cast<const f32x2 *>(p); kp[m] = *reinterpret_cast<const f32x2 *>(p + DP); gp[m] = *reinterpret_cast<const f32x2 *>(p + 2 * DP);
-        }
-      }
-      const float vv = row[3 * DP + wc + mycol], beta = row[3 * DP + VC], kq = row[3 * DP + VC + 1];
-      float x[CL];
+    for (int t = 0; t < CT; t++) {
+      f32x2 kp[NP], qp[NP];
+      ld_vec(vd + t * DP, kp);
+      ld_vec(vd + (CT + t) * DP, qp);
 #pragma unroll
       for (int cc = 0; cc < CL; cc++) {
-        f32x2 a = 0ull, b = 0ull;
+        f32x2 a = mul2(S[cc][0], kp[0]), b = mul2(S[cc][0], qp[0]);
 #pragma unroll
-        for (int q = 0; q < NP; q++) {
-          S[cc][q] = mul2(S[cc][q], gp[q]);
+        for (int q = 1; q < NP; q++) {
           a = fma2(S[cc][q], kp[q], a);
           b = fma2(S[cc][q], qp[q], b);
         }
         float al, ah, bl, bh;
         unpack2(a, al, ah); unpack2(b, bl, bh);
         const float dk = al + ah, dq = bl + bh;
-        x[cc] = (b3 ? dq : dk) + __shfl_xor_sync(0xffffffffu, b3 ? dk : dq, 8);
+        x[t][cc] = (b3 ? dq : dk) + __shfl_xor_sync(0xffffffffu, b3 ? dk : dq, 8);
       }
+    }
 #pragma unroll
-      for (int i = 0; i < CL / 2; i++) x[i] = (b2 ? x[i + CL / 2] : x[i]) + __shfl_xor_sync(0xffffffffu, b2 ? x[i] : x[i + CL / 2], 4);
+    for (int t = 0; t < CT; t++) {
 #pragma unroll
-      for (int i = 0; i < CL / 4; i++) x[i] = (b1 ? x[i + CL / 4] : x[i]) + __shfl_xor_sync(0xffffffffu, b1 ? x[i] : x[i + CL / 4], 2);
-      if (CL == 8) x[0] = (b0 ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, b0 ? x[0] : x[1], 1);
-      else x[0] += __shfl_xor_sync(0xffffffffu, x[0], 1);
-      const float u = beta * (vv - x[0]);  // (lanes 0-7 of a half)
+      for (int i = 0; i < CL / 2; i++) x[t][i] = (b2 ? x[t][i + CL / 2] : x[t][i]) + __shfl_xor_sync(0xffffffffu, b2 ? x[t][i] : x[t][i + CL / 2], 4);
+    }
+#pragma unroll
+    for (int t = 0; t < CT; t++) {
+#pragma unroll
+      for (int i = 0; i < CL / 4; i++) x[t][i] = (b1 ? x[t][i + CL / 4] : x[t][i]) + __shfl_xor_sync(0xffffffffu, b1 ? x[t][i] : x[t][i + CL / 4], 2);
+    }
+#pragma unroll
+    for (int t = 0; t < CT; t++) {
+      if (CL == 8) x[t][0] = (b0 ? x[t][1] : x[t][0]) + __shfl_xor_sync(0xffffffffu, b0 ? x[t][0] : x[t][1], 1);
+      else x[t][0] += __shfl_xor_sync(0xffffffffu, x[t][0], 1);
+    }
+    __syncwarp();
+    float AB[16];
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      const float4 f = *reinterpret_cast<const float4 *>(sc + 4 * j);
+      AB[4 * j] = f.x; AB[4 * j + 1] = f.y; AB[4 * j + 2] = f.z; AB[4 * j + 3] = f.w;
+    }
+    float u[CT];  // (lanes 0-7 of a half)
+#pragma unroll
+    for (int t = 0; t < CT; t++) {
+      float y = raw[t * PT + 3 * DP + wc + mycol] - x[t][0];
+#pragma unroll
+      for (int t2 = 0; t2 < t; t2++) y = fmaf(-AB[t * (t - 1) / 2 + t2], u[t2], y);
+      u[t] = t < ct ? raw[t * PT + 3 * DP + VC] * y : 0.f;
+    }
+    {
+      f32x2 gp[NP];
+      ld_vec(vd + 3 * CT * DP, gp);
+#pragma unroll
+      for (int cc = 0; cc < CL; cc++)
+#pragma unroll
+        for (int q = 0; q < NP; q++) S[cc][q] = mul2(S[cc][q], gp[q]);
+    }
+#pragma unroll
+    for (int t = 0; t < CT; t++) {
+      f32x2 kp[NP];
+      ld_vec(vd + (2 * CT + t) * DP, kp);
 #pragma unroll
       for (int cc = 0; cc < CL; cc++) {
-        const float uc = __shfl_sync(0xffffffffu, u, (lane & 16) | (CL == 8 ? cc : 2 * cc));
+        const float uc = __shfl_sync(0xffffffffu, u[t], (lane & 16) | (CL == 8 ? cc : 2 * cc));
         const f32x2 u2 = pack2(uc, uc);
 #pragma unroll
         for (int q = 0; q < NP; q++) S[cc][q] = fma2(kp[q], u2, S[cc][q]);
       }
-      const float ov = fmaf(__shfl_xor_sync(0xffffffffu, u, 8), kq, x[0]);  // (lanes 8-15)
-      if (b3 && (CL == 8 || !b0)) {
-        if (fin.act) os[tt * VC + wc + mycol] = ov;
-        else if (col0 + mycol < dv) o[(long long)(tok0 + i0 + tt) * H * dv + (long long)h * dv + col0 + mycol] = ov;
+    }
+#pragma unroll
+    for (int t = 0; t < CT; t++) u[t] = __shfl_xor_sync(0xffffffffu, u[t], 8);  // to the lanes that form o
+    if (b3 && (CL == 8 || !b0)) {
+#pragma unroll
+      for (int t = 0; t < CT; t++) {
+        if (t >= ct) break;
+        float ov = x[t][0];
+#pragma unroll
+        for (int t2 = 0; t2 <= t; t2++) ov = fmaf(AB[6 + t * (t + 1) / 2 + t2], u[t2], ov);
+        if (fin.act) os[((ch & 1) * CT + t) * VC + wc + mycol] = ov;
+        else if (col0 + mycol < dv) o[(long long)(tok0 + i0 + t) * H * dv + (long long)h * dv + col0 + mycol] = ov;
       }
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     if (fin.act) {  // a warp finishes a token (columns beyond dv are zero)
       for (int tt = w; tt < ct; tt += NW) {
-        const float *ro = os + tt * VC;
+        const float *ro = os + ((ch & 1) * CT + tt) * VC;
         float ss = 0.f;
         for (int j = lane; j < dv; j += 32) ss = fmaf(ro[j], ro[j], ss);
         const float k = rsqrtf(warp_sum(ss) / (float)dv + fin.eps);
@@ -396,7 +630,6 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
           else st_el<false>(fin.act, t * fin.ld + (long long)h * dv + j, v);
         }
       }
-      if (i0 + kDeltaTok < n) __syncthreads();
     }
   }
 #pragma unroll
@@ -429,12 +662,12 @@ static cudaError_t delta_go(const StackDelta &c, const float *buf, long long ld_
   int nw = std::min(total, 8);
   // long spans: a head's columns are spread over more CTAs while that still brings idle SMs to work
   const long long pairs = (long long)sp.n_spans * c.H;
-  while (max_len > kDeltaTok && nw > 2 && pairs * ((total + nw - 1) / nw) * 2 <= 148) nw = (nw + 1) / 2;
+  while (max_len > 2 * kDeltaTok && nw > 2 && pairs * ((total + nw - 1) / nw) * 2 <= 148) nw = (nw + 1) / 2;
   const int ncb = (total + nw - 1) / nw, VC = nw * CW;
   const DeltaFin fin{ncb == 1 ? act : nullptr, ld_act, gate, norm, c.eps, f32 ? 1 : 0};
   auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const int vec = c.d % 4 == 0 && c.dv % 4 == 0 && ld_b % 4 == 0 && al(buf) && al(dec) && al(state);
-  const size_t shb = ((size_t)2 * kDeltaTok * (3 * 16 * RL + VC + 4) + (fin.act ? (size_t)kDeltaTok * VC : 0)) * sizeof(float);
+  const size_t shb = (size_t)delta_smem_floats<RL>(nw, VC) * sizeof(float);
   static DeviceOnce once;
   DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_delta_kernel<RL, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); }));
   stack_delta_kernel<RL, CL><<<(unsigned)(pairs * ncb), nw * 32, shb, st>>>(c, buf, ld_b, dec, state, sp, o, ncb, vec, fin);

@@ -597,7 +597,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       out_block(m_ + "o", 0, H * dv);
       max_mix = std::max(max_mix, (size_t)H * dv);
       max_dec = std::max(max_dec, (size_t)H * d);
-      max_ssm = std::max(max_ssm, ((size_t)L.conv_ch + G + H + 3) / 4 * 4);
+      max_ssm = std::max(max_ssm, ((size_t)L.conv_ch + H + 3) / 4 * 4);
       max_gz = std::max(max_gz, (size_t)H * dv);
       max_bn[0] = std::max(max_bn[0], (size_t)ra); max_bn[1] = std::max(max_bn[1], (size_t)rg);
     } else if (lc.mixer == DIS_MIX_SSM) {
@@ -1708,7 +1708,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       a.proj = in_src; a.ld = N; a.n_part = in_parts; a.stride = in_stride;
       a.cw = reinterpret_cast<const float *>(L.conv_w.ptr); a.vec = reinterpret_cast<const float *>(L.ssm_vec.ptr); a.cstate = Rn.conv_state;
       a.a2 = L.a2.ptr; a.g2 = L.g2.ptr;
-      a.buf = M.ssm; a.ld_b = ((long long)sd.C + sd.G + sd.H + 3) / 4 * 4; a.dec = M.dec; a.gz = M.gz;
+      a.buf = M.ssm; a.ld_b = ((long long)sd.C + sd.H + 3) / 4 * 4; a.dec = M.dec; a.gz = M.gz;
       if (T > 64) {  // more tokens than the preparation should multiply by itself: the bottlenecks' products as matrix products
         RET_CUDA(launch_stack_delta_pack(sd, a, f32, T, M.bn_a, M.bn_g, stream));
         kl++;

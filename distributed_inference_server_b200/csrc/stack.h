@@ -154,7 +154,7 @@ struct StackDeltaPrep {
   float *cstate = nullptr;        // [slots][taps-1][C]
   const void *a2 = nullptr, *g2 = nullptr;  // [H*d][ra], [H*dv][rg], compute type
   const float *z = nullptr;       // [T][H*d]: the products with a2, when they (and the gate's) were made by matrix products; null: made here
-  float *buf = nullptr;           // [T][ld_b]: q | k | v as they enter the recurrence, k.q [G], beta [H]
+  float *buf = nullptr;           // [T][ld_b]: q | k | v as they enter the recurrence, beta [H]
   long long ld_b = 0;
   float *dec = nullptr;           // [T][H*d]
   float *gz = nullptr;            // [T][H*dv]: the gate's logits (written here when z is null)

@@ -62,6 +62,16 @@ def test_trace_replay_of_a_nifulix_model(tmp_path, dtype, tol):
     _replay(tmp_path, dtype, tol, cfg, N.weights(cfg, seed=3), N.oracle_logits)
 
 
+@pytest.mark.parametrize("dtype,tol", [("float32", 2e-4), ("bfloat16", None)])
+def test_trace_replay_of_a_bunosun_model(tmp_path, dtype, tol):
+    """The same schedule through a looped Bunosun model: windows of 24 and 100 positions against pages of 64, delta-rule states and
+    convolution tails of every loop pass handed on from request to request."""
+    from tests import _bunosun_util as N
+    cfg = N.config([(N.attention(dim=16, vdim=32, window=24, rot=8), N.moe()), (N.delta(), N.moe(groups=None)), (N.attention(window=100), None),
+                    (N.delta(heads=2, kv_heads=1, dim=16, vdim=16, conv=4), N.moe(experts=4, top=1, groups=(2, 1), shared=0))], vocab=90, width=40, loop=(1, 3, 2))
+    _replay(tmp_path, dtype, tol, cfg, N.weights(cfg, seed=3), N.oracle_logits)
+
+
 def _replay(tmp_path, dtype, tol, cfg, W, oracle_logits):
     model = tmp_path / "model"
     model.mkdir()
