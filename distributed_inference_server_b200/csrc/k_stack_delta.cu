@@ -142,7 +142,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
     if (role == 0)
       for (int e = threadIdx.x; e < (t1 - t0) * c.H; e += kDeltaTh) {
         const int t = t0 + e / c.H, h = e % c.H;
-        a.buf[(long long)t * a.ld_b + C + h] = sigmoid_precise(in(t, c.b_off + h));
+        a.buf[(long long)t * a.ld_b + C + c.H * c.d + h] = sigmoid_precise(in(t, c.b_off + h));
       }
     if (ch < C) conv(ch, [&](int t, float v) { a.buf[(long long)t * a.ld_b + ch] = v; });
     return;
@@ -169,7 +169,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
   for (int t = t0; t < t1; t++) {
     const float z = (a.z ? a.z[(long long)t * n + i] : delta_row_dot<WF32>(a.a2, i, sh + (t - t0) * pitch, rank)) + bias;
     const float spl = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-    a.dec[(long long)t * n + i] = expf(-ea * spl);
+    a.buf[(long long)t * a.ld_b + C + i] = expf(-ea * spl);
   }
 }
 // The same for passes with prompts whose sizes let a lane take four neighbouring channels (d and dv multiples of 4, d <= 128, decay
@@ -177,7 +177,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_kernel(StackDelta c
 // and a head's squares are added up across the warp.  Roles as above, without the gate's.
 constexpr int kDeltaWarpTok = 8, kDeltaVecTile = kDeltaWarpTok * kDeltaTh / 32;
 template <int TAPS>
-__global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_vec_kernel(StackDelta c, StackDeltaPrep a, StackSpans sp, int nvb) {
+__global__ void __launch_bounds__(kDeltaTh, 4) stack_delta_prep_vec_kernel(StackDelta c, StackDeltaPrep a, StackSpans sp, int nvb) {
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31, C = c.C;
   const int t0 = blockIdx.x * kDeltaVecTile + w * kDeltaWarpTok, nt = min(kDeltaWarpTok, sp.T - t0);
   if (nt <= 0) return;
@@ -254,7 +254,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_vec_kernel(StackDel
         const float *p = a.proj + (long long)t * a.ld + c.b_off + h;
         float v = p[0];
         for (int k = 1; k < a.n_part; k++) v += p[(long long)k * a.stride];
-        a.buf[(long long)t * a.ld_b + C + h] = sigmoid_precise(v);
+        a.buf[(long long)t * a.ld_b + C + c.H * c.d + h] = sigmoid_precise(v);
       }
     const bool on = ch < C;
     conv(ch, on, [&](int t, float4 v) { if (on) *reinterpret_cast<float4 *>(a.buf + (long long)t * a.ld_b + ch) = v; });
@@ -279,7 +279,7 @@ __global__ void __launch_bounds__(kDeltaTh) stack_delta_prep_vec_kernel(StackDel
       y[e] += bias[e];
       y[e] = expf(-ea * (fmaxf(y[e], 0.f) + log1pf(expf(-fabsf(y[e])))));
     }
-    *reinterpret_cast<float4 *>(a.dec + (long long)(t0 + u) * n + i) = make_float4(y[0], y[1], y[2], y[3]);
+    *reinterpret_cast<float4 *>(a.buf + (long long)(t0 + u) * a.ld_b + C + i) = make_float4(y[0], y[1], y[2], y[3]);
   }
 }
 cudaError_t launch_stack_delta_prep(const StackDelta &c, const StackDeltaPrep &a, bool w_f32, const StackSpans &sp, cudaStream_t st) {
@@ -288,8 +288,8 @@ cudaError_t launch_stack_delta_prep(const StackDelta &c, const StackDeltaPrep &a
   const int single = sp.T == sp.n_spans ? 1 : 0, tile = single ? 1 : 16;
   const int nvb = (c.H * c.dv + kDeltaTh - 1) / kDeltaTh, ndb = (c.H * c.d + kDeltaTh - 1) / kDeltaTh, ngb = a.z ? 0 : (c.H * c.dv + kDeltaTh - 1) / kDeltaTh;
   auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-  if (!single && a.z && c.taps <= 4 && c.d <= 128 && c.d % 4 == 0 && c.dv % 4 == 0 && a.ld % 4 == 0 && a.stride % 4 == 0 && a.ld_b % 4 == 0 && al(a.proj) && al(a.buf) &&
-      al(a.z) && al(a.dec) && al(a.cstate)) {
+  if (!single && a.z && c.taps <= 4 && c.d <= 128 && c.d % 4 == 0 && c.dv % 4 == 0 && a.ld % 4 == 0 && a.stride % 4 == 0 && a.ld_b % 4 == 0 && (c.H * c.d) % 4 == 0 && al(a.proj) && al(a.buf) &&
+      al(a.z) && al(a.cstate)) {
     const dim3 vgrid((sp.T + kDeltaVecTile - 1) / kDeltaVecTile, c.G + nvb + ndb);
     switch (c.taps) {
       case 1: stack_delta_prep_vec_kernel<1><<<vgrid, kDeltaTh, 0, st>>>(c, a, sp, nvb); break;
@@ -359,10 +359,10 @@ cudaError_t launch_stack_delta_pack(const StackDelta &c, const StackDeltaPrep &a
 // order is six multiplications of numbers per column.  G_t k_t, G_t q_t, the suffix products times k_s, A and B of the next four tokens
 // are made while the present ones are worked on (all warps of a CTA share them), and the tokens after those are on their way into
 // shared memory.
-// The columns of S do not touch each other, so a head is cut into blocks of columns that never exchange anything: a warp owns 2 CL
-// columns, its half-warps CL each, and the sixteen lanes of a half share the rows (RL each, taken in pairs by packed fp32 operations).
-// The inner products are added up by a butterfly over the sixteen lanes that halves the values a lane still carries at every step:
-// lanes 0-7 end with a column's products with the k's and solve for u, lanes 8-15 with those with the q's and form o.
+// The columns of S do not touch each other, so a head is cut into blocks of columns that never exchange anything: a warp owns eight
+// columns, each group of eight lanes two of them, and the eight lanes share the rows (RL each, taken in pairs by packed fp32
+// operations).  The inner products are added up by a butterfly over the eight lanes that halves the values a lane still carries at
+// every step: lanes 0-3 end with a column's products with the k's and solve for u, lanes 4-7 with those with the q's and form o.
 // A chunk starts where its span does; tokens beyond the span's end enter as k = q = 0, beta = 0, g = 1.
 // State: [slots][H][dv][d], a column's rows next to each other.
 // fin.act: the CTA holds whole heads, and each token's o of the head is divided by its root mean square, times norm, times
@@ -391,17 +391,20 @@ struct DeltaFin {
 constexpr int kDeltaVec = 3 * kDeltaTok + 1;  // vectors of a chunk: G_t k_t, G_t q_t, suffix products times k_s, G_4
 template <int RL>
 constexpr int delta_smem_floats(int nw, int vc) {  // three chunks as they came, vectors and numbers of two, outputs of two
-  return 3 * kDeltaTok * (3 * 16 * RL + vc + 4) + 2 * kDeltaVec * 16 * RL + 2 * nw * 16 + nw * 16 + 2 * kDeltaTok * vc;
+  return 3 * kDeltaTok * (3 * 8 * RL + vc + 4) + 2 * kDeltaVec * 8 * RL + 2 * nw * 16 + nw * 16 + 2 * kDeltaTok * vc;
 }
-template <int RL, int CL>
-__global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const float *__restrict__ buf, long long ld_b, const float *__restrict__ dec,
-                                                             float *state, StackSpans sp, float *__restrict__ o, int ncb, int vec, DeltaFin fin) {
+constexpr int kDeltaCols = 2;  // columns of a group of eight lanes
+// MW: warps of a CTA at most (fewer leave more registers)
+template <int RL, int MW>
+__global__ void __launch_bounds__(MW * 32, 1) stack_delta_kernel(StackDelta c, const float *__restrict__ buf, int ld_b, float *state, StackSpans sp,
+                                                                 float *__restrict__ o, int ncb, int vec, DeltaFin fin) {
   extern __shared__ __align__(16) float sh[];
-  constexpr int DP = 16 * RL, V = RL < 4 ? RL : 4, NM = RL / V, NP = RL / 2, CW = 2 * CL, CT = kDeltaTok;
+  constexpr int DP = 8 * RL, NM = RL / 4, NP = RL / 2, CL = kDeltaCols, CW = 4 * CL, CT = kDeltaTok;
   const int H = c.H, d = c.d, dv = c.dv;
   const int h = blockIdx.x % H, rest = blockIdx.x / H, cb = rest % ncb, s = rest / ncb;  // heads vary fastest: CTAs that run together read whole rows
   const int tok0 = sp.sp_tok0[s], n = sp.sp_len[s], pos0 = sp.sp_pos0[s], slot = sp.sp_slot[s];
-  const int NW = blockDim.x >> 5, w = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 15, hf = lane >> 4;
+  const int NW = blockDim.x >> 5, w = threadIdx.x >> 5, lane = threadIdx.x & 31, r = lane & 7, grp = lane >> 3;
+  const int NA = min(NW, (d + 31) >> 5);  // warps that prepare chunks
   const int VC = NW * CW, col_cta = cb * VC, nv = min(VC, dv - col_cta);
   const int PT = 3 * DP + VC + 4;  // a token as it comes: q | k | g | v | beta
   float *vecs = sh + 3 * CT * PT;                // [2][kDeltaVec][DP]
@@ -410,42 +413,44 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
   float *os = part + 3 * NW * 16;                // [2][CT][VC]
   for (int i = threadIdx.x; i < delta_smem_floats<RL>(NW, VC); i += blockDim.x) sh[i] = 0.f;  // rows beyond d and columns beyond dv stay zero
   const int kvh = h / (H / c.G);
-  const float *qsrc = buf + kvh * d, *ksrc = buf + (c.G + kvh) * d, *vsrc = buf + 2 * c.G * d + (long long)h * dv + col_cta;
-  const float *gsrc = dec + (long long)h * d, *bsrc = buf + c.C + h;
-  const int nch = (n + CT - 1) / CT;
+  const int nch = (n + CT - 1) / CT, HV = H * dv;
+  // A warp copies whole vectors: q, k, g and v of the chunk's tokens, dealt out from the last warp on (the first ones prepare).  Tokens
+  // beyond the span's end: k = q = 0, beta = 0, g = 1.
+  const int vcol = 2 * c.G * d + h * dv + col_cta, gcol = c.C + h * d, bcol = c.C + H * d + h;
+  const float *rows0 = buf + (long long)tok0 * ld_b;
   auto fetch = [&](int ch) {
-    const int i0 = ch * CT, ct = min(CT, n - i0);
-    float *dst0 = sh + (ch % 3) * CT * PT;
-    const int per = vec ? 4 : 1, dq = d / per, nc = 3 * dq + nv / per;
-    for (int i = threadIdx.x; i < ct * nc; i += blockDim.x) {
-      const int tt = i / nc, e = i - tt * nc;
-      const long long t = tok0 + i0 + tt;
-      float *dst = dst0 + tt * PT;
-      const float *src;
-      if (e < dq) { src = qsrc + t * ld_b + e * per; dst += e * per; }
-      else if (e < 2 * dq) { src = ksrc + t * ld_b + (e - dq) * per; dst += DP + (e - dq) * per; }
-      else if (e < 3 * dq) { src = gsrc + t * (long long)H * d + (e - 2 * dq) * per; dst += 2 * DP + (e - 2 * dq) * per; }
-      else { src = vsrc + t * ld_b + (e - 3 * dq) * per; dst += 3 * DP + (e - 3 * dq) * per; }
-      if (vec) delta_cp16(dst, src);
-      else delta_cp4(dst, src);
+    const int left = n - ch * CT;
+    const float *rows = rows0 + (long long)(ch * CT) * ld_b;
+    float *stage = sh + (ch % 3) * CT * PT;
+    for (int job = NW - 1 - w; job < 4 * CT; job += NW) {
+      const int tt = job >> 2, which = job & 3;
+      float *dst = stage + tt * PT + which * DP;
+      const int len = which == 3 ? nv : d;
+      if (tt < left) {
+        const float *src = rows + tt * ld_b + (which == 0 ? kvh * d : which == 1 ? (c.G + kvh) * d : which == 2 ? gcol : vcol);
+        if (vec) for (int e = lane * 4; e < len; e += 128) delta_cp16(dst + e, src + e);
+        else for (int e = lane; e < len; e += 32) delta_cp4(dst + e, src + e);
+        if (which == 3 && lane == 0) delta_cp4(dst + VC, rows + tt * ld_b + bcol);
+      } else {
+        for (int e = lane; e < len; e += 32) dst[e] = which == 2 ? 1.f : 0.f;
+        if (which == 3 && lane == 0) dst[VC] = 0.f;
+      }
     }
-    for (int tt = threadIdx.x; tt < ct; tt += blockDim.x) delta_cp4(dst0 + tt * PT + 3 * DP + VC, bsrc + (long long)(tok0 + i0 + tt) * ld_b);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   // vectors and numbers of chunk ch, a thread per channel
   auto prepare = [&](int ch) {
-    const int ct = min(CT, n - ch * CT);
+    if (w >= NA) return;
     const float *raw = sh + (ch % 3) * CT * PT;
     float *vd = vecs + (ch & 1) * kDeltaVec * DP;
     float acc[16];
 #pragma unroll
     for (int j = 0; j < 16; j++) acc[j] = 0.f;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) {
+    for (int i = threadIdx.x; i < d; i += NA * 32) {
       float q[CT], k[CT], g[CT];
 #pragma unroll
       for (int t = 0; t < CT; t++) {
-        const bool on = t < ct;
-        q[t] = on ? raw[t * PT + i] : 0.f; k[t] = on ? raw[t * PT + DP + i] : 0.f; g[t] = on ? raw[t * PT + 2 * DP + i] : 1.f;
+        q[t] = raw[t * PT + i]; k[t] = raw[t * PT + DP + i]; g[t] = raw[t * PT + 2 * DP + i];
       }
       float G = 1.f, suf = 1.f;
 #pragma unroll
@@ -480,8 +485,8 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
     acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], 1);
     if (!(lane & 1)) part[((ch & 1) * NW + w) * 16 + (lane >> 1)] = acc[0];
   };
-  // ---- the state: columns col0 + cc, rows r V + 16 V m + e
-  const int wc = w * CW + hf * CL, col0 = col_cta + wc;
+  // ---- the state: columns col0 + cc, rows 4 r + 32 m + e
+  const int wc = w * CW + grp * CL, col0 = col_cta + wc;
   float *st = state + ((long long)slot * H + h) * dv * d;
   f32x2 S[CL][NP];
 #pragma unroll
@@ -491,13 +496,13 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
     const bool on = pos0 > 0 && col0 + cc < dv;
 #pragma unroll
     for (int m = 0; m < NM; m++) {
-      const int i = r * V + 16 * V * m;
-      if (V == 4 && vec) {
+      const int i = r * 4 + 32 * m;
+      if (vec) {
         const float4 f = on && i < d ? *reinterpret_cast<const float4 *>(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-        v[m * V] = f.x; v[m * V + 1] = f.y; v[m * V + (V > 2 ? 2 : 0)] = f.z; v[m * V + (V > 3 ? 3 : 1)] = f.w;
+        v[m * 4] = f.x; v[m * 4 + 1] = f.y; v[m * 4 + 2] = f.z; v[m * 4 + 3] = f.w;
       } else {
 #pragma unroll
-        for (int e = 0; e < V; e++) v[m * V + e] = on && i + e < d ? p[i + e] : 0.f;
+        for (int e = 0; e < 4; e++) v[m * 4 + e] = on && i + e < d ? p[i + e] : 0.f;
       }
     }
 #pragma unroll
@@ -506,10 +511,8 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
   auto ld_vec = [&](const float *p, f32x2 (&x)[NP]) {  // this lane's rows of a vector
 #pragma unroll
     for (int m = 0; m < NM; m++) {
-      if (V == 4) {
-        const ulonglong2 a = *reinterpret_cast<const ulonglong2 *>(p + r * V + 16 * V * m);
-        x[V == 4 ? 2 * m : 0] = a.x; x[V == 4 ? 2 * m + 1 : 0] = a.y;
-      } else x[m] = *reinterpret_cast<const f32x2 *>(p + r * V + 16 * V * m);
+      const ulonglong2 a = *reinterpret_cast<const ulonglong2 *>(p + r * 4 + 32 * m);
+      x[2 * m] = a.x; x[2 * m + 1] = a.y;
     }
   };
   __syncthreads();
@@ -520,16 +523,18 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
   prepare(0);
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  const bool b3 = lane & 8, b2 = lane & 4, b1 = lane & 2, b0 = lane & 1;
-  const int mycol = CL == 8 ? (lane & 7) : (lane & 7) >> 1;  // the column whose sums end in this lane
-  for (int ch = 0; ch < nch; ch++) {
+  const bool b2 = lane & 4, b1 = lane & 2, b0 = lane & 1;
+  const int mycol = (lane >> 1) & 1;  // the column whose sums end in this lane (and its neighbour)
+  const bool writes = b2 && !b0 && (fin.act || col0 + mycol < dv);  // this lane forms outputs
+  float *op = o + (long long)tok0 * HV + h * dv + col0 + mycol;
+  for (int ch = 0; ch < nch; ch++, op += (long long)CT * HV) {
     const int i0 = ch * CT, ct = min(CT, n - i0);
     if (ch + 2 < nch) fetch(ch + 2);
     if (ch + 1 < nch) prepare(ch + 1);
     const float *raw = sh + (ch % 3) * CT * PT, *vd = vecs + (ch & 1) * kDeltaVec * DP;
     if (lane < 16) {
       float v = 0.f;
-      for (int k = 0; k < NW; k++) v += part[((ch & 1) * NW + k) * 16 + lane];
+      for (int k = 0; k < NA; k++) v += part[((ch & 1) * NW + k) * 16 + lane];
       sc[lane] = v;
     }
     float x[CT][CL];
@@ -549,24 +554,13 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
         float al, ah, bl, bh;
         unpack2(a, al, ah); unpack2(b, bl, bh);
         const float dk = al + ah, dq = bl + bh;
-        x[t][cc] = (b3 ? dq : dk) + __shfl_xor_sync(0xffffffffu, b3 ? dk : dq, 8);
+        x[t][cc] = (b2 ? dq : dk) + __shfl_xor_sync(0xffffffffu, b2 ? dk : dq, 4);
       }
     }
 #pragma unroll
-    for (int t = 0; t < CT; t++) {
+    for (int t = 0; t < CT; t++) x[t][0] = (b1 ? x[t][1] : x[t][0]) + __shfl_xor_sync(0xffffffffu, b1 ? x[t][0] : x[t][1], 2);
 #pragma unroll
-      for (int i = 0; i < CL / 2; i++) x[t][i] = (b2 ? x[t][i + CL / 2] : x[t][i]) + __shfl_xor_sync(0xffffffffu, b2 ? x[t][i] : x[t][i + CL / 2], 4);
-    }
-#pragma unroll
-    for (int t = 0; t < CT; t++) {
-#pragma unroll
-      for (int i = 0; i < CL / 4; i++) x[t][i] = (b1 ? x[t][i + CL / 4] : x[t][i]) + __shfl_xor_sync(0xffffffffu, b1 ? x[t][i] : x[t][i + CL / 4], 2);
-    }
-#pragma unroll
-    for (int t = 0; t < CT; t++) {
-      if (CL == 8) x[t][0] = (b0 ? x[t][1] : x[t][0]) + __shfl_xor_sync(0xffffffffu, b0 ? x[t][0] : x[t][1], 1);
-      else x[t][0] += __shfl_xor_sync(0xffffffffu, x[t][0], 1);
-    }
+    for (int t = 0; t < CT; t++) x[t][0] += __shfl_xor_sync(0xffffffffu, x[t][0], 1);
     __syncwarp();
     float AB[16];
 #pragma unroll
@@ -574,13 +568,13 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
       const float4 f = *reinterpret_cast<const float4 *>(sc + 4 * j);
       AB[4 * j] = f.x; AB[4 * j + 1] = f.y; AB[4 * j + 2] = f.z; AB[4 * j + 3] = f.w;
     }
-    float u[CT];  // (lanes 0-7 of a half)
+    float u[CT];  // (lanes 0-3 of a group)
 #pragma unroll
     for (int t = 0; t < CT; t++) {
       float y = raw[t * PT + 3 * DP + wc + mycol] - x[t][0];
 #pragma unroll
       for (int t2 = 0; t2 < t; t2++) y = fmaf(-AB[t * (t - 1) / 2 + t2], u[t2], y);
-      u[t] = t < ct ? raw[t * PT + 3 * DP + VC] * y : 0.f;
+      u[t] = raw[t * PT + 3 * DP + VC] * y;
     }
     {
       f32x2 gp[NP];
@@ -596,23 +590,23 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
       ld_vec(vd + (2 * CT + t) * DP, kp);
 #pragma unroll
       for (int cc = 0; cc < CL; cc++) {
-        const float uc = __shfl_sync(0xffffffffu, u[t], (lane & 16) | (CL == 8 ? cc : 2 * cc));
+        const float uc = __shfl_sync(0xffffffffu, u[t], (lane & 24) | (2 * cc));
         const f32x2 u2 = pack2(uc, uc);
 #pragma unroll
         for (int q = 0; q < NP; q++) S[cc][q] = fma2(kp[q], u2, S[cc][q]);
       }
     }
 #pragma unroll
-    for (int t = 0; t < CT; t++) u[t] = __shfl_xor_sync(0xffffffffu, u[t], 8);  // to the lanes that form o
-    if (b3 && (CL == 8 || !b0)) {
+    for (int t = 0; t < CT; t++) u[t] = __shfl_xor_sync(0xffffffffu, u[t], 4);  // to the lanes that form o
+    {
+      float *dst = fin.act ? os + (ch & 1) * CT * VC + wc + mycol : op;
+      const int step = fin.act ? VC : HV;
 #pragma unroll
       for (int t = 0; t < CT; t++) {
-        if (t >= ct) break;
         float ov = x[t][0];
 #pragma unroll
         for (int t2 = 0; t2 <= t; t2++) ov = fmaf(AB[6 + t * (t + 1) / 2 + t2], u[t2], ov);
-        if (fin.act) os[((ch & 1) * CT + t) * VC + wc + mycol] = ov;
-        else if (col0 + mycol < dv) o[(long long)(tok0 + i0 + t) * H * dv + (long long)h * dv + col0 + mycol] = ov;
+        if (writes && t < ct) dst[t * step] = ov;
       }
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -641,48 +635,53 @@ __global__ void __launch_bounds__(256, 1) stack_delta_kernel(StackDelta c, const
     for (int q = 0; q < NP; q++) unpack2(S[cc][q], v[2 * q], v[2 * q + 1]);
 #pragma unroll
     for (int m = 0; m < NM; m++) {
-      const int i = r * V + 16 * V * m;
-      if (V == 4 && vec) {
-        if (i < d) *reinterpret_cast<float4 *>(p + i) = make_float4(v[m * V], v[m * V + 1], v[m * V + (V > 2 ? 2 : 0)], v[m * V + (V > 3 ? 3 : 1)]);
+      const int i = r * 4 + 32 * m;
+      if (vec) {
+        if (i < d) *reinterpret_cast<float4 *>(p + i) = make_float4(v[m * 4], v[m * 4 + 1], v[m * 4 + 2], v[m * 4 + 3]);
       } else {
 #pragma unroll
-        for (int e = 0; e < V; e++)
-          if (i + e < d) p[i + e] = v[m * V + e];
+        for (int e = 0; e < 4; e++)
+          if (i + e < d) p[i + e] = v[m * 4 + e];
       }
     }
   }
 }
 
-template <int RL, int CL>
-static cudaError_t delta_go(const StackDelta &c, const float *buf, long long ld_b, const float *dec, float *state, const StackSpans &sp, float *o,
-                            int max_len, const float *norm, const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches,
-                            cudaStream_t st) {
-  constexpr int CW = 2 * CL;
-  const int total = (c.dv + CW - 1) / CW;  // warps that hold a head
-  int nw = std::min(total, 8);
-  // long spans: a head's columns are spread over more CTAs while that still brings idle SMs to work
-  const long long pairs = (long long)sp.n_spans * c.H;
-  while (max_len > 2 * kDeltaTok && nw > 2 && pairs * ((total + nw - 1) / nw) * 2 <= 148) nw = (nw + 1) / 2;
-  const int ncb = (total + nw - 1) / nw, VC = nw * CW;
+template <int RL, int MW>
+static cudaError_t delta_go(const StackDelta &c, const float *buf, long long ld_b, float *state, const StackSpans &sp, float *o, int nw, const float *norm,
+                            const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches, cudaStream_t st) {
+  const int total = (c.dv + 4 * kDeltaCols - 1) / (4 * kDeltaCols), ncb = (total + nw - 1) / nw, VC = nw * 4 * kDeltaCols;
   const DeltaFin fin{ncb == 1 ? act : nullptr, ld_act, gate, norm, c.eps, f32 ? 1 : 0};
   auto al = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-  const int vec = c.d % 4 == 0 && c.dv % 4 == 0 && ld_b % 4 == 0 && al(buf) && al(dec) && al(state);
+  const int vec = c.d % 4 == 0 && c.dv % 4 == 0 && ld_b % 4 == 0 && al(buf) && al(state);
   const size_t shb = (size_t)delta_smem_floats<RL>(nw, VC) * sizeof(float);
   static DeviceOnce once;
-  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_delta_kernel<RL, CL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); }));
-  stack_delta_kernel<RL, CL><<<(unsigned)(pairs * ncb), nw * 32, shb, st>>>(c, buf, ld_b, dec, state, sp, o, ncb, vec, fin);
+  DIS_CUDA_TRY(once.run([&] { return cudaFuncSetAttribute(stack_delta_kernel<RL, MW>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); }));
+  stack_delta_kernel<RL, MW><<<(unsigned)((long long)sp.n_spans * c.H * ncb), nw * 32, shb, st>>>(c, buf, (int)ld_b, state, sp, o, ncb, vec, fin);
   DIS_CUDA_TRY(cudaGetLastError());
   *launches += fin.act ? 1 : 2;
   return fin.act ? cudaSuccess : launch_stack_headnorm_silu(o, norm, gate, (long long)c.H * c.dv, act, ld_act, 0, 1.f, f32, sp.T, c.H, c.dv, c.eps, st, true);
 }
-cudaError_t launch_stack_delta(const StackDelta &c, const float *buf, long long ld_b, const float *dec, float *state, const StackSpans &sp, float *o,
-                               int max_len, const float *norm, const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches, cudaStream_t st) {
-#define DIS_DELTA(RL, CL) return delta_go<RL, CL>(c, buf, ld_b, dec, state, sp, o, max_len, norm, gate, act, ld_act, f32, launches, st)
+cudaError_t launch_stack_delta(const StackDelta &c, const float *buf, long long ld_b, float *state, const StackSpans &sp, float *o, int max_len,
+                               const float *norm, const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches, cudaStream_t st) {
   if (sp.T <= 0) return cudaSuccess;
-  if (c.d <= 32) DIS_DELTA(2, 8);
-  if (c.d <= 64) DIS_DELTA(4, 8);
-  if (c.d <= 128) DIS_DELTA(8, 8);
-  if (c.d <= 256) DIS_DELTA(16, 4);
+  // A head's columns in one CTA (its norm and gate then run inside), but for prompts, where a CTA takes at most eight warps and fewer
+  // while halving them still brings idle SMs to work.
+  const int total = (c.dv + 4 * kDeltaCols - 1) / (4 * kDeltaCols);
+  const bool prompts = max_len > 2 * kDeltaTok;
+  int nw = std::min(total, prompts || c.d > 128 ? 8 : 16);
+  while (prompts && nw > 4 && (long long)sp.n_spans * c.H * ((total + nw - 1) / nw) * 2 <= 148) nw = (nw + 1) / 2;
+#define DIS_DELTA(RL, MW) return delta_go<RL, MW>(c, buf, ld_b, state, sp, o, nw, norm, gate, act, ld_act, f32, launches, st)
+  if (nw <= 8) {
+    if (c.d <= 32) DIS_DELTA(4, 8);
+    if (c.d <= 64) DIS_DELTA(8, 8);
+    if (c.d <= 128) DIS_DELTA(16, 8);
+    if (c.d <= 256) DIS_DELTA(32, 8);
+  } else {
+    if (c.d <= 32) DIS_DELTA(4, 16);
+    if (c.d <= 64) DIS_DELTA(8, 16);
+    if (c.d <= 128) DIS_DELTA(16, 16);
+  }
 #undef DIS_DELTA
   return cudaErrorInvalidValue;
 }

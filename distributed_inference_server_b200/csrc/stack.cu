@@ -403,7 +403,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   static StackTensor dummy;  // scalars are written through their own small tensors below
   (void)dummy;
-  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0, lat_row = 0, lat_w[3] = {0, 0, 0}, max_gz = 0, max_bn[2] = {0, 0};
+  size_t max_proj = 1, max_mix = 1, max_act = 1, max_qf = 1, max_vrot = 0, max_dec = 0, max_ssm = 0, max_cq = 0, max_ql = 0, lat_row = 0, lat_w[3] = {0, 0, 0}, max_gz = 0, max_dz = 0, max_bn[2] = {0, 0};
   int max_top = 0, max_e = 0;
   bool any_shared = false;
   size_t max_sff = 0, max_moe[2] = {0, 0};
@@ -596,8 +596,8 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
       ENG_CUDA(tensor(L.w_o, (size_t)W * L.ld_act, M.f32));
       out_block(m_ + "o", 0, H * dv);
       max_mix = std::max(max_mix, (size_t)H * dv);
-      max_dec = std::max(max_dec, (size_t)H * d);
-      max_ssm = std::max(max_ssm, ((size_t)L.conv_ch + H + 3) / 4 * 4);
+      max_dz = std::max(max_dz, (size_t)H * d);
+      max_ssm = std::max(max_ssm, ((size_t)L.conv_ch + H * d + H + 3) / 4 * 4);
       max_gz = std::max(max_gz, (size_t)H * dv);
       max_bn[0] = std::max(max_bn[0], (size_t)ra); max_bn[1] = std::max(max_bn[1], (size_t)rg);
     } else if (lc.mixer == DIS_MIX_SSM) {
@@ -832,7 +832,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   if (max_gz) {
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.gz), cap * max_gz * 4));
-    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.dz), cap * max_dec * 4));
+    ENG_CUDA(alloc(reinterpret_cast<void **>(&M.dz), cap * max_dz * 4));
     ENG_CUDA(alloc(&M.bn_a, cap * max_bn[0] * esz));
     ENG_CUDA(alloc(&M.bn_g, cap * max_bn[1] * esz));
   }
@@ -907,7 +907,7 @@ int Engine::init_stack(const dis_engine_config *c, const dis_stack_config *sc) {
   }
   if (const char *g = getenv("DIS_STACK_PERSIST")) stack_persist = atoi(g) != 0;
   if (!M.f32 && stack_tc) {
-    M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), std::max((size_t)W, std::max(max_gz, max_gz ? max_dec : 0)));
+    M.scratch_elems = 2 * cap * std::max(std::max(max_proj, max_ql), std::max((size_t)W, std::max(max_gz, max_dz)));
     ENG_CUDA(alloc(reinterpret_cast<void **>(&M.scratch), M.scratch_elems * 4));
   }
   ENG_CUDA(alloc(reinterpret_cast<void **>(&M.logits), (size_t)M.max_rows * sc->vocab * 4));
@@ -1708,7 +1708,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
       a.proj = in_src; a.ld = N; a.n_part = in_parts; a.stride = in_stride;
       a.cw = reinterpret_cast<const float *>(L.conv_w.ptr); a.vec = reinterpret_cast<const float *>(L.ssm_vec.ptr); a.cstate = Rn.conv_state;
       a.a2 = L.a2.ptr; a.g2 = L.g2.ptr;
-      a.buf = M.ssm; a.ld_b = ((long long)sd.C + sd.H + 3) / 4 * 4; a.dec = M.dec; a.gz = M.gz;
+      a.buf = M.ssm; a.ld_b = ((long long)sd.C + nz + sd.H + 3) / 4 * 4; a.gz = M.gz;
       if (T > 64) {  // more tokens than the preparation should multiply by itself: the bottlenecks' products as matrix products
         RET_CUDA(launch_stack_delta_pack(sd, a, f32, T, M.bn_a, M.bn_g, stream));
         kl++;
@@ -1720,7 +1720,7 @@ cudaError_t Engine::stack_forward(int T, int n_spans, int n_qb, int R, bool all_
         a.z = M.dz;
       }
       RET_CUDA(launch_stack_delta_prep(sd, a, L.a2.f32, sp, stream));
-      RET_CUDA(launch_stack_delta(sd, M.ssm, a.ld_b, M.dec, Rn.state, sp, M.mix, max_span, reinterpret_cast<const float *>(L.norm_w.ptr), M.gz, M.act,
+      RET_CUDA(launch_stack_delta(sd, M.ssm, a.ld_b, Rn.state, sp, M.mix, max_span, reinterpret_cast<const float *>(L.norm_w.ptr), M.gz, M.act,
                                   L.ld_act, f32, &kl, stream));
       kl += sd.taps > 1 && !single ? 2 : 1;
       n_mix = L.ld_act;

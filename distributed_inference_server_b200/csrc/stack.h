@@ -154,16 +154,15 @@ struct StackDeltaPrep {
   float *cstate = nullptr;        // [slots][taps-1][C]
   const void *a2 = nullptr, *g2 = nullptr;  // [H*d][ra], [H*dv][rg], compute type
   const float *z = nullptr;       // [T][H*d]: the products with a2, when they (and the gate's) were made by matrix products; null: made here
-  float *buf = nullptr;           // [T][ld_b]: q | k | v as they enter the recurrence, beta [H]
+  float *buf = nullptr;           // [T][ld_b]: q | k | v as they enter the recurrence, decays [H*d], beta [H]
   long long ld_b = 0;
-  float *dec = nullptr;           // [T][H*d]
   float *gz = nullptr;            // [T][H*dv]: the gate's logits (written here when z is null)
 };
 // q, k, v, step sizes and decays of the pass's tokens; the convolution's tail moves on
 cudaError_t launch_stack_delta_prep(const StackDelta &c, const StackDeltaPrep &a, bool w_f32, const StackSpans &sp, cudaStream_t st);
 cudaError_t launch_stack_delta_pack(const StackDelta &c, const StackDeltaPrep &a, bool f32, int T, void *ua, void *ug, cudaStream_t st);
 // the recurrence over state [slots][H][dv][d], head norm and gate behind it: act [T][ld_act] (compute type).  o [T][H*dv]: room.  d <= 256
-cudaError_t launch_stack_delta(const StackDelta &c, const float *buf, long long ld_b, const float *dec, float *state, const StackSpans &sp, float *o,
+cudaError_t launch_stack_delta(const StackDelta &c, const float *buf, long long ld_b, float *state, const StackSpans &sp, float *o,
                                int max_len, const float *norm, const float *gate, void *act, long long ld_act, bool f32, uint64_t *launches, cudaStream_t st);
 // out[t][off + h*dv + j] = scale * unit_rms_over_head(o[t][h])[j] * w[j] * silu(gate[t][h*dv + j]); out [T][ldo] compute type; w null: ones.
 // sig: times sigmoid(gate) instead
